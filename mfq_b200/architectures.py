@@ -7,7 +7,8 @@ Runtime code consumes canonical names only (``model.block.N.attention.query.weig
   ``in_proj_ba`` form, ``model.language_model.`` prefix, ``model.visual.*`` kept under ``vision.*``, ``mtp.*`` head);
 * ``deepseek_v3`` / ``glm4_moe``: latent-attention and shared-expert names, sigmoid router bias, and the next-token
   prediction layer these checkpoints append after the last decoder layer (``model.layers.<L>.{enorm,hnorm,eh_proj,
-  shared_head.*}``), which becomes the ``predictor.*`` head.
+  shared_head.*}``), which becomes the ``predictor.*`` head;
+* ``tepetar``: ``l<N>.{mix,mlp,side}.*`` names (``config.json`` names the design under ``architecture``).
 
 :func:`detect_family` picks the family from ``config.json`` (``model_type`` / ``architectures``); :func:`to_canonical`
 renames, stacks per-expert matrices, splits fused tensors and moves the appended prediction layer.  Names match the
@@ -100,6 +101,21 @@ VISION_BLOCK = {
     "mlp.linear_fc1.weight": "mlp.up.weight", "mlp.linear_fc1.bias": "mlp.up.bias",
     "mlp.linear_fc2.weight": "mlp.down.weight", "mlp.linear_fc2.bias": "mlp.down.bias",
 }
+# Tepetar: the design has its own short names; a linear's bias is its name with ``.b`` added
+TEPETAR_TOP = {
+    "embed": "model.token_embedding.weight", "side.embed": "model.token_side.embedding.weight",
+    "final.norm": "model.output_norm.weight", "head": "model.output.weight",
+}
+TEPETAR_LAYER = {
+    "norm1": "attention.post_norm.weight", "norm2": "mlp.post_norm.weight",
+    "mix.q": "attention.query.weight", "mix.k": "attention.key.weight", "mix.v": "attention.value.weight",
+    "mix.o": "attention.output.weight", "mix.q.b": "attention.query.bias", "mix.k.b": "attention.key.bias",
+    "mix.v.b": "attention.value.bias", "mix.o.b": "attention.output.bias", "mix.q.norm": "attention.query_norm.weight",
+    "mix.k.norm": "attention.key_norm.weight", "mix.vmix": "attention.value_mix",
+    "mlp.gate": "mlp.gate.weight", "mlp.up": "mlp.up.weight", "mlp.down": "mlp.down.weight",
+    "side.gate": "token_side.gate.weight", "side.proj": "token_side.projection.weight", "side.norm": "token_side.norm.weight",
+}
+_TEPETAR_LAYER_RE = re.compile(r"^l(\d+)\.(.+)$")
 FAMILY_OF_MODEL_TYPE = {
     "llama": "llama", "mistral": "llama", "qwen2": "llama", "qwen3": "llama", "mixtral": "llama", "qwen2_moe": "llama",
     "qwen3_moe": "llama", "qwen3_next": "qwen3_next", "qwen3_5": "qwen3_next", "qwen3_5_moe": "qwen3_next",
@@ -111,6 +127,8 @@ FAMILY_OF_MODEL_TYPE = {
 def detect_family(hf_config: dict | None, names=()) -> str:
     """Source naming family of a checkpoint: from ``model_type`` (or the text sub-config's), else from its tensor names."""
     cfg = hf_config or {}
+    if str(cfg.get("architecture", "")).lower() == "tepetar":
+        return "tepetar"
     for c in (cfg, cfg.get("text_config") or {}):
         fam = FAMILY_OF_MODEL_TYPE.get(str(c.get("model_type", "")).lower())
         if fam:
@@ -168,6 +186,14 @@ def canonical_name(hf_name: str, nextn_layer: int | None = None) -> tuple[str, i
     return None
 
 
+def tepetar_name(name: str) -> str | None:
+    """Source name of a Tepetar tensor -> canonical name."""
+    if name in TEPETAR_TOP:
+        return TEPETAR_TOP[name]
+    m = _TEPETAR_LAYER_RE.match(name)
+    return f"model.block.{int(m[1])}.{TEPETAR_LAYER[m[2]]}" if m and m[2] in TEPETAR_LAYER else None
+
+
 def split_fused_linear_attention(out: dict[str, np.ndarray], k_heads: int, v_heads: int, head_dim: int) -> None:
     """The hybrid family's fused projections, in place: ``in_proj_qkvz`` holds, per KEY head, the rows
     ``[q (d) | k (d) | v (r d) | z (r d)]`` with ``r = v_heads / k_heads``; ``in_proj_ba`` holds ``[b (r) | a (r)]`` per
@@ -196,6 +222,8 @@ def to_canonical(hf_tensors: dict[str, np.ndarray], hf_config: dict | None = Non
     prediction layer appended after the decoder stack moves under ``predictor.*``.  ``hf_config`` (the checkpoint's
     ``config.json``) selects the family and supplies the geometry those steps need."""
     family = detect_family(hf_config, hf_tensors)
+    if family == "tepetar":
+        return {c: t for c, t in ((tepetar_name(n), t) for n, t in hf_tensors.items()) if c is not None}
     text = dict(hf_config or {})
     text.update(text.get("text_config") or {})
     nextn = None
@@ -241,7 +269,11 @@ def to_canonical(hf_tensors: dict[str, np.ndarray], hf_config: dict | None = Non
 
 def config_from_hf(hf: dict) -> dict:
     """``config.json`` of a Hugging Face model -> the keyword arguments of ``MoeDecoderConfig`` (and of its hybrid and
-    latent-attention extensions); a multimodal wrapper's ``text_config`` is looked through."""
+    latent-attention extensions); a multimodal wrapper's ``text_config`` is looked through.  A design with a configuration
+    of its own (``family`` in the result) gives the fields of that class instead."""
+    if detect_family(hf) == "tepetar":
+        from .models.tepetar import TepetarConfig
+        return TepetarConfig.from_source(hf).to_dict()
     if hf.get("text_config"):
         hf = {**hf, **hf["text_config"]}
     heads = hf.get("num_attention_heads", 32)

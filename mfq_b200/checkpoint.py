@@ -237,16 +237,19 @@ def load_engine(path, device="cuda", *, native_4bit: bool = False, expert_slots:
                 max_seq_len: int = 8192, tp_rank: int = 0, tp_size: int = 1,
                 collective=None, use_graphs: bool = True, kv_budget_bytes: int | None = None,
                 yarn_context_extension: float | None = None, mtp_draft_tokens: int = 0, mtp_adaptive: bool = False, mtp_dynamic_depth: bool = False,
-                lp_rank: int = 0, lp_size: int = 1, layer_split=None, expert_graphs: bool = False):
+                lp_rank: int = 0, lp_size: int = 1, layer_split=None, expert_graphs: bool = False, dtype: str = "auto",
+                num_pages: int | None = None):
     """``.mfq`` -> (engine, tokenizer, config).  ``kv_budget_bytes`` caps the paged KV pool (see ``engine/kv_budget.py``);
     on a GPU it defaults to 90 % of the memory that is free once the weights are resident.  ``yarn_context_extension``
     (> 1) runs the model on that multiple of its trained context with YaRN-scaled rotary frequencies.
     ``mtp_draft_tokens`` (K > 0, only with a checkpoint that carries a ``predictor.*`` head): greedy rows decode by
     draft/verify cycles; ``mtp_adaptive`` parks the cycles while they are slower than plain decoding.
     ``expert_graphs`` (with ``expert_slots``): decode inside CUDA graphs with the experts that are resident and settle
-    misses after the step (``LLMEngine.enable_expert_residency_graphs``); without it such a model decodes eagerly."""
+    misses after the step (``LLMEngine.enable_expert_residency_graphs``); without it such a model decodes eagerly.
+    ``dtype``: element type of weights and activations for the families that offer a choice (``models/registry.py``).
+    ``num_pages``: size of the KV pool in pages (page 0 is the null page), instead of a memory budget."""
     from .engine.llm_engine import LLMEngine
-    from .models.moe_decoder import MoeDecoderConfig, MoeDecoderModel, MoeWeights
+    from .models import registry
     from .server.tokenizer import tokenizer_from_assets
     import contextlib
     if Path(path).is_dir():  # a Hugging Face directory served directly: float tensors, transcoded to FP8 on load
@@ -266,30 +269,22 @@ def load_engine(path, device="cuda", *, native_4bit: bool = False, expert_slots:
             trained = int((raw.get("rope_scaling") or {}).get("original_max_position") or raw.get("max_position") or 8192)
             raw["rope_scaling"] = dict(raw.get("rope_scaling") or {}, factor=float(yarn_context_extension), original_max_position=trained)
             raw["max_position"] = int(trained * yarn_context_extension)
-        if raw.get("kv_lora_rank"):  # latent attention family
-            from .models.mla import MlaConfig, MlaModel, mla_weights_from_tensors
-            if tp_size != 1:
-                raise NotImplementedError("latent-attention checkpoints load on a single rank")
-            cfg = MlaConfig(**{k: v for k, v in raw.items() if k in MlaConfig.__dataclass_fields__})
-            weights = mla_weights_from_tensors(cfg, store, device)
-            model = MlaModel(cfg, weights)
-        else:
-            fields = {f for f in MoeDecoderConfig.__dataclass_fields__}
-            cfg = MoeDecoderConfig(**{k: v for k, v in raw.items() if k in fields})
-            weights = MoeWeights.from_tensors(cfg, store, device, tp_rank, tp_size, expert_slots=expert_slots, native_4bit=native_4bit,
-                                              lp_rank=lp_rank, lp_size=lp_size, layer_split=layer_split)
-            model = MoeDecoderModel(cfg, weights, collective=collective)
+        family = registry.find(raw)
+        family.check_dtype(dtype)
+        cfg, weights, model = family.build(raw, store, registry.LoadOptions(
+            device=device, dtype=dtype, native_4bit=native_4bit, expert_slots=expert_slots, tp_rank=tp_rank, tp_size=tp_size,
+            lp_rank=lp_rank, lp_size=lp_size, layer_split=layer_split, collective=collective))
     # host-tier experts read the routing on the host every step, which a captured graph cannot do; with
     # ``expert_graphs`` the step translates ids on the device instead and the engine settles misses afterwards
-    num_pages = None
-    if kv_budget_bytes is None and str(device).startswith("cuda"):
+    if kv_budget_bytes is None and num_pages is None and str(device).startswith("cuda"):
         from .engine.kv_budget import device_budget
         kv_budget_bytes = device_budget(device)
-    if kv_budget_bytes is not None:
+    if kv_budget_bytes is not None and num_pages is None:
         from .engine.kv_budget import plan
         has_head = getattr(weights, "mtp", None) is not None
         num_pages = plan(budget_bytes=kv_budget_bytes, layers=model.local_layers + int(has_head), kv_heads=model.hk, head_dim=cfg.head_dim,
-                         max_batch=max_batch, max_seq_len=max_seq_len).num_pages
+                         max_batch=max_batch, max_seq_len=max_seq_len,
+                         token_bytes=model.kv_token_bytes() if hasattr(model, "kv_token_bytes") else None).num_pages
     engine = LLMEngine(model, max_batch=max_batch, max_seq_len=max_seq_len, device=device, num_pages=num_pages,
                        use_graphs=use_graphs and (expert_slots is None or expert_graphs),
                        mtp_draft_tokens=mtp_draft_tokens if getattr(weights, "mtp", None) is not None else 0,

@@ -40,8 +40,9 @@ def page_bytes(layers: int, kv_heads: int, head_dim: int) -> int:
 
 
 def plan(*, budget_bytes: int, layers: int, kv_heads: int, head_dim: int, max_batch: int, max_seq_len: int,
-         state_bytes_per_row: int = 0) -> KvPlan:
-    pb = page_bytes(layers, kv_heads, head_dim)
+         state_bytes_per_row: int = 0, token_bytes: int | None = None) -> KvPlan:
+    """``token_bytes``: cache bytes per token of a model whose pages are not the FP8 layout (then the geometry is unused)."""
+    pb = page_bytes(layers, kv_heads, head_dim) if token_bytes is None else token_bytes * PAGE_TOKENS
     per_seq = (max_seq_len + PAGE_TOKENS - 1) // PAGE_TOKENS
     wanted = max_batch * per_seq + 1
     state = state_bytes_per_row * max_batch

@@ -1,6 +1,7 @@
-"""Paged KV cache with FP8 pages.
+"""Paged KV caches: page tables (:class:`PagedTables`) over FP8 pages (:class:`PagedKVCache`) or over unquantized pages whose
+geometry may differ from layer to layer (:class:`PlainPagedKVCache`).
 
-Pool layout per layer (what the CUDA kernels index), chosen so that the decode-attention kernel can fetch a
+FP8 pool layout per layer (what the CUDA kernels index), chosen so that the decode-attention kernel can fetch a
 page with one bulk copy and read tensor-core fragments with single shared-memory loads:
 
 * ``k : [pages, kv_heads, head_dim/64, page_size, 64]`` E4M3 (64-dim chunks, token-major inside a chunk);
@@ -76,13 +77,87 @@ class PageAllocator:
             self.free.append(p)
 
 
-class PagedKVCache:
-    def __init__(self, *, layers: int, kv_heads: int, head_dim: int, num_pages: int, max_seqs: int,
-                 max_pages_per_seq: int, device: torch.device | str, page_size: int = PAGE_SIZE) -> None:
+class PagedTables:
+    """Page allocator and device block table of a cache: what the engine and the kernels' page lookups share, whatever the
+    pages hold."""
+
+    def __init__(self, *, num_pages: int, max_seqs: int, max_pages_per_seq: int, device: torch.device, page_size: int) -> None:
         self.page_size = page_size
         self.num_pages = num_pages
         self.max_pages_per_seq = max_pages_per_seq
+        self.block_table = torch.zeros((max_seqs, max_pages_per_seq), dtype=torch.int32, device=device)
+        self.allocator = PageAllocator(num_pages)
+
+    def assign(self, row: int, seq_id: int, tokens: int) -> None:
+        """Make block-table ``row`` cover ``tokens`` tokens of ``seq_id`` (allocating pages as needed)."""
+        pages = self.allocator.ensure(seq_id, tokens, self.page_size)
+        if len(pages) > self.max_pages_per_seq:
+            raise MemoryError("sequence exceeds max_pages_per_seq")
+        self.block_table[row, : len(pages)] = torch.tensor(pages, dtype=torch.int32)
+
+    def slots(self, seq_id: int, start: int, count: int) -> torch.Tensor:
+        pages = self.allocator.owned[seq_id]
+        pos = torch.arange(start, start + count)
+        page_ids = torch.tensor(pages, dtype=torch.int64)[pos // self.page_size]
+        return (page_ids * self.page_size + pos % self.page_size).to(torch.int32)
+
+    def release(self, seq_id: int) -> None:
+        self.allocator.release(seq_id)
+
+
+@dataclass
+class PlainLayerKV:
+    k: torch.Tensor  # [pages, kv_heads, page_size, dk]
+    v: torch.Tensor  # [pages, kv_heads, page_size, dv]
+    page_size: int
+
+
+class PlainPagedKVCache(PagedTables):
+    """Unquantized pages (bf16 or fp32): per layer ``k [pages, kv_heads, 16, dk]`` and ``v [pages, kv_heads, 16, dv]`` for that
+    layer's ``(kv_heads, dk, dv)``.  Pages start as zeros and only ever hold finite numbers, so a kernel may read the unused
+    slots of a page."""
+
+    def __init__(self, shapes: list[tuple[int, int, int]], dtype: torch.dtype, *, num_pages: int, max_seqs: int,
+                 max_pages_per_seq: int, device: torch.device | str, page_size: int = PAGE_SIZE) -> None:
         dev = torch.device(device)
+        super().__init__(num_pages=num_pages, max_seqs=max_seqs, max_pages_per_seq=max_pages_per_seq, device=dev, page_size=page_size)
+        self.shapes, self.dtype, self.layers = list(shapes), dtype, len(shapes)
+        self.pools = [PlainLayerKV(torch.zeros((num_pages, g, page_size, dk), dtype=dtype, device=dev),
+                                   torch.zeros((num_pages, g, page_size, dv), dtype=dtype, device=dev), page_size)
+                      for g, dk, dv in self.shapes]
+
+    def layer(self, i: int) -> PlainLayerKV:
+        return self.pools[i]
+
+    def bytes_per_token(self) -> int:
+        return sum(g * (dk + dv) for g, dk, dv in self.shapes) * self.dtype.itemsize
+
+    def page_blob_bytes(self, pages: int) -> int:
+        return pages * self.page_size * self.bytes_per_token()
+
+    def export_pages(self, page_ids: list[int]):
+        """All layers' K and V of the given pages as one contiguous uint8 numpy array (host)."""
+        idx = torch.tensor(page_ids, dtype=torch.long, device=self.block_table.device)
+        parts = [t.index_select(0, idx).view(torch.uint8).reshape(-1) for l in self.pools for t in (l.k, l.v)]
+        return torch.cat(parts).cpu().numpy()
+
+    def import_pages(self, page_ids: list[int], blob) -> None:
+        """Inverse of :meth:`export_pages` into (possibly different) physical pages."""
+        idx = torch.tensor(page_ids, dtype=torch.long, device=self.block_table.device)
+        raw, off = torch.from_numpy(blob).to(self.block_table.device), 0
+        for l in self.pools:
+            for t in (l.k, l.v):
+                shape = (len(page_ids),) + tuple(t.shape[1:])
+                nbytes = len(page_ids) * t[0].numel() * t.element_size()
+                t.index_copy_(0, idx, raw[off : off + nbytes].clone().view(t.dtype).view(shape))
+                off += nbytes
+
+
+class PagedKVCache(PagedTables):
+    def __init__(self, *, layers: int, kv_heads: int, head_dim: int, num_pages: int, max_seqs: int,
+                 max_pages_per_seq: int, device: torch.device | str, page_size: int = PAGE_SIZE) -> None:
+        dev = torch.device(device)
+        super().__init__(num_pages=num_pages, max_seqs=max_seqs, max_pages_per_seq=max_pages_per_seq, device=dev, page_size=page_size)
         if page_size != 16 or head_dim % 64:
             raise ValueError("the FP8 page layout needs 16-token pages and a head dim that is a multiple of 64")
         self.head_dim, self.kv_heads, self.layers = head_dim, kv_heads, layers
@@ -90,8 +165,6 @@ class PagedKVCache:
         self.v = torch.zeros((layers, num_pages, kv_heads, head_dim, page_size), dtype=torch.float8_e4m3fn, device=dev)
         self.k_scale = torch.zeros((layers, num_pages, kv_heads, page_size), dtype=torch.float32, device=dev)
         self.v_scale = torch.zeros((layers, num_pages, kv_heads, page_size), dtype=torch.float32, device=dev)
-        self.block_table = torch.zeros((max_seqs, max_pages_per_seq), dtype=torch.int32, device=dev)
-        self.allocator = PageAllocator(num_pages)
 
     def layer(self, i: int) -> LayerKV:
         return LayerKV(self.k[i], self.v[i], self.k_scale[i], self.v_scale[i], self.page_size)
@@ -129,19 +202,3 @@ class PagedKVCache:
 
     def bytes_per_token(self) -> int:
         return self.layers * self.kv_heads * (2 * self.head_dim + 8)
-
-    def assign(self, row: int, seq_id: int, tokens: int) -> None:
-        """Make block-table ``row`` cover ``tokens`` tokens of ``seq_id`` (allocating pages as needed)."""
-        pages = self.allocator.ensure(seq_id, tokens, self.page_size)
-        if len(pages) > self.max_pages_per_seq:
-            raise MemoryError("sequence exceeds max_pages_per_seq")
-        self.block_table[row, : len(pages)] = torch.tensor(pages, dtype=torch.int32)
-
-    def slots(self, seq_id: int, start: int, count: int) -> torch.Tensor:
-        pages = self.allocator.owned[seq_id]
-        pos = torch.arange(start, start + count)
-        page_ids = torch.tensor(pages, dtype=torch.int64)[pos // self.page_size]
-        return (page_ids * self.page_size + pos % self.page_size).to(torch.int32)
-
-    def release(self, seq_id: int) -> None:
-        self.allocator.release(seq_id)

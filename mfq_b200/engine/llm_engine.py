@@ -46,6 +46,22 @@ class GenerationResult:
     new_tokens: int
 
 
+@dataclass
+class PendingPrompt:
+    """A prompt on its way into the cache: admitted by :meth:`LLMEngine.begin_prompt`, read by :meth:`LLMEngine.mixed_step`."""
+
+    ids: torch.Tensor  # the whole prompt, on the device
+    done: int  # tokens in the cache
+    start: int  # ... of which restored from a cache
+    keys: object  # prefix-cache keys
+    params: object
+    generated: int
+
+    @property
+    def total(self) -> int:
+        return self.ids.numel()
+
+
 class LLMEngine:
     def __init__(self, model: LlamaModel, *, max_batch: int = 64, max_seq_len: int = 8192, num_pages: int | None = None,
                  device=None, use_graphs: bool | None = None, mtp_draft_tokens: int = 0, prefill_chunk: int | None = None,
@@ -82,8 +98,11 @@ class LLMEngine:
         pages_per_seq = (max_seq_len + PAGE_SIZE - 1) // PAGE_SIZE
         if num_pages is None:
             num_pages = max_batch * pages_per_seq + 1
-        self.cache = PagedKVCache(layers=getattr(model, "local_layers", cfg.num_layers) + (1 if has_head else 0), kv_heads=model.hk, head_dim=cfg.head_dim, num_pages=num_pages,
-                                  max_seqs=max_batch, max_pages_per_seq=pages_per_seq, device=self.device)
+        pool = dict(num_pages=num_pages, max_seqs=max_batch, max_pages_per_seq=pages_per_seq, device=self.device)
+        if hasattr(model, "make_cache"):  # a model whose pages are not the FP8 layout brings its own cache
+            self.cache = model.make_cache(**pool)
+        else:
+            self.cache = PagedKVCache(layers=getattr(model, "local_layers", cfg.num_layers) + (1 if has_head else 0), kv_heads=model.hk, head_dim=cfg.head_dim, **pool)
         dev = self.device
         self.input_ids = torch.zeros(max_batch, dtype=torch.int32, device=dev)
         self.positions = torch.zeros(max_batch, dtype=torch.int32, device=dev)
@@ -102,6 +121,7 @@ class LLMEngine:
         self.row_seq: dict[int, int] = {}
         self.row_len: dict[int, int] = {}  # host mirror of seq_lens for page management
         self.row_stochastic: dict[int, bool] = {}
+        self.row_prompt: dict[int, PendingPrompt] = {}  # rows whose prompt is still being read (mixed batches)
         self.row_constraint: dict[int, object] = {}  # row -> grammar state of a structured-output request
         self.logit_bias: torch.Tensor | None = None  # [max_batch, vocabulary] bf16, allocated by the first such request
         self._token_bytes, self._constraint_vocab, self._constraint_stop = None, None, ()
@@ -207,6 +227,7 @@ class LLMEngine:
         if seq is not None:
             self.cache.release(seq)
         self.row_len.pop(row, None)
+        self.row_prompt.pop(row, None)
         self.row_stochastic.pop(row, None)
         self.row_constraint.pop(row, None)
 
@@ -238,12 +259,35 @@ class LLMEngine:
         v = logits.shape[1]
         if self.sample_work is None or self.sample_work.shape[1] != v:
             self.sample_work = torch.empty((self.max_batch, v), dtype=torch.float32, device=self.device)
-        fn = ops.lib.lib().mfq_sample
+        fn = ops.lib.lib().mfq_sample_f32 if logits.dtype == torch.float32 else ops.lib.lib().mfq_sample
         fn.argtypes = [C.c_void_p, C.c_int, C.c_int, C.c_int] + [C.c_void_p] * 6
         fn.restype = C.c_int
         rc = fn(logits.data_ptr(), b, v, logits.stride(0), None, self.sample_rows.data_ptr(), self.seq_lens.data_ptr(),
                 self.sample_work.data_ptr(), self.sampled.data_ptr(), ops.lib.stream_ptr())
         ops.lib.check(rc, "sample")
+
+    def _sample_rows(self, logits: torch.Tensor, rows: list[int]) -> torch.Tensor:
+        """Draw one token per entry of ``rows`` from ``logits [len(rows), vocabulary]`` with the rows' own records, constraints
+        and draw counters (``seq_lens``); the tokens also become the rows' ``sampled``."""
+        n, dev = len(rows), self.device
+        idx = torch.tensor(rows, dtype=torch.long).to(dev)
+        if any(r in self.row_constraint for r in rows):
+            bias = self._bias_rows(logits, self.max_batch)
+            self._write_bias(rows)
+            logits = logits + bias.index_select(0, idx)
+        if not any(self.row_stochastic.get(r, False) for r in rows):
+            toks = self.model.sample_greedy(logits)
+        else:
+            held = self.sample_rows, self.seq_lens, self.sampled
+            toks = torch.zeros(n, dtype=torch.int32, device=dev)
+            try:  # the sampler reads records and counters by position: line them up with the logits
+                self.sample_rows, self.seq_lens = held[0].index_select(0, idx), held[1].index_select(0, idx)
+                self.sampled = toks
+                self._sample(logits, n, True)
+            finally:
+                self.sample_rows, self.seq_lens, self.sampled = held
+        self.sampled.index_copy_(0, idx, toks)
+        return toks
 
     def _sample_reference(self, logits: torch.Tensor, b: int) -> None:
         for r in range(b):
@@ -275,41 +319,16 @@ class LLMEngine:
         replayed request); a token constraint re-reads them before it masks the next token."""
         dev = self.device
         self._bind_state()
-        ids = torch.as_tensor(token_ids, dtype=torch.int32)
+        ids, start, keys = self._admit(row, token_ids, params, session)
         n = int(ids.numel())
-        if n + 1 > self.max_seq_len:
-            raise ValueError(f"prompt of {n} tokens exceeds the engine's context of {self.max_seq_len}")
-        if row in self.row_seq:
-            self.release(row)
-        seq_id = self._next_seq_id
-        self._next_seq_id += 1
-        self.row_seq[row] = seq_id
-        try:
-            self.cache.assign(row, seq_id, n + 1)
-        except MemoryError:
-            self.release(row)
-            raise
-        self.set_sampling(row, params)
-        ids = ids.to(dev, non_blocking=True)
+        seq_id = self.row_seq[row]
         state_slots = None
         if self.rec_state is not None:
-            self.rec_state.reset(row)
             state_slots = self.row_ids[row : row + 1]
         last = torch.tensor([n - 1], dtype=torch.int32, device=dev)
-        start, keys = 0, None
-        if session is not None and self.session_cache is not None and not self.mtp_k:
-            start = self.session_cache.restore(self, row, session, [int(t) for t in ids.tolist()])
-        if start == 0:
-            start, keys = self._restore_prefix(seq_id, token_ids, n)
         logits, hidden = self._prefill_span(row, seq_id, ids, start, n, state_slots)
-        self._store_prefix(seq_id, keys, start)
-        self.seq_lens[row] = n
-        self.row_len[row] = n
-        constraint = self._constraint_for(params)
+        constraint = self._prompt_read(row, ids, start, keys, params, generated)
         if constraint is not None:
-            for t in (ids[n - generated :].tolist() if generated else ()):
-                constraint.advance(int(t))
-            self.row_constraint[row] = constraint
             bias = self._bias_rows(logits, self.max_batch)[row : row + 1]
             self._write_bias([row])
             logits = logits + bias
@@ -336,6 +355,155 @@ class LLMEngine:
         if constraint is not None:
             constraint.advance(int(tok))
         return int(tok)
+
+    def _admit(self, row: int, token_ids, params, session):
+        """Give batch row ``row`` a sequence with pages for the prompt and restore what a cache holds of it.  Returns
+        (the prompt on the device, tokens restored, prefix-cache keys)."""
+        ids = torch.as_tensor(token_ids, dtype=torch.int32)
+        n = int(ids.numel())
+        if n + 1 > self.max_seq_len:
+            raise ValueError(f"prompt of {n} tokens exceeds the engine's context of {self.max_seq_len}")
+        seq_id = self.open_row(row, params)
+        try:
+            self.cache.assign(row, seq_id, n + 1)
+        except MemoryError:
+            self.release(row)
+            raise
+        ids = ids.to(self.device, non_blocking=True)
+        start, keys = 0, None
+        if session is not None and self.session_cache is not None and not self.mtp_k:
+            start = self.session_cache.restore(self, row, session, [int(t) for t in ids.tolist()])
+        if start == 0:
+            start, keys = self._restore_prefix(seq_id, token_ids, n)
+        return ids, start, keys
+
+    def _prompt_read(self, row: int, ids, start: int, keys, params, generated: int):
+        """Bookkeeping once every prompt token is in the cache; returns the row's token constraint (or None)."""
+        n = int(ids.numel())
+        self._store_prefix(self.row_seq[row], keys, start)
+        self.seq_lens[row] = n
+        self.row_len[row] = n
+        constraint = self._constraint_for(params)
+        if constraint is not None:
+            for t in (ids[n - generated :].tolist() if generated else ()):
+                constraint.advance(int(t))
+            self.row_constraint[row] = constraint
+        return constraint
+
+    # -- ragged batches: portions of several sequences in one forward ---------------------------------------------------
+    @property
+    def mixed_batches(self) -> bool:
+        """Whether portions of prompts and decoded tokens may share a forward (:meth:`mixed_step`)."""
+        return self.model.ragged and self.mtp_k == 0
+
+    def open_row(self, row: int, params=None) -> int:
+        """Start an empty sequence on batch row ``row`` (ending the one it held); returns its id."""
+        if row in self.row_seq:
+            self.release(row)
+        seq_id = self._next_seq_id
+        self._next_seq_id += 1
+        self.row_seq[row] = seq_id
+        self.row_len[row] = 0
+        self.set_sampling(row, params)
+        if self.rec_state is not None:
+            self.rec_state.reset(row)
+        return seq_id
+
+    def _ragged_step(self, portions, ids: torch.Tensor) -> StepBuffers:
+        """Step of a ragged batch.  ``portions``: ``(row, first position, tokens)``, single tokens first; ``ids`` (device): their
+        tokens one after the other.  Everything the host knows travels in one copy."""
+        rows = [r for r, _, _ in portions]
+        counts = [m for _, _, m in portions]
+        total, b = sum(counts), len(portions)
+        starts = [0]
+        for m in counts:
+            starts.append(starts[-1] + m)
+        host = torch.cat([
+            torch.cat([torch.arange(c, c + m, dtype=torch.int32) for _, c, m in portions]),
+            torch.cat([self.cache.slots(self.row_seq[r], c, m) for r, c, m in portions]),
+            torch.repeat_interleave(torch.arange(b, dtype=torch.int32), torch.tensor(counts)),
+            torch.tensor(starts, dtype=torch.int32), torch.tensor([c + m for _, c, m in portions], dtype=torch.int32),
+            torch.tensor(rows, dtype=torch.int32)])
+        if self.device.type == "cuda":
+            host = host.pin_memory()
+        positions, slots, tok_seq, q_starts, seq_lens, row_ids = host.to(self.device, non_blocking=True).split(
+            [total, total, total, b + 1, b, b])
+        singles = next((i for i, m in enumerate(counts) if m != 1), b)
+        if hasattr(self.model, "decode_splits"):
+            self.model.attn_splits = self.model.decode_splits(max(1, singles), max(c + m for _, c, m in portions))
+        return StepBuffers(input_ids=ids, positions=positions, slots=slots, block_table=self.cache.block_table.index_select(0, row_ids.long()),
+                           seq_lens=seq_lens, cu_seqlens=starts, q_starts=q_starts, tok_seq=tok_seq, max_q=max(counts), num_decode=singles)
+
+    def extend(self, portions, wanted=None) -> torch.Tensor | None:
+        """Append given tokens to open rows, all in one forward: ``portions`` is a list of ``(row, token ids)`` (a row at most
+        once), ``wanted`` a list of places per portion whose logits are asked for.  Returns those logits
+        ``[sum(len(w)), vocabulary]`` in the order of ``portions`` and ``wanted`` (None if nothing is wanted)."""
+        if not self.model.ragged:
+            raise NotImplementedError("this model does not take ragged batches")
+        wanted = [()] * len(portions) if wanted is None else wanted
+        order = sorted(range(len(portions)), key=lambda i: len(portions[i][1]) != 1)  # stable: single tokens first
+        spans, first, at = [], {}, 0
+        for i in order:
+            row, toks = portions[i]
+            start, m = self.row_len[row], len(toks)
+            if m == 0 or start + m > self.max_seq_len:
+                raise ValueError(f"row {row}: {m} tokens after {start} do not fit a context of {self.max_seq_len}")
+            self.cache.assign(row, self.row_seq[row], start + m)
+            spans.append((row, start, m))
+            first[i], at = at, at + m
+        ids = torch.tensor([int(t) for i in order for t in portions[i][1]], dtype=torch.int32).to(self.device)
+        step = self._ragged_step(spans, ids)
+        rows = [first[i] + int(w) for i in range(len(portions)) for w in wanted[i]]
+        pick = torch.tensor(rows or [0], dtype=torch.int32).to(self.device)
+        logits = self._forward_ragged(step, pick)
+        for row, start, m in spans:
+            self.row_len[row] = start + m
+        self.seq_lens.index_copy_(0, torch.tensor([r for r, _, _ in spans]).to(self.device), step.seq_lens)
+        return logits if rows else None
+
+    def _forward_ragged(self, step: StepBuffers, logits_rows: torch.Tensor) -> torch.Tensor:
+        """A batch of single tokens is a decode step; anything else runs as a ragged batch."""
+        prefill = step.num_decode < step.seq_lens.numel()
+        return self.model.forward(step, self.cache, prefill=prefill, logits_rows=logits_rows, gather_logits=False)
+
+    def begin_prompt(self, row: int, token_ids, params=None, session: str | None = None, generated: int = 0) -> int:
+        """Admit a prompt to batch row ``row`` without running it (arguments of :meth:`prefill`); :meth:`mixed_step` reads it in
+        portions.  Returns the number of tokens left to read."""
+        ids, start, keys = self._admit(row, token_ids, params, session)
+        self.row_prompt[row] = PendingPrompt(ids, start, start, keys, params, generated)
+        return self.row_prompt[row].total - start
+
+    def mixed_step(self, decode_rows: list[int], portions: list[tuple[int, int]]) -> dict[int, int]:
+        """One forward that advances every row of ``decode_rows`` by a token and reads the next ``count`` prompt tokens of
+        every ``(row, count)`` in ``portions``.  Returns the new token of each decode row and of each row whose prompt ended."""
+        self._check_pages(decode_rows)
+        spans = [(r, self.row_len[r], 1) for r in decode_rows]
+        spans += sorted(((r, self.row_prompt[r].done, c) for r, c in portions), key=lambda s: s[2] != 1)
+        parts = [self.sampled[r : r + 1] for r in decode_rows]
+        parts += [self.row_prompt[r].ids[a : a + m] for r, a, m in spans[len(decode_rows):]]
+        step = self._ragged_step(spans, torch.cat(parts))
+        answer, places = list(decode_rows), list(range(len(decode_rows)))
+        for (r, a, m), end in zip(spans[len(decode_rows):], step.cu_seqlens[len(decode_rows) + 1 :]):
+            if a + m == self.row_prompt[r].total:
+                answer.append(r)
+                places.append(end - 1)
+        logits = self._forward_ragged(step, torch.tensor(places or [0], dtype=torch.int32).to(self.device))
+        self.seq_lens.index_copy_(0, torch.tensor([r for r, _, _ in spans]).to(self.device), step.seq_lens)
+        for r, a, m in spans:
+            self.row_len[r] = a + m
+        for r, a, m in spans[len(decode_rows):]:
+            p = self.row_prompt[r]
+            p.done = a + m
+            if p.done == p.total:
+                self._prompt_read(r, p.ids, p.start, p.keys, p.params, p.generated)
+                del self.row_prompt[r]
+        if not answer:
+            return {}
+        toks = self._sample_rows(logits, answer).tolist()
+        for r, t in zip(answer, toks):
+            if r in self.row_constraint:
+                self.row_constraint[r].advance(int(t))
+        return {r: int(t) for r, t in zip(answer, toks)}
 
     def save_session(self, row: int, session: str, tokens) -> None:
         """Keep row ``row``'s KV pages (and recurrent state) as the snapshot of conversation ``session``.  ``tokens``
@@ -407,6 +575,13 @@ class LLMEngine:
             c1 = min(end, c0 + self.prefill_chunk)
             m = c1 - c0
             chunk_ids = ids[c0:c1]
+            if self.model.ragged:
+                is_last = c1 == end
+                out = self._forward_ragged(self._ragged_step([(row, c0, m)], chunk_ids),
+                                           torch.tensor([m - 1 if is_last else 0], dtype=torch.int32, device=dev))
+                logits = out if is_last else logits
+                c0 = c1
+                continue
             positions = torch.arange(c0, c1, dtype=torch.int32, device=dev)
             slots = self.cache.slots(seq_id, c0, m).to(dev)
             cu = [0, m]
@@ -462,12 +637,15 @@ class LLMEngine:
             while c0 < n - 1:
                 c1 = min(n, c0 + self.prefill_chunk)
                 m = c1 - c0
-                step = StepBuffers(input_ids=ids[c0:c1], positions=torch.arange(c0, c1, dtype=torch.int32, device=dev),
-                                   slots=self.cache.slots(seq_id, c0, m).to(dev), cu_seqlens=[0, m], state_slots=state_slots,
-                                   past_len=c0, block_table=self.cache.block_table[row : row + 1] if c0 else None)
                 lo, hi = max(start - 1, c0), min(n - 1, c1)          # positions whose NEXT token is scored, in this chunk
                 want = torch.arange(lo - c0, hi - c0, dtype=torch.int32, device=dev) if hi > lo else torch.zeros(1, dtype=torch.int32, device=dev)
-                logits = self.model.forward(step, self.cache, prefill=True, logits_rows=want)
+                if self.model.ragged:
+                    logits = self._forward_ragged(self._ragged_step([(row, c0, m)], ids[c0:c1]), want)
+                else:
+                    step = StepBuffers(input_ids=ids[c0:c1], positions=torch.arange(c0, c1, dtype=torch.int32, device=dev),
+                                       slots=self.cache.slots(seq_id, c0, m).to(dev), cu_seqlens=[0, m], state_slots=state_slots,
+                                       past_len=c0, block_table=self.cache.block_table[row : row + 1] if c0 else None)
+                    logits = self.model.forward(step, self.cache, prefill=True, logits_rows=want)
                 if hi > lo:
                     logp = torch.log_softmax(logits.float(), -1)
                     out += logp.gather(1, ids[lo + 1 : hi + 1].long()[:, None])[:, 0].tolist()
@@ -525,6 +703,8 @@ class LLMEngine:
         """Attention KV splits for the current contexts (host mirror of the row lengths; a graph is kept per value)."""
         from ..ops.kernels import attn_splits_for
         longest = max(self.row_len.values(), default=self.max_seq_len)
+        if hasattr(self.model, "decode_splits"):
+            return self.model.decode_splits(b, min(self.max_seq_len, longest))
         hk = self.model.hk
         rows = max(1, getattr(self.model, "hq", hk) // hk) * q_len
         return attn_splits_for(b, hk, min(self.max_seq_len, longest), getattr(self.model.cfg, "head_dim", 128), rows)

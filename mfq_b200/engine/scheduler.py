@@ -13,7 +13,10 @@ Semantics follow the reference engine so that clients see the same behaviour:
   (``continuous_batch.h:103-125``);
 * prefill and decode alternate; a failure inside one request's prefill fails only that request; a failure of the
   batched decode marks the backend unhealthy and fails every request with ``backend_failure``
-  (``request_executor.h:127-133``).
+  (``request_executor.h:127-133``);
+* a backend that takes mixed batches (``mixed_batches``) is driven without the alternation: while prompts are being read,
+  every step is ONE forward with a token of each decoding row beside portions of the prompts, at most ``mixed_tokens`` prompt
+  tokens in all, so running requests never stall behind a long prompt; otherwise it is a plain batched decode.
 
 The scheduler drives a *backend* with four methods (``prefill``, ``decode``, ``release``, capacity queries), which the
 GPU engine and the test doubles implement; it owns no GPU state itself.
@@ -112,6 +115,9 @@ class Backend(Protocol):
     def decode(self, rows: list[int]) -> dict[int, int | list[int]]: ...  # a list: tokens confirmed by one MTP cycle
     def can_grow(self, row: int) -> bool: ...
     def release(self, row: int) -> None: ...
+    # optional, announced by a true ``mixed_batches``:
+    #   begin_prompt(row, tokens, params, **extra) -> tokens left to read     (admission; takes the prompt's pages)
+    #   mixed_step(decode_rows, [(row, count)]) -> {row: token} of decode rows and of rows whose prompt ended
 
 
 @dataclass
@@ -121,6 +127,7 @@ class SchedulerStats:
     failed: int = 0
     retractions: int = 0
     decode_steps: int = 0
+    mixed_steps: int = 0
     prefill_tokens: int = 0
     decode_tokens: int = 0
     queue_rejections: int = 0
@@ -128,8 +135,10 @@ class SchedulerStats:
 
 class ContinuousBatchScheduler:
     def __init__(self, backend: Backend, *, max_queue: int = 256, queue_timeout: float | None = None,
-                 clock: Callable[[], float] = time.monotonic) -> None:
+                 clock: Callable[[], float] = time.monotonic, mixed_tokens: int = 2048) -> None:
         self.backend = backend
+        self.mixed_tokens = mixed_tokens
+        self.reading: dict[int, int] = {}  # row -> prompt tokens left to read (mixed batches)
         self.max_queue, self.queue_timeout, self.clock = max_queue, queue_timeout, clock
         self.waiting: list[Request] = []
         self.running: dict[int, Request] = {}  # row -> request
@@ -204,6 +213,7 @@ class ContinuousBatchScheduler:
 
     def _release(self, row: int) -> None:
         self.running.pop(row, None)
+        self.reading.pop(row, None)
         self.backend.release(row)
 
     def _free_row(self) -> int | None:
@@ -269,7 +279,10 @@ class ContinuousBatchScheduler:
         return True
 
     # ---- one scheduling step ------------------------------------------------------------------------------------
-    def _try_prefill(self) -> bool:
+    def _try_prefill(self, start=None) -> bool:
+        """Admit the first waiting request, if it fits.  ``start(req, extra)`` begins it (default: run its whole prompt) and
+        returns its first token, or None when there is none yet.  Returns whether a request left the queue."""
+        start = start or (lambda req, extra: self.backend.prefill(req.row, req.context, req.params, **extra))
         for req in self.waiting:
             row = self._free_row()
             if row is None or not self.can_admit(req):
@@ -291,9 +304,10 @@ class ContinuousBatchScheduler:
                     extra["session"] = req.session
                 if req.generated and (req.params.response_format or req.params.logit_bias):  # replay after a retraction: the grammar has to
                     extra["generated"] = len(req.generated)       # re-read what was generated before
-                tok = self.backend.prefill(row, req.context, req.params, **extra)
+                tok = start(req, extra)
             except MemoryError:
                 self.running.pop(row, None)
+                self.reading.pop(row, None)
                 self.backend.release(row)
                 req.row = -1
                 self.waiting.insert(0, req)
@@ -304,15 +318,53 @@ class ContinuousBatchScheduler:
                 self._fail(req, exc)
                 return True
             self.stats.prefill_tokens += len(req.context)
-            if self._accept_token(req, tok):
-                self._snapshot(req)
-                self._release(row)
-                self._finish(req, req.finish_reason)
+            if tok is not None:
+                self._accept_tokens(req, [tok])
             return True
         return False
 
-    def _decode(self) -> None:
-        while self.running and not all(self.backend.can_grow(row) for row in self.running):
+    def _accept_tokens(self, req: Request, toks) -> int:
+        """Record tokens of one step (an MTP cycle confirms several; a stop token or the length cap ends early)."""
+        for n, tok in enumerate(toks, 1):
+            if self._accept_token(req, tok):
+                row = req.row
+                self._snapshot(req)
+                self._release(row)
+                self._finish(req, req.finish_reason)
+                return n
+        return len(toks)
+
+    def _decoding(self) -> list[int]:
+        return sorted(r for r in self.running if r not in self.reading)
+
+    def _begin_reading(self, req: Request, extra: dict) -> None:
+        self.reading[req.row] = self.backend.begin_prompt(req.row, req.context, req.params, **extra)
+
+    def _mixed(self) -> bool:
+        """A step of a backend that takes mixed batches."""
+        while self.waiting and self._try_prefill(self._begin_reading):
+            pass
+        if not self.running:
+            return False
+        if self.reading:
+            self._decode(mixed=True)
+        else:
+            self._decode()
+        return True
+
+    def _portions(self) -> list[tuple[int, int]]:
+        """Prompt portions of the next mixed step, oldest request first."""
+        left, out = self.mixed_tokens, []
+        for row in sorted(self.reading, key=lambda r: self.running[r].id):
+            count = min(left, self.reading[row])
+            if count <= 0:
+                break
+            out.append((row, count))
+            left -= count
+        return out
+
+    def _decode(self, mixed: bool = False) -> None:
+        while not all(self.backend.can_grow(row) for row in self._decoding()):
             if len(self.running) == 1:
                 row, req = next(iter(self.running.items()))
                 self._release(row)
@@ -321,9 +373,13 @@ class ContinuousBatchScheduler:
             self._retract_one()
         if not self.running:
             return
-        rows = sorted(self.running)
+        rows = self._decoding()
         try:
-            out = self.backend.decode(rows)
+            if mixed:
+                portions = self._portions()
+                out = self.backend.mixed_step(rows, portions)
+            else:
+                out = self.backend.decode(rows)
         except Exception as exc:
             self.healthy = False
             for row, req in list(self.running.items()):
@@ -336,24 +392,27 @@ class ContinuousBatchScheduler:
         self.stats.decode_steps += 1
         self.new_token_ratio = max(MIN_NEW_TOKEN_RATIO, self.new_token_ratio -
                                    (INITIAL_NEW_TOKEN_RATIO - MIN_NEW_TOKEN_RATIO) / RATIO_DECAY_STEPS)
+        if mixed:
+            self.stats.mixed_steps += 1
+            for row, count in portions:
+                self.reading[row] -= count
+                if self.reading[row] == 0:
+                    del self.reading[row]
+                    self._accept_tokens(self.running[row], [out[row]])
         for row in rows:
             req = self.running.get(row)
             if req is None:
                 continue
             produced = out[row] if isinstance(out[row], (list, tuple)) else [out[row]]
-            for tok in produced:  # an MTP cycle confirms several tokens; a stop token or the length cap ends early
-                self.stats.decode_tokens += 1
-                if self._accept_token(req, tok):
-                    self._snapshot(req)
-                    self._release(row)
-                    self._finish(req, req.finish_reason)
-                    break
+            self.stats.decode_tokens += self._accept_tokens(req, produced)
 
     def step(self) -> bool:
         """One scheduling step (a prefill or a batched decode).  Returns False when there was nothing to do."""
         if not self.healthy:
             return False
         self._expire()
+        if getattr(self.backend, "mixed_batches", False):
+            return self._mixed()
         did = False
         if self.waiting and (not self._decode_next or not self.running):
             did = self._try_prefill()

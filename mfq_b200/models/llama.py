@@ -239,10 +239,19 @@ class StepBuffers:
     # chunked prefill / restored prefix: tokens of the sequence that are already in the KV pages (the chunk attends to
     # them too); the chunk must then be a single sequence and `block_table` its page-id row ([1, max_pages])
     past_len: int = 0
+    # ragged batches (models with ``ragged = True``): one forward over portions of several sequences.  Sequence ``b`` owns
+    # rows ``q_starts[b] .. q_starts[b + 1] - 1``, has `seq_lens[b]` tokens after this step and the page ids of `block_table[b]`;
+    # the first `num_decode` sequences bring a single token each.
+    q_starts: torch.Tensor | None = None  # [B + 1] int32
+    tok_seq: torch.Tensor | None = None  # [T] int32: the sequence of every row
+    max_q: int = 1  # longest portion
+    num_decode: int = 0
 
 
 class LlamaModel:
     """Stateless forward over :class:`LlamaWeights`; KV state lives in a :class:`PagedKVCache`."""
+
+    ragged = False  # whether one forward may mix portions of several sequences (StepBuffers.q_starts)
 
     def __init__(self, cfg: LlamaConfig, weights: LlamaWeights, collective=None) -> None:
         self.cfg, self.w = cfg, weights

@@ -1,8 +1,12 @@
-"""Builds the in-tree CUDA library ``_mfq_b200_kernels.so`` for sm_100a with plain ``nvcc``.
+"""Builds the in-tree CUDA libraries for sm_100a with plain ``nvcc``.
 
 The kernels expose a C ABI (raw pointers + ``cudaStream_t``) and are loaded with ``ctypes``, so the
-library has no dependency on PyTorch headers, compiles in seconds and cross-compiles on a machine
-without a GPU.  ``python -m mfq_b200.ops.build`` rebuilds it; ``build(force=False)`` is incremental.
+libraries have no dependency on PyTorch headers, compile in seconds and cross-compile on a machine
+without a GPU.  ``python -m mfq_b200.ops.build`` rebuilds them; ``build(force=False)`` is incremental.
+
+* ``_mfq_b200_kernels.so`` -- the FP8 / packed / collective kernels and the engine's bookkeeping;
+* ``_mfq_b200_dense.so`` -- the unquantized path (:data:`DENSE_SOURCES`), on its own so that a model that only needs it
+  can be built in a few seconds (``build(only="dense")``).
 """
 
 from __future__ import annotations
@@ -18,6 +22,8 @@ from pathlib import Path
 HERE = Path(__file__).resolve().parent
 CSRC = HERE / "csrc"
 LIB_PATH = HERE / "_mfq_b200_kernels.so"
+DENSE_LIB_PATH = HERE / "_mfq_b200_dense.so"
+DENSE_SOURCES = ("dense_gemm.cu", "stream_ops.cu", "window_attn.cu", "window_attn_prefill.cu")
 OBJ_DIR = HERE / "build"
 
 NVCC_FLAGS = [
@@ -60,25 +66,38 @@ def _compile_one(src: Path, force: bool) -> tuple[Path, str]:
     return obj, proc.stderr
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
-    """Compile every ``csrc/*.cu`` and link the shared library.  Returns its path."""
+def libraries() -> dict[str, tuple[Path, list[Path]]]:
+    """Library name -> (path, its sources)."""
+    dense = [p for p in sources() if p.name in DENSE_SOURCES]
+    return {"kernels": (LIB_PATH, [p for p in sources() if p not in dense]), "dense": (DENSE_LIB_PATH, dense)}
+
+
+def _link(path: Path, objs: list[Path]) -> None:
+    part = path.with_suffix(f".{os.getpid()}.part")  # a process that loads the library never sees half of it
+    proc = subprocess.run([nvcc_path(), "--shared", "-o", str(part), *map(str, objs)], capture_output=True, text=True)
+    if proc.returncode != 0:
+        raise RuntimeError(f"link failed:\n{proc.stderr}")
+    os.replace(part, path)
+
+
+def build(force: bool = False, verbose: bool = False, only: str | None = None) -> Path:
+    """Compile ``csrc/*.cu`` and link the shared libraries (``only``: just the one of that name).  Returns the path of the
+    library asked for, by default the main one."""
     OBJ_DIR.mkdir(exist_ok=True)
-    srcs = sources()
+    libs = libraries()
+    chosen = libs if only is None else {only: libs[only]}
+    srcs = [s for _, group in chosen.values() for s in group]
     with ThreadPoolExecutor(max_workers=min(8, len(srcs))) as pool:
-        results = list(pool.map(lambda s: _compile_one(s, force), srcs))
-    objs = [str(o) for o, _ in results]
-    log = "".join(text for _, text in results)
+        results = dict(zip(srcs, pool.map(lambda s: _compile_one(s, force), srcs)))
+    log = "".join(text for _, text in results.values())
     if log:
         (OBJ_DIR / "ptxas.log").write_text(log)
-    rebuilt = any(text for _, text in results)
-    if rebuilt or not LIB_PATH.exists():
-        cmd = [nvcc_path(), "--shared", "-o", str(LIB_PATH), *objs]
-        proc = subprocess.run(cmd, capture_output=True, text=True)
-        if proc.returncode != 0:
-            raise RuntimeError(f"link failed:\n{proc.stderr}")
+    for path, group in chosen.values():
+        if any(results[s][1] for s in group) or not path.exists():
+            _link(path, [results[s][0] for s in group])
     if verbose and log:
         print(log, file=sys.stderr)
-    return LIB_PATH
+    return libs[only or "kernels"][0]
 
 
 if __name__ == "__main__":

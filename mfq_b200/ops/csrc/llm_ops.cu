@@ -441,16 +441,20 @@ __global__ void rope_kv_write_kernel(const __nv_bfloat16* __restrict__ qkv, cons
 // ---------------------------------------------------------------------------------------------
 // Greedy sampling: arg-max over the vocabulary, one CTA per row (lowest index wins ties).
 // ---------------------------------------------------------------------------------------------
-__global__ void argmax_kernel(const __nv_bfloat16* __restrict__ logits, int* __restrict__ out, int V, int stride) {
+__device__ __forceinline__ float logit_value(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float logit_value(float v) { return v; }
+
+template <typename T>
+__global__ void argmax_kernel(const T* __restrict__ logits, int* __restrict__ out, int V, int stride) {
   pdl_trigger();
   pdl_wait();
   __shared__ float sv[32];
   __shared__ int si[32];
-  const __nv_bfloat16* row = logits + size_t(blockIdx.x) * stride;
+  const T* row = logits + size_t(blockIdx.x) * stride;
   float best = -FLT_MAX;
   int bi = 0x7fffffff;
   for (int i = threadIdx.x; i < V; i += blockDim.x) {
-    const float v = __bfloat162float(row[i]);
+    const float v = logit_value(row[i]);
     if (v > best) { best = v; bi = i; }
   }
 #pragma unroll
@@ -485,17 +489,18 @@ constexpr int kArgmaxRows = 8192;
 __device__ unsigned long long g_argmax_key[kArgmaxRows];
 __device__ unsigned int g_argmax_count[kArgmaxRows];
 
-__global__ void argmax_split_kernel(const __nv_bfloat16* __restrict__ logits, int* __restrict__ out, int V, int stride) {
+template <typename T>
+__global__ void argmax_split_kernel(const T* __restrict__ logits, int* __restrict__ out, int V, int stride) {
   pdl_trigger();
   pdl_wait();
   __shared__ unsigned long long sk[8];
   const int b = blockIdx.x, seg = blockIdx.y, nseg = gridDim.y;
   const int per = (V + nseg - 1) / nseg;
   const int lo = seg * per, hi = min(V, lo + per);
-  const __nv_bfloat16* row = logits + size_t(b) * stride;
+  const T* row = logits + size_t(b) * stride;
   unsigned long long key = 0ull;
   for (int i = lo + threadIdx.x; i < hi; i += blockDim.x) {
-    const uint32_t u = __float_as_uint(__bfloat162float(row[i]));
+    const uint32_t u = __float_as_uint(logit_value(row[i]));
     const uint32_t ord = (u & 0x80000000u) ? ~u : (u | 0x80000000u);
     const unsigned long long k = (static_cast<unsigned long long>(ord) << 32) | (0xffffffffu - uint32_t(i));
     key = k > key ? k : key;
@@ -641,13 +646,23 @@ extern "C" int mfq_rope_kv_write(const void* qkv, const int* positions, const in
                               theta, kd_out, vd_out, nullptr, nullptr, 0.f, (Hq + 2 * Hk) * D, stream);
 }
 
-extern "C" int mfq_argmax(const void* logits, int* out, int B, int V, int stride, cudaStream_t stream) {
+template <typename T>
+static int launch_argmax(const void* logits, int* out, int B, int V, int stride, cudaStream_t stream) {
   const int segs = V / 4096 > 32 ? 32 : V / 4096;
   if (segs >= 2 && B <= kArgmaxRows && B * segs <= 4096)
-    launch_kernel(argmax_split_kernel, dim3(B, segs), dim3(256), 0, stream, static_cast<const __nv_bfloat16*>(logits), out, V, stride);
+    launch_kernel(argmax_split_kernel<T>, dim3(B, segs), dim3(256), 0, stream, static_cast<const T*>(logits), out, V, stride);
   else
-    launch_kernel(argmax_kernel, dim3(B), dim3(1024), 0, stream, static_cast<const __nv_bfloat16*>(logits), out, V, stride);
+    launch_kernel(argmax_kernel<T>, dim3(B), dim3(1024), 0, stream, static_cast<const T*>(logits), out, V, stride);
   return cudaGetLastError() == cudaSuccess ? 0 : -7;
+}
+
+extern "C" int mfq_argmax(const void* logits, int* out, int B, int V, int stride, cudaStream_t stream) {
+  return launch_argmax<__nv_bfloat16>(logits, out, B, V, stride, stream);
+}
+
+// fp32 logits (models that run in full precision)
+extern "C" int mfq_argmax_f32(const void* logits, int* out, int B, int V, int stride, cudaStream_t stream) {
+  return launch_argmax<float>(logits, out, B, V, stride, stream);
 }
 
 extern "C" int mfq_embed(const int* ids, const void* table, void* out, int T, int H, cudaStream_t stream) {

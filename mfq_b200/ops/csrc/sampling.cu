@@ -47,7 +47,7 @@ __device__ __forceinline__ float uniform01(unsigned long long seed, unsigned lon
   return float(z >> 40) * (1.f / 16777216.f);
 }
 
-// logits [B, V] bf16 (row stride `stride`); counts [B, V] uint16 occurrences of each token in the row's sequence
+// logits [B, V] bf16 or fp32 (row stride `stride`); counts [B, V] uint16 occurrences of each token in the row's sequence
 // (may be null); work [B, V] fp32 scratch; out [B] sampled ids; steps [B] per-row draw counter (read only).
 //
 // Speculative verification (`window` > 1, `draft` given): the B rows are `window` consecutive positions of B / window
@@ -57,8 +57,12 @@ __device__ __forceinline__ float uniform01(unsigned long long seed, unsigned lon
 // distribution and otherwise draws from p with x removed -- the emitted token is then distributed exactly as p.  The
 // last position has no draft and is a plain draw.  Greedy rows return the arg-max either way, so comparing `out` with
 // the draft (what the accept kernel does) is the verification in both modes.
+__device__ __forceinline__ float sample_value(__nv_bfloat16 v) { return __bfloat162float(v); }
+__device__ __forceinline__ float sample_value(float v) { return v; }
+
+template <typename T>
 __global__ void __launch_bounds__(1024)
-sample_kernel(const __nv_bfloat16* __restrict__ logits, int V, int stride, const unsigned short* __restrict__ counts,
+sample_kernel(const T* __restrict__ logits, int V, int stride, const unsigned short* __restrict__ counts,
               const SampleRow* __restrict__ rows, const int* __restrict__ steps, float* __restrict__ work,
               int* __restrict__ out, int window, const int* __restrict__ draft) {
   __shared__ float red[32];
@@ -67,7 +71,7 @@ sample_kernel(const __nv_bfloat16* __restrict__ logits, int V, int stride, const
   const int seq = b / window, pos = b - seq * window;
   const SampleRow r = rows[seq];
   const int x = (draft && pos < window - 1) ? draft[seq * (window - 1) + pos] : -1;
-  const __nv_bfloat16* lr = logits + size_t(b) * stride;
+  const T* lr = logits + size_t(b) * stride;
   float* w = work + size_t(b) * V;
   const unsigned short* cr = counts ? counts + size_t(b) * V : nullptr;
   const bool greedy = r.temperature <= 0.f;
@@ -75,7 +79,7 @@ sample_kernel(const __nv_bfloat16* __restrict__ logits, int V, int stride, const
   float mx = -FLT_MAX;
   int mi = 0x7fffffff;
   for (int i = tid; i < V; i += blockDim.x) {
-    float l = __bfloat162float(lr[i]);
+    float l = sample_value(lr[i]);
     if (cr) {
       const int c = cr[i];
       if (c > 0) {
@@ -185,13 +189,21 @@ sample_kernel(const __nv_bfloat16* __restrict__ logits, int V, int stride, const
 }  // namespace mfq
 
 // rows: device array of B records {temperature, top_k, top_p, presence, frequency, repetition, seed} (see SampleRow).
+template <typename T>
+static int launch_sample(const void* logits, int B, int V, int stride, const void* counts, const void* rows, const int* steps,
+                         float* work, int* out, cudaStream_t stream) {
+  if (B <= 0 || V <= 0) return -1;
+  mfq::sample_kernel<T><<<B, 1024, 0, stream>>>(static_cast<const T*>(logits), V, stride, static_cast<const unsigned short*>(counts),
+                                                static_cast<const mfq::SampleRow*>(rows), steps, work, out, 1, nullptr);
+  return cudaGetLastError() == cudaSuccess ? 0 : -7;
+}
 extern "C" int mfq_sample(const void* logits, int B, int V, int stride, const void* counts, const void* rows,
                           const int* steps, float* work, int* out, cudaStream_t stream) {
-  if (B <= 0 || V <= 0) return -1;
-  mfq::sample_kernel<<<B, 1024, 0, stream>>>(static_cast<const __nv_bfloat16*>(logits), V, stride,
-                                             static_cast<const unsigned short*>(counts),
-                                             static_cast<const mfq::SampleRow*>(rows), steps, work, out, 1, nullptr);
-  return cudaGetLastError() == cudaSuccess ? 0 : -7;
+  return launch_sample<__nv_bfloat16>(logits, B, V, stride, counts, rows, steps, work, out, stream);
+}
+extern "C" int mfq_sample_f32(const void* logits, int B, int V, int stride, const void* counts, const void* rows,
+                              const int* steps, float* work, int* out, cudaStream_t stream) {
+  return launch_sample<float>(logits, B, V, stride, counts, rows, steps, work, out, stream);
 }
 
 // Verification draw for speculative decoding: logits [B * window, V] (window consecutive positions per sequence), rows /
@@ -200,7 +212,7 @@ extern "C" int mfq_sample(const void* logits, int B, int V, int stride, const vo
 extern "C" int mfq_sample_verify(const void* logits, int B, int window, int V, int stride, const void* rows, const int* steps,
                                  const int* draft, float* work, int* out, cudaStream_t stream) {
   if (B <= 0 || V <= 0 || window < 1) return -1;
-  mfq::sample_kernel<<<B * window, 1024, 0, stream>>>(static_cast<const __nv_bfloat16*>(logits), V, stride, nullptr,
+  mfq::sample_kernel<__nv_bfloat16><<<B * window, 1024, 0, stream>>>(static_cast<const __nv_bfloat16*>(logits), V, stride, nullptr,
                                                       static_cast<const mfq::SampleRow*>(rows), steps, work, out, window,
                                                       window > 1 ? draft : nullptr);
   return cudaGetLastError() == cudaSuccess ? 0 : -7;

@@ -1,0 +1,402 @@
+// Sliding-window attention over unquantized pages (K [page][Hk][16][dk], V [page][Hk][16][dv]), one query token per sequence
+// or, in the plain kernel, any number of them.  A query at position i sees the keys j with 0 <= i - j < window.
+//
+//   window_attn_decode_kernel   bf16, one query per sequence.  A CTA serves one (sequence, KV head, KV split); its four warps
+//                               take alternate pages that hold visible keys through private cp.async rings.  The (up to 16)
+//                               query heads of the KV head are the rows of m16n8k16 MMAs: S = Q K^T, probabilities go from
+//                               accumulators straight into the A operand of P V.  Warps (and splits) merge at the end.
+//   window_attn_plain_kernel    a warp per (token, query head), fp32 arithmetic, fp32 or bf16 storage: the full-precision mode.
+#include "window_attn.cuh"
+
+#include <cfloat>
+
+namespace mfq {
+
+constexpr int kWinPage = 16, kWinWarps = 4;
+
+struct WindowDecodeParams {
+  const __nv_bfloat16* q;  // [B, Hq, dk]
+  const __nv_bfloat16* k;
+  const __nv_bfloat16* v;
+  const int* table;     // [B, max_pages]
+  const int* seq_lens;  // length including the query token
+  __nv_bfloat16* out;   // [B, Hq, dv]
+  float* part;          // splits > 1: [B * Hq][splits][dv]
+  float* part_ml;       // [B * Hq][splits][2]
+  int Hq, Hk, dk, dv, max_pages, window, splits, head_tiles;
+  ScoreCap cap;
+};
+
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void win_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
+  __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<uint32_t*>(&h);
+}
+
+// DK / DV: upper bounds of the stored head widths (register arrays); the widths themselves are run-time multiples of 16.
+template <int DK, int DV>
+struct WinCfg {
+  static constexpr int kStages = DK + DV <= 256 ? 3 : 2;
+  static int stage_bytes(int dk, int dv) { return kWinPage * (dk + 8 + dv + 8) * 2; }
+  static int smem_bytes(int dk, int dv) {
+    const int ring = kWinWarps * kStages * stage_bytes(dk, dv), merge = kWinWarps * 16 * (dv + 2) * 4;
+    return ring > merge ? ring : merge;
+  }
+};
+
+template <int DK, int DV>
+__global__ void __launch_bounds__(kWinWarps * 32)
+window_attn_decode_kernel(const WindowDecodeParams p) {
+  pdl_trigger();
+  pdl_wait();
+  extern __shared__ __align__(16) uint8_t win_smem[];
+  constexpr int kStages = WinCfg<DK, DV>::kStages;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int ht = blockIdx.x % p.head_tiles, bg = blockIdx.x / p.head_tiles;
+  const int b = bg / p.Hk, g = bg - b * p.Hk, split = blockIdx.y;
+  const int per = p.Hq / p.Hk, heads = min(16, per - ht * 16);
+  const int head0 = g * per + ht * 16;
+  const int dk = p.dk, dv = p.dv;
+  const int pos = p.seq_lens[b] - 1;
+  const int lo = max(0, pos - p.window + 1);
+  int page0 = lo / kWinPage, page1 = pos >= 0 ? pos / kWinPage + 1 : 0;
+  if (pos < 0) page0 = 0;
+  {
+    const int chunk = (page1 - page0 + p.splits - 1) / p.splits;
+    page0 = page0 + split * chunk;
+    page1 = min(page1, page0 + chunk);
+  }
+  const int kpitch = dk + 8, vpitch = dv + 8;  // odd multiples of 16 bytes apart modulo 128: ldmatrix without conflicts
+  const int stage_bytes = kWinPage * (kpitch + vpitch) * 2;
+  const uint32_t ring = smem_u32(win_smem) + warp * kStages * stage_bytes;
+  const int n = max(0, (page1 - page0 - warp + kWinWarps - 1) / kWinWarps);  // my pages: page0 + warp + 4 i
+  const int* table = p.table + size_t(b) * p.max_pages;
+  const int kch = dk >> 3, vch = dv >> 3;
+  const uint32_t kinv = (65536u + kch - 1) / kch, vinv = (65536u + vch - 1) / vch;  // row = i / chunks for i < 512
+  int ids = 0;  // lane j holds the id of my page (32 block + j)
+  auto fetch = [&](int i) {
+    if ((i & 31) == 0) {
+      const int pg = page0 + warp + kWinWarps * (i + lane);
+      ids = pg < page1 ? table[pg] : 0;
+    }
+    const int page = __shfl_sync(0xffffffffu, ids, i & 31);
+    const uint32_t st = ring + (i % kStages) * stage_bytes;
+    const __nv_bfloat16* ks = p.k + (size_t(page) * p.Hk + g) * (kWinPage * dk);
+    const __nv_bfloat16* vs = p.v + (size_t(page) * p.Hk + g) * (kWinPage * dv);
+    for (int c = lane; c < kWinPage * kch; c += 32) {
+      const int row = (c * kinv) >> 16;
+      cp_async16(st + (row * kpitch + (c - row * kch) * 8) * 2, ks + c * 8);
+    }
+    const uint32_t sv = st + kWinPage * kpitch * 2;
+    for (int c = lane; c < kWinPage * vch; c += 32) {
+      const int row = (c * vinv) >> 16;
+      cp_async16(sv + (row * vpitch + (c - row * vch) * 8) * 2, vs + c * 8);
+    }
+  };
+#pragma unroll
+  for (int i = 0; i < kStages - 1; ++i) {
+    if (i < n) fetch(i);
+    cp_async_commit();
+  }
+  // query fragments: rows r0 = lane / 4 and r0 + 8 of the head tile
+  const int r0 = lane >> 2, t4 = lane & 3;
+  uint32_t qf[DK / 16][4];
+  {
+    const __nv_bfloat16* q0 = p.q + (size_t(b) * p.Hq + head0 + r0) * dk + t4 * 2;
+    const __nv_bfloat16* q1 = q0 + size_t(8) * dk;
+#pragma unroll
+    for (int ks = 0; ks < DK / 16; ++ks) {
+      const bool in = ks * 16 < dk;
+      qf[ks][0] = in && r0 < heads ? *reinterpret_cast<const uint32_t*>(q0 + ks * 16) : 0u;
+      qf[ks][1] = in && r0 + 8 < heads ? *reinterpret_cast<const uint32_t*>(q1 + ks * 16) : 0u;
+      qf[ks][2] = in && r0 < heads ? *reinterpret_cast<const uint32_t*>(q0 + ks * 16 + 8) : 0u;
+      qf[ks][3] = in && r0 + 8 < heads ? *reinterpret_cast<const uint32_t*>(q1 + ks * 16 + 8) : 0u;
+    }
+  }
+  float o[DV / 8][4];
+#pragma unroll
+  for (int i = 0; i < DV / 8; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) o[i][j] = 0.f;
+  float m[2] = {-FLT_MAX, -FLT_MAX}, l[2] = {0.f, 0.f};
+  const int mat = lane >> 3, mrow = lane & 7;
+  const uint32_t k_off = (((mat >> 1) * 8 + mrow) * kpitch + (mat & 1) * 8) * 2;
+  const uint32_t v_off = (((mat & 1) * 8 + mrow) * vpitch + (mat >> 1) * 8) * 2;
+  for (int i = 0; i < n; ++i) {
+    if (i + kStages - 1 < n) fetch(i + kStages - 1);
+    cp_async_commit();
+    cp_async_wait<kStages - 1>();
+    __syncwarp();
+    const uint32_t st = ring + (i % kStages) * stage_bytes, sv = st + kWinPage * kpitch * 2;
+    float s[2][4] = {};
+#pragma unroll
+    for (int ks = 0; ks < DK / 16; ++ks) {
+      if (ks * 16 < dk) {
+        uint32_t kf[4];
+        ldmatrix_x4(st + k_off + ks * 32, kf);
+        win_mma(s[0], qf[ks], kf[0], kf[1]);
+        win_mma(s[1], qf[ks], kf[2], kf[3]);
+      }
+    }
+    const int key0 = (page0 + warp + kWinWarps * i) * kWinPage + t4 * 2;
+    float mx[2] = {-FLT_MAX, -FLT_MAX};
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int key = key0 + nt * 8 + (e & 1);
+        s[nt][e] = key >= lo && key <= pos ? score_any(p.cap, s[nt][e]) : -FLT_MAX;
+        mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
+      }
+    float alpha[2];
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+      const float mn = fmaxf(m[r], mx[r]);  // every page holds a visible key, so mn is a real score
+      alpha[r] = window_exp2(m[r] - mn);
+      m[r] = mn;
+      l[r] *= alpha[r];
+    }
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        s[nt][e] = window_exp2(s[nt][e] - m[e >> 1]);  // hidden keys: exp2 of a huge negative number
+        l[e >> 1] += s[nt][e];
+      }
+    if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
+#pragma unroll
+      for (int d = 0; d < DV / 8; ++d) {
+        o[d][0] *= alpha[0]; o[d][1] *= alpha[0]; o[d][2] *= alpha[1]; o[d][3] *= alpha[1];
+      }
+    }
+    const uint32_t pf[4] = {pack_bf16(s[0][0], s[0][1]), pack_bf16(s[0][2], s[0][3]), pack_bf16(s[1][0], s[1][1]), pack_bf16(s[1][2], s[1][3])};
+#pragma unroll
+    for (int d = 0; d < DV / 16; ++d) {
+      if (d * 16 < dv) {
+        uint32_t vf[4];
+        ldmatrix_x4_trans(sv + v_off + d * 32, vf);
+        win_mma(o[2 * d], pf, vf[0], vf[1]);
+        win_mma(o[2 * d + 1], pf, vf[2], vf[3]);
+      }
+    }
+    __syncwarp();  // the stage is refilled by the next round's fetch
+  }
+  // ----- merge the four warps (then the splits, in a second kernel) -----
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
+    l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+  }
+  cp_async_wait<0>();
+  __syncthreads();
+  float* acc = reinterpret_cast<float*>(win_smem);              // [warp][16][dv]
+  float* ml = acc + kWinWarps * 16 * dv;                        // [warp][16][2]
+  {
+    float* a0 = acc + (warp * 16 + r0) * dv + t4 * 2;
+    float* a1 = a0 + 8 * dv;
+#pragma unroll
+    for (int d = 0; d < DV / 8; ++d) {
+      if (d * 8 < dv) {
+        *reinterpret_cast<float2*>(a0 + d * 8) = make_float2(o[d][0], o[d][1]);
+        *reinterpret_cast<float2*>(a1 + d * 8) = make_float2(o[d][2], o[d][3]);
+      }
+    }
+    if (t4 == 0) {
+      ml[(warp * 16 + r0) * 2] = m[0]; ml[(warp * 16 + r0) * 2 + 1] = l[0];
+      ml[(warp * 16 + r0 + 8) * 2] = m[1]; ml[(warp * 16 + r0 + 8) * 2 + 1] = l[1];
+    }
+  }
+  __syncthreads();
+  for (int r = warp; r < heads; r += kWinWarps) {
+    float mw[kWinWarps], mt = -FLT_MAX, lt = 0.f;
+#pragma unroll
+    for (int w = 0; w < kWinWarps; ++w) { mw[w] = ml[(w * 16 + r) * 2]; mt = fmaxf(mt, mw[w]); }
+#pragma unroll
+    for (int w = 0; w < kWinWarps; ++w) {
+      mw[w] = window_exp2(mw[w] - mt);  // a warp without pages: l = 0, o = 0
+      lt += ml[(w * 16 + r) * 2 + 1] * mw[w];
+    }
+    const size_t orow = size_t(b) * p.Hq + head0 + r;
+    const float inv = p.splits == 1 ? (lt > 0.f ? 1.f / lt : 0.f) : 1.f;
+    for (int c = lane; c < dv; c += 32) {
+      float x = 0.f;
+#pragma unroll
+      for (int w = 0; w < kWinWarps; ++w) x += acc[(w * 16 + r) * dv + c] * mw[w];
+      x *= inv;
+      if (p.splits == 1) p.out[orow * dv + c] = __float2bfloat16(x);
+      else p.part[(orow * p.splits + split) * dv + c] = x;
+    }
+    if (p.splits > 1 && lane == 0) {
+      p.part_ml[(orow * p.splits + split) * 2] = mt;
+      p.part_ml[(orow * p.splits + split) * 2 + 1] = lt;
+    }
+  }
+}
+
+__global__ void window_attn_merge_kernel(const float* __restrict__ part, const float* __restrict__ part_ml,
+                                         __nv_bfloat16* __restrict__ out, int splits, int dv) {
+  pdl_trigger();
+  pdl_wait();
+  const size_t row = blockIdx.x;
+  float mt = -FLT_MAX, lt = 0.f;
+  for (int z = 0; z < splits; ++z) mt = fmaxf(mt, part_ml[(row * splits + z) * 2]);
+  for (int z = 0; z < splits; ++z) lt += part_ml[(row * splits + z) * 2 + 1] * window_exp2(part_ml[(row * splits + z) * 2] - mt);
+  const float inv = lt > 0.f ? 1.f / lt : 0.f;
+  for (int c = threadIdx.x; c < dv; c += blockDim.x) {
+    float x = 0.f;
+    for (int z = 0; z < splits; ++z) x += part[(row * splits + z) * dv + c] * window_exp2(part_ml[(row * splits + z) * 2] - mt);
+    out[row * dv + c] = __float2bfloat16(x * inv);
+  }
+}
+
+template <int DK, int DV>
+static int launch_window_decode(const WindowDecodeParams& p, int B, cudaStream_t stream) {
+  const int smem = WinCfg<DK, DV>::smem_bytes(p.dk, p.dv);
+  static int allowed = 0;
+  if (smem > allowed) {
+    if (cudaFuncSetAttribute(window_attn_decode_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -6;
+    allowed = smem;
+  }
+  launch_kernel(window_attn_decode_kernel<DK, DV>, dim3(B * p.Hk * p.head_tiles, p.splits), dim3(kWinWarps * 32), smem, stream, p);
+  if (p.splits > 1)
+    launch_kernel(window_attn_merge_kernel, dim3(B * p.Hq), dim3(p.dv <= 64 ? 64 : 128), 0, stream, p.part, p.part_ml, p.out, p.splits, p.dv);
+  return cudaGetLastError() == cudaSuccess ? 0 : -7;
+}
+
+// ---------------------------------------------------------------------------------------------
+// A warp per (token, query head).
+// ---------------------------------------------------------------------------------------------
+struct WindowPlainParams {
+  const int* positions;  // [T]
+  const int* tok_seq;    // [T] row of the block table
+  const int* table;
+  int T, Hq, Hk, dk, dv, max_pages, window;
+  float scale, cap;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(128)
+window_attn_plain_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, T* __restrict__ out, const WindowPlainParams p) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ __align__(16) float sq[4][256];
+  __shared__ float sp[4][32];
+  __shared__ int spage[4][32];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int gw = blockIdx.x * 4 + warp;
+  if (gw >= p.T * p.Hq) return;
+  const int t = gw / p.Hq, h = gw - t * p.Hq, g = h / (p.Hq / p.Hk);
+  const int pos = p.positions[t], lo = max(0, pos - p.window + 1);
+  const int* table = p.table + size_t(p.tok_seq[t]) * p.max_pages;
+  if (lane * 8 < p.dk) {
+    float x[8];
+    load8<T>(q + (size_t(t) * p.Hq + h) * p.dk + lane * 8, x);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) sq[warp][lane * 8 + j] = x[j];
+  }
+  __syncwarp();
+  float m = -FLT_MAX, l = 0.f, acc[8] = {};
+  for (int j0 = lo; j0 <= pos; j0 += 32) {
+    const int key = j0 + lane;
+    float s = -FLT_MAX;
+    int page = 0;
+    if (key <= pos) {
+      page = table[key / kWinPage];
+      const T* kr = k + ((size_t(page) * p.Hk + g) * kWinPage + key % kWinPage) * p.dk;
+      float dot = 0.f;
+      for (int c = 0; c < p.dk; c += 8) {
+        float x[8];
+        load8<T>(kr + c, x);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) dot = fmaf(sq[warp][c + j], x[j], dot);
+      }
+      s = dot * p.scale;
+      if (p.cap > 0.f) s = p.cap * tanhf(s / p.cap);
+    }
+    float mx = s;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    const float mn = fmaxf(m, mx), alpha = expf(m - mn);
+    m = mn;
+    const float pr = key <= pos ? expf(s - mn) : 0.f;
+    float sum = pr;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    l = l * alpha + sum;
+    sp[warp][lane] = pr;
+    spage[warp][lane] = page;
+    __syncwarp();
+    if (lane * 8 < p.dv) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) acc[j] *= alpha;
+      const int cnt = min(32, pos - j0 + 1);
+      for (int i = 0; i < cnt; ++i) {
+        float x[8];
+        load8<T>(v + ((size_t(spage[warp][i]) * p.Hk + g) * kWinPage + (j0 + i) % kWinPage) * p.dv + lane * 8, x);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[j] = fmaf(sp[warp][i], x[j], acc[j]);
+      }
+    }
+    __syncwarp();
+  }
+  if (lane * 8 < p.dv) {
+    const float inv = l > 0.f ? 1.f / l : 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) acc[j] *= inv;
+    store8<T>(out + (size_t(t) * p.Hq + h) * p.dv + lane * 8, acc);
+  }
+}
+
+}  // namespace mfq
+
+using namespace mfq;
+
+// One query token per sequence, bf16.  part / part_ml: scratch of B * Hq * splits * dv and * 2 floats (splits > 1).
+extern "C" int mfq_window_attn_decode(const void* q, const void* k, const void* v, const int* table, const int* seq_lens, void* out,
+                                      float* part, float* part_ml, int B, int Hq, int Hk, int dk, int dv, int max_pages, int window,
+                                      float scale, float cap, int splits, cudaStream_t stream) {
+  if (B <= 0 || Hq <= 0 || Hk <= 0 || Hq % Hk || dk % 16 || dv % 16 || dk <= 0 || dv <= 0 || dk > 256 || dv > 256) return -1;
+  if (window <= 0 || !(scale > 0.f) || splits < 1 || (splits > 1 && (!part || !part_ml))) return -1;
+  const WindowDecodeParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k), static_cast<const __nv_bfloat16*>(v),
+                             table, seq_lens, static_cast<__nv_bfloat16*>(out), part, part_ml, Hq, Hk, dk, dv, max_pages, window, splits,
+                             (Hq / Hk + 15) / 16, make_score_cap(scale, cap)};
+#define MFQ_WIN_DV(DK)                                                 \
+  (dv <= 64 ? launch_window_decode<DK, 64>(p, B, stream)               \
+            : dv <= 128 ? launch_window_decode<DK, 128>(p, B, stream) : launch_window_decode<DK, 256>(p, B, stream))
+  return dk <= 64 ? MFQ_WIN_DV(64) : dk <= 128 ? MFQ_WIN_DV(128) : MFQ_WIN_DV(256);
+#undef MFQ_WIN_DV
+}
+
+// Any number of query tokens: token t sits at positions[t] of the sequence in row tok_seq[t] of the block table.
+extern "C" int mfq_window_attn_plain(const void* q, const void* k, const void* v, const int* table, const int* tok_seq,
+                                     const int* positions, void* out, int T_, int Hq, int Hk, int dk, int dv, int max_pages, int window,
+                                     float scale, float cap, int fp32, cudaStream_t stream) {
+  if (T_ <= 0 || Hq <= 0 || Hk <= 0 || Hq % Hk || dk % 8 || dv % 8 || dk > 256 || dv > 256 || window <= 0) return -1;
+  const WindowPlainParams p{positions, tok_seq, table, T_, Hq, Hk, dk, dv, max_pages, window, scale, cap};
+  const dim3 grid(unsigned(((long long)(T_) * Hq + 3) / 4));
+  if (fp32)
+    launch_kernel(window_attn_plain_kernel<float>, grid, dim3(128), 0, stream, static_cast<const float*>(q), static_cast<const float*>(k),
+                  static_cast<const float*>(v), static_cast<float*>(out), p);
+  else
+    launch_kernel(window_attn_plain_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, static_cast<const __nv_bfloat16*>(q),
+                  static_cast<const __nv_bfloat16*>(k), static_cast<const __nv_bfloat16*>(v), static_cast<__nv_bfloat16*>(out), p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -7;
+}

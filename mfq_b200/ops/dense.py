@@ -1,0 +1,120 @@
+"""Unquantized linears and the fp32 residual stream (``csrc/dense_gemm.cu``, ``csrc/stream_ops.cu``).
+
+Activations and weights are bf16, or fp32 throughout; the element type of the weight decides.  Stored widths are rounded up
+(:func:`up`) and the padding is zero, so the kernels need no tails; callers keep the true widths where they matter (norms).
+"""
+
+from __future__ import annotations
+
+import math
+from dataclasses import dataclass
+
+import torch
+
+from .lib import Workspace, check, dense_lib, ptr, stream_ptr
+
+BIAS, GLU, GELU = 0, 1, 2  # epilogues (dense_common.cuh)
+GEMV_ROWS, GEMV_MID_ROWS, GEMV_MID_WEIGHTS = 8, 16, 20 << 20
+
+
+def up(n: int, m: int = 16) -> int:
+    """``n`` rounded up to a multiple of ``m``."""
+    return (n + m - 1) // m * m
+
+
+def is_fp32(dtype: torch.dtype) -> int:
+    if dtype not in (torch.float32, torch.bfloat16):
+        raise TypeError(f"the dense path runs in bfloat16 or float32, not {dtype}")
+    return int(dtype == torch.float32)
+
+
+def plan(m: int, n: int, k: int, sms: int = 148) -> tuple[int, int]:
+    """``(token tile, K splits)`` of a bf16 product ``[m, k] x [n, k]^T``; tile 0 is the weight-streaming kernel.  The split
+    count minimises waves x (K blocks per CTA + ramp) over the clusters of up to 8 CTAs that meet in shared memory."""
+    if m <= GEMV_ROWS or (m <= GEMV_MID_ROWS and n * k <= GEMV_MID_WEIGHTS):
+        return 0, 1
+    rows = math.ceil(n / 128)
+    tile = next((t for t in (16, 32, 64, 128) if m <= t), 0)
+    if not tile:
+        tile = 256 if rows * math.ceil(m / 256) >= 100 else 128
+    tiles, kb = rows * math.ceil(m / tile), math.ceil(k / 64)
+    slots = sms * (2 if tile <= 64 else 1)
+    best, best_cost = 1, None
+    for s in range(1, min(kb, 8) + 1):
+        per = math.ceil(kb / s)
+        if s > 1 and per < 4:
+            break
+        ctas = tiles * math.ceil(kb / per)
+        cost = math.ceil(ctas / slots) * (per + 6) + (3 if s > 1 else 0)
+        if best_cost is None or cost < best_cost:
+            best, best_cost = s, cost
+    return tile, best
+
+
+@dataclass
+class DenseLinear:
+    """``[rows, cols]`` weight (rows a multiple of 16, cols of 8) with an optional fp32 bias.  ``glu``: the rows alternate
+    between 8 gate and 8 up rows (:func:`interleave_glu`) and the output is the clipped GLU of the two, half as wide."""
+
+    w: torch.Tensor
+    bias: torch.Tensor | None = None
+    glu: tuple[float, float] | None = None  # (alpha, limit)
+    input_kind = "dense"
+
+    @property
+    def out_width(self) -> int:
+        return self.w.shape[0] // (2 if self.glu is not None else 1)
+
+    def __call__(self, x: torch.Tensor, *, table: torch.Tensor | None = None, ids: torch.Tensor | None = None,
+                 out: torch.Tensor | None = None, tile: int | None = None, splits: int | None = None) -> torch.Tensor:
+        """``x [M, cols]``.  ``table`` (``[vocabulary, rows]``) with ``ids [M]``: the result is ``gelu_tanh(y) * table[ids]``."""
+        m, n, k = x.shape[0], self.w.shape[0], self.w.shape[1]
+        assert x.shape[1] == k and x.stride(1) == 1 and x.dtype == self.w.dtype and self.w.is_contiguous()
+        if out is None:
+            out = torch.empty((m, self.out_width), dtype=x.dtype, device=x.device)
+        kind, alpha, limit = BIAS, 0.0, 0.0
+        if self.glu is not None:
+            kind, (alpha, limit) = GLU, self.glu
+        elif table is not None:
+            assert table.shape[1] == n and table.is_contiguous() and table.dtype == x.dtype and ids.dtype == torch.int32
+            kind = GELU
+        t, s = plan(m, n, k)
+        t, s = (t if tile is None else tile), (s if splits is None else splits)
+        rc = dense_lib().mfq_dense_linear(ptr(self.w), ptr(x), x.stride(0), ptr(out), out.stride(0), ptr(self.bias), m, n, k, kind,
+                                          alpha, limit, ptr(table), ptr(ids), t, s, is_fp32(x.dtype),
+                                          ptr(Workspace.get(x.device).status), stream_ptr())
+        check(rc, "dense_linear")
+        return out
+
+
+def interleave_glu(gate: torch.Tensor, up_: torch.Tensor) -> torch.Tensor:
+    """Rows of two ``[F, K]`` matrices (F a multiple of 8) as blocks of 8 gate rows followed by the 8 matching up rows."""
+    f, k = gate.shape
+    return torch.stack([gate.reshape(f // 8, 8, k), up_.reshape(f // 8, 8, k)], 1).reshape(2 * f, k).contiguous()
+
+
+def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float):
+    """``(x, act)``: the fp32 stream ``table[ids] * scale`` and its copy in the activation type (the same tensor in fp32)."""
+    t, w = ids.numel(), table.shape[1]
+    x = torch.empty((t, w), dtype=torch.float32, device=table.device)
+    act = None if table.dtype == torch.float32 else torch.empty((t, w), dtype=table.dtype, device=table.device)
+    check(dense_lib().mfq_embed_scaled(ptr(ids), ptr(table), float(scale), ptr(x), ptr(act), t, w, is_fp32(table.dtype), stream_ptr()),
+          "embed_scaled")
+    return x, (x if act is None else act)
+
+
+def norm_add(y: torch.Tensor, weight: torch.Tensor, x: torch.Tensor, act: torch.Tensor, width: int, eps: float) -> None:
+    """In place: ``x += y / sqrt(mean(y^2) + eps) * weight`` (fp32, the mean over ``width`` columns); ``act`` follows ``x``."""
+    m, w = x.shape
+    assert y.shape == x.shape and y.is_contiguous() and x.dtype == torch.float32 and weight.dtype == torch.float32
+    copy = None if act is x else act
+    check(dense_lib().mfq_norm_add(ptr(y), ptr(weight), ptr(x), ptr(copy), m, w, width, float(eps), is_fp32(y.dtype), stream_ptr()),
+          "norm_add")
+
+
+def norm_out(x: torch.Tensor, weight: torch.Tensor, width: int, eps: float, dtype: torch.dtype) -> torch.Tensor:
+    """``x / sqrt(mean(x^2) + eps) * weight`` of the fp32 stream, in ``dtype``."""
+    m, w = x.shape
+    out = torch.empty((m, w), dtype=dtype, device=x.device)
+    check(dense_lib().mfq_norm_out(ptr(x), ptr(weight), ptr(out), m, w, width, float(eps), is_fp32(dtype), stream_ptr()), "norm_out")
+    return out

@@ -293,7 +293,8 @@ def paged_attn_decode(q: torch.Tensor, kv, block_table: torch.Tensor, seq_lens: 
 def argmax(logits: torch.Tensor, *, out=None) -> torch.Tensor:
     b, v = logits.shape
     out = torch.empty(b, dtype=torch.int32, device=logits.device) if out is None else out
-    check(lib().mfq_argmax(ptr(logits), ptr(out), b, v, logits.stride(0), stream_ptr()), "argmax")
+    fn = lib().mfq_argmax_f32 if logits.dtype == torch.float32 else lib().mfq_argmax
+    check(fn(ptr(logits), ptr(out), b, v, logits.stride(0), stream_ptr()), "argmax")
     return out
 
 

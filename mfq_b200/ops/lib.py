@@ -13,7 +13,7 @@ from functools import lru_cache
 
 import torch
 
-from .build import LIB_PATH
+from .build import DENSE_LIB_PATH, LIB_PATH
 
 _vp, _i, _f, _sz = C.c_void_p, C.c_int, C.c_float, C.c_size_t
 
@@ -38,6 +38,7 @@ _SIGNATURES = {
     
     "mfq_paged_attn_decode_mma": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _i, _vp, _vp],
     "mfq_argmax": [_vp, _vp, _i, _i, _i, _vp],
+    "mfq_argmax_f32": [_vp, _vp, _i, _i, _i, _vp],
     "mfq_embed": [_vp, _vp, _vp, _i, _i, _vp],
     "mfq_decode_advance": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _vp],
     "mfq_mtp_prepare": [_vp] * 9 + [_i, _i, _i, _i, _vp],
@@ -52,18 +53,40 @@ _SIGNATURES = {
 }
 
 
-@lru_cache(maxsize=1)
-def lib() -> C.CDLL:
-    if not LIB_PATH.exists():
+# the unquantized path (its own library)
+_DENSE_SIGNATURES = {
+    "mfq_dense_linear": [_vp, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _f, _f, _vp, _vp, _i, _i, _i, _vp, _vp],
+    "mfq_embed_scaled": [_vp, _vp, _f, _vp, _vp, _i, _i, _i, _vp],
+    "mfq_norm_add": [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _vp],
+    "mfq_norm_out": [_vp, _vp, _vp, _i, _i, _i, _f, _i, _vp],
+    "mfq_qkv_finish": [_vp, _i, _vp, _i, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
+    "mfq_window_attn_decode": [_vp] * 8 + [_i, _i, _i, _i, _i, _i, _i, _f, _f, _i, _vp],
+    "mfq_window_attn_plain": [_vp] * 7 + [_i, _i, _i, _i, _i, _i, _i, _f, _f, _i, _vp],
+    "mfq_window_attn_prefill": [_vp] * 7 + [_i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _f, _vp, _vp],
+}
+
+
+def _open(path, signatures) -> C.CDLL:
+    if not path.exists():
         raise RuntimeError(
-            f"{LIB_PATH.name} is not built; run `python -m mfq_b200.ops.build` (needs nvcc) before using GPU ops")
-    handle = C.CDLL(str(LIB_PATH))
-    for name, argtypes in _SIGNATURES.items():
+            f"{path.name} is not built; run `python -m mfq_b200.ops.build` (needs nvcc) before using GPU ops")
+    handle = C.CDLL(str(path))
+    for name, argtypes in signatures.items():
         if hasattr(handle, name):
             fn = getattr(handle, name)
             fn.argtypes = argtypes
             fn.restype = C.c_int
     return handle
+
+
+@lru_cache(maxsize=1)
+def lib() -> C.CDLL:
+    return _open(LIB_PATH, _SIGNATURES)
+
+
+@lru_cache(maxsize=1)
+def dense_lib() -> C.CDLL:
+    return _open(DENSE_LIB_PATH, _DENSE_SIGNATURES)
 
 
 def available() -> bool:
