@@ -380,6 +380,94 @@ def run_hybrid(args) -> dict:
     return result if rank == 0 else {}
 
 
+TEPETAR_SIZES = {  # width, ff, layers, query / KV heads of 128 channels, vocabulary, token-side width
+    "1b": (2048, 8192, 16, 16, 4, 65536, 128),
+    "3b": (3072, 8192, 28, 24, 8, 65536, 128),
+    "8b": (4096, 14336, 32, 32, 8, 128256, 256),
+}
+
+
+def run_tepetar(args) -> dict:
+    """The Tepetar family (bf16, sliding windows, score cap, shared values, token side input) beside the FP8 Llama of equal
+    geometry: prefill of one prompt and decode at batch 1 and ``--batch``, both through the same engine (one GPU)."""
+    import torch
+
+    from mfq_b200 import ops
+    from mfq_b200.engine.llm_engine import LLMEngine
+    from mfq_b200.models.llama import LlamaConfig, LlamaModel, LlamaWeights
+    from mfq_b200.models.tepetar import RandomTensors, TepetarConfig, TepetarModel, TepetarWeights
+
+    if args.gpus != 1:
+        raise SystemExit("--model tepetar runs on one GPU")
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    ops.count_launches(True)
+    ctx, new = args.context, 4 * (args.steps + args.warmup) + 16
+    gen = torch.Generator().manual_seed(1234)
+
+    def timed(fn, steps, warmup):
+        for _ in range(warmup):
+            fn()
+        torch.cuda.synchronize()
+        a, z = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        with ClockSampler(0) as clocks:
+            a.record()
+            for _ in range(steps):
+                fn()
+            z.record()
+            torch.cuda.synchronize()
+        return a.elapsed_time(z) / steps, clocks.summary()
+
+    def measure(model, vocab):
+        engine = LLMEngine(model, max_batch=args.batch, max_seq_len=ctx + new)
+        prompts = [torch.randint(0, vocab, (ctx,), generator=gen) for _ in range(args.batch)]
+        prefill_ms, _ = timed(lambda: engine.prefill(0, prompts[0]), 3, 3)
+        for row, prompt in enumerate(prompts):
+            engine.prefill(row, prompt)
+            engine.grow(row, ctx + new)
+        ms, clocks = timed(lambda: engine.decode_step(args.batch), args.steps, args.warmup)
+        ms1, _ = timed(lambda: engine.decode_step(1), args.steps, args.warmup)
+        host_in = engine.sampled[: args.batch].cpu().pin_memory()
+        host_out = torch.zeros_like(host_in).pin_memory()
+        e2e, _ = timed(lambda: engine.step_host(host_in, host_out), args.steps, args.warmup)
+        ops.Workspace.get(dev).check()
+        return {"prefill_tok_s": round(ctx / prefill_ms * 1e3, 1), "prefill_ms": round(prefill_ms, 3),
+                "decode_ms": round(ms, 4), "decode_tok_s": round(args.batch / ms * 1e3, 1), "decode_ms_bs1": round(ms1, 4),
+                "decode_tok_s_bs1": round(1e3 / ms1, 1), "e2e_tok_s": round(args.batch / e2e * 1e3, 1), "clocks": clocks,
+                "launches_per_step": engine.launches_per_step.get(args.batch)}
+
+    table = {}
+    for size in (args.size.split(",") if args.size else ["1b", "8b"]):
+        width, ff, layers, hq, hk, vocab, side = TEPETAR_SIZES[size]
+        if args.tiny:
+            width, ff, layers, hq, hk, vocab = 256, 512, 2, 4, 2, 1024
+        for window in (int(w) for w in args.window.split(",")):
+            cfg = TepetarConfig.uniform(vocab_size=vocab, hidden_size=width, num_layers=layers, heads=hq, kv_heads=hk, dim=128, vdim=128,
+                                        window=window, ff=ff, side_dim=side)
+            weights = TepetarWeights(cfg, RandomTensors(cfg, dev), dev)
+            row = {"params_b": round(cfg.param_count() / 1e9, 3), "weights_gb": round(weights.nbytes() / 1e9, 2),
+                   **measure(TepetarModel(cfg, weights), vocab)}
+            table[f"tepetar-{size}-w{window}"] = row
+            print(f"[bench] tepetar-{size}-w{window} {json.dumps(row)}", file=sys.stderr, flush=True)
+            del weights
+            torch.cuda.empty_cache()
+        cfg = LlamaConfig(vocab_size=vocab, hidden_size=width, intermediate_size=ff, num_layers=layers, num_heads=hq, num_kv_heads=hk)
+        row = {"params_b": round(cfg.param_count() / 1e9, 3), **measure(LlamaModel(cfg, LlamaWeights.random_init(cfg, dev)), vocab)}
+        table[f"llama-fp8-{size}"] = row
+        print(f"[bench] llama-fp8-{size} {json.dumps(row)}", file=sys.stderr, flush=True)
+        torch.cuda.empty_cache()
+    name, first = next(iter(table.items()))
+    return {"metric": f"decode_tok_s_bs{args.batch}", "value": first["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
+            "warmup": args.warmup, "ms_per_step": first["decode_ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+            "dtype": "bf16 weights/activations/KV, fp32 stream, norms and scores", "impl": "ours",
+            "data": "synthetic (uniform random token ids, random-init weights)",
+            "config": {"model": name, "global_batch": args.batch, "seq_len": ctx, "parallelism": "dp1",
+                       "l2": "inputs larger than L2 (every step streams all weights)"},
+            "clocks": first["clocks"],
+            "e2e": {"value": first["e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 4 * args.batch, "d2h_bytes_per_step": 4 * args.batch},
+            "gpu_launches": (first["launches_per_step"] or 0) * args.steps, "extra": table}
+
+
 def run_reference(args) -> dict:
     from baseline import reference_arm
     return reference_arm.run(args)
@@ -405,15 +493,18 @@ def main() -> None:
     ap.add_argument("--profile-steps", type=int, default=0,
                     help="after the timed region, run this many batched decode steps between cudaProfilerStart/Stop")
     ap.add_argument("--tiny", action="store_true", help="tiny model, for checking the harness itself")
-    ap.add_argument("--model", choices=["llama8b", "hybrid80b"], default="llama8b",
-                    help="llama8b: the flagship; hybrid80b: the Gated-DeltaNet + MoE hybrid with an MTP head (one GPU)")
+    ap.add_argument("--model", choices=["llama8b", "hybrid80b", "tepetar"], default="llama8b",
+                    help="llama8b: the flagship; hybrid80b: the Gated-DeltaNet + MoE hybrid with an MTP head (one GPU); "
+                         "tepetar: that family in bf16 beside the FP8 Llama of equal geometry (one GPU)")
+    ap.add_argument("--size", default="", help="tepetar: comma separated sizes out of " + ", ".join(TEPETAR_SIZES) + " (default 1b,8b)")
+    ap.add_argument("--window", default="4096,1024", help="tepetar: comma separated window sizes")
     args = ap.parse_args()
     if args.warmup < 3:
         args.warmup = 3
     if args.impl == "reference":
         out = run_reference(args)
     else:
-        out = run_hybrid(args) if args.model == "hybrid80b" else run_ours(args)
+        out = {"hybrid80b": run_hybrid, "tepetar": run_tepetar}.get(args.model, run_ours)(args)
     if out:
         print(json.dumps(out), flush=True)
 

@@ -534,7 +534,7 @@ def _cmd_serve(args) -> int:
         slots = args.moe_gpu_cache_slots
         if slots is None and cache_gb:
             slots = _expert_slots_for(path, cache_gb)
-        engine, tok, _cfg = load_engine(path, device, max_batch=args.continuous_batching, max_seq_len=ctx_size, **tp,
+        engine, tok, _cfg = load_engine(path, device, max_batch=args.continuous_batching, max_seq_len=ctx_size, **tp, dtype=args.dtype,
                                         native_4bit=args.native_4bit, expert_slots=slots,
                                         expert_graphs=getattr(args, "moe_cache_graphs", False),
                                         kv_budget_bytes=int(kv_gb * (1 << 30)) if kv_gb else None,
@@ -635,6 +635,7 @@ def _serve_with_worker(args, service, device) -> int:
     command = [sys.executable, "-m", "mfq_b200.cli", "runtime", "--model", args.model, "--device", device,
                "--continuous-batching", str(args.continuous_batching), "--ctx-size", str(args.ctx_size),
                "--max-queue", str(args.max_queue), "--queue-timeout", str(args.queue_timeout),
+               "--dtype", args.dtype,
                *(["--native-4bit"] if args.native_4bit else []),
                *(["--yarn-context-extension", str(args.yarn_context_extension)] if args.yarn_context_extension else [])]
     service.add_worker_model(args.model_name or Path(args.model).stem, command, tokenizer_from_assets(assets, vocab),
@@ -660,7 +661,7 @@ def _cmd_runtime(args) -> int:
     sys.stdout = sys.stderr  # anything printed while serving must not corrupt the frame stream
     service = ModelService(max_queue=args.max_queue, queue_timeout=args.queue_timeout)
     engine, tok, _cfg = load_engine(args.model, device, max_batch=args.continuous_batching, max_seq_len=args.ctx_size,
-                                    native_4bit=args.native_4bit, yarn_context_extension=args.yarn_context_extension)
+                                    dtype=args.dtype, native_4bit=args.native_4bit, yarn_context_extension=args.yarn_context_extension)
     service.add_model(args.model_name or Path(args.model).stem, engine, tok)
     try:
         StdioTransport(service, sys.stdin, out).serve()
@@ -676,7 +677,8 @@ def _cmd_profile(args) -> int:
     from .checkpoint import load_engine
     from .utils.profiler import PROFILER, profile_engine
     device = args.device or ("cuda" if torch.cuda.is_available() else "cpu")
-    engine, _tok, cfg = load_engine(args.model, device, max_batch=1, max_seq_len=args.prompt_tokens + args.decode_tokens + 8)
+    engine, _tok, cfg = load_engine(args.model, device, max_batch=1, max_seq_len=args.prompt_tokens + args.decode_tokens + 8,
+                                    dtype=args.dtype)
     vocab = int(cfg.vocab_size)
     ids = torch.tensor([3 + (i * 7919) % (vocab - 8) for i in range(args.prompt_tokens)], dtype=torch.int32)
     profile_engine(engine, ids, args.decode_tokens, args.filter)
@@ -923,6 +925,8 @@ def build_parser() -> argparse.ArgumentParser:
     s.add_argument("--access-log", action="store_true")
     s.add_argument("--native-4bit", action="store_true",
                    help="run NINT (<= 4 code bits) / MXFP4 projections through the 4-bit in-pipeline-decode GEMM instead of FP8")
+    s.add_argument("--dtype", choices=["auto", "bfloat16", "float32"], default="auto",
+                   help="element type of weights and activations, for model families that offer a choice")
     s.add_argument("--moe-gpu-cache-slots", type=int, default=None,
                    help="keep routed experts in pinned host memory behind an HBM arena of this many slots per layer")
     s.add_argument("--moe-cache-graphs", action="store_true",
@@ -986,6 +990,8 @@ def build_parser() -> argparse.ArgumentParser:
     pf.add_argument("--decode-tokens", type=int, default=8)
     pf.add_argument("--filter", default="", help="comma separated name pieces to keep (e.g. attn,ffn.down)")
     pf.add_argument("--device")
+    pf.add_argument("--dtype", choices=["auto", "bfloat16", "float32"], default="auto",
+                    help="element type of weights and activations, for model families that offer a choice")
     pf.set_defaults(fn=_cmd_profile)
     rt = sub.add_parser("runtime", help="serve one model over newline-delimited JSON frames on stdin / stdout")
     rt.add_argument("--model", required=True)
@@ -998,6 +1004,8 @@ def build_parser() -> argparse.ArgumentParser:
     rt.add_argument("--native-4bit", action="store_true")
     rt.add_argument("--yarn-context-extension", type=float, default=None)
     rt.add_argument("--device")
+    rt.add_argument("--dtype", choices=["auto", "bfloat16", "float32"], default="auto",
+                    help="element type of weights and activations, for model families that offer a choice")
     rt.set_defaults(fn=_cmd_runtime)
     be = sub.add_parser("bench", help="run the flagship benchmark (arguments are passed through to bench.py)")
     be.add_argument("rest", nargs=argparse.REMAINDER)

@@ -135,9 +135,10 @@ class SchedulerStats:
 
 class ContinuousBatchScheduler:
     def __init__(self, backend: Backend, *, max_queue: int = 256, queue_timeout: float | None = None,
-                 clock: Callable[[], float] = time.monotonic, mixed_tokens: int = 2048) -> None:
+                 clock: Callable[[], float] = time.monotonic, mixed_tokens: int | None = None) -> None:
+        """``mixed_tokens``: most prompt tokens a mixed step reads (default 2048, or the backend's prefill chunk if smaller)."""
         self.backend = backend
-        self.mixed_tokens = mixed_tokens
+        self.mixed_tokens = mixed_tokens or min(2048, getattr(backend, "prefill_chunk", 2048))
         self.reading: dict[int, int] = {}  # row -> prompt tokens left to read (mixed batches)
         self.max_queue, self.queue_timeout, self.clock = max_queue, queue_timeout, clock
         self.waiting: list[Request] = []

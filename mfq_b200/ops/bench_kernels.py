@@ -161,12 +161,89 @@ def bench_small(m: int, h: int, i: int, reps: int) -> list[dict]:
     return out
 
 
+def bench_dense(m: int, n: int, k: int, reps: int, glu: bool = False, tile=None, splits=None) -> dict:
+    """Unquantized (bf16) product, optionally with the clipped-GLU output stage."""
+    from . import dense
+    copies = max(1, min(16, math.ceil(4 * L2_BYTES / (2 * n * k))))
+    lin = [dense.DenseLinear((torch.randn((n, k), device="cuda") * k ** -0.5).to(torch.bfloat16),
+                             torch.zeros(n, device="cuda"), (1.702, 7.0) if glu else None) for _ in range(copies)]
+    x = torch.randn((m, k), device="cuda").to(torch.bfloat16)
+    out = torch.empty((m, lin[0].out_width), device="cuda", dtype=torch.bfloat16)
+    ms = time_ms(lambda i: lin[i % copies](x, out=out, tile=tile, splits=splits), reps)
+    t, sp = dense.plan(m, n, k)
+    return {"kernel": "dense_gemv" if (t if tile is None else tile) == 0 else "dense_gemm", "m": m, "n": n, "k": k, "us": ms * 1e3,
+            "gbs": 2 * (n * k + m * k + out.numel()) / ms / 1e6, "tflops": 2 * m * n * k / ms / 1e9,
+            "tile": t if tile is None else tile, "splits": sp if splits is None else splits}
+
+
+def _plain_cache(batch: int, ctx: int, hk: int, d: int, e: int, layers: int):
+    from ..engine.kv_cache import PlainPagedKVCache
+    pages_per = math.ceil(ctx / 16)
+    cache = PlainPagedKVCache([(hk, d, e)] * layers, torch.bfloat16, num_pages=batch * pages_per + 1, max_seqs=batch,
+                              max_pages_per_seq=pages_per, device="cuda")
+    for pool in cache.pools:
+        pool.k.normal_()
+        pool.v.normal_()
+    for b in range(batch):
+        cache.assign(b, b, ctx)
+    return cache
+
+
+def bench_window_decode(batch: int, ctx: int, hq: int, hk: int, d: int, window: int, cap: float, reps: int, splits=None) -> dict:
+    """One token per sequence over unquantized pages; every key inside the window is read once."""
+    from . import window_attn
+    seen = min(ctx, window)
+    layers = max(1, min(32, math.ceil(4 * L2_BYTES / (batch * seen * hk * d * 4))))
+    cache = _plain_cache(batch, ctx, hk, d, d, layers)
+    q = torch.randn((batch, hq, d), device="cuda").to(torch.bfloat16)
+    sl = torch.full((batch,), ctx, dtype=torch.int32, device="cuda")
+    out = torch.empty_like(q)
+    splits = window_attn.decode_splits(batch, hk, seen) if splits is None else splits
+    ms = time_ms(lambda i: window_attn.decode(q, cache.layer(i % layers), cache.block_table, sl, window=window, scale=0.088, cap=cap,
+                                              splits=splits, out=out), reps)
+    return {"kernel": "window_attn_decode", "batch": batch, "ctx": ctx, "hq": hq, "hk": hk, "d": d, "window": window, "cap": cap,
+            "splits": splits, "us": ms * 1e3, "gbs": batch * seen * hk * d * 4 / ms / 1e6}
+
+
+def bench_window_prefill(t: int, hq: int, hk: int, d: int, window: int, cap: float, reps: int) -> dict:
+    from . import window_attn
+    cache = _plain_cache(1, t, hk, d, d, 1)
+    q = torch.randn((t, hq, d), device="cuda").to(torch.bfloat16)
+    out = torch.empty_like(q)
+    starts, lens = (torch.tensor(v, dtype=torch.int32, device="cuda") for v in ([0, t], [t]))
+    ms = time_ms(lambda _: window_attn.prefill(q, cache.layer(0), cache.block_table, starts, lens, t, window=window, scale=0.088, cap=cap,
+                                               out=out), reps)
+    w = min(window, t)
+    pairs = w * (w + 1) // 2 + (t - w) * w  # visible (query, key) pairs
+    return {"kernel": "window_attn_prefill", "t": t, "hq": hq, "hk": hk, "d": d, "window": window, "cap": cap, "us": ms * 1e3,
+            "tflops": 4 * pairs * hq * d / ms / 1e9}
+
+
+def bench_dense_small(m: int, h: int, reps: int) -> list[dict]:
+    """The fp32 stream and the per-head stage (32 / 8 heads of 128)."""
+    from . import dense, window_attn
+    y = torch.randn((m, h), device="cuda").to(torch.bfloat16)
+    x, act, w = torch.randn((m, h), device="cuda"), torch.empty_like(y), torch.ones(h, device="cuda")
+    ms = time_ms(lambda _: dense.norm_add(y, w, x, act, h, 1e-5), reps)
+    rows = [{"kernel": "norm_add", "m": m, "h": h, "us": ms * 1e3, "gbs": m * h * 12 / ms / 1e6}]
+    hq, hk, d = 32, 8, 128
+    cache = _plain_cache(1, m, hk, d, d, 1)
+    qkv = torch.randn((m, (hq + 2 * hk) * d), device="cuda").to(torch.bfloat16)
+    first = torch.randn((m, hk * d), device="cuda").to(torch.bfloat16)
+    pos, slots, one = torch.arange(m, dtype=torch.int32, device="cuda"), cache.slots(0, 0, m).cuda(), torch.ones(d, device="cuda")
+    rope = window_attn.rope_table(5e5, d, m, "cuda")
+    ms = time_ms(lambda _: window_attn.qkv_finish(qkv, cache.layer(0), pos, slots, heads=hq, kv_heads=hk, dim=d, q_norm=one, k_norm=one,
+                                                  rope=rope, rot=d, eps=1e-5, v_first=first, mix=0.5), reps)
+    rows.append({"kernel": "qkv_finish", "t": m, "us": ms * 1e3, "gbs": m * ((hq + 2 * hk) * d * 4 + hk * d * 2) / ms / 1e6})
+    return rows
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--json", default="")
     ap.add_argument("--reps", type=int, default=20)
     ap.add_argument("--quick", action="store_true")
-    ap.add_argument("--only", default="", help="comma separated kernel families: gemm,w4,attn,mla,small,prefill")
+    ap.add_argument("--only", default="", help="comma separated kernel families: gemm,w4,attn,mla,small,prefill,dense")
     ap.add_argument("--tp", type=int, default=1, help="time one rank's shard of a tensor-parallel group of this size")
     args = ap.parse_args()
     pk = peaks()
@@ -205,6 +282,20 @@ def main() -> None:
     for t in (1024, 4096) if want("prefill") else ():
         rows += bench_prefill(t, 32, 8, args.reps)
         rows += bench_prefill(t, 16, 2, args.reps, d=256)[:1]
+    for m in ((1, 64) if args.quick else (1, 16, 64, 512, 4096)) if want("dense") else ():
+        for name, n, k in shapes:
+            if name == "lm_head" and m > 64:
+                continue
+            rows.append({**bench_dense(m, n, k, args.reps, glu=name == "gate_up"), "name": name})
+    if want("dense"):
+        for batch in (1, 64):
+            for window, cap in ((4096, 0.0), (4096, 50.0), (1024, 50.0)):
+                rows.append(bench_window_decode(batch, 4096, 32, 8, 128, window, cap, args.reps))
+        for t in (1024, 4096):
+            for window, cap in ((1 << 30, 0.0), (1 << 30, 50.0), (1024, 50.0)):
+                rows.append(bench_window_prefill(t, 32, 8, 128, window, cap, args.reps))
+        for m in (1, 64, 4096):
+            rows += bench_dense_small(m, 4096, args.reps)
     for r in rows:
         if "gbs" in r:
             r["hbm_frac"] = r["gbs"] / pk["hbm_gbs"]
