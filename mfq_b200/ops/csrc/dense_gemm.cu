@@ -272,6 +272,20 @@ dense_gemv_kernel(const __nv_bfloat16* __restrict__ w, const __nv_bfloat16* __re
   }
 }
 
+template <int NT>
+static int launch_dense_gemv(const void* w, const void* x, int ldx, const DenseParams& p, cudaStream_t stream) {
+  // The loads in flight live in L1.  On an SM that a kernel with much shared memory leaves behind, L1 would stay small and
+  // the stream slow, so this kernel asks for a small shared-memory carve-out.
+  static bool set = false;
+  if (!set) {
+    if (cudaFuncSetAttribute(dense_gemv_kernel<NT>, cudaFuncAttributePreferredSharedMemoryCarveout, 15 * NT) != cudaSuccess) return -6;
+    set = true;
+  }
+  launch_kernel(dense_gemv_kernel<NT>, dim3(p.N / 16), dim3(256), 0, stream, static_cast<const __nv_bfloat16*>(w),
+                static_cast<const __nv_bfloat16*>(x), ldx, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -7;
+}
+
 // ---------------------------------------------------------------------------------------------
 // fp32 operands: 64 tokens x 64 rows per CTA, 16-wide K steps, 4 x 4 outputs per thread.
 // ---------------------------------------------------------------------------------------------
@@ -337,11 +351,7 @@ extern "C" int mfq_dense_linear(const void* w, const void* x, int ldx, void* out
   }
   if (token_tile == 0) {
     if (M > 16) return -1;
-    auto* wp = static_cast<const __nv_bfloat16*>(w);
-    auto* xp = static_cast<const __nv_bfloat16*>(x);
-    if (M <= 8) launch_kernel(dense_gemv_kernel<1>, dim3(N / 16), dim3(256), 0, stream, wp, xp, ldx, p);
-    else launch_kernel(dense_gemv_kernel<2>, dim3(N / 16), dim3(256), 0, stream, wp, xp, ldx, p);
-    return cudaGetLastError() == cudaSuccess ? 0 : -7;
+    return M <= 8 ? launch_dense_gemv<1>(w, x, ldx, p, stream) : launch_dense_gemv<2>(w, x, ldx, p, stream);
   }
   switch (token_tile) {
     case 16: return launch_dense_gemm<16>(p, w, x, ldx, splits, stream);

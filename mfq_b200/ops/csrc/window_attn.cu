@@ -52,7 +52,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
 // DK / DV: upper bounds of the stored head widths (register arrays); the widths themselves are run-time multiples of 16.
 template <int DK, int DV>
 struct WinCfg {
-  static constexpr int kStages = DK + DV <= 256 ? 3 : 2;
+  static constexpr int kStages = 2;  // two pages per warp in flight leave room for three CTAs per SM at 128 + 128 channels
   static int stage_bytes(int dk, int dv) { return kWinPage * (dk + 8 + dv + 8) * 2; }
   static int smem_bytes(int dk, int dv) {
     const int ring = kWinWarps * kStages * stage_bytes(dk, dv), merge = kWinWarps * 16 * (dv + 2) * 4;

@@ -14,7 +14,7 @@ import torch
 from .lib import Workspace, check, dense_lib, ptr, stream_ptr
 
 BIAS, GLU, GELU = 0, 1, 2  # epilogues (dense_common.cuh)
-GEMV_ROWS, GEMV_MID_ROWS, GEMV_MID_WEIGHTS = 8, 16, 20 << 20
+GEMV_ROWS, GEMV_MID_ROWS, GEMV_MID_WEIGHTS = 8, 16, 8 << 20
 
 
 def up(n: int, m: int = 16) -> int:
@@ -28,27 +28,36 @@ def is_fp32(dtype: torch.dtype) -> int:
     return int(dtype == torch.float32)
 
 
+def _most_splits(tiles: int, blocks: int, small: bool, sms: int) -> int:
+    """Most K splits worth taking: the clusters must all be resident at once, every CTA keeps 8 K blocks.  Where one CTA fills
+    an SM, clusters do not pack every SM of a GPC: 128 CTAs fit, 96 in clusters of more than 4."""
+    best = 1
+    for s in range(2, 9):
+        room = sms if small else (96 if s > 4 else 128)
+        if tiles * s <= room and blocks // s >= 8:
+            best = s
+    return best
+
+
 def plan(m: int, n: int, k: int, sms: int = 148) -> tuple[int, int]:
-    """``(token tile, K splits)`` of a bf16 product ``[m, k] x [n, k]^T``; tile 0 is the weight-streaming kernel.  The split
-    count minimises waves x (K blocks per CTA + ramp) over the clusters of up to 8 CTAs that meet in shared memory."""
+    """``(token tile, K splits)`` of a bf16 product ``[m, k] x [n, k]^T``; tile 0 is the weight-streaming kernel.  Fitted to a
+    sweep on B200 over the projections of 1B- and 8B-sized layers at 16 .. 4096 tokens: up to 128 tokens the weights are read
+    once whatever the split, so the grid is filled; beyond that a wave of 256-token tiles costs about 7 + 0.35 us per K block,
+    of 128-token tiles 5 + 0.30 us, and meeting in a cluster 5 / 3 us."""
     if m <= GEMV_ROWS or (m <= GEMV_MID_ROWS and n * k <= GEMV_MID_WEIGHTS):
         return 0, 1
-    rows = math.ceil(n / 128)
-    tile = next((t for t in (16, 32, 64, 128) if m <= t), 0)
-    if not tile:
-        tile = 256 if rows * math.ceil(m / 256) >= 100 else 128
-    tiles, kb = rows * math.ceil(m / tile), math.ceil(k / 64)
-    slots = sms * (2 if tile <= 64 else 1)
-    best, best_cost = 1, None
-    for s in range(1, min(kb, 8) + 1):
-        per = math.ceil(kb / s)
-        if s > 1 and per < 4:
-            break
-        ctas = tiles * math.ceil(kb / per)
-        cost = math.ceil(ctas / slots) * (per + 6) + (3 if s > 1 else 0)
-        if best_cost is None or cost < best_cost:
-            best, best_cost = s, cost
-    return tile, best
+    rows, blocks = math.ceil(n / 128), math.ceil(k / 64)
+    for tile in (16, 32, 64, 128):
+        if m <= tile:
+            return tile, _most_splits(rows, blocks, tile <= 64, sms)
+    best, best_cost = (128, 1), None
+    for tile, ramp, per_block, meet in ((128, 5.0, 0.30, 3.0), (256, 7.0, 0.35, 5.0)):
+        tiles = rows * math.ceil(m / tile)
+        for s in range(1, _most_splits(tiles, blocks, False, sms) + 1):
+            cost = math.ceil(tiles * s / sms) * (ramp + per_block * math.ceil(blocks / s)) + (meet if s > 1 else 0.0)
+            if best_cost is None or cost < best_cost:
+                best, best_cost = (tile, s), cost
+    return best
 
 
 @dataclass

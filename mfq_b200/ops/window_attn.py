@@ -41,8 +41,17 @@ def qkv_finish(qkv: torch.Tensor, kv, positions, slots, *, heads: int, kv_heads:
 
 
 def decode_splits(batch: int, kv_heads: int, keys: int) -> int:
-    """KV splits per (sequence, KV head): as many as one wave of three CTAs per SM holds, at least 128 keys each."""
-    return max(1, min(148 * 3 // max(1, batch * kv_heads), keys // 128, 16))
+    """KV splits per (sequence, KV head) over ``keys`` visible keys: least waves of three CTAs per SM times keys per CTA, at
+    least 160 keys per split while one wave holds all CTAs and 256 beyond that."""
+    n, slots = max(1, batch * kv_heads), 148 * 3
+    best, best_cost = 1, None
+    for s in range(1, 25):
+        if s > 1 and keys // s < (160 if n * s <= slots else 256):
+            break
+        cost = -(-n * s // slots) * keys / s + 8 * s
+        if best_cost is None or cost < best_cost:
+            best, best_cost = s, cost
+    return best
 
 
 def decode(q: torch.Tensor, kv, block_table, seq_lens, *, window: int, scale: float, cap: float, splits: int = 1, out=None):
