@@ -7,7 +7,9 @@ for a multi-pass capture to finish in about a minute) and exits.  Cases: ``gemm_
 64 sequences), ``moe_dispatch`` (expert-parallel dispatch + combine kernels at world 1, 4096 tokens), ``gemv_decode``
 (the weight-streaming FP8 kernel, M=1, N=28672, K=4096), ``attn_prefill_d256`` (T=2048, 16 query / 2 KV heads of 256),
 ``gdn_prefill`` (the long-row Gated DeltaNet path, 2048 tokens, 32 heads), ``mla_decode`` (latent-cache decode attention), ``packed_decode`` / ``packed_decode_bs1`` (the
-packed-expert product at 64 tokens / one token, 512 experts).
+packed-expert product at 64 tokens / one token, 512 experts), ``window_decode`` / ``window_prefill`` (attention over
+unquantized pages with a 1024-token window and a score cap: 64 sequences of 4096 tokens, one prompt of 2048), ``dense_prefill``
+(unquantized product, M=4096, N=K=4096).
 """
 
 from __future__ import annotations
@@ -170,11 +172,40 @@ def packed_decode(tokens: int = 64) -> None:
         packed.packed_gemv_grouped(pe, x, plan, gather=True)
 
 
+def window_decode() -> None:
+    from . import bench_kernels, window_attn
+    cache = bench_kernels._plain_cache(64, 4096, 8, 128, 128, 3)  # 1 GB of pages per launch, a quarter of it inside the window
+    q = torch.randn((64, 32, 128), device="cuda").to(torch.bfloat16)
+    lens = torch.full((64,), 4096, dtype=torch.int32, device="cuda")
+    for i in range(3):
+        window_attn.decode(q, cache.layer(i), cache.block_table, lens, window=1024, scale=0.088, cap=50.0,
+                           splits=window_attn.decode_splits(64, 8, 1024))
+
+
+def window_prefill() -> None:
+    from . import bench_kernels, window_attn
+    t = 2048
+    cache = bench_kernels._plain_cache(1, t, 8, 128, 128, 1)
+    q = torch.randn((t, 32, 128), device="cuda").to(torch.bfloat16)
+    starts, lens = (torch.tensor(v, dtype=torch.int32, device="cuda") for v in ([0, t], [t]))
+    for _ in range(3):
+        window_attn.prefill(q, cache.layer(0), cache.block_table, starts, lens, t, window=1024, scale=0.088, cap=50.0)
+
+
+def dense_prefill() -> None:
+    from . import dense
+    lin = [dense.DenseLinear(torch.randn((4096, 4096), device="cuda").to(torch.bfloat16)) for _ in range(3)]
+    x = torch.randn((4096, 4096), device="cuda").to(torch.bfloat16)
+    for i in range(3):
+        lin[i](x)
+
+
 CASES = {"gemm_prefill": lambda: gemm(4096, 4096, 4096), "gemm_decode": lambda: gemm(64, 28672, 4096),
          "gemm_decode_splitk": lambda: gemm(64, 4096, 14336),
          "attn_decode": attn_decode, "attn_prefill": attn_prefill, "w4_decode": lambda: w4_gemm(64, 28672, 4096),
          "w4_prefill": lambda: w4_gemm(4096, 4096, 4096), "gdn_decode": gdn_decode, "moe_dispatch": moe_dispatch,
-         "gemv_decode": lambda: gemm(1, 28672, 4096), "packed_decode": packed_decode, "packed_decode_bs1": lambda: packed_decode(1), "attn_prefill_d256": attn_prefill_d256, "gdn_prefill": gdn_prefill, "mla_decode": mla_decode}
+         "gemv_decode": lambda: gemm(1, 28672, 4096), "packed_decode": packed_decode, "packed_decode_bs1": lambda: packed_decode(1), "attn_prefill_d256": attn_prefill_d256, "gdn_prefill": gdn_prefill, "mla_decode": mla_decode,
+         "window_decode": window_decode, "window_prefill": window_prefill, "dense_prefill": dense_prefill}
 
 if __name__ == "__main__":
     CASES[sys.argv[1]]()

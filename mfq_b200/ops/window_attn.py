@@ -41,17 +41,17 @@ def qkv_finish(qkv: torch.Tensor, kv, positions, slots, *, heads: int, kv_heads:
 
 
 def decode_splits(batch: int, kv_heads: int, keys: int) -> int:
-    """KV splits per (sequence, KV head) over ``keys`` visible keys: least waves of three CTAs per SM times keys per CTA, at
-    least 160 keys per split while one wave holds all CTAs and 256 beyond that."""
+    """KV splits per (sequence, KV head) over ``keys`` visible keys, fitted to a sweep on B200 (batch 1 .. 128, windows 1024 and
+    4096): a batch that leaves SMs free takes the most splits that keep the grid below 400 CTAs (at most 16, 64 keys each); one
+    that comes near a wave of three CTAs per SM evens its last wave out with up to 5 splits of at least 256 keys; more is not
+    split."""
     n, slots = max(1, batch * kv_heads), 148 * 3
-    best, best_cost = 1, None
-    for s in range(1, 25):
-        if s > 1 and keys // s < (160 if n * s <= slots else 256):
-            break
-        cost = -(-n * s // slots) * keys / s + 8 * s
-        if best_cost is None or cost < best_cost:
-            best, best_cost = s, cost
-    return best
+    if n <= 200:
+        return max(1, min(400 // n, keys // 64, 16))
+    if n > 600:
+        return 1
+    choices = [s for s in range(1, 6) if s == 1 or keys // s >= 256]
+    return min(choices, key=lambda s: -(-n * s // slots) * keys / s + 20 * s)
 
 
 def decode(q: torch.Tensor, kv, block_table, seq_lens, *, window: int, scale: float, cap: float, splits: int = 1, out=None):
