@@ -127,6 +127,13 @@ class TepetarConfig:
                           v_mix, ff, limit)
         return cls(vocab_size, hidden_size, [layer] * num_layers, embed_scale, norm_eps, side_dim, name)
 
+    def kv_shapes(self) -> list[tuple[int, int, int]]:
+        """Per layer: (KV heads, stored key width, stored value width)."""
+        return [(l.kv_heads, up(l.dim), up(l.vdim)) for l in self.layers]
+
+    def kv_token_bytes(self, element_bytes: int) -> int:
+        return sum(g * (dk + dv) for g, dk, dv in self.kv_shapes()) * element_bytes
+
     def param_count(self) -> int:
         h, total = self.hidden_size, 2 * self.vocab_size * self.hidden_size
         for l in self.layers:
@@ -279,15 +286,11 @@ class TepetarModel(LlamaModel):
         self._rows: torch.Tensor | None = None
 
     # -- cache ------------------------------------------------------------------------------------------------------
-    def kv_shapes(self) -> list[tuple[int, int, int]]:
-        """Per layer: (KV heads, stored key width, stored value width)."""
-        return [(l.kv_heads, up(l.dim), up(l.vdim)) for l in self.cfg.layers]
-
     def kv_token_bytes(self) -> int:
-        return sum(g * (dk + dv) for g, dk, dv in self.kv_shapes()) * self.w.embed.element_size()
+        return self.cfg.kv_token_bytes(self.w.embed.element_size())
 
     def make_cache(self, *, num_pages: int, max_seqs: int, max_pages_per_seq: int, device) -> PlainPagedKVCache:
-        cache = PlainPagedKVCache(self.kv_shapes(), self.w.dtype, num_pages=num_pages, max_seqs=max_seqs,
+        cache = PlainPagedKVCache(self.cfg.kv_shapes(), self.w.dtype, num_pages=num_pages, max_seqs=max_seqs,
                                   max_pages_per_seq=max_pages_per_seq, device=device)
         n = max_pages_per_seq * cache.page_size  # positions an engine with this cache can reach
         for l in self.cfg.layers:

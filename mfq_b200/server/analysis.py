@@ -147,6 +147,9 @@ def model_memory(cfg: dict, weight_bytes: int, *, batch: int = 1, context: int =
     tp = max(1, int(tensor_parallel))
     pages = batch * math.ceil(context / PAGE_TOKENS) + 1
     kv = pages * page_bytes(p["attention_layers"], max(1, hk // tp), d)
+    if cfg.get("family") == "tepetar":  # bf16 pages, every layer its own geometry
+        from ..models.tepetar import TepetarConfig
+        kv = pages * PAGE_TOKENS * TepetarConfig.from_dict(cfg).kv_token_bytes(2)
     lin_v = _cfg_int(cfg, "linear_num_value_heads")
     state = 0
     if lin_v:

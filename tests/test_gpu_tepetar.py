@@ -183,6 +183,29 @@ def test_greedy_generation_through_engine_and_scheduler(tmp_path):
     check_status()
 
 
+def test_command_line_runtime_serves_the_checkpoint(tmp_path):
+    """`mfq runtime` on the checkpoint's own directory: ready, two prompts at once, shutdown."""
+    import json
+    import subprocess
+    import sys
+    from pathlib import Path
+    cfg = cases.config([cases.layer()] * 2, vocab=300)
+    path = cases.write(tmp_path / "m", cfg, cases.weights(cfg))
+    ask = lambda i, n: {"v": 1, "id": i, "op": "generate", "params": {"model": "m", "input": {"benchmark_prompt_tokens": n},
+                                                                      "sampling": {"temperature": 0.0, "max_new_tokens": 6}, "stream": False}}
+    frames = [ask("a", 37), ask("b", 90), {"v": 1, "op": "shutdown"}]
+    run = subprocess.run([sys.executable, "-m", "mfq_b200.cli", "runtime", "--model", str(path), "--dtype", "float32", "--ctx-size", "256",
+                          "--continuous-batching", "4"], input="".join(json.dumps(f) + "\n" for f in frames), capture_output=True,
+                         text=True, timeout=240, cwd=Path(__file__).resolve().parents[1])
+    said = [json.loads(l) for l in run.stdout.splitlines()]
+    assert run.returncode == 0, run.stderr[-2000:]
+    results = {f["id"]: f["data"] for f in said if f["type"] == "result"}
+    assert said[0]["type"] == "ready" and not [f for f in said if f["type"] == "error"]
+    for i, n in (("a", 37), ("b", 90)):
+        usage = results[i]["usage"]
+        assert usage["prompt_tokens"] == n and (usage["completion_tokens"] == 6 or results[i]["finish_reason"] == "stop")
+
+
 def test_sampling_scoring_and_retraction(tmp_path):
     """Seeded sampling does not depend on how the prompt was read; scores are the oracle's log probabilities; a pool that is too
     small retracts and still finishes."""

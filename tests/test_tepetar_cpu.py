@@ -155,6 +155,14 @@ def test_decode_splits_leave_pages_for_everyone():
                 assert 1 <= s <= 16 and (s == 1 or keys // s >= 64)
 
 
+def test_memory_of_a_deployment_counts_unquantized_pages():
+    from mfq_b200.models.tepetar import TepetarConfig
+    from mfq_b200.server.analysis import model_memory
+    cfg = TepetarConfig.from_source(cases.uneven()).to_dict()
+    per_token = 2 * (4 * (48 + 32) + 2 * (32 + 32) + (80 + 64) + 2 * (32 + 32) + 2 * (16 + 32))
+    assert model_memory(cfg, 1000, batch=2, context=64)["per_gpu"]["kv_cache"] == (2 * 4 + 1) * 16 * per_token
+
+
 # -- pages ----------------------------------------------------------------------------------------------------------
 def test_unquantized_pages_move_between_caches():
     from mfq_b200.engine.kv_cache import PlainPagedKVCache
