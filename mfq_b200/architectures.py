@@ -8,7 +8,7 @@ Runtime code consumes canonical names only (``model.block.N.attention.query.weig
 * ``deepseek_v3`` / ``glm4_moe``: latent-attention and shared-expert names, sigmoid router bias, and the next-token
   prediction layer these checkpoints append after the last decoder layer (``model.layers.<L>.{enorm,hnorm,eh_proj,
   shared_head.*}``), which becomes the ``predictor.*`` head;
-* ``tepetar``: ``l<N>.{mix,mlp,side}.*`` names (``config.json`` names the design under ``architecture``).
+* ``tepetar``, ``kamedra``: ``l<N>.{mix,mlp,side}.*`` names (``config.json`` names the design under ``architecture``).
 
 :func:`detect_family` picks the family from ``config.json`` (``model_type`` / ``architectures``); :func:`to_canonical`
 renames, stacks per-expert matrices, splits fused tensors and moves the appended prediction layer.  Names match the
@@ -115,7 +115,22 @@ TEPETAR_LAYER = {
     "mlp.gate": "mlp.gate.weight", "mlp.up": "mlp.up.weight", "mlp.down": "mlp.down.weight",
     "side.gate": "token_side.gate.weight", "side.proj": "token_side.projection.weight", "side.norm": "token_side.norm.weight",
 }
-_TEPETAR_LAYER_RE = re.compile(r"^l(\d+)\.(.+)$")
+# Kamedra: the same short names; what a layer's ``mix.*`` tensors are depends on its mixer
+KAMEDRA_TOP = {"embed": "model.token_embedding.weight", "final.norm": "model.output_norm.weight"}
+KAMEDRA_LAYER = {
+    "norm1": "attention.norm.weight", "norm2": "mlp.norm.weight", "mlp.gate": "mlp.gate.weight", "mlp.up": "mlp.up.weight",
+    "mlp.down": "mlp.down.weight",
+}
+KAMEDRA_MIXER = {
+    "attention": {"q": "attention.query.weight", "k": "attention.key.weight", "v": "attention.value.weight",
+                  "o": "attention.output.weight", "lq1": "attention.lambda_q1", "lk1": "attention.lambda_k1",
+                  "lq2": "attention.lambda_q2", "lk2": "attention.lambda_k2"},
+    "gla": {"q": "linear_attention.query.weight", "k": "linear_attention.key.weight", "v": "linear_attention.value.weight",
+            "g": "linear_attention.gate.weight", "o": "linear_attention.output.weight", "norm": "linear_attention.norm.weight",
+            "a1": "linear_attention.decay_a.weight", "a2": "linear_attention.decay_b.weight",
+            "a2.b": "linear_attention.decay_b.bias"},
+}
+_OWN_LAYER_RE = re.compile(r"^l(\d+)\.(.+)$")
 FAMILY_OF_MODEL_TYPE = {
     "llama": "llama", "mistral": "llama", "qwen2": "llama", "qwen3": "llama", "mixtral": "llama", "qwen2_moe": "llama",
     "qwen3_moe": "llama", "qwen3_next": "qwen3_next", "qwen3_5": "qwen3_next", "qwen3_5_moe": "qwen3_next",
@@ -127,8 +142,9 @@ FAMILY_OF_MODEL_TYPE = {
 def detect_family(hf_config: dict | None, names=()) -> str:
     """Source naming family of a checkpoint: from ``model_type`` (or the text sub-config's), else from its tensor names."""
     cfg = hf_config or {}
-    if str(cfg.get("architecture", "")).lower() == "tepetar":
-        return "tepetar"
+    own = str(cfg.get("architecture", "")).lower()
+    if own in ("tepetar", "kamedra"):
+        return own
     for c in (cfg, cfg.get("text_config") or {}):
         fam = FAMILY_OF_MODEL_TYPE.get(str(c.get("model_type", "")).lower())
         if fam:
@@ -190,8 +206,19 @@ def tepetar_name(name: str) -> str | None:
     """Source name of a Tepetar tensor -> canonical name."""
     if name in TEPETAR_TOP:
         return TEPETAR_TOP[name]
-    m = _TEPETAR_LAYER_RE.match(name)
+    m = _OWN_LAYER_RE.match(name)
     return f"model.block.{int(m[1])}.{TEPETAR_LAYER[m[2]]}" if m and m[2] in TEPETAR_LAYER else None
+
+
+def kamedra_name(name: str, mixers: list[str]) -> str | None:
+    """Source name of a Kamedra tensor -> canonical name; ``mixers``: the kind of every layer."""
+    if name in KAMEDRA_TOP:
+        return KAMEDRA_TOP[name]
+    m = _OWN_LAYER_RE.match(name)
+    if not m or int(m[1]) >= len(mixers):
+        return None
+    known = KAMEDRA_LAYER | {"mix." + k: v for k, v in KAMEDRA_MIXER.get(mixers[int(m[1])], {}).items()}
+    return f"model.block.{int(m[1])}.{known[m[2]]}" if m[2] in known else None
 
 
 def split_fused_linear_attention(out: dict[str, np.ndarray], k_heads: int, v_heads: int, head_dim: int) -> None:
@@ -224,6 +251,9 @@ def to_canonical(hf_tensors: dict[str, np.ndarray], hf_config: dict | None = Non
     family = detect_family(hf_config, hf_tensors)
     if family == "tepetar":
         return {c: t for c, t in ((tepetar_name(n), t) for n, t in hf_tensors.items()) if c is not None}
+    if family == "kamedra":
+        mixers = [l.get("type") for l in hf_config["layers"]]
+        return {c: t for c, t in ((kamedra_name(n, mixers), t) for n, t in hf_tensors.items()) if c is not None}
     text = dict(hf_config or {})
     text.update(text.get("text_config") or {})
     nextn = None
@@ -271,9 +301,13 @@ def config_from_hf(hf: dict) -> dict:
     """``config.json`` of a Hugging Face model -> the keyword arguments of ``MoeDecoderConfig`` (and of its hybrid and
     latent-attention extensions); a multimodal wrapper's ``text_config`` is looked through.  A design with a configuration
     of its own (``family`` in the result) gives the fields of that class instead."""
-    if detect_family(hf) == "tepetar":
+    family = detect_family(hf)
+    if family == "tepetar":
         from .models.tepetar import TepetarConfig
         return TepetarConfig.from_source(hf).to_dict()
+    if family == "kamedra":
+        from .models.kamedra import KamedraConfig
+        return KamedraConfig.from_source(hf).to_dict()
     if hf.get("text_config"):
         hf = {**hf, **hf["text_config"]}
     heads = hf.get("num_attention_heads", 32)

@@ -284,7 +284,8 @@ def load_engine(path, device="cuda", *, native_4bit: bool = False, expert_slots:
         has_head = getattr(weights, "mtp", None) is not None
         num_pages = plan(budget_bytes=kv_budget_bytes, layers=model.local_layers + int(has_head), kv_heads=model.hk, head_dim=cfg.head_dim,
                          max_batch=max_batch, max_seq_len=max_seq_len,
-                         token_bytes=model.kv_token_bytes() if hasattr(model, "kv_token_bytes") else None).num_pages
+                         token_bytes=model.kv_token_bytes() if hasattr(model, "kv_token_bytes") else None,
+                         state_bytes_per_row=model.state_bytes_per_row() if hasattr(model, "state_bytes_per_row") else 0).num_pages
     engine = LLMEngine(model, max_batch=max_batch, max_seq_len=max_seq_len, device=device, num_pages=num_pages,
                        use_graphs=use_graphs and (expert_slots is None or expert_graphs),
                        mtp_draft_tokens=mtp_draft_tokens if getattr(weights, "mtp", None) is not None else 0,

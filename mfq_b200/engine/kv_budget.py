@@ -47,7 +47,7 @@ def plan(*, budget_bytes: int, layers: int, kv_heads: int, head_dim: int, max_ba
     wanted = max_batch * per_seq + 1
     state = state_bytes_per_row * max_batch
     room = budget_bytes - state
-    fit = room // pb if room > 0 else 0
+    fit = (room // pb if pb else wanted) if room > 0 else 0  # a model without pages needs their numbers only
     if fit < per_seq + 1:
         need = state + (per_seq + 1) * pb
         raise MemoryError(f"KV budget of {budget_bytes / 2**30:.2f} GiB cannot hold one sequence of {max_seq_len} tokens "

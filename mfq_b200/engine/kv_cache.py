@@ -139,7 +139,7 @@ class PlainPagedKVCache(PagedTables):
         """All layers' K and V of the given pages as one contiguous uint8 numpy array (host)."""
         idx = torch.tensor(page_ids, dtype=torch.long, device=self.block_table.device)
         parts = [t.index_select(0, idx).view(torch.uint8).reshape(-1) for l in self.pools for t in (l.k, l.v)]
-        return torch.cat(parts).cpu().numpy()
+        return torch.cat(parts or [torch.empty(0, dtype=torch.uint8)]).cpu().numpy()
 
     def import_pages(self, page_ids: list[int], blob) -> None:
         """Inverse of :meth:`export_pages` into (possibly different) physical pages."""

@@ -432,7 +432,8 @@ class LLMEngine:
         if hasattr(self.model, "decode_splits"):
             self.model.attn_splits = self.model.decode_splits(max(1, singles), max(c + m for _, c, m in portions))
         return StepBuffers(input_ids=ids, positions=positions, slots=slots, block_table=self.cache.block_table.index_select(0, row_ids.long()),
-                           seq_lens=seq_lens, cu_seqlens=starts, q_starts=q_starts, tok_seq=tok_seq, max_q=max(counts), num_decode=singles)
+                           seq_lens=seq_lens, state_slots=row_ids if self.rec_state is not None else None, cu_seqlens=starts,
+                           q_starts=q_starts, tok_seq=tok_seq, max_q=max(counts), num_decode=singles)
 
     def extend(self, portions, wanted=None) -> torch.Tensor | None:
         """Append given tokens to open rows, all in one forward: ``portions`` is a list of ``(row, token ids)`` (a row at most
@@ -463,6 +464,7 @@ class LLMEngine:
 
     def _forward_ragged(self, step: StepBuffers, logits_rows: torch.Tensor) -> torch.Tensor:
         """A batch of single tokens is a decode step; anything else runs as a ragged batch."""
+        self._bind_state()
         prefill = step.num_decode < step.seq_lens.numel()
         return self.model.forward(step, self.cache, prefill=prefill, logits_rows=logits_rows, gather_logits=False)
 
@@ -777,7 +779,7 @@ class LLMEngine:
             side.wait_stream(torch.cuda.current_stream())
             saved = (self.seq_lens.clone(), self.sampled.clone())
             saved_draft = self.draft.clone() if keep_head else None
-            saved_rec = (self.rec_state.conv.clone(), self.rec_state.state.clone()) if self.rec_state is not None else None
+            saved_rec = self.rec_state.save() if self.rec_state is not None else None
             with torch.cuda.stream(side):
                 for _ in range(2):
                     self._decode_body(b, stochastic, constrained, keep_head)
@@ -795,8 +797,7 @@ class LLMEngine:
             if saved_draft is not None:
                 self.draft.copy_(saved_draft)
             if saved_rec is not None:  # the recurrent state cannot be "rewritten later" like KV rows: put it back
-                self.rec_state.conv.copy_(saved_rec[0])
-                self.rec_state.state.copy_(saved_rec[1])
+                self.rec_state.load(saved_rec)
             self.graphs[key] = g
         g.replay()
 
@@ -930,7 +931,7 @@ class LLMEngine:
             side = torch.cuda.Stream(device=self.device)
             side.wait_stream(torch.cuda.current_stream())
             saved = [t.clone() for t in (self.seq_lens, self.sampled, self.draft, self.mtp_counters)]
-            saved_rec = (self.rec_state.conv.clone(), self.rec_state.state.clone()) if self.rec_state is not None else None
+            saved_rec = self.rec_state.save() if self.rec_state is not None else None
             with torch.cuda.stream(side):
                 for _ in range(2):
                     self._mtp_body(b, depth, nxt, stochastic)
@@ -943,8 +944,7 @@ class LLMEngine:
             for dst, src in zip((self.seq_lens, self.sampled, self.draft, self.mtp_counters), saved):
                 dst.copy_(src)
             if saved_rec is not None:
-                self.rec_state.conv.copy_(saved_rec[0])
-                self.rec_state.state.copy_(saved_rec[1])
+                self.rec_state.load(saved_rec)
             self.mtp_graphs[key] = g
         g.replay()
 

@@ -22,7 +22,7 @@ import torch
 class Snapshot:
     tokens: list[int]
     pages: np.ndarray  # export of the pages that hold `tokens` (whole pages)
-    recurrent: tuple[torch.Tensor, torch.Tensor] | None  # (conv, state) of the row, on the host
+    recurrent: tuple[torch.Tensor, ...] | None  # the row's slot of every state tensor, on the host
     nbytes: int
 
 
@@ -41,7 +41,7 @@ class SessionSnapshotCache:
         pages = engine.cache.export_pages(engine.cache.allocator.owned[seq][:n_pages])
         rec = None
         if engine.rec_state is not None:
-            rec = (engine.rec_state.conv[:, row].detach().cpu().clone(), engine.rec_state.state[:, row].detach().cpu().clone())
+            rec = engine.rec_state.export_slot(row)
         nbytes = pages.nbytes + (sum(t.numel() * t.element_size() for t in rec) if rec else 0)
         self.drop(session)
         self.entries[session] = Snapshot(list(tokens), pages, rec, nbytes)
@@ -74,8 +74,7 @@ class SessionSnapshotCache:
         n_pages = (n + ps - 1) // ps
         engine.cache.import_pages(engine.cache.allocator.owned[seq][:n_pages], snap.pages)
         if snap.recurrent is not None:
-            engine.rec_state.conv[:, row].copy_(snap.recurrent[0])
-            engine.rec_state.state[:, row].copy_(snap.recurrent[1])
+            engine.rec_state.import_slot(row, snap.recurrent)
         self.stats["restored"] += 1
         self.stats["tokens_skipped"] += n
         return n

@@ -25,6 +25,7 @@ import numpy as np
 import torch
 
 from .. import ops
+from ..engine.recurrent_state import RecurrentState
 from ..ops import gdn
 from ..ops import reference as ref
 from ..utils.profiler import scope
@@ -87,8 +88,10 @@ class HybridLayer(MoeLayer):
     gated: bool = False  # qkv rows are followed by the output-gate projection
 
 
-class GdnState:
+class GdnState(RecurrentState):
     """Recurrent state of the linear-attention layers for ``slots`` sequences (slot = engine batch row)."""
+
+    slot_dim = 1
 
     def __init__(self, cfg: HybridConfig, slots: int, device, tp: int = 1) -> None:
         hv, d = cfg.linear_v_heads // tp, cfg.linear_head_dim
@@ -97,12 +100,8 @@ class GdnState:
         self.index = {i: j for j, i in enumerate(i for i in range(cfg.num_layers) if cfg.is_linear(i))}
         self.conv = torch.zeros((n, slots, 3, c), dtype=torch.float32, device=device)
         self.state = torch.zeros((n, slots, hv, d, d), dtype=torch.float32, device=device)
-
+        super().__init__([self.conv, self.state])
         self._ckpt: dict[tuple[int, int], tuple[torch.Tensor, torch.Tensor]] = {}
-
-    def reset(self, slot: int) -> None:
-        self.conv[:, slot].zero_()
-        self.state[:, slot].zero_()
 
     def checkpoints(self, rows: int, window: int):
         """Per-layer verify-window checkpoints ``(conv [n, rows, L, 3, C], state [n, rows, L, Hv, d, d])`` (allocated once

@@ -48,15 +48,19 @@ class Family:
             raise UnsupportedDtype(f"models of the {self.name} family do not run in {dtype} (available: {', '.join(self.dtypes)})")
 
 
-def _build_tepetar(raw: dict, store, o: LoadOptions):
-    from .tepetar import TepetarConfig, TepetarModel, TepetarWeights
-    if o.tp_size != 1 or o.lp_size != 1:
-        raise NotImplementedError("Tepetar checkpoints load on a single rank")
-    if raw.get("rope_scaling"):
-        raise ValueError("this family has no rotary context extension")
-    cfg = TepetarConfig.from_dict(raw)
-    weights = TepetarWeights(cfg, store, o.device, DTYPES["bfloat16" if o.dtype == "auto" else o.dtype])
-    return cfg, weights, TepetarModel(cfg, weights, collective=o.collective)
+def _unquantized(name: str, config: str, weights: str, model: str):
+    """Builder of a family of the unquantized path, from the classes in ``models/<name>.py``."""
+    def build(raw: dict, store, o: LoadOptions):
+        from importlib import import_module
+        module = import_module(f"{__package__}.{name}")
+        if o.tp_size != 1 or o.lp_size != 1:
+            raise NotImplementedError(f"{name} checkpoints load on a single rank")
+        if raw.get("rope_scaling"):
+            raise ValueError("this family has no rotary context extension")
+        cfg = getattr(module, config).from_dict(raw)
+        w = getattr(module, weights)(cfg, store, o.device, DTYPES["bfloat16" if o.dtype == "auto" else o.dtype])
+        return cfg, w, getattr(module, model)(cfg, w, collective=o.collective)
+    return Family(name, lambda raw: raw.get("family") == name, build, ("auto", "bfloat16", "float32"), ("dense",))
 
 
 def _build_mla(raw: dict, store, o: LoadOptions):
@@ -77,7 +81,8 @@ def _build_moe_decoder(raw: dict, store, o: LoadOptions):
 
 
 FAMILIES = (
-    Family("tepetar", lambda raw: raw.get("family") == "tepetar", _build_tepetar, ("auto", "bfloat16", "float32"), ("dense",)),
+    _unquantized("tepetar", "TepetarConfig", "TepetarWeights", "TepetarModel"),
+    _unquantized("kamedra", "KamedraConfig", "KamedraWeights", "KamedraModel"),
     Family("latent attention", lambda raw: bool(raw.get("kv_lora_rank")), _build_mla),
     Family("decoder", lambda raw: True, _build_moe_decoder),  # dense and mixture-of-experts decoders
 )

@@ -21,11 +21,12 @@ from dataclasses import asdict, dataclass, field
 
 import torch
 
-from ..engine.kv_cache import PlainPagedKVCache
 from ..ops import dense, window_attn
 from ..ops.dense import DenseLinear, up
 from ..utils.profiler import scope
-from .llama import LlamaModel, StepBuffers
+from . import unquantized
+from .llama import StepBuffers
+from .unquantized import TensorReader, UnquantizedModel, fit
 
 GLU_ALPHA = 1.702
 
@@ -131,6 +132,13 @@ class TepetarConfig:
         """Per layer: (KV heads, stored key width, stored value width)."""
         return [(l.kv_heads, up(l.dim), up(l.vdim)) for l in self.layers]
 
+    def rotations(self) -> set[tuple[float, int]]:
+        return {(l.rot_base, l.rot_dims) for l in self.layers}
+
+    def key_spans(self) -> list[tuple[int, int, int]]:
+        """Per layer: (KV heads, window, kept first keys)."""
+        return [(l.kv_heads, l.window, 0) for l in self.layers]
+
     def kv_token_bytes(self, element_bytes: int) -> int:
         return sum(g * (dk + dv) for g, dk, dv in self.kv_shapes()) * element_bytes
 
@@ -159,15 +167,6 @@ class TepetarLayer:
     side_norm: torch.Tensor | None
 
 
-def _fit(t: torch.Tensor, *shape: int) -> torch.Tensor:
-    """``t`` in the leading corner of a zero tensor of ``shape``."""
-    if tuple(t.shape) == shape:
-        return t
-    out = torch.zeros(shape, dtype=t.dtype, device=t.device)
-    out[tuple(slice(0, n) for n in t.shape)] = t
-    return out
-
-
 class TepetarWeights:
     """Weights in the layout the kernels read (widths rounded up, padding zero), on one device in one element type."""
 
@@ -175,24 +174,11 @@ class TepetarWeights:
 
     def __init__(self, cfg: TepetarConfig, tensors, device, dtype: torch.dtype = torch.bfloat16) -> None:
         """``tensors``: canonical name -> checkpoint tensor (anything ``formats.dequantize`` reads, or a torch tensor)."""
-        from .moe_decoder import _to_float
-        dense.is_fp32(dtype)
+        r = TensorReader(tensors, device, dtype)
         self.dtype = dtype
-        dev = torch.device(device)
         w = up(cfg.hidden_size)
-
-        def get(name: str) -> torch.Tensor:
-            t = tensors[name]
-            return t.to(dev) if isinstance(t, torch.Tensor) else _to_float(t, dev)
-
-        def vec(name: str, n: int, offset: float = 0.0) -> torch.Tensor:
-            return _fit(get(name).float().reshape(-1) + offset, n).contiguous()
-
-        def linear(name: str, rows: int, cols: int, bias: bool = False, **kw) -> DenseLinear:
-            t = _fit(get(name + ".weight").to(dtype), rows, cols).contiguous()
-            return DenseLinear(t, vec(name + ".bias", rows) if bias else None, **kw)
-
-        self.embed = _fit(get("model.token_embedding.weight").to(dtype), cfg.vocab_size, w).contiguous()
+        get, vec, linear = r.get, r.vec, r.linear
+        self.embed = r.matrix("model.token_embedding.weight", cfg.vocab_size, w)
         self.lm_head = linear("model.output", up(cfg.vocab_size), w)
         self.final_norm = vec("model.output_norm.weight", w, 1.0)
         side, sp = cfg.side_dim, up(cfg.side_dim)
@@ -203,21 +189,19 @@ class TepetarWeights:
             dk, dv = up(l.dim), up(l.vdim)
             parts, biases = [], []
             for name, heads, d, dp in (("query", l.heads, l.dim, dk), ("key", l.kv_heads, l.dim, dk), ("value", l.kv_heads, l.vdim, dv)):
-                t = get(p + f"attention.{name}.weight").to(dtype).reshape(heads, d, cfg.hidden_size)
-                parts.append(_fit(t, heads, dp, w).reshape(heads * dp, w))
-                biases.append(_fit(get(p + f"attention.{name}.bias").float().reshape(heads, d), heads, dp).reshape(-1))
-            out = get(p + "attention.output.weight").to(dtype).reshape(cfg.hidden_size, l.heads, l.vdim)
-            o_proj = DenseLinear(_fit(out, w, l.heads, dv).reshape(w, l.heads * dv).contiguous(), vec(p + "attention.output.bias", w))
+                parts.append(r.heads(p + f"attention.{name}.weight", heads, d, dp, cfg.hidden_size, w).reshape(heads * dp, w))
+                biases.append(fit(get(p + f"attention.{name}.bias").float().reshape(heads, d), heads, dp).reshape(-1))
+            o_proj = DenseLinear(r.from_heads(p + "attention.output.weight", cfg.hidden_size, w, l.heads, l.vdim, dv),
+                                 vec(p + "attention.output.bias", w))
             gate_up = down = mlp_norm = None
             if l.ff:
                 fp = up(l.ff, 8)
-                gate, up_ = (_fit(get(p + f"mlp.{n}.weight").to(dtype), fp, w) for n in ("gate", "up"))
-                gate_up = DenseLinear(dense.interleave_glu(gate, up_), glu=(GLU_ALPHA, l.limit))
+                gate_up = r.glu(p + "mlp.", fp, w, (GLU_ALPHA, l.limit))
                 down, mlp_norm = linear(p + "mlp.down", w, fp), vec(p + "mlp.post_norm.weight", w, 1.0)
             side_w = [None] * 4
             if side:
                 side_w = [linear(p + "token_side.gate", sp, w),
-                          _fit(table[:, i * side : (i + 1) * side].to(dtype), cfg.vocab_size, sp).contiguous(),
+                          fit(table[:, i * side : (i + 1) * side].to(dtype), cfg.vocab_size, sp).contiguous(),
                           linear(p + "token_side.projection", w, sp), vec(p + "token_side.norm.weight", w)]
             self.layers.append(TepetarLayer(
                 DenseLinear(torch.cat(parts).contiguous(), torch.cat(biases).contiguous()), vec(p + "attention.query_norm.weight", dk),
@@ -253,67 +237,25 @@ def tensor_shapes(cfg: TepetarConfig) -> dict[str, tuple[int, ...]]:
     return out
 
 
-class RandomTensors:
-    """Seeded N(0, std) tensors of a configuration, drawn when they are asked for (no second copy of a large model)."""
+class RandomTensors(unquantized.RandomTensors):
+    """Seeded random tensors of a configuration."""
 
     def __init__(self, cfg: TepetarConfig, device, seed: int = 0, std: float = 0.02) -> None:
-        self.shapes, self.device, self.std = tensor_shapes(cfg), torch.device(device), std
-        self.gen = torch.Generator(device=self.device).manual_seed(seed)
-
-    def __getitem__(self, name: str) -> torch.Tensor:
-        t = torch.randn(self.shapes[name], generator=self.gen, device=self.device, dtype=torch.float32)
-        if name.endswith(("query_norm.weight", "key_norm.weight", "token_side.norm.weight")):
-            return 1 + 0.1 * t
-        return (t * self.std).to(torch.bfloat16)
+        super().__init__(tensor_shapes(cfg), device, seed, std, ("query_norm.weight", "key_norm.weight", "token_side.norm.weight"))
 
 
-class TepetarModel(LlamaModel):
-    """Stateless forward over :class:`TepetarWeights`; keys and values live in a :class:`PlainPagedKVCache`."""
-
-    ragged = True
-
+class TepetarModel(UnquantizedModel):
     def __init__(self, cfg: TepetarConfig, weights: TepetarWeights, collective=None) -> None:
-        if collective is not None:
-            raise NotImplementedError("this family runs on a single rank")
-        if weights.embed.device.type != "cuda":
-            raise RuntimeError("this family runs on a CUDA device only")
-        self.cfg, self.w, self.tp, self.collective = cfg, weights, 1, None
-        self.hq, self.hk = cfg.num_heads, cfg.num_kv_heads
-        self.attn_splits = 1
+        super().__init__(cfg, weights, collective)
         mixed = [i for i, l in enumerate(cfg.layers) if l.v_mix]
         self.first_mixed = mixed[0] if mixed else -1
-        self._rope: dict[tuple[float, int], torch.Tensor] = {}
-        self._rows: torch.Tensor | None = None
-
-    # -- cache ------------------------------------------------------------------------------------------------------
-    def kv_token_bytes(self) -> int:
-        return self.cfg.kv_token_bytes(self.w.embed.element_size())
-
-    def make_cache(self, *, num_pages: int, max_seqs: int, max_pages_per_seq: int, device) -> PlainPagedKVCache:
-        cache = PlainPagedKVCache(self.cfg.kv_shapes(), self.w.dtype, num_pages=num_pages, max_seqs=max_seqs,
-                                  max_pages_per_seq=max_pages_per_seq, device=device)
-        n = max_pages_per_seq * cache.page_size  # positions an engine with this cache can reach
-        for l in self.cfg.layers:
-            key = (l.rot_base, l.rot_dims)
-            if l.rot_dims and (key not in self._rope or self._rope[key].shape[0] < n):
-                self._rope[key] = window_attn.rope_table(*key, n, self.w.embed.device)
-        return cache
-
-    def decode_splits(self, batch: int, longest: int) -> int:
-        """Upper bound of the KV splits of a decode step at the current contexts (every layer caps it by its window)."""
-        return max(window_attn.decode_splits(batch, l.kv_heads, min(longest, l.window)) for l in self.cfg.layers)
 
     # -- forward ----------------------------------------------------------------------------------------------------
     def _attend(self, q, kv, l: LayerSpec, step: StepBuffers, prefill: bool):
         t = q.shape[0]
         how = dict(window=l.window, scale=l.scale, cap=l.softcap)
         if q.dtype == torch.float32:
-            seq = step.tok_seq
-            if seq is None:  # a decode step: one row per sequence
-                if self._rows is None or self._rows.numel() < t:
-                    self._rows = torch.arange(max(t, 256), dtype=torch.int32, device=q.device)
-                seq = self._rows[:t]
-            return window_attn.plain(q, kv, step.block_table, seq, step.positions, **how)
+            return window_attn.plain(q, kv, step.block_table, self._sequence_of_rows(step, t), step.positions, **how)
         singles = step.num_decode if prefill else t
         out = torch.empty((t, l.heads, kv.v.shape[-1]), dtype=q.dtype, device=q.device)
         if singles:

@@ -23,7 +23,7 @@ HERE = Path(__file__).resolve().parent
 CSRC = HERE / "csrc"
 LIB_PATH = HERE / "_mfq_b200_kernels.so"
 DENSE_LIB_PATH = HERE / "_mfq_b200_dense.so"
-DENSE_SOURCES = ("dense_gemm.cu", "stream_ops.cu", "window_attn.cu", "window_attn_prefill.cu")
+DENSE_SOURCES = ("dense_gemm.cu", "stream_ops.cu", "window_attn.cu", "window_attn_prefill.cu", "gla.cu", "gla_chunk.cu")
 OBJ_DIR = HERE / "build"
 
 NVCC_FLAGS = [

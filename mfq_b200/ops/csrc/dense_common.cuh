@@ -63,12 +63,16 @@ enum : int {
   kDenseBias = 0,   // out[t, n] = v + bias[n]
   kDenseGlu = 1,    // weight rows packed in blocks of 16 = 8 gate rows | 8 up rows: out = clipped GLU, half as wide
   kDenseGelu = 2,   // out[t, n] = gelu_tanh(v + bias[n]) * table[ids[t], n]
+  kDenseGeluGlu = 3,  // rows packed as for kDenseGlu: out = gelu_tanh(gate) * up, half as wide
+  kDenseSoftcap = 4,  // out[t, n] = limit * tanh((v + bias[n]) / limit)
+  kDenseAdd = 5,      // x[t, n] += v + bias[n] on the fp32 stream x = out
 };
+__host__ __device__ constexpr bool dense_is_glu(int kind) { return kind == kDenseGlu || kind == kDenseGeluGlu; }
 
 struct DenseEpilogue {
   int kind;
   const float* bias;  // [N] or null
-  float alpha, limit;  // GLU: y = g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit)
+  float alpha, limit;  // GLU: y = g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit); soft cap: limit
   const void* table;   // GELU: [tokens of the vocabulary, N] in the activation type
   const int* ids;
   void* out;
@@ -83,8 +87,8 @@ __device__ __forceinline__ float gelu_tanh(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
-// One output item of token `t`: 8 packed rows from `n0` (kDenseBias, kDenseGelu) or 16 (kDenseGlu).  `load(n, v)` fetches
-// the finished fp32 sums of rows n .. n + 7.
+// One output item of token `t`: 8 packed rows from `n0`, or 16 for the GLU kinds.  `load(n, v)` fetches the finished fp32 sums
+// of rows n .. n + 7.
 template <typename T, typename Load>
 __device__ __forceinline__ void dense_store_item(const DenseEpilogue& e, int t, int n0, Load&& load) {
   float v[8];
@@ -95,8 +99,17 @@ __device__ __forceinline__ void dense_store_item(const DenseEpilogue& e, int t, 
 #pragma unroll
     for (int i = 0; i < 8; ++i) v[i] += b[i];
   }
+  if (e.kind == kDenseAdd) {
+    float* x = static_cast<float*>(e.out) + size_t(t) * e.ldo + n0;
+    float r[8];
+    load8<float>(x, r);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) r[i] += v[i];
+    store8<float>(x, r);
+    return;
+  }
   T* out = static_cast<T*>(e.out) + size_t(t) * e.ldo;
-  if (e.kind == kDenseGlu) {
+  if (dense_is_glu(e.kind)) {
     float u[8];
     load(n0 + 8, u);
     if (e.bias) {
@@ -106,7 +119,7 @@ __device__ __forceinline__ void dense_store_item(const DenseEpilogue& e, int t, 
       for (int i = 0; i < 8; ++i) u[i] += b[i];
     }
 #pragma unroll
-    for (int i = 0; i < 8; ++i) v[i] = clipped_glu(v[i], u[i], e.alpha, e.limit);
+    for (int i = 0; i < 8; ++i) v[i] = e.kind == kDenseGlu ? clipped_glu(v[i], u[i], e.alpha, e.limit) : gelu_tanh(v[i]) * u[i];
     store8<T>(out + (n0 >> 1), v);
     return;
   }
@@ -115,6 +128,10 @@ __device__ __forceinline__ void dense_store_item(const DenseEpilogue& e, int t, 
     load8<T>(static_cast<const T*>(e.table) + size_t(e.ids[t]) * e.ldo + n0, g);
 #pragma unroll
     for (int i = 0; i < 8; ++i) v[i] = gelu_tanh(v[i]) * g[i];
+  }
+  if (e.kind == kDenseSoftcap) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = e.limit * tanhf(v[i] / e.limit);
   }
   store8<T>(out + n0, v);
 }

@@ -12,8 +12,8 @@
 //                       two m16n8k16 MMAs, the activation fragment uses the same K assignment, so the product is exact.
 //   dense_sgemm_kernel  fp32 operands on the FMA units (64 x 64 tiles): the full-precision mode of a model.
 //
-// The output stage (bias, clipped GLU over interleaved gate / up rows, GELU times a per-token table row) is shared by the
-// three kernels (dense_common.cuh).  Waits are bounded as everywhere (common.cuh).
+// The output stage (bias, a gated unit over interleaved gate / up rows, GELU times a per-token table row, soft cap, addition to
+// the fp32 stream) is shared by the three kernels (dense_common.cuh).  Waits are bounded as everywhere (common.cuh).
 #include "dense_common.cuh"
 
 namespace mfq {
@@ -147,7 +147,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_const
   const int tl = min(BT, p.M - t0), nl = min(kDnTileN, p.N - n0);
   const bool all_ok = splits > 1 || *abort_flag == 0;
   if (all_ok) {
-    const int width = p.epi.kind == kDenseGlu ? 16 : 8;  // N is a multiple of 16
+    const int width = dense_is_glu(p.epi.kind) ? 16 : 8;  // N is a multiple of 16
     const int per = nl / width, items = tl * per;
     const uint32_t tile_addr = smem_u32(tile);
     for (int i = blockIdx.z * kDnThreads + threadIdx.x; i < items; i += splits * kDnThreads) {
@@ -257,7 +257,7 @@ dense_gemv_kernel(const __nv_bfloat16* __restrict__ w, const __nv_bfloat16* __re
     red[warp][g + 8][c + 1] = acc[nt][3];
   }
   __syncthreads();
-  const int width = p.epi.kind == kDenseGlu ? 16 : 8, per = 16 / width;
+  const int width = dense_is_glu(p.epi.kind) ? 16 : 8, per = 16 / width;
   for (int i = threadIdx.x; i < p.M * per; i += 256) {
     const int t = i / per, n = (i - t * per) * width;
     dense_store_item<__nv_bfloat16>(p.epi, t, n0 + n, [&](int row, float(&v)[8]) {
@@ -325,7 +325,7 @@ dense_sgemm_kernel(const float* __restrict__ w, const float* __restrict__ x, int
     for (int j = 0; j < 4; ++j) tile[tt + i][tn + j] = acc[i][j];
   __syncthreads();
   const int tl = min(64, p.M - t0), nl = min(64, p.N - n0);
-  const int width = p.epi.kind == kDenseGlu ? 16 : 8, per = nl / width;
+  const int width = dense_is_glu(p.epi.kind) ? 16 : 8, per = nl / width;
   for (int i = tid; i < tl * per; i += 256) {
     const int t = i / per, n = (i - t * per) * width;
     dense_store_item<float>(p.epi, t0 + t, n0 + n, [&](int row, float(&v)[8]) { load8<float>(&tile[t][row - n0], v); });
@@ -341,8 +341,9 @@ extern "C" int mfq_dense_linear(const void* w, const void* x, int ldx, void* out
                                 int splits, int fp32, int* status, cudaStream_t stream) {
   using namespace mfq;
   if (M <= 0 || N <= 0 || K <= 0 || N % 16 || K % 8 || ldx % 8 || ldx < K || ldo % 8) return -1;
-  if (epilogue < kDenseBias || epilogue > kDenseGelu || (epilogue == kDenseGelu && (!table || !ids))) return -1;
-  if (ldo < (epilogue == kDenseGlu ? N / 2 : N)) return -1;
+  if (epilogue < kDenseBias || epilogue > kDenseAdd || (epilogue == kDenseGelu && (!table || !ids))) return -1;
+  if (epilogue == kDenseSoftcap && !(limit > 0.f)) return -1;
+  if (ldo < (dense_is_glu(epilogue) ? N / 2 : N)) return -1;
   const DenseParams p{DenseEpilogue{epilogue, bias, alpha, limit, table, ids, out, ldo}, status, M, N, K, 0};
   if (fp32) {
     launch_kernel(dense_sgemm_kernel, dim3((N + 63) / 64, (M + 63) / 64), dim3(256), 0, stream, static_cast<const float*>(w),

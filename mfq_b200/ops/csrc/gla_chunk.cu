@@ -1,0 +1,555 @@
+// Gated linear attention over prompt portions in 64-token chunks, bf16 (see gla.cuh for the recurrence).
+//
+// With b_t the running sum of g inside a chunk, S_0 the state before it and C its length,
+//     o_t = (2^b_t q_t)^T S_0 + sum_{s <= t} A_ts v_s,       A_ts = sum_c q_tc k_sc 2^(b_tc - b_sc)
+//     S_C = diag(2^b_C) S_0 + U,                             U    = sum_s (2^(b_C - b_s) k_s) v_s^T
+// so all that is sequential is one multiply-add per state element and chunk.  Three kernels:
+//
+//   gla_chunk_local    a CTA per (chunk, head): decays and their running sum b, and U
+//   gla_chunk_state    a thread per eight state elements: replaces every U by the S_0 of its chunk, advances the state
+//   gla_chunk_output   a CTA per (chunk, head): A, then O = A V + (2^b q)^T S_0, per-head norm and gate
+//
+// Exponents never overflow: A is formed in 16 x 16 blocks relative to b before the block's first row, where both factors are at
+// most 1 below the diagonal; a diagonal block whose own decay spans more than 2^-100 is summed term by term instead.
+// Precision: the recurrence is kept to fp32 level on bf16 tensor cores by splitting every fp32 operand into two bf16 numbers
+// (16 significant bits): 2^(b_C - b) k, 2^b q, the factors of A, A itself and S_0; v is bf16 as projected.  The 16-row
+// products here are too small for 128-row tcgen05 tiles, and their operands are made in registers, so they run as mma.sync.
+#include "gla.cuh"
+
+namespace mfq {
+namespace {
+
+constexpr int kGc = 64, kGcThreads = 256, kGcMaxDk = 256, kGcMaxDv = 512;
+constexpr float kGcSpan = 100.f;
+
+struct GlaChunkParams {
+  GlaShape s;
+  const __nv_bfloat16* proj;  // [T, row_stride]
+  const __nv_bfloat16* w2;    // [H dk, rank]
+  const float* bias;          // [H dk]
+  const float* norm_w;        // [dv]
+  __nv_bfloat16* y;           // [T, H dv]
+  const int* starts;          // [B + 1] first token of every portion
+  const int* slot;            // [B]
+  float* state;               // [slots, H, dk, dv]
+  float* cum;                 // [T, H dk]           b
+  float* u;                   // [chunks, H, dk, dv] U, then S_0 as [hi x 8 | lo x 8] bf16 per eight elements
+  float* gam;                 // [chunks, H, dk]     2^b_C
+};
+
+__device__ __forceinline__ float gc_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void gc_cp16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void gc_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void gc_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+__device__ __forceinline__ void gc_ldm(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void gc_ldm_t(uint32_t addr, uint32_t (&r)[4]) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ void gc_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// (x, y) as a pair of bf16 numbers and the pair of what they leave
+__device__ __forceinline__ void gc_split(float x, float y, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(x - __low2float(h), y - __high2float(h));
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+__device__ __forceinline__ float2 gc_pair(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+
+// A CTA's chunk: tokens t0 .. t0 + n - 1; `index` numbers the chunks of all portions without overlap.
+struct GlaChunkAt {
+  int t0, n;
+  size_t index;
+};
+__device__ __forceinline__ bool gc_locate(const GlaChunkParams& p, int chunk, int b, GlaChunkAt& at) {
+  const int r0 = p.starts[b], len = p.starts[b + 1] - r0;
+  at.t0 = r0 + chunk * kGc;
+  at.n = min(kGc, len - chunk * kGc);
+  at.index = size_t((r0 - p.starts[0]) / kGc + b + chunk);
+  return at.n > 0 && p.slot[b] >= 0;
+}
+
+__host__ __device__ constexpr int gc_groups(int dk) { return dk <= 32 ? 8 : dk <= 64 ? 4 : dk <= 128 ? 2 : 1; }
+
+struct GlaLocalSmem {
+  int b, k, v, tot, bytes;
+};
+__host__ __device__ inline GlaLocalSmem gc_local_smem(int dk, int dv, int rank) {
+  GlaLocalSmem m{};
+  m.b = 0;                                                   // [64][dk + 8] fp32
+  m.k = m.b + kGc * (dk + 8) * 4;                            // hi, lo [64][dk + 8] bf16; before that a^T [rank][68] fp32
+  const int kbytes = 2 * kGc * (dk + 8) * 2, abytes = rank * 68 * 4;
+  m.v = m.k + (kbytes > abytes ? kbytes : abytes);           // [64][dv + 8] bf16
+  m.tot = m.v + kGc * (dv + 8) * 2;                          // [256] fp32
+  m.bytes = m.tot + 1024;
+  return m;
+}
+
+__global__ void __launch_bounds__(kGcThreads)
+gla_chunk_local_kernel(const GlaChunkParams p) {
+  pdl_trigger();
+  extern __shared__ __align__(16) uint8_t gc_sm[];
+  pdl_wait();
+  GlaChunkAt at;
+  if (!gc_locate(p, blockIdx.x, blockIdx.z, at)) return;
+  const int h = blockIdx.y, H = p.s.H, dk = p.s.dk, dv = p.s.dv, rank = p.s.rank;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const GlaLocalSmem m = gc_local_smem(dk, dv, rank);
+  float* b_s = reinterpret_cast<float*>(gc_sm + m.b);
+  float* a_s = reinterpret_cast<float*>(gc_sm + m.k);
+  __nv_bfloat16* k_hi = reinterpret_cast<__nv_bfloat16*>(gc_sm + m.k);
+  __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(gc_sm + m.v);
+  float* tot = reinterpret_cast<float*>(gc_sm + m.tot);
+  const int bp = dk + 8, kp = dk + 8, vp = dv + 8;
+  __nv_bfloat16* k_lo = k_hi + kGc * kp;
+  const __nv_bfloat16* rows = p.proj + size_t(at.t0) * p.s.row_stride;
+  {
+    const __nv_bfloat16* v = rows + 2 * H * dk + h * dv;
+    const int per = dv / 8;
+    for (int i = tid; i < kGc * per; i += kGcThreads) {
+      const int t = i / per, c = (i - t * per) * 8;
+      if (t < at.n) gc_cp16(v_s + t * vp + c, v + size_t(t) * p.s.row_stride + c);
+      else *reinterpret_cast<uint4*>(v_s + t * vp + c) = make_uint4(0, 0, 0, 0);
+    }
+    gc_commit();
+    const __nv_bfloat16* a = rows + 2 * H * (dk + dv);
+    const int aper = rank / 8;
+    for (int i = tid; i < kGc * aper; i += kGcThreads) {
+      const int t = i / aper, r = (i - t * aper) * 8;
+      float x[8] = {};
+      if (t < at.n) load8<__nv_bfloat16>(a + size_t(t) * p.s.row_stride + r, x);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) a_s[(r + j) * 68 + t] = x[j];
+    }
+  }
+  __syncthreads();
+  // ----- decays: a thread takes one key channel of 64 / TG tokens -----
+  const int TG = gc_groups(dk), len = kGc / TG, c = tid % dk, tg = tid / dk;
+  const bool live = tg < TG;
+  if (live) {
+    const __nv_bfloat16* w = p.w2 + size_t(h * dk + c) * rank;
+    const float bias = p.bias[h * dk + c];
+    float run = 0.f;
+    for (int t = tg * len; t < tg * len + len; t += 8) {
+      float z[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) z[j] = bias;
+      for (int r = 0; r < rank; r += 8) {
+        float x[8];
+        load8<__nv_bfloat16>(w + r, x);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const float4 lo = *reinterpret_cast<const float4*>(a_s + (r + e) * 68 + t), hi = *reinterpret_cast<const float4*>(a_s + (r + e) * 68 + t + 4);
+          z[0] = fmaf(x[e], lo.x, z[0]); z[1] = fmaf(x[e], lo.y, z[1]); z[2] = fmaf(x[e], lo.z, z[2]); z[3] = fmaf(x[e], lo.w, z[3]);
+          z[4] = fmaf(x[e], hi.x, z[4]); z[5] = fmaf(x[e], hi.y, z[5]); z[6] = fmaf(x[e], hi.z, z[6]); z[7] = fmaf(x[e], hi.w, z[7]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        run += t + j < at.n ? log2_sigmoid(z[j]) * p.s.inv_tau : 0.f;
+        b_s[(t + j) * bp + c] = run;
+      }
+    }
+    tot[tg * dk + c] = run;
+  }
+  __syncthreads();
+  if (live) {
+    float off = 0.f;
+    for (int g = 0; g < tg; ++g) off += tot[g * dk + c];
+    for (int t = tg * len; t < tg * len + len; ++t) {
+      const float b = b_s[t * bp + c] + off;
+      b_s[t * bp + c] = b;
+      if (t < at.n) p.cum[size_t(at.t0 + t) * (H * dk) + h * dk + c] = b;
+    }
+    if (tg == TG - 1) p.gam[(at.index * H + h) * dk + c] = exp2f(b_s[(kGc - 1) * bp + c]);
+  }
+  __syncthreads();
+  {
+    const __nv_bfloat16* k = rows + (H + h) * dk;
+    const int per = dk / 2;
+    for (int i = tid; i < kGc * per; i += kGcThreads) {
+      const int t = i / per, ch = (i - t * per) * 2;
+      float2 x = make_float2(0.f, 0.f);
+      if (t < at.n) {
+        x = gc_pair(k + size_t(t) * p.s.row_stride + ch);
+        const float2 b = *reinterpret_cast<const float2*>(b_s + t * bp + ch), e = *reinterpret_cast<const float2*>(b_s + (kGc - 1) * bp + ch);
+        x.x *= gc_exp2(e.x - b.x);
+        x.y *= gc_exp2(e.y - b.y);
+      }
+      gc_split(x.x, x.y, *reinterpret_cast<uint32_t*>(k_hi + t * kp + ch), *reinterpret_cast<uint32_t*>(k_lo + t * kp + ch));
+    }
+  }
+  gc_wait<0>();
+  __syncthreads();
+  // ----- U = (2^(b_C - b) k)^T V: jobs of 16 rows x 64 columns -----
+  float* u = p.u + (at.index * H + h) * size_t(dk) * dv;
+  const int mat = lane >> 3, mrow = lane & 7, g = lane >> 2, t4 = lane & 3;
+  const int nbs = (dv + 63) / 64;
+  const int steps = (at.n + 15) / 16;
+  for (int job = warp; job < (dk / 16) * nbs; job += kGcThreads / 32) {
+    const int m0 = job / nbs * 16, n0 = (job % nbs) * 64, tiles = min(8, (dv - n0) / 8);
+    float acc[8][4] = {};
+    for (int ks = 0; ks < steps; ++ks) {
+      uint32_t hi[4], lo[4];
+      const int off = (ks * 16 + (mat >> 1) * 8 + mrow) * kp + m0 + (mat & 1) * 8;
+      gc_ldm_t(smem_u32(k_hi + off), hi);
+      gc_ldm_t(smem_u32(k_lo + off), lo);
+#pragma unroll
+      for (int nt = 0; nt < 8; nt += 2) {
+        if (nt < tiles) {  // tiles is even: dv is a multiple of 16
+          uint32_t v[4];
+          gc_ldm_t(smem_u32(v_s + (ks * 16 + (mat & 1) * 8 + mrow) * vp + n0 + nt * 8 + (mat >> 1) * 8), v);
+          gc_mma(acc[nt], hi, v[0], v[1]);
+          gc_mma(acc[nt], lo, v[0], v[1]);
+          gc_mma(acc[nt + 1], hi, v[2], v[3]);
+          gc_mma(acc[nt + 1], lo, v[2], v[3]);
+        }
+      }
+    }
+#pragma unroll
+    for (int nt = 0; nt < 8; ++nt) {
+      if (nt < tiles) {
+        float* d = u + size_t(m0 + g) * dv + n0 + nt * 8 + t4 * 2;
+        *reinterpret_cast<float2*>(d) = make_float2(acc[nt][0], acc[nt][1]);
+        *reinterpret_cast<float2*>(d + size_t(8) * dv) = make_float2(acc[nt][2], acc[nt][3]);
+      }
+    }
+  }
+}
+
+__global__ void __launch_bounds__(128)
+gla_chunk_state_kernel(const GlaChunkParams p) {
+  pdl_trigger();
+  pdl_wait();
+  const int h = blockIdx.y, b = blockIdx.z, H = p.s.H, dk = p.s.dk, dv = p.s.dv;
+  const int slot = p.slot[b], r0 = p.starts[b], len = p.starts[b + 1] - r0;
+  const int e = (blockIdx.x * 128 + threadIdx.x) * 8;
+  if (slot < 0 || e >= dk * dv) return;
+  const int chunks = (len + kGc - 1) / kGc, row = e / dv;
+  const size_t first = size_t((r0 - p.starts[0]) / kGc + b), step = size_t(H) * dk * dv;
+  float* u = p.u + (first * H + h) * size_t(dk) * dv + e;
+  const float* gam = p.gam + (first * H + h) * dk + row;
+  float* st = p.state + (size_t(slot) * H + h) * dk * dv + e;
+  float s[8];
+  load8<float>(st, s);
+  constexpr int kAhead = 4;
+  for (int c0 = 0; c0 < chunks; c0 += kAhead) {
+    float x[kAhead][8], gm[kAhead];
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i)
+      if (c0 + i < chunks) {
+        load8<float>(u + (c0 + i) * step, x[i]);
+        gm[i] = gam[size_t(c0 + i) * H * dk];
+      }
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i)
+      if (c0 + i < chunks) {
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) gc_split(s[2 * j], s[2 * j + 1], hi[j], lo[j]);
+        uint4* d = reinterpret_cast<uint4*>(u + (c0 + i) * step);
+        d[0] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        d[1] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) s[j] = fmaf(gm[i], s[j], x[i][j]);
+      }
+  }
+  store8<float>(st, s);
+}
+
+struct GlaOutputSmem {
+  int b, q, a, v, ss, bytes;
+};
+__host__ __device__ inline GlaOutputSmem gc_output_smem(int dk, int dv) {
+  GlaOutputSmem m{};
+  m.b = 0;                                             // b [64][dk + 8] fp32, then two stages of S_0: [16][dv * 4 + 16 bytes]
+  const int bb = kGc * (dk + 8) * 4, sb = 2 * 16 * (dv * 4 + 16);
+  m.q = m.b + (bb > sb ? bb : sb);                     // q, k [64][dk + 8] bf16, then hi, lo of 2^b q
+  m.a = m.q + 2 * kGc * (dk + 8) * 2;                  // A hi, lo [64][72] bf16
+  m.v = m.a + 2 * kGc * 72 * 2;                        // [64][dv + 8] bf16
+  m.ss = m.v + kGc * (dv + 8) * 2;                     // [2][64] fp32
+  m.bytes = m.ss + 512;
+  return m;
+}
+
+// NT: upper bound of the 8-column tiles of a warp (dv / 16)
+template <int NT>
+__global__ void __launch_bounds__(kGcThreads, NT <= 8 ? 2 : 1)
+gla_chunk_output_kernel(const GlaChunkParams p) {
+  pdl_trigger();
+  extern __shared__ __align__(16) uint8_t gc_sm[];
+  pdl_wait();
+  GlaChunkAt at;
+  if (!gc_locate(p, blockIdx.x, blockIdx.z, at)) return;
+  const int h = blockIdx.y, H = p.s.H, dk = p.s.dk, dv = p.s.dv;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int mat = lane >> 3, mrow = lane & 7, g = lane >> 2, t4 = lane & 3;
+  const GlaOutputSmem m = gc_output_smem(dk, dv);
+  float* b_s = reinterpret_cast<float*>(gc_sm + m.b);
+  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(gc_sm + m.q);
+  __nv_bfloat16* a_hi = reinterpret_cast<__nv_bfloat16*>(gc_sm + m.a);
+  __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(gc_sm + m.v);
+  float* ss_s = reinterpret_cast<float*>(gc_sm + m.ss);
+  const int bp = dk + 8, kp = dk + 8, vp = dv + 8, ap = 72;
+  __nv_bfloat16* k_s = q_s + kGc * kp;
+  __nv_bfloat16* a_lo = a_hi + kGc * ap;
+  const __nv_bfloat16* rows = p.proj + size_t(at.t0) * p.s.row_stride;
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  {
+    const float* cum = p.cum + size_t(at.t0) * (H * dk) + h * dk;
+    const int bper = dk / 4;
+    for (int i = tid; i < kGc * bper; i += kGcThreads) {  // rows past the end repeat the last one
+      const int t = i / bper, c = (i - t * bper) * 4;
+      gc_cp16(b_s + t * bp + c, cum + size_t(min(t, at.n - 1)) * (H * dk) + c);
+    }
+    const int per = dk / 8;
+    for (int i = tid; i < 2 * kGc * per; i += kGcThreads) {
+      const int which = i / (kGc * per), j = i - which * kGc * per, t = j / per, c = (j - t * per) * 8;
+      __nv_bfloat16* d = (which ? k_s : q_s) + t * kp + c;
+      if (t < at.n) gc_cp16(d, rows + size_t(t) * p.s.row_stride + (which * H + h) * dk + c);
+      else *reinterpret_cast<uint4*>(d) = zero;
+    }
+    gc_commit();
+    const int vper = dv / 8;
+    for (int i = tid; i < kGc * vper; i += kGcThreads) {
+      const int t = i / vper, c = (i - t * vper) * 8;
+      if (t < at.n) gc_cp16(v_s + t * vp + c, rows + size_t(t) * p.s.row_stride + 2 * H * dk + h * dv + c);
+      else *reinterpret_cast<uint4*>(v_s + t * vp + c) = zero;
+    }
+    gc_commit();
+  }
+  gc_wait<1>();
+  __syncthreads();
+  // ----- A: warp = (row block I, one half of the column blocks J <= I) -----
+  const int ksteps = dk / 16;
+  bool wide = false;
+  {
+    const int I = warp & 3, J0 = warp < 4 ? 0 : (I + 2) / 2, J1 = warp < 4 ? (I + 2) / 2 : I + 1;  // blocks J0 .. J1 - 1
+    float acc[2][2][4] = {};
+    const float* ref = b_s + (16 * I - 1) * bp;
+    for (int ks = 0; ks < ksteps; ++ks) {
+      uint32_t hi[4], lo[4];
+      float2 rf[2];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int c = ks * 16 + e * 8 + t4 * 2;
+        rf[e] = I ? *reinterpret_cast<const float2*>(ref + c) : make_float2(0.f, 0.f);
+        const float2 last = *reinterpret_cast<const float2*>(b_s + (16 * I + 15) * bp + c);
+        wide = wide || rf[e].x - last.x > kGcSpan || rf[e].y - last.y > kGcSpan;
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int t = 16 * I + r * 8 + g;
+          const float2 q = gc_pair(q_s + t * kp + c), b = *reinterpret_cast<const float2*>(b_s + t * bp + c);
+          gc_split(q.x * p.s.scale * gc_exp2(b.x - rf[e].x), q.y * p.s.scale * gc_exp2(b.y - rf[e].y), hi[e * 2 + r], lo[e * 2 + r]);
+        }
+      }
+#pragma unroll
+      for (int jj = 0; jj < 2; ++jj) {
+        if (J0 + jj < J1) {
+#pragma unroll
+          for (int nt = 0; nt < 2; ++nt) {
+            uint32_t kh[2], kl[2];
+            const int s = 16 * (J0 + jj) + nt * 8 + g;
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              const int c = ks * 16 + e * 8 + t4 * 2;
+              const float2 k = gc_pair(k_s + s * kp + c), b = *reinterpret_cast<const float2*>(b_s + s * bp + c);
+              gc_split(k.x * gc_exp2(rf[e].x - b.x), k.y * gc_exp2(rf[e].y - b.y), kh[e], kl[e]);
+            }
+            gc_mma(acc[jj][nt], hi, kh[0], kh[1]);
+            gc_mma(acc[jj][nt], lo, kh[0], kh[1]);
+            gc_mma(acc[jj][nt], hi, kl[0], kl[1]);
+          }
+        }
+      }
+    }
+#pragma unroll
+    for (int jj = 0; jj < 2; ++jj) {
+      if (J0 + jj < J1) {
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+          for (int r = 0; r < 2; ++r) {
+            const int t = 16 * I + r * 8 + g, s = 16 * (J0 + jj) + nt * 8 + t4 * 2;
+            gc_split(s <= t ? acc[jj][nt][2 * r] : 0.f, s + 1 <= t ? acc[jj][nt][2 * r + 1] : 0.f,
+                     *reinterpret_cast<uint32_t*>(a_hi + t * ap + s), *reinterpret_cast<uint32_t*>(a_lo + t * ap + s));
+          }
+      }
+    }
+  }
+  if (__syncthreads_or(wide)) {  // diagonal blocks term by term
+    for (int i = tid; i < 4 * 256; i += kGcThreads) {
+      const int t = (i >> 8) * 16 + ((i >> 4) & 15), s = (i >> 8) * 16 + (i & 15);
+      if (s > t) continue;
+      float x = 0.f;
+      for (int c = 0; c < dk; ++c)
+        x += __bfloat162float(q_s[t * kp + c]) * __bfloat162float(k_s[s * kp + c]) * gc_exp2(b_s[t * bp + c] - b_s[s * bp + c]);
+      x *= p.s.scale;
+      const __nv_bfloat16 hi = __float2bfloat16(x);
+      a_hi[t * ap + s] = hi;
+      a_lo[t * ap + s] = __float2bfloat16(x - __bfloat162float(hi));
+    }
+    __syncthreads();
+  }
+  // ----- 2^b q, in the place of q and k -----
+  {
+    const int per = dk / 2;
+    for (int i = tid; i < kGc * per; i += kGcThreads) {
+      const int t = i / per, c = (i - t * per) * 2;
+      const float2 q = gc_pair(q_s + t * kp + c), b = *reinterpret_cast<const float2*>(b_s + t * bp + c);
+      gc_split(q.x * p.s.scale * gc_exp2(b.x), q.y * p.s.scale * gc_exp2(b.y), *reinterpret_cast<uint32_t*>(q_s + t * kp + c),
+               *reinterpret_cast<uint32_t*>(k_s + t * kp + c));
+    }
+  }
+  __syncthreads();
+  // ----- O: warp = (16 tokens, half of the value columns) -----
+  const uint8_t* s0 = reinterpret_cast<const uint8_t*>(p.u + (at.index * H + h) * size_t(dk) * dv);
+  const int spitch = dv * 4 + 16;
+  auto fetch = [&](int ks) {
+    uint8_t* d = gc_sm + m.b + (ks & 1) * 16 * spitch;
+    const int per = dv / 4;  // 16-byte pieces of a row
+    for (int i = tid; i < 16 * per; i += kGcThreads) {
+      const int r = i / per, c = i - r * per;
+      gc_cp16(d + r * spitch + c * 16, s0 + (size_t(ks) * 16 + r) * dv * 4 + c * 16);
+    }
+  };
+  fetch(0);
+  gc_commit();
+  if (ksteps > 1) fetch(1);
+  gc_commit();
+  gc_wait<2>();  // V
+  __syncthreads();
+  const int mt = warp & 3, half = warp >> 2, tiles = dv / 16;
+  const int col0 = half * (dv / 2);
+  float o[NT][4];
+#pragma unroll
+  for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) o[nt][e] = 0.f;
+  const int frag = (mt * 16 + (mat & 1) * 8 + mrow), fk = (mat >> 1) * 8;
+  for (int ks = 0; ks <= mt; ++ks) {
+    uint32_t hi[4], lo[4];
+    gc_ldm(smem_u32(a_hi + frag * ap + ks * 16 + fk), hi);
+    gc_ldm(smem_u32(a_lo + frag * ap + ks * 16 + fk), lo);
+#pragma unroll
+    for (int nt = 0; nt < NT; nt += 2) {
+      if (nt < tiles) {
+        uint32_t v[4];  // the second tile of the last pair may lie past the half: it is not used then
+        gc_ldm_t(smem_u32(v_s + (ks * 16 + (mat & 1) * 8 + mrow) * vp + col0 + nt * 8 + (mat >> 1) * 8), v);
+        gc_mma(o[nt], hi, v[0], v[1]);
+        gc_mma(o[nt], lo, v[0], v[1]);
+        if (nt + 1 < tiles) {
+          gc_mma(o[nt + 1], hi, v[2], v[3]);
+          gc_mma(o[nt + 1], lo, v[2], v[3]);
+        }
+      }
+    }
+  }
+  for (int ks = 0; ks < ksteps; ++ks) {
+    gc_wait<1>();
+    __syncthreads();
+    uint32_t hi[4], lo[4];
+    gc_ldm(smem_u32(q_s + frag * kp + ks * 16 + fk), hi);
+    gc_ldm(smem_u32(k_s + frag * kp + ks * 16 + fk), lo);
+    const uint32_t st = smem_u32(gc_sm + m.b) + (ks & 1) * 16 * spitch + ((mat & 1) * 8 + mrow) * spitch + col0 * 4 + (mat >> 1) * 16;
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) {
+      if (nt < tiles) {
+        uint32_t s[4];  // hi of rows 0-7, 8-15, then lo
+        gc_ldm_t(st + nt * 32, s);
+        gc_mma(o[nt], hi, s[0], s[1]);
+        gc_mma(o[nt], lo, s[0], s[1]);
+        gc_mma(o[nt], hi, s[2], s[3]);
+      }
+    }
+    __syncthreads();
+    if (ks + 2 < ksteps) fetch(ks + 2);
+    gc_commit();
+  }
+  // ----- norm over the head's value channels, gate -----
+  float sq[2] = {0.f, 0.f};
+#pragma unroll
+  for (int nt = 0; nt < NT; ++nt) {
+    if (nt < tiles) {
+      sq[0] += o[nt][0] * o[nt][0] + o[nt][1] * o[nt][1];
+      sq[1] += o[nt][2] * o[nt][2] + o[nt][3] * o[nt][3];
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    sq[r] += __shfl_xor_sync(0xffffffffu, sq[r], 1);
+    sq[r] += __shfl_xor_sync(0xffffffffu, sq[r], 2);
+    if (t4 == 0) ss_s[half * kGc + mt * 16 + r * 8 + g] = sq[r];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int t = mt * 16 + r * 8 + g;
+    if (t >= at.n) continue;
+    const float f = rsqrtf((ss_s[t] + ss_s[kGc + t]) * p.s.inv_dv + p.s.eps);
+    const __nv_bfloat16* gate = rows + size_t(t) * p.s.row_stride + 2 * H * dk + (H + h) * dv;
+    __nv_bfloat16* y = p.y + (size_t(at.t0 + t) * H + h) * dv;
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) {
+      if (nt < tiles) {
+        const int c = col0 + nt * 8 + t4 * 2;
+        const float2 gt = gc_pair(gate + c), w = *reinterpret_cast<const float2*>(p.norm_w + c);
+        *reinterpret_cast<__nv_bfloat162*>(y + c) =
+            __floats2bfloat162_rn(o[nt][2 * r] * f * w.x * silu_of(gt.x), o[nt][2 * r + 1] * f * w.y * silu_of(gt.y));
+      }
+    }
+  }
+}
+
+template <int NT>
+int launch_gla_output(const GlaChunkParams& p, dim3 grid, cudaStream_t stream) {
+  const int smem = gc_output_smem(p.s.dk, p.s.dv).bytes;
+  static int allowed = 0;
+  if (smem > allowed) {
+    if (cudaFuncSetAttribute(gla_chunk_output_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -6;
+    allowed = smem;
+  }
+  return launch_kernel(gla_chunk_output_kernel<NT>, grid, dim3(kGcThreads), smem, stream, p) == cudaSuccess ? 0 : -7;
+}
+
+}  // namespace
+}  // namespace mfq
+
+using namespace mfq;
+
+// Portions of B sequences (tokens starts[b] .. starts[b + 1] - 1 of proj and y), longest `max_q`.  With chunks = T / 64 + B, T the
+// tokens of all portions: cum [tokens of proj, H dk], u [chunks, H, dk, dv] and gam [chunks, H, dk] are fp32 scratch.
+// Returns -5 for sizes that do not fit (callers use the token-by-token kernel).
+extern "C" int mfq_gla_chunk(const void* proj, const void* w2, const float* bias, const float* norm_w, void* y, float* state,
+                             const int* slot, const int* starts, float* cum, float* u, float* gam, int B, int max_q, int H, int dk, int dv,
+                             int real_dv, int rank, int row_stride, float scale, float inv_tau, float eps, cudaStream_t stream) {
+  if (B <= 0 || B > 65535 || max_q <= 0 || H <= 0 || H > 65535 || dk <= 0 || dv <= 0 || dk % 16 || dv % 16 || rank <= 0 || rank % 8) return -1;
+  if (real_dv <= 0 || real_dv > dv || row_stride < 2 * H * (dk + dv) + rank || row_stride % 8) return -1;
+  const int local = gc_local_smem(dk, dv, rank).bytes;
+  if (dk > kGcMaxDk || dv > kGcMaxDv || local > 227 * 1024 || gc_output_smem(dk, dv).bytes > 227 * 1024) return -5;
+  const GlaChunkParams p{GlaShape{H, dk, dv, rank, row_stride, scale, inv_tau, 1.f / float(real_dv), eps}, static_cast<const __nv_bfloat16*>(proj),
+                         static_cast<const __nv_bfloat16*>(w2), bias, norm_w, static_cast<__nv_bfloat16*>(y), starts, slot, state, cum, u, gam};
+  const dim3 grid((max_q + kGc - 1) / kGc, H, B);
+  static int allowed = 0;
+  if (local > allowed) {
+    if (cudaFuncSetAttribute(gla_chunk_local_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, local) != cudaSuccess) return -6;
+    allowed = local;
+  }
+  launch_kernel(gla_chunk_local_kernel, grid, dim3(kGcThreads), local, stream, p);
+  launch_kernel(gla_chunk_state_kernel, dim3((dk * dv / 8 + 127) / 128, H, B), dim3(128), 0, stream, p);
+  const int rc = dv <= 64 ? launch_gla_output<4>(p, grid, stream) : dv <= 128 ? launch_gla_output<8>(p, grid, stream)
+               : dv <= 256 ? launch_gla_output<16>(p, grid, stream) : launch_gla_output<32>(p, grid, stream);
+  return rc == 0 && cudaGetLastError() == cudaSuccess ? 0 : (rc ? rc : -7);
+}

@@ -1,11 +1,12 @@
-// fp32 residual stream of a decoder whose sublayers are normalised on their OUTPUT, and the per-head stage between the
-// q/k/v projection and attention, for activations in bf16 or fp32.
+// fp32 residual stream of a decoder (sublayers normalised on their input or on their output), and the per-head stage between
+// the q/k/v projection and attention, for activations in bf16 or fp32.
 //
 //   embed_scaled      x = table[id] * scale              -> fp32 stream + copy in the activation type
 //   norm_add          x += rms_norm(y) * w               -> fp32 stream + copy in the activation type, one pass over y and x
-//   norm_out          h = rms_norm(x) * w                -> activation type (input of the LM head)
+//   norm_out          h = rms_norm(x) * w                -> activation type (input of a sublayer or of the LM head)
 //   qkv_finish        per head: RMS norm of q and k, rotation of the leading channels, blending of v with the values another
 //                     layer computed for the same token, K / V into their pages
+//   map_difference    differential attention: rms_norm(a1 - lambda a2) * scale of every head
 //
 // "rms_norm" divides by sqrt(mean(x^2) + eps) over the model's true width; weights arrive in fp32 in the form they multiply
 // with.  Padding columns hold zeros and stay zero because their weights are zero.
@@ -101,13 +102,14 @@ norm_out_kernel(const float* __restrict__ x, const float* __restrict__ w, T* __r
 }
 
 // ---------------------------------------------------------------------------------------------
-// qkv rows [Hq * dk | Hk * dk | Hk * dv] (dk, dv: head widths as stored, multiples of 16; d: the true q / k width the norm
-// averages over).  `L` lanes (a power of two) share a head, 8 channels each; a warp takes 32 / L heads of one token.
-// The rotation reads (cos, sin) of the token's position from a table [positions][rot / 2] and its partner channel from
-// shared memory.  Pages: K [page][Hk][16][dk], V [page][Hk][16][dv]; slot < 0: the token is not cached.
+// qkv rows [Hq * dk | Hk * maps * dk | Hk * dv] (dk, dv: head widths as stored, multiples of 16; d: the true q / k width the
+// norm averages over; Hq counts every query map).  `L` lanes (a power of two) share a head, 8 channels each; a warp takes 32 / L
+// heads of one token.  The rotation reads (cos, sin) of the token's position from a table [positions][rot / 2]; channel i turns
+// with i + rot / 2 (read from shared memory), or with its neighbour (`pairs`).  Pages: K [page][Hk][16][maps * dk],
+// V [page][Hk][16][dv]; slot < 0: the token is not cached.  No pages: rows hold queries only.
 // ---------------------------------------------------------------------------------------------
 struct QkvFinishParams {
-  int T, Hq, Hk, d, dk, dv, rot, row_stride, page_size, L, table_rows;
+  int T, Hq, Hk, maps, d, dk, dv, rot, pairs, row_stride, page_size, L, table_rows;
   float eps, lambda;        // lambda: share of the other layer's values
   int first_stride;         // row stride of `v_first`
   const float* q_norm;
@@ -126,17 +128,17 @@ qkv_finish_kernel(const T* __restrict__ qkv, const T* __restrict__ v_first, T* _
   __shared__ float sh[8][32 * 8];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int per_warp = 32 / p.L, sub = lane / p.L, c = lane - sub * p.L;  // c: my 8-channel chunk
-  const int heads = p.Hq + 2 * p.Hk;
+  const int keys = k_pages ? p.Hk * p.maps : 0, heads = p.Hq + keys + (k_pages ? p.Hk : 0);
   const int groups = (heads + per_warp - 1) / per_warp;  // head groups of a token
   const int gw = blockIdx.x * 8 + warp;
   if (gw >= p.T * groups) return;  // whole warps leave together
   const int t = gw / groups, h = (gw - t * groups) * per_warp + sub;
   const bool live_head = h < heads;
-  const bool is_q = h < p.Hq, is_v = h >= p.Hq + p.Hk;
+  const bool is_q = h < p.Hq, is_v = h >= p.Hq + keys;
   const int width = is_v ? p.dv : p.dk;
   const bool mine = live_head && c * 8 < width;
   const T* row = qkv + size_t(t) * p.row_stride;
-  const int col = is_v ? (p.Hq + p.Hk) * p.dk + (h - p.Hq - p.Hk) * p.dv : h * p.dk;
+  const int col = is_v ? (p.Hq + keys) * p.dk + (h - p.Hq - keys) * p.dv : h * p.dk;
   float v[8];
   if (mine) {
     load8<T>(row + col + c * 8, v);
@@ -164,8 +166,20 @@ qkv_finish_kernel(const T* __restrict__ qkv, const T* __restrict__ v_first, T* _
   if (!is_v && c * 8 < p.rot) {
     const int half = p.rot >> 1, pos = min(p.positions[t], p.table_rows - 1);
     const float2* tab = p.rope + size_t(pos) * half;
+    if (p.pairs) {
+#pragma unroll
+      for (int j = 0; j < 8; j += 2) {
+        if (c * 8 + j < p.rot) {
+          const float2 cs = tab[(c * 8 + j) >> 1];
+          const float a = v[j], b = v[j + 1];
+          v[j] = a * cs.x - b * cs.y;
+          v[j + 1] = b * cs.x + a * cs.y;
+        }
+      }
+    }
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
+      if (p.pairs) break;
       const int i = c * 8 + j;
       if (i < half) {
         const float2 cs = tab[i];
@@ -184,10 +198,11 @@ qkv_finish_kernel(const T* __restrict__ qkv, const T* __restrict__ v_first, T* _
   if (slot < 0) return;
   const int page = slot / p.page_size, off = slot - page * p.page_size;
   if (!is_v) {
-    store8<T>(k_pages + ((size_t(page) * p.Hk + (h - p.Hq)) * p.page_size + off) * p.dk + c * 8, v);
+    const int g = (h - p.Hq) / p.maps, m = h - p.Hq - g * p.maps;
+    store8<T>(k_pages + (((size_t(page) * p.Hk + g) * p.page_size + off) * p.maps + m) * p.dk + c * 8, v);
     return;
   }
-  const int g = h - p.Hq - p.Hk;
+  const int g = h - p.Hq - keys;
   if (v_first) {
     float f[8];
     load8<T>(v_first + size_t(t) * p.first_stride + g * p.dv + c * 8, f);
@@ -195,6 +210,41 @@ qkv_finish_kernel(const T* __restrict__ qkv, const T* __restrict__ v_first, T* _
     for (int j = 0; j < 8; ++j) v[j] = (1.f - p.lambda) * v[j] + p.lambda * f[j];
   }
   store8<T>(v_pages + ((size_t(page) * p.Hk + g) * p.page_size + off) * p.dv + c * 8, v);
+}
+
+// ---------------------------------------------------------------------------------------------
+// a [T][G][2][per][dv] (both maps of every head) -> out [T][G * per][dv]: y = a1 - lambda a2, out = scale * y / sqrt(mean(y^2) + eps),
+// the mean over the `d` real channels (the others are zeros).  A warp per (token, head).
+// ---------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256)
+map_difference_kernel(const T* __restrict__ a, T* __restrict__ out, int pairs, int H, int per, int dv, float inv_d, float lambda,
+                      float scale, float eps) {
+  pdl_trigger();
+  pdl_wait();
+  const int pair = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (pair >= pairs) return;
+  const int t = pair / H, h = pair - t * H, g = h / per, j = h - g * per;
+  const bool mine = lane * 8 < dv;
+  float y[8] = {};
+  if (mine) {
+    const T* a1 = a + ((size_t(t) * H + g * per) * 2 + j) * dv + lane * 8;
+    float b[8];
+    load8<T>(a1, y);
+    load8<T>(a1 + size_t(per) * dv, b);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) y[i] -= lambda * b[i];
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) ss += y[i] * y[i];
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (!mine) return;
+  const float f = rsqrtf(ss * inv_d + eps) * scale;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) y[i] *= f;
+  store8<T>(out + size_t(pair) * dv + lane * 8, y);
 }
 
 static int stream_threads(int W) {
@@ -243,18 +293,31 @@ extern "C" int mfq_norm_out(const float* x, const float* w, void* out, int M, in
   return cudaGetLastError() == cudaSuccess ? 0 : -7;
 }
 
+extern "C" int mfq_map_difference(const void* a, void* out, int T_, int H, int per, int dv, int d, float lambda, float scale, float eps,
+                                  int fp32, cudaStream_t stream) {
+  if (T_ <= 0 || H <= 0 || per <= 0 || H % per || dv % 8 || dv <= 0 || dv > 256 || d <= 0 || d > dv) return -1;
+  const long long pairs = (long long)(T_) * H;
+  if (pairs > 0x7fffffff) return -1;
+  MFQ_BY_TYPE(fp32, launch_kernel(map_difference_kernel<T>, dim3(unsigned((pairs + 7) / 8)), dim3(256), 0, stream,
+                                  static_cast<const T*>(a), static_cast<T*>(out), int(pairs), H, per, dv, 1.f / float(d), lambda, scale, eps));
+  return cudaGetLastError() == cudaSuccess ? 0 : -7;
+}
+
+// k_pages null: the rows hold the Hq query heads only (Hk, dv unused)
 extern "C" int mfq_qkv_finish(const void* qkv, int row_stride, const void* v_first, int first_stride, float lambda, void* q_out,
                               void* k_pages, void* v_pages, const int* positions, const int* slots, const float* q_norm,
-                              const float* k_norm, const float* rope, int table_rows, int T_, int Hq, int Hk, int d, int dk, int dv,
-                              int rot, int page_size, float eps, int fp32, cudaStream_t stream) {
-  if (T_ <= 0 || Hq <= 0 || Hk <= 0 || Hq % Hk || dk % 16 || dv % 16 || dk > 256 || dv > 256 || d <= 0 || d > dk) return -1;
-  if (row_stride % 8 || row_stride < (Hq + Hk) * dk + Hk * dv || (v_first && first_stride % 8)) return -1;
-  if (rot < 0 || rot % 2 || rot > d || (rot > 0 && (!rope || table_rows <= 0)) || page_size <= 0) return -1;
+                              const float* k_norm, const float* rope, int table_rows, int T_, int Hq, int Hk, int maps, int d, int dk,
+                              int dv, int rot, int pairs, int page_size, float eps, int fp32, cudaStream_t stream) {
+  if (!k_pages) { Hk = 0; dv = 0; v_first = nullptr; }
+  if (T_ <= 0 || Hq <= 0 || maps <= 0 || dk % 16 || dk <= 0 || dk > 256 || d <= 0 || d > dk) return -1;
+  if (k_pages && (Hk <= 0 || Hq % (Hk * maps) || dv % 16 || dv <= 0 || dv > 256 || page_size <= 0 || !v_pages || !slots)) return -1;
+  if (row_stride % 8 || row_stride < (Hq + Hk * maps) * dk + Hk * dv || (v_first && first_stride % 8)) return -1;
+  if (rot < 0 || rot % 2 || rot > d || (rot > 0 && (!rope || table_rows <= 0))) return -1;
   int L = 1;
   while (L * 8 < max(dk, dv)) L *= 2;
-  QkvFinishParams p{T_, Hq, Hk, d, dk, dv, rot, row_stride, page_size, L, table_rows, eps, lambda, first_stride, q_norm, k_norm,
+  QkvFinishParams p{T_, Hq, Hk, maps, d, dk, dv, rot, pairs, row_stride, page_size, L, table_rows, eps, lambda, first_stride, q_norm, k_norm,
                     reinterpret_cast<const float2*>(rope), positions, slots};
-  const int heads = Hq + 2 * Hk, per_warp = 32 / L;
+  const int heads = Hq + Hk * (maps + 1), per_warp = 32 / L;
   const long long warps = (long long)(T_) * ((heads + per_warp - 1) / per_warp);
   MFQ_BY_TYPE(fp32, launch_kernel(qkv_finish_kernel<T>, dim3(unsigned((warps + 7) / 8)), dim3(256), 0, stream, static_cast<const T*>(qkv),
                                   static_cast<const T*>(v_first), static_cast<T*>(q_out), static_cast<T*>(k_pages),

@@ -1,10 +1,14 @@
-// Sliding-window attention over unquantized pages (K [page][Hk][16][dk], V [page][Hk][16][dv]), one query token per sequence
-// or, in the plain kernel, any number of them.  A query at position i sees the keys j with 0 <= i - j < window.
+// Sliding-window attention over unquantized pages (K [page][Hk][16][maps * dk], V [page][Hk][16][dv]), one query token per
+// sequence or, in the plain kernel, any number of them.  A query at position i sees the keys j with 0 <= i - j < window, and of
+// the first `keep` keys every one up to i.  With two maps (differential attention) a KV head has two key vectors and one value
+// vector per token; queries are ordered [KV head][map][query head of the KV head].
 //
 //   window_attn_decode_kernel   bf16, one query per sequence.  A CTA serves one (sequence, KV head, KV split); its four warps
 //                               take alternate pages that hold visible keys through private cp.async rings.  The (up to 16)
-//                               query heads of the KV head are the rows of m16n8k16 MMAs: S = Q K^T, probabilities go from
-//                               accumulators straight into the A operand of P V.  Warps (and splits) merge at the end.
+//                               queries of the KV head are the rows of m16n8k16 MMAs: S = Q K^T, probabilities go from
+//                               accumulators straight into the A operand of P V.  Queries of both maps share the rows (and the
+//                               values): a row is zero on the key channels of the other map.  Warps (and splits) merge at the end.
+//   window_attn_merge_kernel    sums the splits; with two maps also the normalised difference of a head's maps
 //   window_attn_plain_kernel    a warp per (token, query head), fp32 arithmetic, fp32 or bf16 storage: the full-precision mode.
 #include "window_attn.cuh"
 
@@ -15,15 +19,15 @@ namespace mfq {
 constexpr int kWinPage = 16, kWinWarps = 4;
 
 struct WindowDecodeParams {
-  const __nv_bfloat16* q;  // [B, Hq, dk]
+  const __nv_bfloat16* q;  // [B, Hq, dk]; Hq counts the queries of all maps
   const __nv_bfloat16* k;
   const __nv_bfloat16* v;
   const int* table;     // [B, max_pages]
   const int* seq_lens;  // length including the query token
   __nv_bfloat16* out;   // [B, Hq, dv]
-  float* part;          // splits > 1: [B * Hq][splits][dv]
+  float* part;          // splits > 1 or maps > 1: [B * Hq][splits][dv]
   float* part_ml;       // [B * Hq][splits][2]
-  int Hq, Hk, dk, dv, max_pages, window, splits, head_tiles;
+  int Hq, Hk, maps, dk, dv, max_pages, window, keep, splits, head_tiles;
   ScoreCap cap;
 };
 
@@ -49,7 +53,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
   return *reinterpret_cast<uint32_t*>(&h);
 }
 
-// DK / DV: upper bounds of the stored head widths (register arrays); the widths themselves are run-time multiples of 16.
+// DK / DV: upper bounds of the stored widths of a KV head (register arrays); the widths themselves are run-time multiples of 16.
 template <int DK, int DV>
 struct WinCfg {
   static constexpr int kStages = 2;  // two pages per warp in flight leave room for three CTAs per SM at 128 + 128 channels
@@ -72,11 +76,12 @@ window_attn_decode_kernel(const WindowDecodeParams p) {
   const int b = bg / p.Hk, g = bg - b * p.Hk, split = blockIdx.y;
   const int per = p.Hq / p.Hk, heads = min(16, per - ht * 16);
   const int head0 = g * per + ht * 16;
-  const int dk = p.dk, dv = p.dv;
+  const int map_dk = p.dk, dk = p.maps * p.dk, dv = p.dv;  // dk: channels of a key row, all maps
   const int pos = p.seq_lens[b] - 1;
   const int lo = max(0, pos - p.window + 1);
-  int page0 = lo / kWinPage, page1 = pos >= 0 ? pos / kWinPage + 1 : 0;
-  if (pos < 0) page0 = 0;
+  // pages are counted over the visible ones: `kept` pages of first tokens that lie before the window, then the window's
+  const int first = pos >= 0 ? lo / kWinPage : 0, kept = min((p.keep + kWinPage - 1) / kWinPage, first), skip = first - kept;
+  int page0 = 0, page1 = pos >= 0 ? pos / kWinPage + 1 - skip : 0;
   {
     const int chunk = (page1 - page0 + p.splits - 1) / p.splits;
     page0 = page0 + split * chunk;
@@ -93,7 +98,7 @@ window_attn_decode_kernel(const WindowDecodeParams p) {
   auto fetch = [&](int i) {
     if ((i & 31) == 0) {
       const int pg = page0 + warp + kWinWarps * (i + lane);
-      ids = pg < page1 ? table[pg] : 0;
+      ids = pg < page1 ? table[pg < kept ? pg : pg + skip] : 0;
     }
     const int page = __shfl_sync(0xffffffffu, ids, i & 31);
     const uint32_t st = ring + (i % kStages) * stage_bytes;
@@ -118,15 +123,19 @@ window_attn_decode_kernel(const WindowDecodeParams p) {
   const int r0 = lane >> 2, t4 = lane & 3;
   uint32_t qf[DK / 16][4];
   {
-    const __nv_bfloat16* q0 = p.q + (size_t(b) * p.Hq + head0 + r0) * dk + t4 * 2;
-    const __nv_bfloat16* q1 = q0 + size_t(8) * dk;
+    // a row's own map covers the key channels c0 .. c0 + map_dk - 1
+    const int of_map = per / p.maps;
+    const int c0 = (ht * 16 + r0) / of_map * map_dk, c1 = (ht * 16 + r0 + 8) / of_map * map_dk;
+    const __nv_bfloat16* q0 = p.q + (size_t(b) * p.Hq + head0 + r0) * map_dk + t4 * 2 - c0;
+    const __nv_bfloat16* q1 = p.q + (size_t(b) * p.Hq + head0 + r0 + 8) * map_dk + t4 * 2 - c1;
 #pragma unroll
     for (int ks = 0; ks < DK / 16; ++ks) {
-      const bool in = ks * 16 < dk;
-      qf[ks][0] = in && r0 < heads ? *reinterpret_cast<const uint32_t*>(q0 + ks * 16) : 0u;
-      qf[ks][1] = in && r0 + 8 < heads ? *reinterpret_cast<const uint32_t*>(q1 + ks * 16) : 0u;
-      qf[ks][2] = in && r0 < heads ? *reinterpret_cast<const uint32_t*>(q0 + ks * 16 + 8) : 0u;
-      qf[ks][3] = in && r0 + 8 < heads ? *reinterpret_cast<const uint32_t*>(q1 + ks * 16 + 8) : 0u;
+      const bool in0 = r0 < heads && ks * 16 >= c0 && ks * 16 < c0 + map_dk;
+      const bool in1 = r0 + 8 < heads && ks * 16 >= c1 && ks * 16 < c1 + map_dk;
+      qf[ks][0] = in0 ? *reinterpret_cast<const uint32_t*>(q0 + ks * 16) : 0u;
+      qf[ks][1] = in1 ? *reinterpret_cast<const uint32_t*>(q1 + ks * 16) : 0u;
+      qf[ks][2] = in0 ? *reinterpret_cast<const uint32_t*>(q0 + ks * 16 + 8) : 0u;
+      qf[ks][3] = in1 ? *reinterpret_cast<const uint32_t*>(q1 + ks * 16 + 8) : 0u;
     }
   }
   float o[DV / 8][4];
@@ -154,14 +163,15 @@ window_attn_decode_kernel(const WindowDecodeParams p) {
         win_mma(s[1], qf[ks], kf[2], kf[3]);
       }
     }
-    const int key0 = (page0 + warp + kWinWarps * i) * kWinPage + t4 * 2;
+    const int pg = page0 + warp + kWinWarps * i;
+    const int key0 = (pg < kept ? pg : pg + skip) * kWinPage + t4 * 2;
     float mx[2] = {-FLT_MAX, -FLT_MAX};
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = key0 + nt * 8 + (e & 1);
-        s[nt][e] = key >= lo && key <= pos ? score_any(p.cap, s[nt][e]) : -FLT_MAX;
+        s[nt][e] = (key >= lo || key < p.keep) && key <= pos ? score_any(p.cap, s[nt][e]) : -FLT_MAX;
         mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
       }
     float alpha[2];
@@ -235,49 +245,73 @@ window_attn_decode_kernel(const WindowDecodeParams p) {
       lt += ml[(w * 16 + r) * 2 + 1] * mw[w];
     }
     const size_t orow = size_t(b) * p.Hq + head0 + r;
-    const float inv = p.splits == 1 ? (lt > 0.f ? 1.f / lt : 0.f) : 1.f;
+    const bool whole = p.splits == 1 && p.maps == 1;
+    const float inv = whole ? (lt > 0.f ? 1.f / lt : 0.f) : 1.f;
     for (int c = lane; c < dv; c += 32) {
       float x = 0.f;
 #pragma unroll
       for (int w = 0; w < kWinWarps; ++w) x += acc[(w * 16 + r) * dv + c] * mw[w];
       x *= inv;
-      if (p.splits == 1) p.out[orow * dv + c] = __float2bfloat16(x);
+      if (whole) p.out[orow * dv + c] = __float2bfloat16(x);
       else p.part[(orow * p.splits + split) * dv + c] = x;
     }
-    if (p.splits > 1 && lane == 0) {
+    if (!whole && lane == 0) {
       p.part_ml[(orow * p.splits + split) * 2] = mt;
       p.part_ml[(orow * p.splits + split) * 2 + 1] = lt;
     }
   }
 }
 
-__global__ void window_attn_merge_kernel(const float* __restrict__ part, const float* __restrict__ part_ml,
-                                         __nv_bfloat16* __restrict__ out, int splits, int dv) {
+// A CTA per (sequence, output head).  Two maps: y = a1 - lambda a2, out = scale * y / sqrt(mean(y^2) + eps).
+struct WindowMergeParams {
+  int splits, dv, heads, of_map, maps;  // heads: output heads; of_map: query heads per KV head
+  float lambda, scale, eps, inv_d;
+};
+
+__global__ void __launch_bounds__(128)
+window_attn_merge_kernel(const float* __restrict__ part, const float* __restrict__ part_ml, __nv_bfloat16* __restrict__ out,
+                         const WindowMergeParams p) {
   pdl_trigger();
   pdl_wait();
-  const size_t row = blockIdx.x;
-  float mt = -FLT_MAX, lt = 0.f;
-  for (int z = 0; z < splits; ++z) mt = fmaxf(mt, part_ml[(row * splits + z) * 2]);
-  for (int z = 0; z < splits; ++z) lt += part_ml[(row * splits + z) * 2 + 1] * window_exp2(part_ml[(row * splits + z) * 2] - mt);
-  const float inv = lt > 0.f ? 1.f / lt : 0.f;
-  for (int c = threadIdx.x; c < dv; c += blockDim.x) {
-    float x = 0.f;
-    for (int z = 0; z < splits; ++z) x += part[(row * splits + z) * dv + c] * window_exp2(part_ml[(row * splits + z) * 2] - mt);
-    out[row * dv + c] = __float2bfloat16(x * inv);
+  __shared__ float red[33];
+  const int b = blockIdx.x / p.heads, h = blockIdx.x - b * p.heads, g = h / p.of_map;
+  float y[2] = {0.f, 0.f};  // channels threadIdx.x and threadIdx.x + 128
+  for (int m = 0; m < p.maps; ++m) {
+    const size_t row = (size_t(b) * p.heads + g * p.of_map) * p.maps + m * p.of_map + h - g * p.of_map;
+    const float* ml = part_ml + row * p.splits * 2;
+    float mt = -FLT_MAX, lt = 0.f;
+    for (int z = 0; z < p.splits; ++z) mt = fmaxf(mt, ml[z * 2]);
+    for (int z = 0; z < p.splits; ++z) lt += ml[z * 2 + 1] * window_exp2(ml[z * 2] - mt);
+    const float inv = (lt > 0.f ? 1.f / lt : 0.f) * (m == 0 ? 1.f : -p.lambda);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int c = threadIdx.x + i * 128;
+      if (c >= p.dv) continue;
+      float x = 0.f;
+      for (int z = 0; z < p.splits; ++z) x += part[(row * p.splits + z) * p.dv + c] * window_exp2(ml[z * 2] - mt);
+      y[i] += x * inv;
+    }
+  }
+  float f = 1.f;
+  if (p.maps == 2) f = rsqrtf(dense_block_sum(y[0] * y[0] + y[1] * y[1], red) * p.inv_d + p.eps) * p.scale;
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int c = threadIdx.x + i * 128;
+    if (c < p.dv) out[size_t(blockIdx.x) * p.dv + c] = __float2bfloat16(y[i] * f);
   }
 }
 
 template <int DK, int DV>
-static int launch_window_decode(const WindowDecodeParams& p, int B, cudaStream_t stream) {
-  const int smem = WinCfg<DK, DV>::smem_bytes(p.dk, p.dv);
+static int launch_window_decode(const WindowDecodeParams& p, const WindowMergeParams& mp, int B, cudaStream_t stream) {
+  const int smem = WinCfg<DK, DV>::smem_bytes(p.dk * p.maps, p.dv);
   static int allowed = 0;
   if (smem > allowed) {
     if (cudaFuncSetAttribute(window_attn_decode_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -6;
     allowed = smem;
   }
   launch_kernel(window_attn_decode_kernel<DK, DV>, dim3(B * p.Hk * p.head_tiles, p.splits), dim3(kWinWarps * 32), smem, stream, p);
-  if (p.splits > 1)
-    launch_kernel(window_attn_merge_kernel, dim3(B * p.Hq), dim3(p.dv <= 64 ? 64 : 128), 0, stream, p.part, p.part_ml, p.out, p.splits, p.dv);
+  if (p.splits > 1 || p.maps > 1)
+    launch_kernel(window_attn_merge_kernel, dim3(B * mp.heads), dim3(128), 0, stream, p.part, p.part_ml, p.out, mp);
   return cudaGetLastError() == cudaSuccess ? 0 : -7;
 }
 
@@ -288,7 +322,7 @@ struct WindowPlainParams {
   const int* positions;  // [T]
   const int* tok_seq;    // [T] row of the block table
   const int* table;
-  int T, Hq, Hk, dk, dv, max_pages, window;
+  int T, Hq, Hk, maps, dk, dv, max_pages, window, keep;
   float scale, cap;
 };
 
@@ -303,8 +337,8 @@ window_attn_plain_kernel(const T* __restrict__ q, const T* __restrict__ k, const
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int gw = blockIdx.x * 4 + warp;
   if (gw >= p.T * p.Hq) return;
-  const int t = gw / p.Hq, h = gw - t * p.Hq, g = h / (p.Hq / p.Hk);
-  const int pos = p.positions[t], lo = max(0, pos - p.window + 1);
+  const int t = gw / p.Hq, h = gw - t * p.Hq, per = p.Hq / p.Hk, g = h / per, map = (h - g * per) / (per / p.maps);
+  const int pos = p.positions[t], lo = max(0, pos - p.window + 1), kept = min(p.keep, lo), skip = lo - kept;
   const int* table = p.table + size_t(p.tok_seq[t]) * p.max_pages;
   if (lane * 8 < p.dk) {
     float x[8];
@@ -314,13 +348,13 @@ window_attn_plain_kernel(const T* __restrict__ q, const T* __restrict__ k, const
   }
   __syncwarp();
   float m = -FLT_MAX, l = 0.f, acc[8] = {};
-  for (int j0 = lo; j0 <= pos; j0 += 32) {
-    const int key = j0 + lane;
+  for (int j0 = 0; j0 <= pos - skip; j0 += 32) {  // over the visible keys: the kept ones before the window, then the window
+    const int key = j0 + lane < kept ? j0 + lane : j0 + lane + skip;
     float s = -FLT_MAX;
     int page = 0;
     if (key <= pos) {
       page = table[key / kWinPage];
-      const T* kr = k + ((size_t(page) * p.Hk + g) * kWinPage + key % kWinPage) * p.dk;
+      const T* kr = k + (((size_t(page) * p.Hk + g) * kWinPage + key % kWinPage) * p.maps + map) * p.dk;
       float dot = 0.f;
       for (int c = 0; c < p.dk; c += 8) {
         float x[8];
@@ -347,10 +381,11 @@ window_attn_plain_kernel(const T* __restrict__ q, const T* __restrict__ k, const
     if (lane * 8 < p.dv) {
 #pragma unroll
       for (int j = 0; j < 8; ++j) acc[j] *= alpha;
-      const int cnt = min(32, pos - j0 + 1);
+      const int cnt = min(32, pos - skip - j0 + 1);
       for (int i = 0; i < cnt; ++i) {
         float x[8];
-        load8<T>(v + ((size_t(spage[warp][i]) * p.Hk + g) * kWinPage + (j0 + i) % kWinPage) * p.dv + lane * 8, x);
+        const int key_i = j0 + i < kept ? j0 + i : j0 + i + skip;
+        load8<T>(v + ((size_t(spage[warp][i]) * p.Hk + g) * kWinPage + key_i % kWinPage) * p.dv + lane * 8, x);
 #pragma unroll
         for (int j = 0; j < 8; ++j) acc[j] = fmaf(sp[warp][i], x[j], acc[j]);
       }
@@ -369,28 +404,37 @@ window_attn_plain_kernel(const T* __restrict__ q, const T* __restrict__ k, const
 
 using namespace mfq;
 
-// One query token per sequence, bf16.  part / part_ml: scratch of B * Hq * splits * dv and * 2 floats (splits > 1).
+// One query token per sequence, bf16; Hq counts the queries of all maps.  part / part_ml: scratch of B * Hq * splits * dv and * 2
+// floats (splits > 1 or maps > 1).  Two maps: out [B, Hq / 2, dv] is the normalised difference (see the merge kernel; `d` real
+// value channels).
 extern "C" int mfq_window_attn_decode(const void* q, const void* k, const void* v, const int* table, const int* seq_lens, void* out,
-                                      float* part, float* part_ml, int B, int Hq, int Hk, int dk, int dv, int max_pages, int window,
-                                      float scale, float cap, int splits, cudaStream_t stream) {
-  if (B <= 0 || Hq <= 0 || Hk <= 0 || Hq % Hk || dk % 16 || dv % 16 || dk <= 0 || dv <= 0 || dk > 256 || dv > 256) return -1;
-  if (window <= 0 || !(scale > 0.f) || splits < 1 || (splits > 1 && (!part || !part_ml))) return -1;
+                                      float* part, float* part_ml, int B, int Hq, int Hk, int maps, int dk, int dv, int max_pages, int window,
+                                      int keep, float scale, float cap, int splits, float lambda, float out_scale, float eps, int d,
+                                      cudaStream_t stream) {
+  if (B <= 0 || Hq <= 0 || Hk <= 0 || maps < 1 || maps > 2 || Hq % (Hk * maps) || dk % 16 || dv % 16 || dk <= 0 || dv <= 0) return -1;
+  if (dk * maps > 512 || dv > 256 || keep < 0 || (maps > 1 && (d <= 0 || d > dv))) return -1;
+  if (window <= 0 || !(scale > 0.f) || splits < 1 || ((splits > 1 || maps > 1) && (!part || !part_ml))) return -1;
   const WindowDecodeParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k), static_cast<const __nv_bfloat16*>(v),
-                             table, seq_lens, static_cast<__nv_bfloat16*>(out), part, part_ml, Hq, Hk, dk, dv, max_pages, window, splits,
-                             (Hq / Hk + 15) / 16, make_score_cap(scale, cap)};
-#define MFQ_WIN_DV(DK)                                                 \
-  (dv <= 64 ? launch_window_decode<DK, 64>(p, B, stream)               \
-            : dv <= 128 ? launch_window_decode<DK, 128>(p, B, stream) : launch_window_decode<DK, 256>(p, B, stream))
-  return dk <= 64 ? MFQ_WIN_DV(64) : dk <= 128 ? MFQ_WIN_DV(128) : MFQ_WIN_DV(256);
+                             table, seq_lens, static_cast<__nv_bfloat16*>(out), part, part_ml, Hq, Hk, maps, dk, dv, max_pages, window, keep,
+                             splits, (Hq / Hk + 15) / 16, make_score_cap(scale, cap)};
+  const WindowMergeParams mp{splits, dv, Hq / maps, Hq / Hk / maps, maps, lambda, out_scale, eps, maps > 1 ? 1.f / float(d) : 0.f};
+  const int kw = dk * maps;
+#define MFQ_WIN_DV(DK)                                                     \
+  (dv <= 64 ? launch_window_decode<DK, 64>(p, mp, B, stream)               \
+            : dv <= 128 ? launch_window_decode<DK, 128>(p, mp, B, stream) : launch_window_decode<DK, 256>(p, mp, B, stream))
+  if (kw > 256) return launch_window_decode<512, 256>(p, mp, B, stream);
+  return kw <= 64 ? MFQ_WIN_DV(64) : kw <= 128 ? MFQ_WIN_DV(128) : MFQ_WIN_DV(256);
 #undef MFQ_WIN_DV
 }
 
-// Any number of query tokens: token t sits at positions[t] of the sequence in row tok_seq[t] of the block table.
+// Any number of query tokens: token t sits at positions[t] of the sequence in row tok_seq[t] of the block table.  Writes the
+// output of every map.
 extern "C" int mfq_window_attn_plain(const void* q, const void* k, const void* v, const int* table, const int* tok_seq,
-                                     const int* positions, void* out, int T_, int Hq, int Hk, int dk, int dv, int max_pages, int window,
-                                     float scale, float cap, int fp32, cudaStream_t stream) {
-  if (T_ <= 0 || Hq <= 0 || Hk <= 0 || Hq % Hk || dk % 8 || dv % 8 || dk > 256 || dv > 256 || window <= 0) return -1;
-  const WindowPlainParams p{positions, tok_seq, table, T_, Hq, Hk, dk, dv, max_pages, window, scale, cap};
+                                     const int* positions, void* out, int T_, int Hq, int Hk, int maps, int dk, int dv, int max_pages,
+                                     int window, int keep, float scale, float cap, int fp32, cudaStream_t stream) {
+  if (T_ <= 0 || Hq <= 0 || Hk <= 0 || maps < 1 || Hq % (Hk * maps) || dk % 8 || dv % 8 || dk > 256 || dv > 256 || window <= 0 || keep < 0)
+    return -1;
+  const WindowPlainParams p{positions, tok_seq, table, T_, Hq, Hk, maps, dk, dv, max_pages, window, keep, scale, cap};
   const dim3 grid(unsigned(((long long)(T_) * Hq + 3) / 4));
   if (fp32)
     launch_kernel(window_attn_plain_kernel<float>, grid, dim3(128), 0, stream, static_cast<const float*>(q), static_cast<const float*>(k),

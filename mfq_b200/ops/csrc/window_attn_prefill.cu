@@ -1,15 +1,17 @@
 // Sliding-window attention of prompt portions on tcgen05 tensor cores, bf16, straight from the pages.
 //
 // A batch holds portions of several sequences; the keys and values of their tokens, and of everything before them, are in
-// the pages already.  One CTA = (sequence, run of query tokens, KV head).  The tile's 128 rows are (token, query head of the
+// the pages already.  One CTA = (sequence, run of query tokens, KV head, map).  The tile's 128 rows are (token, query head of the
 // KV head) pairs, so short portions fill it and keys are loaded once per group of heads; row r = token * heads + head, which is
-// the order a 3-D TMA box {64 channels, heads, tokens} of q [T, Hq, dk] delivers.  Per block of KB keys (KB / 16 pages, each
-// one TMA box per 64 channels, page ids from the block table):
+// the order a 3-D TMA box {64 channels, heads, tokens} of q [T, Hq, dk] delivers.  With two maps (differential attention; heads
+// ordered [KV head][map][head of the KV head]) a CTA takes one map: its half of the key row, and the shared values.  Per block of
+// KB keys (KB / 16 pages, each one TMA box per 64 channels, page ids from the block table):
 //   S = Q K^T      tcgen05.mma kind::f16, double-buffered in TMEM
 //   P = softmax    8 warps, two threads per row; the scores' soft cap is a fused polynomial where all of a warp's scores are
 //                  small against the cap, else the exact exponential form; masks only on blocks that need them
 //   O_blk = P V    V as MN-major operand; folded into fp32 registers under the running maximum
-// Only key blocks that some query of the tile can see are visited.  Head widths are multiples of 16 up to 256; channels past a
+// Only key blocks that some query of the tile can see are visited: the pages of the kept first tokens, then those of the window;
+// blocks count these pages without the gap between the two.  Head widths are multiples of 16 up to 256; channels past a
 // width arrive as zeros (TMA fills them).  Pages past the sequence's last are replaced by the last one, so that every byte the
 // tensor core reads is a number (hidden keys have weight zero, and zero times a number is zero).
 #include "window_attn.cuh"
@@ -36,7 +38,7 @@ struct WindowPrefillParams {
   const int* table;     // [B, max_pages]
   __nv_bfloat16* out;   // [T, Hq, dv]
   int* status;
-  int Hq, Hk, dk, dv, max_pages, window, per, tokens;  // per: query heads per KV head; tokens: query tokens per tile
+  int Hq, Hk, maps, dk, dv, max_pages, window, keep, per, tokens;  // per: query heads per KV head and map; tokens: query tokens per tile
   ScoreCap cap;
 };
 
@@ -48,7 +50,8 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
   constexpr int kHalf = KB / 2;      // key columns of a softmax thread
   constexpr int kOut = VS * 32;      // output channels of a softmax thread
   pdl_wait();
-  const int seq = blockIdx.y, kvh = blockIdx.z;
+  const int seq = blockIdx.y, group = blockIdx.z, kvh = group / p.maps;  // group: (KV head, map)
+  const int k_x = (group - kvh * p.maps) * p.dk;                         // first key channel of the map
   const int row0 = p.q_starts[seq], q_len = p.q_starts[seq + 1] - row0;
   const int tiles = (q_len + p.tokens - 1) / p.tokens;
   if (int(blockIdx.x) >= tiles) return;
@@ -57,8 +60,8 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
   const int pos0 = p.seq_lens[seq] - q_len + tok0, pos_last = pos0 + n_tok - 1;
   const int* table = p.table + size_t(seq) * p.max_pages;
   const int first_page = max(0, pos0 - p.window + 1) / kWpPage, last_page = pos_last / kWpPage;
-  const int key_base = first_page * kWpPage;
-  const int nblk = (pos_last - key_base) / KB + 1;
+  const int kept = min((p.keep + kWpPage - 1) / kWpPage, first_page), skip = first_page - kept;  // pages before / not visited
+  const int nblk = (pos_last - skip * kWpPage) / KB + 1;
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -106,7 +109,7 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       tma_prefetch_desc(&tmap_q); tma_prefetch_desc(&tmap_k); tma_prefetch_desc(&tmap_v);
       mbar_expect_tx(q_full, uint32_t(DS) * p.per * p.tokens * 128u);  // boxes are always full: rows past the tensor are zeros
       for (int d = 0; d < DS; ++d)
-        tma_load_3d(sQ + d * (kWpRows * 128), &tmap_q, q_full, d * 64, kvh * p.per, row0 + tok0);
+        tma_load_3d(sQ + d * (kWpRows * 128), &tmap_q, q_full, d * 64, group * p.per, row0 + tok0);
       for (int j = 0; j < nblk; ++j) {
         const int s = j & 1;
         if (!mbar_wait(&kv_empty[s], ((j >> 1) & 1) ^ 1, abort_flag, p.status, kStatusTimeoutProducer)) break;
@@ -115,10 +118,11 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
         mbar_expect_tx(&kv_full[s], Cfg::kStage);
 #pragma unroll 1
         for (int i = 0; i < KB / kWpPage; ++i) {
-          const int page = table[min(first_page + j * (KB / kWpPage) + i, last_page)];
+          const int nth = j * (KB / kWpPage) + i;
+          const int page = table[min(nth < kept ? nth : nth + skip, last_page)];
           const int row = (page * p.Hk + kvh) * kWpPage;
 #pragma unroll
-          for (int d = 0; d < DS; ++d) tma_load_2d(k + d * Cfg::kKSlab + i * (kWpPage * 128), &tmap_k, &kv_full[s], d * 64, row);
+          for (int d = 0; d < DS; ++d) tma_load_2d(k + d * Cfg::kKSlab + i * (kWpPage * 128), &tmap_k, &kv_full[s], k_x + d * 64, row);
 #pragma unroll
           for (int d = 0; d < VS; ++d) tma_load_2d(v + d * Cfg::kKSlab + i * (kWpPage * 128), &tmap_v, &kv_full[s], d * 64, row);
         }
@@ -183,9 +187,10 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       ok = __all_sync(0xffffffffu, mbar_wait(&s_full[sb], (j >> 1) & 1, abort_flag, p.status, kStatusTimeoutEpilogue));
       if (!ok) break;
       tc_fence_after();
-      const int block0 = key_base + j * KB, key0 = block0 + half * kHalf;
-      // a mask is needed where the block reaches past the FIRST query or starts before the LAST query's window
-      const bool masked = block0 + KB - 1 > pos0 || block0 < pos_last - p.window + 1;
+      // places count visited keys; the key at place n is n before the gap (n < kept pages), n + gap after it
+      const int place0 = j * KB + half * kHalf, split = kept * kWpPage, gap = skip * kWpPage;
+      // a mask is needed where the block holds kept pages, reaches past the FIRST query or starts before the LAST query's window
+      const bool masked = j * KB < split || j * KB + gap + KB - 1 > pos0 || j * KB + gap < pos_last - p.window + 1;
       const uint32_t tS = tmem_base + sb * KB + lane_base + half * kHalf;
       float mx = -FLT_MAX, big = 0.f;
 #pragma unroll
@@ -204,8 +209,8 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const float s = __uint_as_float(r[i]);
-            const int key = key0 + c + i;
-            const bool see = key <= q_pos && key >= lo;
+            const int n = place0 + c + i, key = n < split ? n : n + gap;
+            const bool see = key <= q_pos && (key >= lo || key < p.keep);
             mx = fmaxf(mx, see ? s : -FLT_MAX);
             big = fmaxf(big, see ? fabsf(s) : 0.f);
           }
@@ -247,7 +252,10 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
         tmem_ld_32x32(tS + c, r);
         tmem_wait_ld();
         float pr[32];
-        if (small) {
+        if (p.cap.out == 0.f) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) pr[i] = window_exp2(fmaf(__uint_as_float(r[i]), p.cap.scale_log2, -m_new));
+        } else if (small) {
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const float s = __uint_as_float(r[i]), t = s * s;
@@ -261,8 +269,8 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
         if (masked) {
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
-            const int key = key0 + c + i;
-            pr[i] = key <= q_pos && key >= lo ? pr[i] : 0.f;
+            const int n = place0 + c + i, key = n < split ? n : n + gap;
+            pr[i] = key <= q_pos && (key >= lo || key < p.keep) ? pr[i] : 0.f;
           }
         }
         const int col = half * kHalf + c;
@@ -297,7 +305,7 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
         tc_fence_after();
         const float l_tot = l_run + s_max[(4 + (half ^ 1)) * kWpRows + row];
         const float inv = l_tot > 0.f ? 1.f / l_tot : 0.f;
-        const int head = kvh * p.per + row - tok * p.per;
+        const int head = group * p.per + row - tok * p.per;
         __nv_bfloat16* dst = p.out + (size_t(row0 + tok0 + tok) * p.Hq + head) * p.dv + half * kOut;
 #pragma unroll
         for (int c = 0; c < kOut; c += 32) {
@@ -332,14 +340,14 @@ static int launch_window_prefill(const WindowPrefillParams& p, const void* q, co
   CUtensorMap tq, tk, tv;
   if (make_tmap_3d(&tq, q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, p.dk, p.Hq, T, uint64_t(p.dk) * 2, uint64_t(p.Hq) * p.dk * 2, 64, p.per, p.tokens)) return -2;
   const uint64_t rows = uint64_t(pages) * p.Hk * kWpPage;
-  if (make_tmap_2d(&tk, k, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows, p.dk, uint64_t(p.dk) * 2, kWpPage, 64)) return -3;
+  if (make_tmap_2d(&tk, k, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows, p.maps * p.dk, uint64_t(p.maps) * p.dk * 2, kWpPage, 64)) return -3;
   if (make_tmap_2d(&tv, v, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows, p.dv, uint64_t(p.dv) * 2, kWpPage, 64)) return -4;
   static bool attr = false;
   if (!attr) {
     if (cudaFuncSetAttribute(window_attn_prefill_kernel<DS, VS, KB>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmem) != cudaSuccess) return -6;
     attr = true;
   }
-  const dim3 grid((max_q + p.tokens - 1) / p.tokens, B, p.Hk);
+  const dim3 grid((max_q + p.tokens - 1) / p.tokens, B, p.Hk * p.maps);
   launch_kernel(window_attn_prefill_kernel<DS, VS, KB>, grid, dim3(kWpThreads), Cfg::kSmem, stream, tq, tk, tv, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -7;
 }
@@ -349,15 +357,18 @@ static int launch_window_prefill(const WindowPrefillParams& p, const void* q, co
 using namespace mfq;
 
 // Portions of B sequences, longest `max_q` tokens.  q [T, Hq, dk] and out [T, Hq, dv] hold the tokens of all portions (rows
-// q_starts[b] .. q_starts[b + 1] - 1 belong to sequence b), `pages` is the number of pages of the pools.
+// q_starts[b] .. q_starts[b + 1] - 1 belong to sequence b), Hq counts the queries of all maps, `pages` is the number of pages of
+// the pools.
 extern "C" int mfq_window_attn_prefill(const void* q, const void* k, const void* v, const int* table, const int* q_starts,
-                                       const int* seq_lens, void* out, int T, int B, int max_q, int Hq, int Hk, int dk, int dv,
-                                       int pages, int max_pages, int window, float scale, float cap, int* status, cudaStream_t stream) {
-  if (T <= 0 || B <= 0 || B > 65535 || max_q <= 0 || Hq <= 0 || Hk <= 0 || Hk > 65535 || Hq % Hk || Hq / Hk > kWpRows) return -1;
+                                       const int* seq_lens, void* out, int T, int B, int max_q, int Hq, int Hk, int maps, int dk, int dv,
+                                       int pages, int max_pages, int window, int keep, float scale, float cap, int* status,
+                                       cudaStream_t stream) {
+  if (T <= 0 || B <= 0 || B > 65535 || max_q <= 0 || Hq <= 0 || Hk <= 0 || maps < 1 || maps > 2 || Hk * maps > 65535) return -1;
+  if (Hq % (Hk * maps) || Hq / (Hk * maps) > kWpRows || keep < 0) return -1;
   if (dk % 16 || dv % 16 || dk <= 0 || dv <= 0 || dk > 256 || dv > 256 || window <= 0 || !(scale > 0.f)) return -1;
-  const int per = Hq / Hk;
-  const WindowPrefillParams p{q_starts, seq_lens, table, static_cast<__nv_bfloat16*>(out), status, Hq, Hk, dk, dv, max_pages, window,
-                              per, kWpRows / per, make_score_cap(scale, cap)};
+  const int per = Hq / (Hk * maps);
+  const WindowPrefillParams p{q_starts, seq_lens, table, static_cast<__nv_bfloat16*>(out), status, Hq, Hk, maps, dk, dv, max_pages, window,
+                              keep, per, kWpRows / per, make_score_cap(scale, cap)};
   const int ds = (dk + 63) / 64, vs = (dv + 63) / 64;
 #define MFQ_WP(DS, VS, KB) return launch_window_prefill<DS, VS, KB>(p, q, k, v, T, pages, B, max_q, stream)
   if (ds == 1 && vs == 1) MFQ_WP(1, 1, 128);

@@ -13,7 +13,7 @@ import torch
 
 from .lib import Workspace, check, dense_lib, ptr, stream_ptr
 
-BIAS, GLU, GELU = 0, 1, 2  # epilogues (dense_common.cuh)
+BIAS, GLU, GELU, GELU_GLU, SOFTCAP, ADD = range(6)  # epilogues (dense_common.cuh)
 GEMV_ROWS, GEMV_MID_ROWS, GEMV_MID_WEIGHTS = 8, 16, 8 << 20
 
 
@@ -63,11 +63,11 @@ def plan(m: int, n: int, k: int, sms: int = 148) -> tuple[int, int]:
 @dataclass
 class DenseLinear:
     """``[rows, cols]`` weight (rows a multiple of 16, cols of 8) with an optional fp32 bias.  ``glu``: the rows alternate
-    between 8 gate and 8 up rows (:func:`interleave_glu`) and the output is the clipped GLU of the two, half as wide."""
+    between 8 gate and 8 up rows (:func:`interleave_glu`) and the output is the gated unit of the two, half as wide."""
 
     w: torch.Tensor
     bias: torch.Tensor | None = None
-    glu: tuple[float, float] | None = None  # (alpha, limit)
+    glu: tuple[float, float] | str | None = None  # (alpha, limit) of the clipped GLU, or "gelu": gelu_tanh(gate) * up
     input_kind = "dense"
 
     @property
@@ -75,15 +75,26 @@ class DenseLinear:
         return self.w.shape[0] // (2 if self.glu is not None else 1)
 
     def __call__(self, x: torch.Tensor, *, table: torch.Tensor | None = None, ids: torch.Tensor | None = None,
-                 out: torch.Tensor | None = None, tile: int | None = None, splits: int | None = None) -> torch.Tensor:
-        """``x [M, cols]``.  ``table`` (``[vocabulary, rows]``) with ``ids [M]``: the result is ``gelu_tanh(y) * table[ids]``."""
+                 softcap: float = 0.0, add_to: torch.Tensor | None = None, out: torch.Tensor | None = None, tile: int | None = None,
+                 splits: int | None = None) -> torch.Tensor:
+        """``x [M, cols]``.  ``table`` (``[vocabulary, rows]``) with ``ids [M]``: the result is ``gelu_tanh(y) * table[ids]``;
+        ``softcap`` c > 0: ``c tanh(y / c)``; ``add_to``: ``y`` is added to this fp32 stream, which is also the result."""
         m, n, k = x.shape[0], self.w.shape[0], self.w.shape[1]
         assert x.shape[1] == k and x.stride(1) == 1 and x.dtype == self.w.dtype and self.w.is_contiguous()
-        if out is None:
+        if add_to is not None:
+            assert self.glu is None and add_to.dtype == torch.float32 and add_to.shape == (m, n) and add_to.stride(1) == 1
+            out = add_to
+        elif out is None:
             out = torch.empty((m, self.out_width), dtype=x.dtype, device=x.device)
         kind, alpha, limit = BIAS, 0.0, 0.0
-        if self.glu is not None:
+        if self.glu == "gelu":
+            kind = GELU_GLU
+        elif self.glu is not None:
             kind, (alpha, limit) = GLU, self.glu
+        elif add_to is not None:
+            kind = ADD
+        elif softcap > 0:
+            kind, limit = SOFTCAP, softcap
         elif table is not None:
             assert table.shape[1] == n and table.is_contiguous() and table.dtype == x.dtype and ids.dtype == torch.int32
             kind = GELU
@@ -102,11 +113,12 @@ def interleave_glu(gate: torch.Tensor, up_: torch.Tensor) -> torch.Tensor:
     return torch.stack([gate.reshape(f // 8, 8, k), up_.reshape(f // 8, 8, k)], 1).reshape(2 * f, k).contiguous()
 
 
-def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float):
-    """``(x, act)``: the fp32 stream ``table[ids] * scale`` and its copy in the activation type (the same tensor in fp32)."""
+def embed_scaled(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0, copy: bool = True):
+    """``(x, act)``: the fp32 stream ``table[ids] * scale`` and its copy in the activation type (the same tensor in fp32, or
+    without ``copy``)."""
     t, w = ids.numel(), table.shape[1]
     x = torch.empty((t, w), dtype=torch.float32, device=table.device)
-    act = None if table.dtype == torch.float32 else torch.empty((t, w), dtype=table.dtype, device=table.device)
+    act = None if table.dtype == torch.float32 or not copy else torch.empty((t, w), dtype=table.dtype, device=table.device)
     check(dense_lib().mfq_embed_scaled(ptr(ids), ptr(table), float(scale), ptr(x), ptr(act), t, w, is_fp32(table.dtype), stream_ptr()),
           "embed_scaled")
     return x, (x if act is None else act)

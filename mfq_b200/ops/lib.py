@@ -59,10 +59,13 @@ _DENSE_SIGNATURES = {
     "mfq_embed_scaled": [_vp, _vp, _f, _vp, _vp, _i, _i, _i, _vp],
     "mfq_norm_add": [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _vp],
     "mfq_norm_out": [_vp, _vp, _vp, _i, _i, _i, _f, _i, _vp],
-    "mfq_qkv_finish": [_vp, _i, _vp, _i, _f, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp],
-    "mfq_window_attn_decode": [_vp] * 8 + [_i, _i, _i, _i, _i, _i, _i, _f, _f, _i, _vp],
-    "mfq_window_attn_plain": [_vp] * 7 + [_i, _i, _i, _i, _i, _i, _i, _f, _f, _i, _vp],
-    "mfq_window_attn_prefill": [_vp] * 7 + [_i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _f, _vp, _vp],
+    "mfq_qkv_finish": [_vp, _i, _vp, _i, _f] + [_vp] * 8 + [_i] * 11 + [_f, _i, _vp],
+    "mfq_map_difference": [_vp, _vp, _i, _i, _i, _i, _i, _f, _f, _f, _i, _vp],
+    "mfq_window_attn_decode": [_vp] * 8 + [_i] * 9 + [_f, _f, _i, _f, _f, _f, _i, _vp],
+    "mfq_window_attn_plain": [_vp] * 7 + [_i] * 9 + [_f, _f, _i, _vp],
+    "mfq_window_attn_prefill": [_vp] * 7 + [_i] * 12 + [_f, _f, _vp, _vp],
+    "mfq_gla_recurrent": [_vp] * 8 + [_i] * 8 + [_f, _f, _f, _i, _vp],
+    "mfq_gla_chunk": [_vp] * 11 + [_i] * 8 + [_f, _f, _f, _vp],
 }
 
 

@@ -1,12 +1,20 @@
-"""Attention over unquantized pages with a sliding window and an optional score cap (``csrc/window_attn*.cu``), and the
-per-head stage in front of it (``csrc/stream_ops.cu``).
+"""Attention over unquantized pages with a sliding window, kept first tokens, an optional score cap and one or two maps
+(``csrc/window_attn*.cu``), and the per-head stage in front of it (``csrc/stream_ops.cu``).
 
-A query at position ``i`` sees the keys ``j`` with ``0 <= i - j < window``; a score is ``q . k * scale``, then
-``cap * tanh(score / cap)`` (``cap`` 0: no cap).  Pages: ``k [pages, Hk, 16, dk]``, ``v [pages, Hk, 16, dv]``, widths multiples
-of 16 up to 256.  bf16 runs on tensor cores (one kernel for portions of prompts, one for single tokens), fp32 on a plain kernel.
+A query at position ``i`` sees the keys ``j <= i`` with ``i - j < window`` or ``j < keep``; a score is ``q . k * scale``, then
+``cap * tanh(score / cap)`` (``cap`` 0: no cap).  Pages: ``k [pages, Hk, 16, maps * dk]``, ``v [pages, Hk, 16, dv]``, widths
+``dk`` and ``dv`` multiples of 16 up to 256.  bf16 runs on tensor cores (one kernel for portions of prompts, one for single
+tokens), fp32 on a plain kernel.
+
+Two maps (differential attention): every query and KV head has two query / key vectors that attend on their own over the same
+values; a head's output is ``rms(a1 - lambda a2) * scale`` (:class:`Difference`).  Queries are ordered ``[KV head][map][query
+head of the KV head]``.
 """
 
 from __future__ import annotations
+
+import math
+from dataclasses import dataclass
 
 import torch
 
@@ -17,27 +25,73 @@ MAX_HEAD = 256
 NO_WINDOW = 1 << 30
 
 
-def rope_table(base: float, dims: int, positions: int, device) -> torch.Tensor:
-    """``[positions, dims / 2, 2]`` fp32 (cos, sin) of ``p * base^(-2i / dims)``, evaluated in double precision."""
-    freq = torch.tensor([float(base) ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64, device=device)
+@dataclass(frozen=True)
+class Difference:
+    """How the two maps of a head are combined."""
+
+    weight: float  # lambda
+    scale: float
+    eps: float
+    dim: int  # real value channels
+
+
+@dataclass(frozen=True)
+class FrequencyScaling:
+    """Rotation frequencies for contexts longer than the original one: frequencies that turn less than ``low`` times over the
+    original context are divided by ``factor``, those that turn more than ``high`` times are kept, with a linear blend between."""
+
+    factor: float
+    low: float
+    high: float
+    original: float
+
+    def __call__(self, f: float) -> float:
+        turns = self.original * f / (2 * math.pi)
+        if turns > self.high:
+            return f
+        if turns < self.low:
+            return f / self.factor
+        s = (turns - self.low) / (self.high - self.low) if self.high > self.low else 1.0
+        return (1 - s) * f / self.factor + s * f
+
+
+def rope_table(base: float, dims: int, positions: int, device, scaling: FrequencyScaling | None = None) -> torch.Tensor:
+    """``[positions, dims / 2, 2]`` fp32 (cos, sin) of ``p * f_i``, ``f_i = base^(-2i / dims)`` (scaled), in double precision."""
+    freq = [float(base) ** (-2.0 * i / dims) for i in range(dims // 2)]
+    freq = torch.tensor([scaling(f) for f in freq] if scaling is not None else freq, dtype=torch.float64, device=device)
     a = torch.arange(positions, dtype=torch.float64, device=device)[:, None] * freq
     return torch.stack([a.cos(), a.sin()], -1).float().contiguous()
 
 
 def qkv_finish(qkv: torch.Tensor, kv, positions, slots, *, heads: int, kv_heads: int, dim: int, q_norm, k_norm, rope, rot: int,
-               eps: float, v_first: torch.Tensor | None = None, mix: float = 0.0) -> torch.Tensor:
-    """Per-head RMS norm of q and k (over ``dim`` channels), rotation of the leading ``rot`` channels, K and V into their
-    pages; returns ``q [T, heads, dk]``.  ``v_first`` (``[T, kv_heads * dv]``, rows may be strided): the cached values are
-    ``(1 - mix) v + mix v_first``."""
+               eps: float, v_first: torch.Tensor | None = None, mix: float = 0.0, maps: int = 1, pairs: bool = False,
+               dk: int | None = None) -> torch.Tensor:
+    """Per-head RMS norm of q and k (over ``dim`` channels; no norm without weights), rotation of the leading ``rot`` channels
+    (``i`` with ``i + rot / 2``, or with its neighbour: ``pairs``), K and V into their pages; returns ``q [T, maps * heads, dk]``.
+    ``v_first`` (``[T, kv_heads * dv]``, rows may be strided): the cached values are ``(1 - mix) v + mix v_first``.  ``kv`` None:
+    the rows hold queries only (of stored width ``dk``)."""
     t = qkv.shape[0]
-    dk, dv = kv.k.shape[-1], kv.v.shape[-1]
-    q = torch.empty((t, heads, dk), dtype=qkv.dtype, device=qkv.device)
+    if kv is not None:
+        dk, dv, page = kv.k.shape[-1] // maps, kv.v.shape[-1], kv.page_size
+    else:
+        dv = page = 0
+    q = torch.empty((t, maps * heads, dk), dtype=qkv.dtype, device=qkv.device)
     rc = dense_lib().mfq_qkv_finish(ptr(qkv), qkv.stride(0), ptr(v_first), v_first.stride(0) if v_first is not None else 0, float(mix),
-                                    ptr(q), ptr(kv.k), ptr(kv.v), ptr(positions), ptr(slots), ptr(q_norm), ptr(k_norm), ptr(rope),
-                                    rope.shape[0] if rope is not None else 0, t, heads, kv_heads, dim, dk, dv, rot, kv.page_size,
-                                    float(eps), is_fp32(qkv.dtype), stream_ptr())
+                                    ptr(q), ptr(kv.k) if kv is not None else None, ptr(kv.v) if kv is not None else None, ptr(positions),
+                                    ptr(slots), ptr(q_norm), ptr(k_norm), ptr(rope), rope.shape[0] if rope is not None else 0, t,
+                                    maps * heads, kv_heads, maps, dim, dk, dv, rot, int(pairs), page, float(eps), is_fp32(qkv.dtype),
+                                    stream_ptr())
     check(rc, "qkv_finish")
     return q
+
+
+def difference(a: torch.Tensor, kv_heads: int, d: Difference, out: torch.Tensor | None = None) -> torch.Tensor:
+    """``a [T, 2 * H, dv]`` (both maps of every head, in query order) -> ``[T, H, dv]``."""
+    t, rows, dv = a.shape
+    out = torch.empty((t, rows // 2, dv), dtype=a.dtype, device=a.device) if out is None else out
+    check(dense_lib().mfq_map_difference(ptr(a), ptr(out), t, rows // 2, rows // 2 // kv_heads, dv, d.dim, d.weight, d.scale, d.eps,
+                                         is_fp32(a.dtype), stream_ptr()), "map_difference")
+    return out
 
 
 def decode_splits(batch: int, kv_heads: int, keys: int) -> int:
@@ -54,40 +108,52 @@ def decode_splits(batch: int, kv_heads: int, keys: int) -> int:
     return min(choices, key=lambda s: -(-n * s // slots) * keys / s + 20 * s)
 
 
-def decode(q: torch.Tensor, kv, block_table, seq_lens, *, window: int, scale: float, cap: float, splits: int = 1, out=None):
-    """One query token per sequence (bf16): ``q [B, Hq, dk]`` -> ``[B, Hq, dv]``; ``seq_lens`` count the query token."""
+def decode(q: torch.Tensor, kv, block_table, seq_lens, *, window: int, scale: float, cap: float, keep: int = 0,
+           diff: Difference | None = None, splits: int = 1, out=None):
+    """One query token per sequence (bf16): ``q [B, Hq, dk]`` -> ``[B, Hq, dv]``, or ``[B, Hq / 2, dv]`` with ``diff``;
+    ``seq_lens`` count the query token."""
     b, hq, dk = q.shape
     hk, dv = kv.k.shape[1], kv.v.shape[-1]
-    out = torch.empty((b, hq, dv), dtype=q.dtype, device=q.device) if out is None else out
+    maps = 1 if diff is None else 2
+    out = torch.empty((b, hq // maps, dv), dtype=q.dtype, device=q.device) if out is None else out
     ws = Workspace.get(q.device)
-    assert splits == 1 or (b * hq * splits * dv <= ws.attn_acc.numel() and b * hq * splits * 2 <= ws.attn_ml.numel())
+    parts = splits > 1 or maps > 1
+    assert kv.k.shape[-1] == maps * dk
+    assert not parts or (b * hq * splits * dv <= ws.attn_acc.numel() and b * hq * splits * 2 <= ws.attn_ml.numel())
+    how = (diff.weight, diff.scale, diff.eps, diff.dim) if diff is not None else (0.0, 1.0, 0.0, dv)
     rc = dense_lib().mfq_window_attn_decode(ptr(q), ptr(kv.k), ptr(kv.v), ptr(block_table), ptr(seq_lens), ptr(out), ptr(ws.attn_acc),
-                                            ptr(ws.attn_ml), b, hq, hk, dk, dv, block_table.stride(0), window, float(scale), float(cap),
-                                            splits, stream_ptr())
-    check(rc, "window_attn_decode", 2 if splits > 1 else 1)
+                                            ptr(ws.attn_ml), b, hq, hk, maps, dk, dv, block_table.stride(0), window, keep, float(scale),
+                                            float(cap), splits, *how, stream_ptr())
+    check(rc, "window_attn_decode", 2 if parts else 1)
     return out
 
 
-def prefill(q: torch.Tensor, kv, block_table, q_starts, seq_lens, max_q: int, *, window: int, scale: float, cap: float, out=None):
+def prefill(q: torch.Tensor, kv, block_table, q_starts, seq_lens, max_q: int, *, window: int, scale: float, cap: float, keep: int = 0,
+            maps: int = 1, out=None):
     """Portions of several sequences (bf16): rows ``q_starts[b] .. q_starts[b + 1] - 1`` of ``q [T, Hq, dk]`` are the last
-    tokens of a sequence of ``seq_lens[b]``.  ``max_q``: the longest portion (host)."""
+    tokens of a sequence of ``seq_lens[b]``.  ``max_q``: the longest portion (host).  Writes the output of every map."""
     t, hq, dk = q.shape
     hk, dv = kv.k.shape[1], kv.v.shape[-1]
     out = torch.empty((t, hq, dv), dtype=q.dtype, device=q.device) if out is None else out
     rc = dense_lib().mfq_window_attn_prefill(ptr(q), ptr(kv.k), ptr(kv.v), ptr(block_table), ptr(q_starts), ptr(seq_lens), ptr(out), t,
-                                             seq_lens.numel(), max_q, hq, hk, dk, dv, kv.k.shape[0], block_table.stride(0), window,
-                                             float(scale), float(cap), ptr(Workspace.get(q.device).status), stream_ptr())
+                                             seq_lens.numel(), max_q, hq, hk, maps, dk, dv, kv.k.shape[0], block_table.stride(0), window,
+                                             keep, float(scale), float(cap), ptr(Workspace.get(q.device).status), stream_ptr())
     check(rc, "window_attn_prefill")
     return out
 
 
-def plain(q: torch.Tensor, kv, block_table, tok_seq, positions, *, window: int, scale: float, cap: float):
+def plain(q: torch.Tensor, kv, block_table, tok_seq, positions, *, window: int, scale: float, cap: float, keep: int = 0, maps: int = 1):
     """The same in fp32 arithmetic for any mix of tokens: token ``t`` is at ``positions[t]`` of sequence ``tok_seq[t]``."""
     t, hq, dk = q.shape
     hk, dv = kv.k.shape[1], kv.v.shape[-1]
     out = torch.empty((t, hq, dv), dtype=q.dtype, device=q.device)
     rc = dense_lib().mfq_window_attn_plain(ptr(q), ptr(kv.k), ptr(kv.v), ptr(block_table), ptr(tok_seq), ptr(positions), ptr(out), t, hq,
-                                           hk, dk, dv, block_table.stride(0), window, float(scale), float(cap), is_fp32(q.dtype),
-                                           stream_ptr())
+                                           hk, maps, dk, dv, block_table.stride(0), window, keep, float(scale), float(cap),
+                                           is_fp32(q.dtype), stream_ptr())
     check(rc, "window_attn_plain")
     return out
+
+
+def visible_keys(length: int, window: int, keep: int) -> int:
+    """Most keys a query of a sequence of ``length`` tokens sees."""
+    return min(length, window + keep)

@@ -147,11 +147,15 @@ def model_memory(cfg: dict, weight_bytes: int, *, batch: int = 1, context: int =
     tp = max(1, int(tensor_parallel))
     pages = batch * math.ceil(context / PAGE_TOKENS) + 1
     kv = pages * page_bytes(p["attention_layers"], max(1, hk // tp), d)
+    state = 0
     if cfg.get("family") == "tepetar":  # bf16 pages, every layer its own geometry
         from ..models.tepetar import TepetarConfig
         kv = pages * PAGE_TOKENS * TepetarConfig.from_dict(cfg).kv_token_bytes(2)
+    elif cfg.get("family") == "kamedra":  # the same, plus a recurrent state per sequence
+        from ..models.kamedra import KamedraConfig
+        own = KamedraConfig.from_dict(cfg)
+        kv, state = pages * PAGE_TOKENS * own.kv_token_bytes(2), batch * own.state_bytes()
     lin_v = _cfg_int(cfg, "linear_num_value_heads")
-    state = 0
     if lin_v:
         lin_layers = p["layers"] - p["attention_layers"]
         dk, dv = _cfg_int(cfg, "linear_key_head_dim", default=128), _cfg_int(cfg, "linear_value_head_dim", default=128)
