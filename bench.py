@@ -387,25 +387,29 @@ TEPETAR_SIZES = {  # width, ff, layers, query / KV heads of 128 channels, vocabu
 }
 
 
-def run_tepetar(args) -> dict:
-    """The Tepetar family (bf16, sliding windows, score cap, shared values, token side input) beside the FP8 Llama of equal
-    geometry: prefill of one prompt and decode at batch 1 and ``--batch``, both through the same engine (one GPU)."""
-    import torch
+KAMEDRA_SIZES = {  # width, ff, layers, query / KV heads (two maps of 64 channels, values of 128), linear heads (128 x 256), vocabulary
+    "1b": (2048, 8192, 16, 16, 4, 8, 65536),
+    "3b": (3072, 8192, 28, 24, 8, 12, 65536),
+    "8b": (4096, 14336, 32, 32, 8, 16, 128256),
+}
 
-    from mfq_b200 import ops
-    from mfq_b200.engine.llm_engine import LLMEngine
-    from mfq_b200.models.llama import LlamaConfig, LlamaModel, LlamaWeights
-    from mfq_b200.models.tepetar import RandomTensors, TepetarConfig, TepetarModel, TepetarWeights
 
-    if args.gpus != 1:
-        raise SystemExit("--model tepetar runs on one GPU")
-    dev = torch.device("cuda", 0)
-    torch.cuda.set_device(dev)
-    ops.count_launches(True)
-    ctx, new = args.context, 4 * (args.steps + args.warmup) + 16
-    gen = torch.Generator().manual_seed(1234)
+class FamilyBench:
+    """Prefill of one prompt and decode at batch 1 and ``--batch`` of several models through the same engine (one GPU)."""
 
-    def timed(fn, steps, warmup):
+    def __init__(self, args) -> None:
+        import torch
+
+        from mfq_b200 import ops
+        if args.gpus != 1:
+            raise SystemExit(f"--model {args.model} runs on one GPU")
+        self.args, self.dev, self.table = args, torch.device("cuda", 0), {}
+        torch.cuda.set_device(self.dev)
+        ops.count_launches(True)
+        self.gen = torch.Generator().manual_seed(1234)
+
+    def _timed(self, fn, steps, warmup):
+        import torch
         for _ in range(warmup):
             fn()
         torch.cuda.synchronize()
@@ -418,54 +422,99 @@ def run_tepetar(args) -> dict:
             torch.cuda.synchronize()
         return a.elapsed_time(z) / steps, clocks.summary()
 
-    def measure(model, vocab):
+    def add(self, name: str, model, vocab: int, **facts) -> None:
+        import torch
+
+        from mfq_b200 import ops
+        from mfq_b200.engine.llm_engine import LLMEngine
+        args, ctx = self.args, self.args.context
+        new = 4 * (args.steps + args.warmup) + 16
         engine = LLMEngine(model, max_batch=args.batch, max_seq_len=ctx + new)
-        prompts = [torch.randint(0, vocab, (ctx,), generator=gen) for _ in range(args.batch)]
-        prefill_ms, _ = timed(lambda: engine.prefill(0, prompts[0]), 3, 3)
+        prompts = [torch.randint(0, vocab, (ctx,), generator=self.gen) for _ in range(args.batch)]
+        prefill_ms, _ = self._timed(lambda: engine.prefill(0, prompts[0]), 3, 3)
         for row, prompt in enumerate(prompts):
             engine.prefill(row, prompt)
             engine.grow(row, ctx + new)
-        ms, clocks = timed(lambda: engine.decode_step(args.batch), args.steps, args.warmup)
-        ms1, _ = timed(lambda: engine.decode_step(1), args.steps, args.warmup)
+        ms, clocks = self._timed(lambda: engine.decode_step(args.batch), args.steps, args.warmup)
+        ms1, _ = self._timed(lambda: engine.decode_step(1), args.steps, args.warmup)
         host_in = engine.sampled[: args.batch].cpu().pin_memory()
         host_out = torch.zeros_like(host_in).pin_memory()
-        e2e, _ = timed(lambda: engine.step_host(host_in, host_out), args.steps, args.warmup)
-        ops.Workspace.get(dev).check()
-        return {"prefill_tok_s": round(ctx / prefill_ms * 1e3, 1), "prefill_ms": round(prefill_ms, 3),
-                "decode_ms": round(ms, 4), "decode_tok_s": round(args.batch / ms * 1e3, 1), "decode_ms_bs1": round(ms1, 4),
-                "decode_tok_s_bs1": round(1e3 / ms1, 1), "e2e_tok_s": round(args.batch / e2e * 1e3, 1), "clocks": clocks,
-                "launches_per_step": engine.launches_per_step.get(args.batch)}
+        e2e, _ = self._timed(lambda: engine.step_host(host_in, host_out), args.steps, args.warmup)
+        ops.Workspace.get(self.dev).check()
+        row = {**facts, "prefill_tok_s": round(ctx / prefill_ms * 1e3, 1), "prefill_ms": round(prefill_ms, 3),
+               "decode_ms": round(ms, 4), "decode_tok_s": round(args.batch / ms * 1e3, 1), "decode_ms_bs1": round(ms1, 4),
+               "decode_tok_s_bs1": round(1e3 / ms1, 1), "e2e_tok_s": round(args.batch / e2e * 1e3, 1), "clocks": clocks,
+               "launches_per_step": engine.launches_per_step.get(args.batch)}
+        self.table[name] = row
+        print(f"[bench] {name} {json.dumps(row)}", file=sys.stderr, flush=True)
+        del engine
+        torch.cuda.empty_cache()
 
-    table = {}
+    def result(self) -> dict:
+        args = self.args
+        name, first = next(iter(self.table.items()))
+        return {"metric": f"decode_tok_s_bs{args.batch}", "value": first["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
+                "warmup": args.warmup, "ms_per_step": first["decode_ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+                "dtype": "bf16 weights/activations/KV, fp32 stream, norms and scores", "impl": "ours",
+                "data": "synthetic (uniform random token ids, random-init weights)",
+                "config": {"model": name, "global_batch": args.batch, "seq_len": args.context, "parallelism": "dp1",
+                           "l2": "inputs larger than L2 (every step streams all weights)"},
+                "clocks": first["clocks"],
+                "e2e": {"value": first["e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 4 * args.batch, "d2h_bytes_per_step": 4 * args.batch},
+                "gpu_launches": (first["launches_per_step"] or 0) * args.steps, "extra": self.table}
+
+
+def _facts(cfg, weights=None) -> dict:
+    out = {"params_b": round(cfg.param_count() / 1e9, 3)}
+    return out if weights is None else {**out, "weights_gb": round(weights.nbytes() / 1e9, 2)}
+
+
+def _tepetar(dev, width, ff, layers, hq, hk, vocab, side, window):
+    from mfq_b200.models.tepetar import RandomTensors, TepetarConfig, TepetarModel, TepetarWeights
+    cfg = TepetarConfig.uniform(vocab_size=vocab, hidden_size=width, num_layers=layers, heads=hq, kv_heads=hk, dim=128, vdim=128,
+                                window=window, ff=ff, side_dim=side)
+    weights = TepetarWeights(cfg, RandomTensors(cfg, dev), dev)
+    return TepetarModel(cfg, weights), _facts(cfg, weights)
+
+
+def run_tepetar(args) -> dict:
+    """The Tepetar family (bf16, sliding windows, score cap, shared values, token side input) beside the FP8 Llama of equal
+    geometry."""
+    from mfq_b200.models.llama import LlamaConfig, LlamaModel, LlamaWeights
+    bench = FamilyBench(args)
     for size in (args.size.split(",") if args.size else ["1b", "8b"]):
         width, ff, layers, hq, hk, vocab, side = TEPETAR_SIZES[size]
         if args.tiny:
             width, ff, layers, hq, hk, vocab = 256, 512, 2, 4, 2, 1024
         for window in (int(w) for w in args.window.split(",")):
-            cfg = TepetarConfig.uniform(vocab_size=vocab, hidden_size=width, num_layers=layers, heads=hq, kv_heads=hk, dim=128, vdim=128,
-                                        window=window, ff=ff, side_dim=side)
-            weights = TepetarWeights(cfg, RandomTensors(cfg, dev), dev)
-            row = {"params_b": round(cfg.param_count() / 1e9, 3), "weights_gb": round(weights.nbytes() / 1e9, 2),
-                   **measure(TepetarModel(cfg, weights), vocab)}
-            table[f"tepetar-{size}-w{window}"] = row
-            print(f"[bench] tepetar-{size}-w{window} {json.dumps(row)}", file=sys.stderr, flush=True)
-            del weights
-            torch.cuda.empty_cache()
+            model, facts = _tepetar(bench.dev, width, ff, layers, hq, hk, vocab, side, window)
+            bench.add(f"tepetar-{size}-w{window}", model, vocab, **facts)
+            del model
         cfg = LlamaConfig(vocab_size=vocab, hidden_size=width, intermediate_size=ff, num_layers=layers, num_heads=hq, num_kv_heads=hk)
-        row = {"params_b": round(cfg.param_count() / 1e9, 3), **measure(LlamaModel(cfg, LlamaWeights.random_init(cfg, dev)), vocab)}
-        table[f"llama-fp8-{size}"] = row
-        print(f"[bench] llama-fp8-{size} {json.dumps(row)}", file=sys.stderr, flush=True)
-        torch.cuda.empty_cache()
-    name, first = next(iter(table.items()))
-    return {"metric": f"decode_tok_s_bs{args.batch}", "value": first["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
-            "warmup": args.warmup, "ms_per_step": first["decode_ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
-            "dtype": "bf16 weights/activations/KV, fp32 stream, norms and scores", "impl": "ours",
-            "data": "synthetic (uniform random token ids, random-init weights)",
-            "config": {"model": name, "global_batch": args.batch, "seq_len": ctx, "parallelism": "dp1",
-                       "l2": "inputs larger than L2 (every step streams all weights)"},
-            "clocks": first["clocks"],
-            "e2e": {"value": first["e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 4 * args.batch, "d2h_bytes_per_step": 4 * args.batch},
-            "gpu_launches": (first["launches_per_step"] or 0) * args.steps, "extra": table}
+        bench.add(f"llama-fp8-{size}", LlamaModel(cfg, LlamaWeights.random_init(cfg, bench.dev)), vocab, **_facts(cfg))
+    return bench.result()
+
+
+def run_kamedra(args) -> dict:
+    """The Kamedra family (bf16; every fourth layer differential attention in a window with 64 kept tokens, the others gated
+    linear attention) beside the Tepetar of equal width, depth, feed-forward, heads and window."""
+    from mfq_b200.models.kamedra import AttentionSpec, GlaSpec, KamedraConfig, KamedraModel, KamedraWeights, RandomTensors
+    bench = FamilyBench(args)
+    for size in (args.size.split(",") if args.size else ["1b", "8b"]):
+        width, ff, layers, hq, hk, hl, vocab = KAMEDRA_SIZES[size]
+        if args.tiny:
+            width, ff, layers, hq, hk, hl, vocab = 256, 512, 4, 4, 2, 2, 1024
+        for window in (int(w) for w in args.window.split(",")):
+            attention = AttentionSpec(hq, hk, 64, 128, 0.125, 0.5, window=window, keep=64, rot_dims=64, rot_base=5e5)
+            cfg = KamedraConfig.periodic(vocab_size=vocab, hidden_size=width, num_layers=layers, attention=attention,
+                                         linear=GlaSpec(hl, 128, 256, 16.0, rank=16), ff=ff)
+            weights = KamedraWeights(cfg, RandomTensors(cfg, bench.dev), bench.dev)
+            bench.add(f"kamedra-{size}-w{window}", KamedraModel(cfg, weights), vocab, **_facts(cfg, weights))
+            del weights
+            model, facts = _tepetar(bench.dev, width, ff, layers, hq, hk, vocab, 128, window)
+            bench.add(f"tepetar-{size}-w{window}", model, vocab, **facts)
+            del model
+    return bench.result()
 
 
 def run_reference(args) -> dict:
@@ -493,18 +542,19 @@ def main() -> None:
     ap.add_argument("--profile-steps", type=int, default=0,
                     help="after the timed region, run this many batched decode steps between cudaProfilerStart/Stop")
     ap.add_argument("--tiny", action="store_true", help="tiny model, for checking the harness itself")
-    ap.add_argument("--model", choices=["llama8b", "hybrid80b", "tepetar"], default="llama8b",
+    ap.add_argument("--model", choices=["llama8b", "hybrid80b", "tepetar", "kamedra"], default="llama8b",
                     help="llama8b: the flagship; hybrid80b: the Gated-DeltaNet + MoE hybrid with an MTP head (one GPU); "
-                         "tepetar: that family in bf16 beside the FP8 Llama of equal geometry (one GPU)")
-    ap.add_argument("--size", default="", help="tepetar: comma separated sizes out of " + ", ".join(TEPETAR_SIZES) + " (default 1b,8b)")
-    ap.add_argument("--window", default="4096,1024", help="tepetar: comma separated window sizes")
+                         "tepetar: that family in bf16 beside the FP8 Llama of equal geometry (one GPU); "
+                         "kamedra: that family in bf16 beside the Tepetar of equal geometry (one GPU)")
+    ap.add_argument("--size", default="", help="tepetar, kamedra: comma separated sizes out of " + ", ".join(TEPETAR_SIZES) + " (default 1b,8b)")
+    ap.add_argument("--window", default="4096,1024", help="tepetar, kamedra: comma separated window sizes")
     args = ap.parse_args()
     if args.warmup < 3:
         args.warmup = 3
     if args.impl == "reference":
         out = run_reference(args)
     else:
-        out = {"hybrid80b": run_hybrid, "tepetar": run_tepetar}.get(args.model, run_ours)(args)
+        out = {"hybrid80b": run_hybrid, "tepetar": run_tepetar, "kamedra": run_kamedra}.get(args.model, run_ours)(args)
     if out:
         print(json.dumps(out), flush=True)
 

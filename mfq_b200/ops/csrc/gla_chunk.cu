@@ -19,7 +19,7 @@
 namespace mfq {
 namespace {
 
-constexpr int kGc = 64, kGcThreads = 256, kGcMaxDk = 256, kGcMaxDv = 512;
+constexpr int kGc = 64, kGcThreads = 512, kGcWarps = kGcThreads / 32, kGcMaxDk = 256, kGcMaxDv = 512;
 constexpr float kGcSpan = 100.f;
 
 struct GlaChunkParams {
@@ -42,6 +42,13 @@ __device__ __forceinline__ float gc_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+// log2(sigmoid(z)) and silu to a few units of 2^-23 (absolute, relative)
+__device__ __forceinline__ float gc_log2_sigmoid(float z) {
+  float y;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(1.f + gc_exp2(-1.4426950408889634f * fabsf(z))));
+  return fmaf(1.4426950408889634f, fminf(z, 0.f), -y);
+}
+__device__ __forceinline__ float gc_silu(float x) { return __fdividef(x, 1.f + gc_exp2(-1.4426950408889634f * fmaxf(x, -80.f))); }
 __device__ __forceinline__ void gc_cp16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
@@ -55,7 +62,7 @@ __device__ __forceinline__ void gc_ldm_t(uint32_t addr, uint32_t (&r)[4]) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
 __device__ __forceinline__ void gc_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
@@ -81,23 +88,35 @@ __device__ __forceinline__ bool gc_locate(const GlaChunkParams& p, int chunk, in
   return at.n > 0 && p.slot[b] >= 0;
 }
 
-__host__ __device__ constexpr int gc_groups(int dk) { return dk <= 32 ? 8 : dk <= 64 ? 4 : dk <= 128 ? 2 : 1; }
+__host__ __device__ constexpr int gc_groups(int dk) { return dk <= 64 ? 8 : dk <= 128 ? 4 : 2; }
+
+// 64 rows of `width` bf16 (a multiple of 16) to shared memory, two rows of a warp at a time; rows from `n` on are zeros.
+__device__ __forceinline__ void gc_rows(__nv_bfloat16* dst, int pitch, const __nv_bfloat16* src, int stride, int width, int n, int warp, int lane) {
+  const int per = width / 8;
+  for (int t0 = warp * 2; t0 < kGc; t0 += 2 * kGcWarps)
+    for (int i = lane; i < 2 * per; i += 32) {
+      const int t = t0 + (i >= per), c = (i >= per ? i - per : i) * 8;
+      if (t < n) gc_cp16(dst + t * pitch + c, src + size_t(t) * stride + c);
+      else *reinterpret_cast<uint4*>(dst + t * pitch + c) = make_uint4(0, 0, 0, 0);
+    }
+}
 
 struct GlaLocalSmem {
-  int b, k, v, tot, bytes;
+  int b, k, lo, v, tot, bytes;
 };
 __host__ __device__ inline GlaLocalSmem gc_local_smem(int dk, int dv, int rank) {
   GlaLocalSmem m{};
   m.b = 0;                                                   // [64][dk + 8] fp32
-  m.k = m.b + kGc * (dk + 8) * 4;                            // hi, lo [64][dk + 8] bf16; before that a^T [rank][68] fp32
-  const int kbytes = 2 * kGc * (dk + 8) * 2, abytes = rank * 68 * 4;
-  m.v = m.k + (kbytes > abytes ? kbytes : abytes);           // [64][dv + 8] bf16
-  m.tot = m.v + kGc * (dv + 8) * 2;                          // [256] fp32
-  m.bytes = m.tot + 1024;
+  m.k = m.b + kGc * (dk + 8) * 4;                            // a^T [rank][68] fp32, then hi [64][dk + 8] bf16
+  const int half = kGc * (dk + 8) * 2, abytes = rank * 68 * 4;
+  m.lo = m.k + (half > abytes ? half : abytes);              // k, then lo [64][dk + 8] bf16
+  m.v = m.lo + half;                                         // [64][dv + 8] bf16
+  m.tot = m.v + kGc * (dv + 8) * 2;                          // [512] fp32
+  m.bytes = m.tot + kGcThreads * 4;
   return m;
 }
 
-__global__ void __launch_bounds__(kGcThreads)
+__global__ void __launch_bounds__(kGcThreads, 2)
 gla_chunk_local_kernel(const GlaChunkParams p) {
   pdl_trigger();
   extern __shared__ __align__(16) uint8_t gc_sm[];
@@ -113,16 +132,12 @@ gla_chunk_local_kernel(const GlaChunkParams p) {
   __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(gc_sm + m.v);
   float* tot = reinterpret_cast<float*>(gc_sm + m.tot);
   const int bp = dk + 8, kp = dk + 8, vp = dv + 8;
-  __nv_bfloat16* k_lo = k_hi + kGc * kp;
+  __nv_bfloat16* k_lo = reinterpret_cast<__nv_bfloat16*>(gc_sm + m.lo);
   const __nv_bfloat16* rows = p.proj + size_t(at.t0) * p.s.row_stride;
   {
-    const __nv_bfloat16* v = rows + 2 * H * dk + h * dv;
-    const int per = dv / 8;
-    for (int i = tid; i < kGc * per; i += kGcThreads) {
-      const int t = i / per, c = (i - t * per) * 8;
-      if (t < at.n) gc_cp16(v_s + t * vp + c, v + size_t(t) * p.s.row_stride + c);
-      else *reinterpret_cast<uint4*>(v_s + t * vp + c) = make_uint4(0, 0, 0, 0);
-    }
+    gc_rows(k_lo, kp, rows + (H + h) * dk, p.s.row_stride, dk, at.n, warp, lane);
+    gc_commit();
+    gc_rows(v_s, vp, rows + 2 * H * dk + h * dv, p.s.row_stride, dv, at.n, warp, lane);
     gc_commit();
     const __nv_bfloat16* a = rows + 2 * H * (dk + dv);
     const int aper = rank / 8;
@@ -158,7 +173,7 @@ gla_chunk_local_kernel(const GlaChunkParams p) {
       }
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
-        run += t + j < at.n ? log2_sigmoid(z[j]) * p.s.inv_tau : 0.f;
+        run += t + j < at.n ? gc_log2_sigmoid(z[j]) * p.s.inv_tau : 0.f;
         b_s[(t + j) * bp + c] = run;
       }
     }
@@ -175,51 +190,49 @@ gla_chunk_local_kernel(const GlaChunkParams p) {
     }
     if (tg == TG - 1) p.gam[(at.index * H + h) * dk + c] = exp2f(b_s[(kGc - 1) * bp + c]);
   }
+  gc_wait<1>();
   __syncthreads();
-  {
-    const __nv_bfloat16* k = rows + (H + h) * dk;
-    const int per = dk / 2;
-    for (int i = tid; i < kGc * per; i += kGcThreads) {
-      const int t = i / per, ch = (i - t * per) * 2;
-      float2 x = make_float2(0.f, 0.f);
-      if (t < at.n) {
-        x = gc_pair(k + size_t(t) * p.s.row_stride + ch);
-        const float2 b = *reinterpret_cast<const float2*>(b_s + t * bp + ch), e = *reinterpret_cast<const float2*>(b_s + (kGc - 1) * bp + ch);
-        x.x *= gc_exp2(e.x - b.x);
-        x.y *= gc_exp2(e.y - b.y);
-      }
+  for (int ch = lane * 2; ch < dk; ch += 64) {
+    const float2 e = *reinterpret_cast<const float2*>(b_s + (kGc - 1) * bp + ch);
+#pragma unroll
+    for (int i = 0; i < kGc / kGcWarps; ++i) {
+      const int t = warp + kGcWarps * i;
+      float2 x = gc_pair(k_lo + t * kp + ch);
+      const float2 b = *reinterpret_cast<const float2*>(b_s + t * bp + ch);
+      x.x *= gc_exp2(e.x - b.x);
+      x.y *= gc_exp2(e.y - b.y);
       gc_split(x.x, x.y, *reinterpret_cast<uint32_t*>(k_hi + t * kp + ch), *reinterpret_cast<uint32_t*>(k_lo + t * kp + ch));
     }
   }
   gc_wait<0>();
   __syncthreads();
-  // ----- U = (2^(b_C - b) k)^T V: jobs of 16 rows x 64 columns -----
+  // ----- U = (2^(b_C - b) k)^T V: jobs of 16 rows x 32 columns -----
   float* u = p.u + (at.index * H + h) * size_t(dk) * dv;
   const int mat = lane >> 3, mrow = lane & 7, g = lane >> 2, t4 = lane & 3;
-  const int nbs = (dv + 63) / 64;
+  const int nbs = (dv + 31) / 32;
   const int steps = (at.n + 15) / 16;
-  for (int job = warp; job < (dk / 16) * nbs; job += kGcThreads / 32) {
-    const int m0 = job / nbs * 16, n0 = (job % nbs) * 64, tiles = min(8, (dv - n0) / 8);
-    float acc[8][4] = {};
+  for (int job = warp; job < (dk / 16) * nbs; job += kGcWarps) {
+    const int m0 = job / nbs * 16, n0 = (job % nbs) * 32, tiles = min(4, (dv - n0) / 8);  // 2 or 4: dv is a multiple of 16
+    float acc[4][4] = {};
     for (int ks = 0; ks < steps; ++ks) {
-      uint32_t hi[4], lo[4];
+      uint32_t hi[4], lo[4], v[2][4];
       const int off = (ks * 16 + (mat >> 1) * 8 + mrow) * kp + m0 + (mat & 1) * 8;
       gc_ldm_t(smem_u32(k_hi + off), hi);
       gc_ldm_t(smem_u32(k_lo + off), lo);
 #pragma unroll
-      for (int nt = 0; nt < 8; nt += 2) {
-        if (nt < tiles) {  // tiles is even: dv is a multiple of 16
-          uint32_t v[4];
-          gc_ldm_t(smem_u32(v_s + (ks * 16 + (mat & 1) * 8 + mrow) * vp + n0 + nt * 8 + (mat >> 1) * 8), v);
-          gc_mma(acc[nt], hi, v[0], v[1]);
-          gc_mma(acc[nt], lo, v[0], v[1]);
-          gc_mma(acc[nt + 1], hi, v[2], v[3]);
-          gc_mma(acc[nt + 1], lo, v[2], v[3]);
-        }
-      }
+      for (int i = 0; i < 2; ++i)
+        if (2 * i < tiles) gc_ldm_t(smem_u32(v_s + (ks * 16 + (mat & 1) * 8 + mrow) * vp + n0 + i * 16 + (mat >> 1) * 8), v[i]);
+#pragma unroll
+      for (int part = 0; part < 2; ++part)  // all tiles between two additions to the same one
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+          if (2 * i < tiles) {
+            gc_mma(acc[2 * i], part ? lo : hi, v[i][0], v[i][1]);
+            gc_mma(acc[2 * i + 1], part ? lo : hi, v[i][2], v[i][3]);
+          }
     }
 #pragma unroll
-    for (int nt = 0; nt < 8; ++nt) {
+    for (int nt = 0; nt < 4; ++nt) {
       if (nt < tiles) {
         float* d = u + size_t(m0 + g) * dv + n0 + nt * 8 + t4 * 2;
         *reinterpret_cast<float2*>(d) = make_float2(acc[nt][0], acc[nt][1]);
@@ -270,23 +283,24 @@ gla_chunk_state_kernel(const GlaChunkParams p) {
 }
 
 struct GlaOutputSmem {
-  int b, q, a, v, ss, bytes;
+  int b, q, a, v, ss, bytes, stages;
 };
 __host__ __device__ inline GlaOutputSmem gc_output_smem(int dk, int dv) {
   GlaOutputSmem m{};
-  m.b = 0;                                             // b [64][dk + 8] fp32, then two stages of S_0: [16][dv * 4 + 16 bytes]
-  const int bb = kGc * (dk + 8) * 4, sb = 2 * 16 * (dv * 4 + 16);
+  m.b = 0;                                             // b [64][dk + 8] fp32, then stages of S_0: [16][dv * 4 + 16 bytes]
+  const int bb = kGc * (dk + 8) * 4, stage = 16 * (dv * 4 + 16), sb = 2 * stage;
+  m.stages = bb >= 4 * stage ? 4 : 2;
   m.q = m.b + (bb > sb ? bb : sb);                     // q, k [64][dk + 8] bf16, then hi, lo of 2^b q
-  m.a = m.q + 2 * kGc * (dk + 8) * 2;                  // A hi, lo [64][72] bf16
+  m.a = m.q + 2 * kGc * (dk + 8) * 2;                  // partial sums of A [64][72] fp32, then A hi, lo [64][72] bf16
   m.v = m.a + 2 * kGc * 72 * 2;                        // [64][dv + 8] bf16
-  m.ss = m.v + kGc * (dv + 8) * 2;                     // [2][64] fp32
-  m.bytes = m.ss + 512;
+  m.ss = m.v + kGc * (dv + 8) * 2;                     // [4][64] fp32
+  m.bytes = m.ss + 1024;
   return m;
 }
 
-// NT: upper bound of the 8-column tiles of a warp (dv / 16)
+// NT: upper bound of the 8-column tiles of a warp (dv / 32)
 template <int NT>
-__global__ void __launch_bounds__(kGcThreads, NT <= 8 ? 2 : 1)
+__global__ void __launch_bounds__(kGcThreads, NT <= 4 ? 2 : 1)
 gla_chunk_output_kernel(const GlaChunkParams p) {
   pdl_trigger();
   extern __shared__ __align__(16) uint8_t gc_sm[];
@@ -306,40 +320,28 @@ gla_chunk_output_kernel(const GlaChunkParams p) {
   __nv_bfloat16* k_s = q_s + kGc * kp;
   __nv_bfloat16* a_lo = a_hi + kGc * ap;
   const __nv_bfloat16* rows = p.proj + size_t(at.t0) * p.s.row_stride;
-  const uint4 zero = make_uint4(0, 0, 0, 0);
   {
     const float* cum = p.cum + size_t(at.t0) * (H * dk) + h * dk;
-    const int bper = dk / 4;
-    for (int i = tid; i < kGc * bper; i += kGcThreads) {  // rows past the end repeat the last one
-      const int t = i / bper, c = (i - t * bper) * 4;
-      gc_cp16(b_s + t * bp + c, cum + size_t(min(t, at.n - 1)) * (H * dk) + c);
-    }
-    const int per = dk / 8;
-    for (int i = tid; i < 2 * kGc * per; i += kGcThreads) {
-      const int which = i / (kGc * per), j = i - which * kGc * per, t = j / per, c = (j - t * per) * 8;
-      __nv_bfloat16* d = (which ? k_s : q_s) + t * kp + c;
-      if (t < at.n) gc_cp16(d, rows + size_t(t) * p.s.row_stride + (which * H + h) * dk + c);
-      else *reinterpret_cast<uint4*>(d) = zero;
-    }
-    gc_commit();
-    const int vper = dv / 8;
-    for (int i = tid; i < kGc * vper; i += kGcThreads) {
-      const int t = i / vper, c = (i - t * vper) * 8;
-      if (t < at.n) gc_cp16(v_s + t * vp + c, rows + size_t(t) * p.s.row_stride + 2 * H * dk + h * dv + c);
-      else *reinterpret_cast<uint4*>(v_s + t * vp + c) = zero;
-    }
+    for (int t = warp; t < kGc; t += kGcWarps)  // rows past the end repeat the last one
+      for (int c = lane * 4; c < dk; c += 128) gc_cp16(b_s + t * bp + c, cum + size_t(min(t, at.n - 1)) * (H * dk) + c);
+    gc_rows(q_s, kp, rows + h * dk, p.s.row_stride, dk, at.n, warp, lane);
+    gc_rows(k_s, kp, rows + (H + h) * dk, p.s.row_stride, dk, at.n, warp, lane);
+    gc_rows(v_s, vp, rows + 2 * H * dk + h * dv, p.s.row_stride, dv, at.n, warp, lane);
     gc_commit();
   }
-  gc_wait<1>();
+  gc_wait<0>();
   __syncthreads();
-  // ----- A: warp = (row block I, one half of the column blocks J <= I) -----
+  // ----- A: warp = (row block I, one half of the column blocks J <= I, even or odd 16-channel steps); the second half of the
+  //       columns is taken in reverse, so that every scheduler gets short and long row blocks -----
   const int ksteps = dk / 16;
   bool wide = false;
   {
-    const int I = warp & 3, J0 = warp < 4 ? 0 : (I + 2) / 2, J1 = warp < 4 ? (I + 2) / 2 : I + 1;  // blocks J0 .. J1 - 1
+    const bool upper = warp & 4, odd = warp & 8;
+    const int I = upper ? 3 - (warp & 3) : warp & 3, J0 = upper ? (I + 2) / 2 : 0, J1 = upper ? I + 1 : (I + 2) / 2;  // J0 .. J1 - 1
+    float* part = reinterpret_cast<float*>(a_hi);
     float acc[2][2][4] = {};
     const float* ref = b_s + (16 * I - 1) * bp;
-    for (int ks = 0; ks < ksteps; ++ks) {
+    for (int ks = odd; ks < ksteps && J0 < J1; ks += 2) {
       uint32_t hi[4], lo[4];
       float2 rf[2];
 #pragma unroll
@@ -358,36 +360,48 @@ gla_chunk_output_kernel(const GlaChunkParams p) {
 #pragma unroll
       for (int jj = 0; jj < 2; ++jj) {
         if (J0 + jj < J1) {
+          uint32_t kh[2][2], kl[2][2];
 #pragma unroll
           for (int nt = 0; nt < 2; ++nt) {
-            uint32_t kh[2], kl[2];
             const int s = 16 * (J0 + jj) + nt * 8 + g;
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
               const int c = ks * 16 + e * 8 + t4 * 2;
               const float2 k = gc_pair(k_s + s * kp + c), b = *reinterpret_cast<const float2*>(b_s + s * bp + c);
-              gc_split(k.x * gc_exp2(rf[e].x - b.x), k.y * gc_exp2(rf[e].y - b.y), kh[e], kl[e]);
+              gc_split(k.x * gc_exp2(rf[e].x - b.x), k.y * gc_exp2(rf[e].y - b.y), kh[nt][e], kl[nt][e]);
             }
-            gc_mma(acc[jj][nt], hi, kh[0], kh[1]);
-            gc_mma(acc[jj][nt], lo, kh[0], kh[1]);
-            gc_mma(acc[jj][nt], hi, kl[0], kl[1]);
           }
+          gc_mma(acc[jj][0], hi, kh[0][0], kh[0][1]);
+          gc_mma(acc[jj][1], hi, kh[1][0], kh[1][1]);
+          gc_mma(acc[jj][0], lo, kh[0][0], kh[0][1]);
+          gc_mma(acc[jj][1], lo, kh[1][0], kh[1][1]);
+          gc_mma(acc[jj][0], hi, kl[0][0], kl[0][1]);
+          gc_mma(acc[jj][1], hi, kl[1][0], kl[1][1]);
         }
       }
     }
+    auto each = [&](auto&& f) {  // f(pair of sums, row, first column) over my blocks
 #pragma unroll
-    for (int jj = 0; jj < 2; ++jj) {
-      if (J0 + jj < J1) {
+      for (int jj = 0; jj < 2; ++jj)
+        if (J0 + jj < J1)
 #pragma unroll
-        for (int nt = 0; nt < 2; ++nt)
+          for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-          for (int r = 0; r < 2; ++r) {
-            const int t = 16 * I + r * 8 + g, s = 16 * (J0 + jj) + nt * 8 + t4 * 2;
-            gc_split(s <= t ? acc[jj][nt][2 * r] : 0.f, s + 1 <= t ? acc[jj][nt][2 * r + 1] : 0.f,
-                     *reinterpret_cast<uint32_t*>(a_hi + t * ap + s), *reinterpret_cast<uint32_t*>(a_lo + t * ap + s));
-          }
-      }
-    }
+            for (int r = 0; r < 2; ++r) f(acc[jj][nt][2 * r], acc[jj][nt][2 * r + 1], 16 * I + r * 8 + g, 16 * (J0 + jj) + nt * 8 + t4 * 2);
+    };
+    if (odd) each([&](float x, float y, int t, int s) { *reinterpret_cast<float2*>(part + t * ap + s) = make_float2(x, y); });
+    __syncthreads();
+    if (!odd)
+      each([&](float& x, float& y, int t, int s) {
+        const float2 o = *reinterpret_cast<const float2*>(part + t * ap + s);
+        x = s <= t ? x + o.x : 0.f;
+        y = s + 1 <= t ? y + o.y : 0.f;
+      });
+    __syncthreads();
+    if (!odd)
+      each([&](float x, float y, int t, int s) {
+        gc_split(x, y, *reinterpret_cast<uint32_t*>(a_hi + t * ap + s), *reinterpret_cast<uint32_t*>(a_lo + t * ap + s));
+      });
   }
   if (__syncthreads_or(wide)) {  // diagonal blocks term by term
     for (int i = tid; i < 4 * 256; i += kGcThreads) {
@@ -405,34 +419,28 @@ gla_chunk_output_kernel(const GlaChunkParams p) {
   }
   // ----- 2^b q, in the place of q and k -----
   {
-    const int per = dk / 2;
-    for (int i = tid; i < kGc * per; i += kGcThreads) {
-      const int t = i / per, c = (i - t * per) * 2;
-      const float2 q = gc_pair(q_s + t * kp + c), b = *reinterpret_cast<const float2*>(b_s + t * bp + c);
-      gc_split(q.x * p.s.scale * gc_exp2(b.x), q.y * p.s.scale * gc_exp2(b.y), *reinterpret_cast<uint32_t*>(q_s + t * kp + c),
-               *reinterpret_cast<uint32_t*>(k_s + t * kp + c));
-    }
+    for (int t = warp; t < kGc; t += kGcWarps)
+      for (int c = lane * 2; c < dk; c += 64) {
+        const float2 q = gc_pair(q_s + t * kp + c), b = *reinterpret_cast<const float2*>(b_s + t * bp + c);
+        gc_split(q.x * p.s.scale * gc_exp2(b.x), q.y * p.s.scale * gc_exp2(b.y), *reinterpret_cast<uint32_t*>(q_s + t * kp + c),
+                 *reinterpret_cast<uint32_t*>(k_s + t * kp + c));
+      }
   }
   __syncthreads();
-  // ----- O: warp = (16 tokens, half of the value columns) -----
+  // ----- O: warp = (16 tokens, every fourth 8-column tile of the values) -----
   const uint8_t* s0 = reinterpret_cast<const uint8_t*>(p.u + (at.index * H + h) * size_t(dk) * dv);
   const int spitch = dv * 4 + 16;
+  const int ahead = m.stages - 1;  // stages (a power of two) in flight while one is used
   auto fetch = [&](int ks) {
-    uint8_t* d = gc_sm + m.b + (ks & 1) * 16 * spitch;
-    const int per = dv / 4;  // 16-byte pieces of a row
-    for (int i = tid; i < 16 * per; i += kGcThreads) {
-      const int r = i / per, c = i - r * per;
-      gc_cp16(d + r * spitch + c * 16, s0 + (size_t(ks) * 16 + r) * dv * 4 + c * 16);
-    }
+    uint8_t* d = gc_sm + m.b + (ks & ahead) * 16 * spitch;
+    for (int c = lane * 16; c < dv * 4; c += 512) gc_cp16(d + warp * spitch + c, s0 + (size_t(ks) * 16 + warp) * dv * 4 + c);  // 16 warps, 16 rows
   };
-  fetch(0);
-  gc_commit();
-  if (ksteps > 1) fetch(1);
-  gc_commit();
-  gc_wait<2>();  // V
-  __syncthreads();
-  const int mt = warp & 3, half = warp >> 2, tiles = dv / 16;
-  const int col0 = half * (dv / 2);
+  for (int ks = 0; ks < ahead; ++ks) {
+    if (ks < ksteps) fetch(ks);
+    gc_commit();
+  }
+  const int mt = warp & 4 ? 3 - (warp & 3) : warp & 3, quarter = warp >> 2, tiles = (dv / 8 - quarter + 3) / 4;
+  auto col = [&](int i) { return (quarter + 4 * i) * 8; };  // first column of my i-th tile
   float o[NT][4];
 #pragma unroll
   for (int nt = 0; nt < NT; ++nt)
@@ -444,39 +452,50 @@ gla_chunk_output_kernel(const GlaChunkParams p) {
     gc_ldm(smem_u32(a_hi + frag * ap + ks * 16 + fk), hi);
     gc_ldm(smem_u32(a_lo + frag * ap + ks * 16 + fk), lo);
 #pragma unroll
-    for (int nt = 0; nt < NT; nt += 2) {
-      if (nt < tiles) {
-        uint32_t v[4];  // the second tile of the last pair may lie past the half: it is not used then
-        gc_ldm_t(smem_u32(v_s + (ks * 16 + (mat & 1) * 8 + mrow) * vp + col0 + nt * 8 + (mat >> 1) * 8), v);
-        gc_mma(o[nt], hi, v[0], v[1]);
-        gc_mma(o[nt], lo, v[0], v[1]);
-        if (nt + 1 < tiles) {
-          gc_mma(o[nt + 1], hi, v[2], v[3]);
-          gc_mma(o[nt + 1], lo, v[2], v[3]);
-        }
-      }
+    for (int n0 = 0; n0 < NT; n0 += 4) {
+      uint32_t v[2][4];
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+        if (n0 + 2 * i < tiles)  // a second tile past the last is the first one again, and not used
+          gc_ldm_t(smem_u32(v_s + (ks * 16 + (mat & 1) * 8 + mrow) * vp + col(min(n0 + 2 * i + (mat >> 1), tiles - 1))), v[i]);
+#pragma unroll
+      for (int part = 0; part < 2; ++part)
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if (n0 + i < tiles) gc_mma(o[n0 + i], part ? lo : hi, v[i >> 1][(i & 1) * 2], v[i >> 1][(i & 1) * 2 + 1]);
     }
   }
+  // gates of my places, requested while S_0 arrives
+  uint32_t gate[2][NT];
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int t = mt * 16 + r * 8 + g;
+    const __nv_bfloat16* src = rows + size_t(min(t, at.n - 1)) * p.s.row_stride + 2 * H * dk + (H + h) * dv + t4 * 2;
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) gate[r][nt] = nt < tiles ? *reinterpret_cast<const uint32_t*>(src + col(nt)) : 0u;
+  }
   for (int ks = 0; ks < ksteps; ++ks) {
-    gc_wait<1>();
-    __syncthreads();
+    if (ahead == 3) gc_wait<2>();
+    else gc_wait<0>();
+    __syncthreads();  // step ks has arrived, and everyone is done with step ks - 1
+    if (ks + ahead < ksteps) fetch(ks + ahead);
+    gc_commit();
     uint32_t hi[4], lo[4];
     gc_ldm(smem_u32(q_s + frag * kp + ks * 16 + fk), hi);
     gc_ldm(smem_u32(k_s + frag * kp + ks * 16 + fk), lo);
-    const uint32_t st = smem_u32(gc_sm + m.b) + (ks & 1) * 16 * spitch + ((mat & 1) * 8 + mrow) * spitch + col0 * 4 + (mat >> 1) * 16;
+    const uint32_t st = smem_u32(gc_sm + m.b) + (ks & ahead) * 16 * spitch + ((mat & 1) * 8 + mrow) * spitch + quarter * 32 + (mat >> 1) * 16;
 #pragma unroll
-    for (int nt = 0; nt < NT; ++nt) {
-      if (nt < tiles) {
-        uint32_t s[4];  // hi of rows 0-7, 8-15, then lo
-        gc_ldm_t(st + nt * 32, s);
-        gc_mma(o[nt], hi, s[0], s[1]);
-        gc_mma(o[nt], lo, s[0], s[1]);
-        gc_mma(o[nt], hi, s[2], s[3]);
-      }
+    for (int n0 = 0; n0 < NT; n0 += 4) {
+      uint32_t s[4][4];  // hi of rows 0-7, 8-15, then lo
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (n0 + i < tiles) gc_ldm_t(st + (n0 + i) * 128, s[i]);
+#pragma unroll
+      for (int part = 0; part < 3; ++part)  // all tiles between two additions to the same one
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if (n0 + i < tiles) gc_mma(o[n0 + i], part == 1 ? lo : hi, s[i][part == 2 ? 2 : 0], s[i][part == 2 ? 3 : 1]);
     }
-    __syncthreads();
-    if (ks + 2 < ksteps) fetch(ks + 2);
-    gc_commit();
   }
   // ----- norm over the head's value channels, gate -----
   float sq[2] = {0.f, 0.f};
@@ -491,23 +510,22 @@ gla_chunk_output_kernel(const GlaChunkParams p) {
   for (int r = 0; r < 2; ++r) {
     sq[r] += __shfl_xor_sync(0xffffffffu, sq[r], 1);
     sq[r] += __shfl_xor_sync(0xffffffffu, sq[r], 2);
-    if (t4 == 0) ss_s[half * kGc + mt * 16 + r * 8 + g] = sq[r];
+    if (t4 == 0) ss_s[quarter * kGc + mt * 16 + r * 8 + g] = sq[r];
   }
   __syncthreads();
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     const int t = mt * 16 + r * 8 + g;
     if (t >= at.n) continue;
-    const float f = rsqrtf((ss_s[t] + ss_s[kGc + t]) * p.s.inv_dv + p.s.eps);
-    const __nv_bfloat16* gate = rows + size_t(t) * p.s.row_stride + 2 * H * dk + (H + h) * dv;
+    const float f = rsqrtf((ss_s[t] + ss_s[kGc + t] + ss_s[2 * kGc + t] + ss_s[3 * kGc + t]) * p.s.inv_dv + p.s.eps);
     __nv_bfloat16* y = p.y + (size_t(at.t0 + t) * H + h) * dv;
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) {
       if (nt < tiles) {
-        const int c = col0 + nt * 8 + t4 * 2;
-        const float2 gt = gc_pair(gate + c), w = *reinterpret_cast<const float2*>(p.norm_w + c);
+        const int c = col(nt) + t4 * 2;
+        const float2 gt = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gate[r][nt])), w = *reinterpret_cast<const float2*>(p.norm_w + c);
         *reinterpret_cast<__nv_bfloat162*>(y + c) =
-            __floats2bfloat162_rn(o[nt][2 * r] * f * w.x * silu_of(gt.x), o[nt][2 * r + 1] * f * w.y * silu_of(gt.y));
+            __floats2bfloat162_rn(o[nt][2 * r] * f * w.x * gc_silu(gt.x), o[nt][2 * r + 1] * f * w.y * gc_silu(gt.y));
       }
     }
   }
@@ -549,7 +567,7 @@ extern "C" int mfq_gla_chunk(const void* proj, const void* w2, const float* bias
   }
   launch_kernel(gla_chunk_local_kernel, grid, dim3(kGcThreads), local, stream, p);
   launch_kernel(gla_chunk_state_kernel, dim3((dk * dv / 8 + 127) / 128, H, B), dim3(128), 0, stream, p);
-  const int rc = dv <= 64 ? launch_gla_output<4>(p, grid, stream) : dv <= 128 ? launch_gla_output<8>(p, grid, stream)
-               : dv <= 256 ? launch_gla_output<16>(p, grid, stream) : launch_gla_output<32>(p, grid, stream);
+  const int rc = dv <= 128 ? launch_gla_output<4>(p, grid, stream) : dv <= 256 ? launch_gla_output<8>(p, grid, stream)
+                                                                          : launch_gla_output<16>(p, grid, stream);
   return rc == 0 && cudaGetLastError() == cudaSuccess ? 0 : (rc ? rc : -7);
 }
