@@ -161,18 +161,19 @@ def bench_small(m: int, h: int, i: int, reps: int) -> list[dict]:
     return out
 
 
-def bench_dense(m: int, n: int, k: int, reps: int, glu: bool = False, tile=None, splits=None) -> dict:
-    """Unquantized (bf16) product, optionally with the clipped-GLU output stage."""
+def bench_dense(m: int, n: int, k: int, reps: int, stage: str = "", tile=None, splits=None) -> dict:
+    """Unquantized (bf16) product with an output stage: "" (bias), "clipped" / "gelu" (gated unit), "add" (to the fp32 stream)."""
     from . import dense
     copies = max(1, min(16, math.ceil(4 * L2_BYTES / (2 * n * k))))
     lin = [dense.DenseLinear((torch.randn((n, k), device="cuda") * k ** -0.5).to(torch.bfloat16),
-                             torch.zeros(n, device="cuda"), (1.702, 7.0) if glu else None) for _ in range(copies)]
+                             torch.zeros(n, device="cuda"), {"clipped": (1.702, 7.0), "gelu": "gelu"}.get(stage)) for _ in range(copies)]
     x = torch.randn((m, k), device="cuda").to(torch.bfloat16)
-    out = torch.empty((m, lin[0].out_width), device="cuda", dtype=torch.bfloat16)
-    ms = time_ms(lambda i: lin[i % copies](x, out=out, tile=tile, splits=splits), reps)
+    add = stage == "add"
+    out = torch.zeros((m, lin[0].out_width), device="cuda", dtype=torch.float32 if add else torch.bfloat16)
+    ms = time_ms(lambda i: lin[i % copies](x, tile=tile, splits=splits, **{"add_to" if add else "out": out}), reps)
     t, sp = dense.plan(m, n, k)
-    return {"kernel": "dense_gemv" if (t if tile is None else tile) == 0 else "dense_gemm", "m": m, "n": n, "k": k, "us": ms * 1e3,
-            "gbs": 2 * (n * k + m * k + out.numel()) / ms / 1e6, "tflops": 2 * m * n * k / ms / 1e9,
+    return {"kernel": "dense_gemv" if (t if tile is None else tile) == 0 else "dense_gemm", "m": m, "n": n, "k": k, "stage": stage, "us": ms * 1e3,
+            "gbs": (2 * (n * k + m * k) + out.numel() * (8 if add else 2)) / ms / 1e6, "tflops": 2 * m * n * k / ms / 1e9,
             "tile": t if tile is None else tile, "splits": sp if splits is None else splits}
 
 
@@ -238,12 +239,74 @@ def bench_dense_small(m: int, h: int, reps: int) -> list[dict]:
     return rows
 
 
+def bench_two_maps(batch: int, ctx: int, h: int, hk: int, d: int, e: int, window: int, keep: int, reps: int) -> list[dict]:
+    """Differential attention (two maps of ``d`` channels, values of ``e``): one token per sequence, or for batch 0 one prompt of
+    ``ctx`` tokens and the difference of the maps."""
+    from . import window_attn
+    seen, diff = window_attn.visible_keys(ctx, window, keep), window_attn.Difference(0.5, 0.5, 1e-6, e)
+    how = dict(window=window, keep=keep, scale=d ** -0.5, cap=0.0)
+    shape = {"heads": h, "hk": hk, "d": d, "e": e, "window": window, "keep": keep}
+    if batch:
+        layers = max(1, min(32, math.ceil(4 * L2_BYTES / (batch * seen * hk * (2 * d + e) * 2))))
+        cache = _plain_cache(batch, ctx, hk, 2 * d, e, layers)
+        q = torch.randn((batch, 2 * h, d), device="cuda").to(torch.bfloat16)
+        sl = torch.full((batch,), ctx, dtype=torch.int32, device="cuda")
+        splits = window_attn.decode_splits(batch, hk, seen)
+        ms = time_ms(lambda i: window_attn.decode(q, cache.layer(i % layers), cache.block_table, sl, diff=diff, splits=splits, **how), reps)
+        return [{"kernel": "window_attn_decode (two maps, difference)", "batch": batch, "ctx": ctx, **shape, "splits": splits, "us": ms * 1e3,
+                 "gbs": batch * seen * hk * (2 * d + e) * 2 / ms / 1e6}]
+    cache = _plain_cache(1, ctx, hk, 2 * d, e, 1)
+    q = torch.randn((ctx, 2 * h, d), device="cuda").to(torch.bfloat16)
+    starts, lens = (torch.tensor(v, dtype=torch.int32, device="cuda") for v in ([0, ctx], [ctx]))
+    maps = torch.empty((ctx, 2 * h, e), device="cuda", dtype=torch.bfloat16)
+    ms = time_ms(lambda _: window_attn.prefill(q, cache.layer(0), cache.block_table, starts, lens, ctx, maps=2, out=maps, **how), reps)
+    pairs = sum(min(i + 1, window + min(keep, max(0, i + 1 - window))) for i in range(ctx))
+    out = window_attn.difference(maps, hk, diff)
+    md = time_ms(lambda _: window_attn.difference(maps, hk, diff, out=out), reps)
+    return [{"kernel": "window_attn_prefill (two maps)", "t": ctx, **shape, "us": ms * 1e3, "tflops": 2 * pairs * 2 * h * (d + e) / ms / 1e9},
+            {"kernel": "map_difference", "t": ctx, **shape, "us": md * 1e3, "gbs": ctx * h * e * 6 / md / 1e6}]
+
+
+def bench_gla(batch: int, tokens: int, h: int, dk: int, dv: int, reps: int) -> dict:
+    """Gated linear attention: ``tokens`` 1: a decode step of ``batch`` sequences, else one prompt in chunks."""
+    from . import gla
+    geo = gla.Geometry(h, dk, dv, dk, dv, 16, 16.0, 1e-6)
+    w2, bias = (torch.randn((h * dk, 16), device="cuda") * 0.25).to(torch.bfloat16), torch.randn(h * dk, device="cuda") + 2
+    norm, slots = torch.ones(dv, device="cuda"), torch.arange(batch, dtype=torch.int32, device="cuda")
+    proj = torch.randn((batch * tokens, geo.width), device="cuda").to(torch.bfloat16)
+    row = batch * tokens * (geo.width + h * dv) * 2
+    if tokens == 1:
+        layers = max(1, min(32, math.ceil(4 * L2_BYTES / (batch * h * dk * dv * 4))))
+        states = [torch.zeros((batch, h, dk, dv), device="cuda") for _ in range(layers)]
+        ms = time_ms(lambda i: gla.recurrent(proj, w2, bias, norm, states[i % layers], slots, geo), reps)
+        return {"kernel": "gla_recurrent", "batch": batch, "h": h, "dk": dk, "dv": dv, "us": ms * 1e3,
+                "gbs": (batch * h * dk * dv * 8 + row) / ms / 1e6}
+    state, starts = torch.zeros((1, h, dk, dv), device="cuda"), torch.tensor([0, tokens], dtype=torch.int32, device="cuda")
+    ms = time_ms(lambda _: gla.chunked(proj, w2, bias, norm, state, slots, geo, starts, tokens), reps)
+    return {"kernel": "gla_chunk (three kernels)", "t": tokens, "h": h, "dk": dk, "dv": dv, "us": ms * 1e3, "gbs": row / ms / 1e6}
+
+
+def bench_gdn(batch: int, tokens: int, reps: int) -> dict:
+    """Gated DeltaNet at 16 key / 32 value heads of 128, the same way (without its convolution)."""
+    from . import gdn
+    hk, hv, d = 16, 32, 128
+    n = batch * tokens
+    qkv, z = torch.randn((n, (2 * hk + hv) * d), device="cuda"), torch.randn((n, hv * d), device="cuda").to(torch.bfloat16)
+    a, zero, one = torch.randn((n, hv), device="cuda").to(torch.bfloat16), torch.zeros(hv, device="cuda"), torch.ones(d, device="cuda")
+    layers = max(1, min(32, math.ceil(4 * L2_BYTES / (batch * hv * d * d * 4)))) if tokens == 1 else 1
+    states = [torch.zeros((batch, hv, d, d), device="cuda") for _ in range(layers)]
+    slots = torch.arange(batch, dtype=torch.int32, device="cuda")
+    ms = time_ms(lambda i: gdn.recurrent(qkv, z, a, a, zero, zero, one, states[i % layers], slots, tokens, hk, hv), reps)
+    bytes_ = n * ((2 * hk + hv) * d * 4 + hv * d * 4) + (batch * hv * d * d * 8 if tokens == 1 else 0)
+    return {"kernel": "gdn_recurrent" if tokens == 1 else "gdn_chunk (three kernels)", "batch": batch, "t": tokens, "us": ms * 1e3, "gbs": bytes_ / ms / 1e6}
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--json", default="")
     ap.add_argument("--reps", type=int, default=20)
     ap.add_argument("--quick", action="store_true")
-    ap.add_argument("--only", default="", help="comma separated kernel families: gemm,w4,attn,mla,small,prefill,dense")
+    ap.add_argument("--only", default="", help="comma separated kernel families: gemm,w4,attn,mla,small,prefill,dense,maps,gla")
     ap.add_argument("--tp", type=int, default=1, help="time one rank's shard of a tensor-parallel group of this size")
     args = ap.parse_args()
     pk = peaks()
@@ -286,7 +349,7 @@ def main() -> None:
         for name, n, k in shapes:
             if name == "lm_head" and m > 64:
                 continue
-            rows.append({**bench_dense(m, n, k, args.reps, glu=name == "gate_up"), "name": name})
+            rows.append({**bench_dense(m, n, k, args.reps, "clipped" if name == "gate_up" else ""), "name": name})
     if want("dense"):
         for batch in (1, 64):
             for window, cap in ((4096, 0.0), (4096, 50.0), (1024, 50.0)):
@@ -296,6 +359,24 @@ def main() -> None:
                 rows.append(bench_window_prefill(t, 32, 8, 128, window, cap, args.reps))
         for m in (1, 64, 4096):
             rows += bench_dense_small(m, 4096, args.reps)
+    if want("maps"):
+        for d, e, h in ((64, 128, 32), (128, 256, 16)):
+            for window, keep in ((4096, 0), (1024, 64)):
+                for batch in (1, 64, 0):
+                    rows += bench_two_maps(batch, 4096, h, 8, d, e, window, keep, args.reps)
+        for m in (1, 64, 4096):
+            for name, n, k, stage in (("o_proj", 4096, 4096, "add"), ("gate_up", 28672, 4096, "gelu"), ("down", 4096, 14336, "add")):
+                rows.append({**bench_dense(m, n, k, args.reps, stage), "name": name})
+        from . import dense
+        for m in (1, 64, 4096):
+            x, w = torch.randn((m, 4096), device="cuda"), torch.ones(4096, device="cuda")
+            ms = time_ms(lambda _: dense.norm_out(x, w, 4096, 1e-5, torch.bfloat16), args.reps)
+            rows.append({"kernel": "norm_out", "m": m, "h": 4096, "us": ms * 1e3, "gbs": m * 4096 * 6 / ms / 1e6})
+    if want("gla"):
+        for batch, tokens in ((1, 1), (64, 1), (1, 2048), (1, 4096)):
+            for h, dk, dv in ((32, 128, 128), (16, 128, 256)):
+                rows.append(bench_gla(batch, tokens, h, dk, dv, args.reps))
+            rows.append(bench_gdn(batch, tokens, args.reps))
     for r in rows:
         if "gbs" in r:
             r["hbm_frac"] = r["gbs"] / pk["hbm_gbs"]

@@ -257,7 +257,7 @@ gla_chunk_state_kernel(const GlaChunkParams p) {
   float* st = p.state + (size_t(slot) * H + h) * dk * dv + e;
   float s[8];
   load8<float>(st, s);
-  constexpr int kAhead = 4;
+  constexpr int kAhead = 8;
   for (int c0 = 0; c0 < chunks; c0 += kAhead) {
     float x[kAhead][8], gm[kAhead];
 #pragma unroll

@@ -200,7 +200,45 @@ def dense_prefill() -> None:
         lin[i](x)
 
 
-CASES = {"gemm_prefill": lambda: gemm(4096, 4096, 4096), "gemm_decode": lambda: gemm(64, 28672, 4096),
+def two_maps_decode() -> None:
+    from . import bench_kernels, window_attn
+    cache = bench_kernels._plain_cache(64, 4096, 8, 128, 128, 3)
+    q = torch.randn((64, 64, 64), device="cuda").to(torch.bfloat16)
+    lens = torch.full((64,), 4096, dtype=torch.int32, device="cuda")
+    for i in range(3):
+        window_attn.decode(q, cache.layer(i), cache.block_table, lens, window=1024, keep=64, scale=0.125, cap=0.0,
+                           diff=window_attn.Difference(0.5, 0.5, 1e-6, 128), splits=window_attn.decode_splits(64, 8, 1088))
+
+
+def two_maps_prefill() -> None:
+    from . import bench_kernels, window_attn
+    t = 2048
+    cache = bench_kernels._plain_cache(1, t, 8, 128, 128, 1)
+    q = torch.randn((t, 64, 64), device="cuda").to(torch.bfloat16)
+    starts, lens = (torch.tensor(v, dtype=torch.int32, device="cuda") for v in ([0, t], [t]))
+    for _ in range(3):
+        maps = window_attn.prefill(q, cache.layer(0), cache.block_table, starts, lens, t, window=1024, keep=64, scale=0.125, cap=0.0, maps=2)
+        window_attn.difference(maps, 8, window_attn.Difference(0.5, 0.5, 1e-6, 128))
+
+
+def gla_case(tokens: int, batch: int) -> None:
+    """16 heads with a 128 x 256 state: a prompt of `tokens` tokens in chunks, or (tokens 1) a decode step of `batch` sequences."""
+    from . import gla
+    h, dk, dv = 16, 128, 256
+    geo = gla.Geometry(h, dk, dv, dk, dv, 16, 16.0, 1e-6)
+    w2, bias = (torch.randn((h * dk, 16), device="cuda") * 0.25).to(torch.bfloat16), torch.randn(h * dk, device="cuda") + 2
+    proj, norm = torch.randn((batch * tokens, geo.width), device="cuda").to(torch.bfloat16), torch.ones(dv, device="cuda")
+    slots, starts = torch.arange(batch, dtype=torch.int32, device="cuda"), torch.tensor([0, tokens], dtype=torch.int32, device="cuda")
+    for _ in range(3):
+        state = torch.zeros((batch, h, dk, dv), device="cuda")
+        if tokens == 1:
+            gla.recurrent(proj, w2, bias, norm, state, slots, geo)
+        else:
+            gla.chunked(proj, w2, bias, norm, state, slots, geo, starts, tokens)
+
+
+CASES = {"two_maps_decode": two_maps_decode, "two_maps_prefill": two_maps_prefill, "gla_decode": lambda: gla_case(1, 64),
+         "gla_prefill": lambda: gla_case(2048, 1), "gemm_prefill": lambda: gemm(4096, 4096, 4096), "gemm_decode": lambda: gemm(64, 28672, 4096),
          "gemm_decode_splitk": lambda: gemm(64, 4096, 14336),
          "attn_decode": attn_decode, "attn_prefill": attn_prefill, "w4_decode": lambda: w4_gemm(64, 28672, 4096),
          "w4_prefill": lambda: w4_gemm(4096, 4096, 4096), "gdn_decode": gdn_decode, "moe_dispatch": moe_dispatch,

@@ -99,8 +99,28 @@ def _cfg_int(cfg: dict, *names, default: int = 0) -> int:
     return default
 
 
+def _own_family(cfg: dict):
+    """``(configuration object, its tensor shapes)`` of a family whose layers may all differ (None for the others)."""
+    if cfg.get("family") == "tepetar":
+        from ..models.tepetar import TepetarConfig as Config, tensor_shapes
+    elif cfg.get("family") == "kamedra":
+        from ..models.kamedra import KamedraConfig as Config, tensor_shapes
+    else:
+        return None
+    own = Config.from_dict(cfg)
+    return own, tensor_shapes(own)
+
+
 def model_parameters(cfg: dict) -> dict:
     """Counts from a model configuration (canonical keys of ``model_config.json``; Hugging Face spellings accepted)."""
+    own = _own_family(cfg)
+    if own is not None:
+        groups: dict[str, int] = {}
+        for name, shape in own[1].items():
+            groups[group_of(name)] = groups.get(group_of(name), 0) + math.prod(shape)
+        total = sum(groups.values())
+        return {"groups": groups, "total": total, "active_per_token": total, "experts": None, "top_k": None, "layers": own[0].num_layers,
+                "attention_layers": len(own[0].key_spans())}
     h = _cfg_int(cfg, "hidden_size")
     layers = _cfg_int(cfg, "num_layers", "num_hidden_layers")
     hq = _cfg_int(cfg, "num_heads", "num_attention_heads")
@@ -148,13 +168,10 @@ def model_memory(cfg: dict, weight_bytes: int, *, batch: int = 1, context: int =
     pages = batch * math.ceil(context / PAGE_TOKENS) + 1
     kv = pages * page_bytes(p["attention_layers"], max(1, hk // tp), d)
     state = 0
-    if cfg.get("family") == "tepetar":  # bf16 pages, every layer its own geometry
-        from ..models.tepetar import TepetarConfig
-        kv = pages * PAGE_TOKENS * TepetarConfig.from_dict(cfg).kv_token_bytes(2)
-    elif cfg.get("family") == "kamedra":  # the same, plus a recurrent state per sequence
-        from ..models.kamedra import KamedraConfig
-        own = KamedraConfig.from_dict(cfg)
-        kv, state = pages * PAGE_TOKENS * own.kv_token_bytes(2), batch * own.state_bytes()
+    own = _own_family(cfg)
+    if own is not None:  # bf16 pages, every layer its own geometry; perhaps a recurrent state per sequence
+        kv = pages * PAGE_TOKENS * own[0].kv_token_bytes(2)
+        state = batch * own[0].state_bytes() if hasattr(own[0], "state_bytes") else 0
     lin_v = _cfg_int(cfg, "linear_num_value_heads")
     if lin_v:
         lin_layers = p["layers"] - p["attention_layers"]

@@ -200,11 +200,14 @@ def test_weights_as_stored_compute_the_same_products(dtype):
 
 def test_memory_of_a_deployment_counts_pages_and_state():
     from mfq_b200.models.kamedra import KamedraConfig
-    from mfq_b200.server.analysis import model_memory
+    from mfq_b200.server.analysis import model_memory, model_parameters
     cfg = KamedraConfig.from_source(cases.uneven()).to_dict()
     got = model_memory(cfg, 1000, batch=2, context=64)["per_gpu"]
     assert got["kv_cache"] == (2 * 4 + 1) * 16 * 2 * (2 * (64 + 32) + 96 + 80 + 32 + 16)
     assert got["recurrent_state"] == 2 * 4 * (3 * 32 * 48 + 2 * 48 * 112)
+    counts = model_parameters(cfg)
+    assert counts["attention_layers"] == 5 and counts["groups"]["dense_mlp"] == 3 * 104 * (72 + 40 + 56) + 3 * 104
+    assert counts["groups"]["embeddings"] == 150 * 104 and "head" not in counts["groups"]
 
 
 def test_budget_sets_the_state_aside_and_takes_models_without_pages():
