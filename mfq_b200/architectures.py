@@ -8,7 +8,7 @@ Runtime code consumes canonical names only (``model.block.N.attention.query.weig
 * ``deepseek_v3`` / ``glm4_moe``: latent-attention and shared-expert names, sigmoid router bias, and the next-token
   prediction layer these checkpoints append after the last decoder layer (``model.layers.<L>.{enorm,hnorm,eh_proj,
   shared_head.*}``), which becomes the ``predictor.*`` head;
-* ``tepetar``, ``kamedra``: ``l<N>.{mix,mlp,side}.*`` names (``config.json`` names the design under ``architecture``).
+* ``tepetar``, ``kamedra``, ``bufolorn``: ``l<N>.{mix,mlp,side}.*`` names (``config.json`` names the design under ``architecture``).
 
 :func:`detect_family` picks the family from ``config.json`` (``model_type`` / ``architectures``); :func:`to_canonical`
 renames, stacks per-expert matrices, splits fused tensors and moves the appended prediction layer.  Names match the
@@ -130,6 +130,37 @@ KAMEDRA_MIXER = {
             "a1": "linear_attention.decay_a.weight", "a2": "linear_attention.decay_b.weight",
             "a2.b": "linear_attention.decay_b.bias"},
 }
+# Bufolorn: the same short names; the experts' matrices (``mlp.e<N>.*``) are stacked
+BUFOLORN_TOP = {
+    "embed": "model.token_embedding.weight", "final.norm": "model.output_norm.weight", "final.norm.b": "model.output_norm.bias",
+    "head": "model.output.weight",
+}
+_UNIT = ("gate", "up", "down")
+BUFOLORN_LAYER = {
+    "norm1": "norm.weight", "norm1.b": "norm.bias", "mlp.router": "mlp.router.weight", "mlp.correction": "mlp.router.bias",
+    **{f"mlp.{n}": f"mlp.{n}.weight" for n in _UNIT}, **{f"mlp.shared.{n}": f"mlp.shared_expert.{n}.weight" for n in _UNIT},
+}
+BUFOLORN_MIXER = {
+    "latent_attention": {"q": "attention.query.weight", "dkv": "attention.latent.weight", "dkv.norm": "attention.latent_norm.weight",
+                         "uk": "attention.key_up.weight", "uv": "attention.value_up.weight", "o": "attention.output.weight"},
+    "parallel": {
+        **{f"left.{k}": f"attention.{n}.weight" for k, n in (("q", "query"), ("k", "key"), ("v", "value"), ("o", "output"))},
+        **{f"left.{k}.b": f"attention.{n}.bias" for k, n in (("q", "query"), ("k", "key"), ("v", "value"), ("o", "output"))},
+        "left.rel": "attention.distance.bias", "left.sink": "attention.sink",
+        **{f"right.{k}": f"time_mixing.{n}.weight" for k, n in (("r", "receptance"), ("k", "key"), ("v", "value"), ("g", "gate"), ("o", "output"))},
+        **{f"right.mu.{k}": f"time_mixing.{n}_mix" for k, n in (("r", "receptance"), ("k", "key"), ("v", "value"), ("g", "gate"), ("w", "decay"))},
+        "right.w1": "time_mixing.decay_a.weight", "right.w2": "time_mixing.decay_b.weight", "right.w0": "time_mixing.decay_b.bias",
+        "right.u": "time_mixing.bonus", "right.norm": "time_mixing.norm.weight",
+    },
+    "channel_delta": {
+        **{k: f"linear_attention.{n}.weight" for k, n in (("q", "query"), ("k", "key"), ("v", "value"), ("o", "output"))},
+        **{f"{k}.conv": f"linear_attention.{n}_conv.weight" for k, n in (("q", "query"), ("k", "key"), ("v", "value"))},
+        "b": "linear_attention.beta.weight", "A_log": "linear_attention.a", "dt_bias": "linear_attention.dt_bias",
+        "norm": "linear_attention.norm.weight", "a1": "linear_attention.decay_a.weight", "a2": "linear_attention.decay_b.weight",
+        "g1": "linear_attention.gate_a.weight", "g2": "linear_attention.gate_b.weight",
+    },
+}
+_OWN_EXPERT_RE = re.compile(r"^mlp\.e(\d+)\.(gate|up|down)$")
 _OWN_LAYER_RE = re.compile(r"^l(\d+)\.(.+)$")
 FAMILY_OF_MODEL_TYPE = {
     "llama": "llama", "mistral": "llama", "qwen2": "llama", "qwen3": "llama", "mixtral": "llama", "qwen2_moe": "llama",
@@ -143,7 +174,7 @@ def detect_family(hf_config: dict | None, names=()) -> str:
     """Source naming family of a checkpoint: from ``model_type`` (or the text sub-config's), else from its tensor names."""
     cfg = hf_config or {}
     own = str(cfg.get("architecture", "")).lower()
-    if own in ("tepetar", "kamedra"):
+    if own in ("tepetar", "kamedra", "bufolorn"):
         return own
     for c in (cfg, cfg.get("text_config") or {}):
         fam = FAMILY_OF_MODEL_TYPE.get(str(c.get("model_type", "")).lower())
@@ -221,6 +252,20 @@ def kamedra_name(name: str, mixers: list[str]) -> str | None:
     return f"model.block.{int(m[1])}.{known[m[2]]}" if m[2] in known else None
 
 
+def bufolorn_name(name: str, mixers: list[str]) -> tuple[str, int | None] | None:
+    """Source name of a Bufolorn tensor -> (canonical name, expert index or None); ``mixers``: the kind of every layer."""
+    if name in BUFOLORN_TOP:
+        return BUFOLORN_TOP[name], None
+    m = _OWN_LAYER_RE.match(name)
+    if not m or int(m[1]) >= len(mixers):
+        return None
+    block, e = f"model.block.{int(m[1])}.", _OWN_EXPERT_RE.match(m[2])
+    if e:
+        return f"{block}mlp.experts.{e[2]}.weight", int(e[1])
+    known = BUFOLORN_LAYER | {"mix." + k: v for k, v in BUFOLORN_MIXER.get(mixers[int(m[1])], {}).items()}
+    return (block + known[m[2]], None) if m[2] in known else None
+
+
 def split_fused_linear_attention(out: dict[str, np.ndarray], k_heads: int, v_heads: int, head_dim: int) -> None:
     """The hybrid family's fused projections, in place: ``in_proj_qkvz`` holds, per KEY head, the rows
     ``[q (d) | k (d) | v (r d) | z (r d)]`` with ``r = v_heads / k_heads``; ``in_proj_ba`` holds ``[b (r) | a (r)]`` per
@@ -243,6 +288,24 @@ def split_fused_linear_attention(out: dict[str, np.ndarray], k_heads: int, v_hea
         out[base + "alpha.weight"] = np.ascontiguousarray(per[:, r:].reshape(-1, w.shape[-1]))
 
 
+def _renamed_and_stacked(tensors: dict[str, np.ndarray], rename) -> dict[str, np.ndarray]:
+    """Tensors under the names ``rename`` gives (name, expert index or None), those of experts stacked; without the ones it drops."""
+    out: dict[str, np.ndarray] = {}
+    experts: dict[str, dict[int, np.ndarray]] = {}
+    for name, t in tensors.items():
+        mapped = rename(name)
+        if mapped is None:
+            continue
+        cname, e = mapped
+        if e is None:
+            out[cname] = t
+        else:
+            experts.setdefault(cname, {})[e] = t
+    for cname, parts in experts.items():
+        out[cname] = np.stack([parts[i] for i in range(len(parts))])
+    return out
+
+
 def to_canonical(hf_tensors: dict[str, np.ndarray], hf_config: dict | None = None) -> dict[str, np.ndarray]:
     """Rename a Hugging Face state dict; per-expert matrices are stacked into ``[experts, out, in]`` tensors, a fused
     ``gate_up`` expert tensor is split into ``gate`` and ``up``, fused linear-attention projections are split, and the
@@ -254,24 +317,15 @@ def to_canonical(hf_tensors: dict[str, np.ndarray], hf_config: dict | None = Non
     if family == "kamedra":
         mixers = [l.get("type") for l in hf_config["layers"]]
         return {c: t for c, t in ((kamedra_name(n, mixers), t) for n, t in hf_tensors.items()) if c is not None}
+    if family == "bufolorn":
+        mixers = [l.get("type") for l in hf_config["layers"]]
+        return _renamed_and_stacked(hf_tensors, lambda n: bufolorn_name(n, mixers))
     text = dict(hf_config or {})
     text.update(text.get("text_config") or {})
     nextn = None
     if family in ("deepseek_v3", "glm4_moe") and text.get("num_hidden_layers") and text.get("num_nextn_predict_layers", 0):
         nextn = int(text["num_hidden_layers"])
-    out: dict[str, np.ndarray] = {}
-    experts: dict[str, dict[int, np.ndarray]] = {}
-    for name, t in hf_tensors.items():
-        mapped = canonical_name(name, nextn)
-        if mapped is None:
-            continue
-        cname, e = mapped
-        if e is None:
-            out[cname] = t
-        else:
-            experts.setdefault(cname, {})[e] = t
-    for cname, parts in experts.items():
-        out[cname] = np.stack([parts[i] for i in range(len(parts))])
+    out = _renamed_and_stacked(hf_tensors, lambda n: canonical_name(n, nextn))
     for cname in [n for n in out if n.endswith("mlp.experts.gate_up.weight")]:
         fused = out.pop(cname)
         half = fused.shape[1] // 2
@@ -308,6 +362,9 @@ def config_from_hf(hf: dict) -> dict:
     if family == "kamedra":
         from .models.kamedra import KamedraConfig
         return KamedraConfig.from_source(hf).to_dict()
+    if family == "bufolorn":
+        from .models.bufolorn import BufolornConfig
+        return BufolornConfig.from_source(hf).to_dict()
     if hf.get("text_config"):
         hf = {**hf, **hf["text_config"]}
     heads = hf.get("num_attention_heads", 32)

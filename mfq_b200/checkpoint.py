@@ -135,7 +135,7 @@ def quantize_tensors(tensors: dict[str, np.ndarray], *, dense: str = "nint4", ex
         if progress:
             progress(name)
         a = np.asarray(t, dtype=np.float32)
-        keep = a.ndim < 2 or "norm" in name or "router" in name or name.endswith(".bias")
+        keep = a.ndim < 2 or "norm" in name or "router" in name or name.endswith((".bias", ".bonus")) or "_conv." in name
         profile = dense_profile
         if widths is not None and name in widths:
             profile = None if widths[name] is None else parse_profiles(f"NINT{widths[name]}")[0]

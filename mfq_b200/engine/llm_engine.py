@@ -433,7 +433,8 @@ class LLMEngine:
             self.model.attn_splits = self.model.decode_splits(max(1, singles), max(c + m for _, c, m in portions))
         return StepBuffers(input_ids=ids, positions=positions, slots=slots, block_table=self.cache.block_table.index_select(0, row_ids.long()),
                            seq_lens=seq_lens, state_slots=row_ids if self.rec_state is not None else None, cu_seqlens=starts,
-                           q_starts=q_starts, tok_seq=tok_seq, max_q=max(counts), num_decode=singles)
+                           q_starts=q_starts, tok_seq=tok_seq, max_q=max(counts), num_decode=singles,
+                           portions=[(c, m) for _, c, m in portions])
 
     def extend(self, portions, wanted=None) -> torch.Tensor | None:
         """Append given tokens to open rows, all in one forward: ``portions`` is a list of ``(row, token ids)`` (a row at most

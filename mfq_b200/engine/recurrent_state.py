@@ -43,11 +43,12 @@ class RecurrentState:
 
 
 class LayerStates(RecurrentState):
-    """fp32 state ``[slots, *shape]`` of each layer in ``shapes`` (layer index -> shape of one sequence's state)."""
+    """fp32 state ``[slots, *shape]`` of each entry of ``shapes``: layer index, or (layer index, part) where a layer keeps several
+    things, -> shape of one sequence's state."""
 
-    def __init__(self, shapes: dict[int, tuple[int, ...]], slots: int, device) -> None:
+    def __init__(self, shapes: dict, slots: int, device) -> None:
         self.by_layer = {i: torch.zeros((slots, *shape), dtype=torch.float32, device=device) for i, shape in shapes.items()}
         super().__init__(list(self.by_layer.values()))
 
-    def layer(self, i: int) -> torch.Tensor:
+    def layer(self, i) -> torch.Tensor:
         return self.by_layer[i]

@@ -246,6 +246,8 @@ class StepBuffers:
     tok_seq: torch.Tensor | None = None  # [T] int32: the sequence of every row
     max_q: int = 1  # longest portion
     num_decode: int = 0
+    portions: list[tuple[int, int]] = field(default_factory=list)  # host: (first position, tokens) of every sequence
+    plans: dict = field(default_factory=dict)  # what layers derive from the portions, kept for the layers alike
 
 
 class LlamaModel:

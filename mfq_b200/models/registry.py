@@ -83,6 +83,7 @@ def _build_moe_decoder(raw: dict, store, o: LoadOptions):
 FAMILIES = (
     _unquantized("tepetar", "TepetarConfig", "TepetarWeights", "TepetarModel"),
     _unquantized("kamedra", "KamedraConfig", "KamedraWeights", "KamedraModel"),
+    _unquantized("bufolorn", "BufolornConfig", "BufolornWeights", "BufolornModel"),
     Family("latent attention", lambda raw: bool(raw.get("kv_lora_rank")), _build_mla),
     Family("decoder", lambda raw: True, _build_moe_decoder),  # dense and mixture-of-experts decoders
 )

@@ -96,5 +96,11 @@ class YarnScaling:
         ramp = ((i - low) / (high - low)).clamp(0.0, 1.0)
         return base * ((1.0 - ramp) + ramp / self.factor)
 
+    def frequencies(self, rot: int, theta: float) -> list[float]:
+        """The same in double precision."""
+        low, high = self.correction_range(rot, theta)
+        ramp = [min(max((i - low) / max(high - low, 0.001), 0.0), 1.0) for i in range(rot // 2)]
+        return [float(theta) ** (-2.0 * i / rot) * (r / self.factor + 1.0 - r) for i, r in enumerate(ramp)]
+
     def max_position(self) -> int:
         return int(self.original_max_position * self.factor)

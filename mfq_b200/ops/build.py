@@ -23,7 +23,9 @@ HERE = Path(__file__).resolve().parent
 CSRC = HERE / "csrc"
 LIB_PATH = HERE / "_mfq_b200_kernels.so"
 DENSE_LIB_PATH = HERE / "_mfq_b200_dense.so"
-DENSE_SOURCES = ("dense_gemm.cu", "stream_ops.cu", "window_attn.cu", "window_attn_prefill.cu", "gla.cu", "gla_chunk.cu")
+DENSE_SOURCES = ("dense_gemm.cu", "dense_moe.cu", "stream_ops.cu", "mix_ops.cu", "window_attn.cu", "window_attn_prefill.cu",
+                 "window_attn_prefill_bias.cu", "latent_attn.cu", "gla.cu", "gla_chunk.cu", "delta.cu", "delta_chunk.cu", "moe_route.cu")
+SHARED_SOURCES = ("moe_route.cu",)  # part of the main library too
 OBJ_DIR = HERE / "build"
 
 NVCC_FLAGS = [
@@ -69,7 +71,7 @@ def _compile_one(src: Path, force: bool) -> tuple[Path, str]:
 def libraries() -> dict[str, tuple[Path, list[Path]]]:
     """Library name -> (path, its sources)."""
     dense = [p for p in sources() if p.name in DENSE_SOURCES]
-    return {"kernels": (LIB_PATH, [p for p in sources() if p not in dense]), "dense": (DENSE_LIB_PATH, dense)}
+    return {"kernels": (LIB_PATH, [p for p in sources() if p not in dense or p.name in SHARED_SOURCES]), "dense": (DENSE_LIB_PATH, dense)}
 
 
 def _link(path: Path, objs: list[Path]) -> None:
@@ -86,14 +88,14 @@ def build(force: bool = False, verbose: bool = False, only: str | None = None) -
     OBJ_DIR.mkdir(exist_ok=True)
     libs = libraries()
     chosen = libs if only is None else {only: libs[only]}
-    srcs = [s for _, group in chosen.values() for s in group]
+    srcs = sorted({s for _, group in chosen.values() for s in group})
     with ThreadPoolExecutor(max_workers=min(8, len(srcs))) as pool:
         results = dict(zip(srcs, pool.map(lambda s: _compile_one(s, force), srcs)))
     log = "".join(text for _, text in results.values())
     if log:
         (OBJ_DIR / "ptxas.log").write_text(log)
     for path, group in chosen.values():
-        if any(results[s][1] for s in group) or not path.exists():
+        if not path.exists() or any(results[s][1] or results[s][0].stat().st_mtime > path.stat().st_mtime for s in group):
             _link(path, [results[s][0] for s in group])
     if verbose and log:
         print(log, file=sys.stderr)

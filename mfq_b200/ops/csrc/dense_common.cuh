@@ -65,14 +65,19 @@ enum : int {
   kDenseGelu = 2,   // out[t, n] = gelu_tanh(v + bias[n]) * table[ids[t], n]
   kDenseGeluGlu = 3,  // rows packed as for kDenseGlu: out = gelu_tanh(gate) * up, half as wide
   kDenseSoftcap = 4,  // out[t, n] = limit * tanh((v + bias[n]) / limit)
-  kDenseAdd = 5,      // x[t, n] += v + bias[n] on the fp32 stream x = out
+  kDenseAdd = 5,      // x[t, n] += alpha * (v + bias[n]) on the fp32 stream x = out
+  kDenseReluGlu = 6,  // rows packed as for kDenseGlu: out = max(gate, 0) * up, half as wide
+  kDenseSiluGlu = 7,  // ... out = silu(gate) * up
+  kDenseFloat = 8,    // fp32 out[t, n] = v + bias[n]
 };
-__host__ __device__ constexpr bool dense_is_glu(int kind) { return kind == kDenseGlu || kind == kDenseGeluGlu; }
+__host__ __device__ constexpr bool dense_is_glu(int kind) {
+  return kind == kDenseGlu || kind == kDenseGeluGlu || kind == kDenseReluGlu || kind == kDenseSiluGlu;
+}
 
 struct DenseEpilogue {
   int kind;
   const float* bias;  // [N] or null
-  float alpha, limit;  // GLU: y = g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit); soft cap: limit
+  float alpha, limit;  // GLU: y = g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit); soft cap: limit; add: alpha
   const void* table;   // GELU: [tokens of the vocabulary, N] in the activation type
   const int* ids;
   void* out;
@@ -85,6 +90,14 @@ __device__ __forceinline__ float clipped_glu(float gate, float up, float alpha, 
 }
 __device__ __forceinline__ float gelu_tanh(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+__device__ __forceinline__ float gated_unit(const DenseEpilogue& e, float gate, float up) {
+  switch (e.kind) {
+    case kDenseGlu: return clipped_glu(gate, up, e.alpha, e.limit);
+    case kDenseGeluGlu: return gelu_tanh(gate) * up;
+    case kDenseReluGlu: return fmaxf(gate, 0.f) * up;
+    default: return gate / (1.f + expf(-gate)) * up;
+  }
 }
 
 // One output item of token `t`: 8 packed rows from `n0`, or 16 for the GLU kinds.  `load(n, v)` fetches the finished fp32 sums
@@ -104,8 +117,12 @@ __device__ __forceinline__ void dense_store_item(const DenseEpilogue& e, int t, 
     float r[8];
     load8<float>(x, r);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) r[i] += v[i];
+    for (int i = 0; i < 8; ++i) r[i] = fmaf(e.alpha, v[i], r[i]);
     store8<float>(x, r);
+    return;
+  }
+  if (e.kind == kDenseFloat) {
+    store8<float>(static_cast<float*>(e.out) + size_t(t) * e.ldo + n0, v);
     return;
   }
   T* out = static_cast<T*>(e.out) + size_t(t) * e.ldo;
@@ -119,7 +136,7 @@ __device__ __forceinline__ void dense_store_item(const DenseEpilogue& e, int t, 
       for (int i = 0; i < 8; ++i) u[i] += b[i];
     }
 #pragma unroll
-    for (int i = 0; i < 8; ++i) v[i] = e.kind == kDenseGlu ? clipped_glu(v[i], u[i], e.alpha, e.limit) : gelu_tanh(v[i]) * u[i];
+    for (int i = 0; i < 8; ++i) v[i] = gated_unit(e, v[i], u[i]);
     store8<T>(out + (n0 >> 1), v);
     return;
   }

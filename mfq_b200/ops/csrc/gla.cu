@@ -42,7 +42,8 @@ gla_recurrent_kernel(const T* __restrict__ proj, const T* __restrict__ w2, const
   float* q_s = gla_sm;           // [dk]
   float* k_s = q_s + dk;         // [dk]
   float* d_s = k_s + dk;         // [dk] decay
-  float* a_s = d_s + dk;         // [rank]
+  float* u_s = d_s + dk;         // [dk] bonus
+  float* a_s = u_s + dk;         // [rank]
   float* v_s = a_s + rank;       // [cols]
   float* part = v_s + cols;      // [R][cols]
   __shared__ float red[33];
@@ -79,7 +80,8 @@ gla_recurrent_kernel(const T* __restrict__ proj, const T* __restrict__ w2, const
 #pragma unroll
         for (int j = 0; j < 8; ++j) z = fmaf(x[j], a_s[r + j], z);
       }
-      d_s[i] = exp2f(log2_sigmoid(z) * p.s.inv_tau);
+      d_s[i] = exp2f(gla_log2_decay(p.s, z));
+      if (p.s.bonus) u_s[i] = p.s.bonus[h * dk + i];
     }
     __syncthreads();
     if (worker) {
@@ -96,10 +98,17 @@ gla_recurrent_kernel(const T* __restrict__ proj, const T* __restrict__ w2, const
           if (i0 + i < mine) {
             const int r = rg + R * (i0 + i);
             const float q = q_s[r], k = k_s[r], d = d_s[r];
+            if (p.s.bonus) {  // read-out before the write
+              const float uk = u_s[r] * k;
+              o.x = fmaf(q, fmaf(uk, v.x, s[i].x), o.x); o.y = fmaf(q, fmaf(uk, v.y, s[i].y), o.y);
+              o.z = fmaf(q, fmaf(uk, v.z, s[i].z), o.z); o.w = fmaf(q, fmaf(uk, v.w, s[i].w), o.w);
+            }
             s[i].x = fmaf(d, s[i].x, k * v.x); s[i].y = fmaf(d, s[i].y, k * v.y);
             s[i].z = fmaf(d, s[i].z, k * v.z); s[i].w = fmaf(d, s[i].w, k * v.w);
-            o.x = fmaf(q, s[i].x, o.x); o.y = fmaf(q, s[i].y, o.y);
-            o.z = fmaf(q, s[i].z, o.z); o.w = fmaf(q, s[i].w, o.w);
+            if (!p.s.bonus) {
+              o.x = fmaf(q, s[i].x, o.x); o.y = fmaf(q, s[i].y, o.y);
+              o.z = fmaf(q, s[i].z, o.z); o.w = fmaf(q, s[i].w, o.w);
+            }
             *reinterpret_cast<float4*>(st + size_t(r) * dv) = s[i];
           }
         }
@@ -124,7 +133,7 @@ gla_recurrent_kernel(const T* __restrict__ proj, const T* __restrict__ w2, const
     const float f = rsqrtf(ss * p.s.inv_dv + p.s.eps);
     for (int c = tid; c < cols; c += kGlaThreads) {
       const float gate = to_float(row[2 * H * dk + (H + h) * dv + c_base + c]);
-      y[(size_t(t) * H + h) * dv + c_base + c] = from_float<T>(part[c] * f * norm_w[c_base + c] * silu_of(gate));
+      y[(size_t(t) * H + h) * dv + c_base + c] = from_float<T>(part[c] * f * norm_w[h * p.s.norm_stride + c_base + c] * silu_of(gate));
     }
     __syncthreads();  // the token's vectors are replaced next
   }
@@ -134,7 +143,7 @@ gla_recurrent_kernel(const T* __restrict__ proj, const T* __restrict__ w2, const
 template <typename T>
 static int launch_gla_recurrent(const void* proj, const void* w2, const float* bias, const float* norm_w, void* y,
                                 const GlaRecurrentParams& p, int B, cudaStream_t stream) {
-  const int smem = (3 * p.s.dk + p.s.rank + (1 + p.rows) * (p.s.dv / p.split)) * 4;
+  const int smem = (4 * p.s.dk + p.s.rank + (1 + p.rows) * (p.s.dv / p.split)) * 4;
   if (smem > 200 * 1024) return -5;
   static int allowed = 48 * 1024;
   if (smem > allowed) {
@@ -154,16 +163,19 @@ static int launch_gla_recurrent(const void* proj, const void* w2, const float* b
 
 using namespace mfq;
 
-// proj [T, row_stride] as in gla.cuh; w2 [H * dk, rank]; bias [H * dk] and norm_w [dv] fp32; y [T, H * dv]; state fp32
+// proj [T, row_stride] as in gla.cuh; w2 [H * dk, rank]; bias and bonus (may be null) [H * dk] and norm_w [dv] (norm_stride 0) or
+// [H, dv] fp32; y [T, H * dv]; state fp32
 // [slots, H, dk, dv].  starts null: one token per sequence.  split: cluster size over a head's columns.
 extern "C" int mfq_gla_recurrent(const void* proj, const void* w2, const float* bias, const float* norm_w, void* y, float* state,
                                  const int* slot, const int* starts, int B, int H, int dk, int dv, int real_dv, int rank,
-                                 int row_stride, int split, float scale, float inv_tau, float eps, int fp32, cudaStream_t stream) {
+                                 int row_stride, int split, float scale, float inv_tau, float eps, int decay, int norm_stride,
+                                 const float* bonus, int fp32, cudaStream_t stream) {
+  if (decay < kGlaSigmoid || decay > kGlaExp || (norm_stride && norm_stride != dv)) return -1;
   if (B <= 0 || B > 65535 || H <= 0 || dk <= 0 || dv <= 0 || dk % 16 || dv % 16 || rank <= 0 || rank % 8 || real_dv <= 0 || real_dv > dv) return -1;
   if (row_stride < 2 * H * (dk + dv) + rank || row_stride % 8 || split < 1 || split > kGlaMaxSplit || dv % (4 * split)) return -1;
   const int groups = dv / split / 4;
   if (groups > kGlaThreads) return -1;
-  GlaRecurrentParams p{GlaShape{H, dk, dv, rank, row_stride, scale, inv_tau, 1.f / float(real_dv), eps}, starts, slot, state, split,
+  GlaRecurrentParams p{GlaShape{H, dk, dv, rank, row_stride, scale, inv_tau, 1.f / float(real_dv), eps, decay, norm_stride, bonus}, starts, slot, state, split,
                        min(dk, kGlaThreads / groups)};
   return fp32 ? launch_gla_recurrent<float>(proj, w2, bias, norm_w, y, p, B, stream)
               : launch_gla_recurrent<__nv_bfloat16>(proj, w2, bias, norm_w, y, p, B, stream);

@@ -9,12 +9,17 @@
 //   gla_chunk_state    a thread per eight state elements: replaces every U by the S_0 of its chunk, advances the state
 //   gla_chunk_output   a CTA per (chunk, head): A, then O = A V + (2^b q)^T S_0, per-head norm and gate
 //
+// With a bonus u the query of token t stands before its own write: b_(t-1) takes the place of b_t beside q, A is strictly lower
+// triangular, and its diagonal is sum_c q_tc u_c k_tc.
+//
 // Exponents never overflow: A is formed in 16 x 16 blocks relative to b before the block's first row, where both factors are at
 // most 1 below the diagonal; a diagonal block whose own decay spans more than 2^-100 is summed term by term instead.
 // Precision: the recurrence is kept to fp32 level on bf16 tensor cores by splitting every fp32 operand into two bf16 numbers
 // (16 significant bits): 2^(b_C - b) k, 2^b q, the factors of A, A itself and S_0; v is bf16 as projected.  The 16-row
 // products here are too small for 128-row tcgen05 tiles, and their operands are made in registers, so they run as mma.sync.
 #include "gla.cuh"
+
+#include <type_traits>
 
 namespace mfq {
 namespace {
@@ -47,6 +52,10 @@ __device__ __forceinline__ float gc_log2_sigmoid(float z) {
   float y;
   asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(1.f + gc_exp2(-1.4426950408889634f * fabsf(z))));
   return fmaf(1.4426950408889634f, fminf(z, 0.f), -y);
+}
+__device__ __forceinline__ float gc_log2_decay(const GlaShape& s, float z) {
+  if (s.decay == kGlaSigmoid) return gc_log2_sigmoid(z) * s.inv_tau;
+  return fmaxf(-1.4426950408889634f * gc_exp2(1.4426950408889634f * z), kGlaFloor);
 }
 __device__ __forceinline__ float gc_silu(float x) { return __fdividef(x, 1.f + gc_exp2(-1.4426950408889634f * fmaxf(x, -80.f))); }
 __device__ __forceinline__ void gc_cp16(void* dst, const void* src) {
@@ -173,7 +182,7 @@ gla_chunk_local_kernel(const GlaChunkParams p) {
       }
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
-        run += t + j < at.n ? gc_log2_sigmoid(z[j]) * p.s.inv_tau : 0.f;
+        run += t + j < at.n ? gc_log2_decay(p.s, z[j]) : 0.f;
         b_s[(t + j) * bp + c] = run;
       }
     }
@@ -299,7 +308,7 @@ __host__ __device__ inline GlaOutputSmem gc_output_smem(int dk, int dv) {
 }
 
 // NT: upper bound of the 8-column tiles of a warp (dv / 32)
-template <int NT>
+template <int NT, bool kBonus>
 __global__ void __launch_bounds__(kGcThreads, NT <= 4 ? 2 : 1)
 gla_chunk_output_kernel(const GlaChunkParams p) {
   pdl_trigger();
@@ -331,6 +340,23 @@ gla_chunk_output_kernel(const GlaChunkParams p) {
   }
   gc_wait<0>();
   __syncthreads();
+  auto b_query = [&](int t, int c) {  // b of the state that token t reads, channels c and c + 1
+    if (!kBonus) return *reinterpret_cast<const float2*>(b_s + t * bp + c);
+    return t ? *reinterpret_cast<const float2*>(b_s + (t - 1) * bp + c) : make_float2(0.f, 0.f);
+  };
+  if (kBonus) {  // diagonal of A, kept where the norm's sums go later
+    for (int t = warp; t < kGc; t += kGcWarps) {
+      float x = 0.f;
+      for (int c = lane * 2; c < dk; c += 64) {
+        const float2 q = gc_pair(q_s + t * kp + c), k = gc_pair(k_s + t * kp + c), u = *reinterpret_cast<const float2*>(p.s.bonus + h * dk + c);
+        x = fmaf(q.x * k.x, u.x, fmaf(q.y * k.y, u.y, x));
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) x += __shfl_xor_sync(0xffffffffu, x, o);
+      if (lane == 0) ss_s[t] = x * p.s.scale;
+    }
+    __syncthreads();
+  }
   // ----- A: warp = (row block I, one half of the column blocks J <= I, even or odd 16-channel steps); the second half of the
   //       columns is taken in reverse, so that every scheduler gets short and long row blocks -----
   const int ksteps = dk / 16;
@@ -353,7 +379,7 @@ gla_chunk_output_kernel(const GlaChunkParams p) {
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
           const int t = 16 * I + r * 8 + g;
-          const float2 q = gc_pair(q_s + t * kp + c), b = *reinterpret_cast<const float2*>(b_s + t * bp + c);
+          const float2 q = gc_pair(q_s + t * kp + c), b = b_query(t, c);
           gc_split(q.x * p.s.scale * gc_exp2(b.x - rf[e].x), q.y * p.s.scale * gc_exp2(b.y - rf[e].y), hi[e * 2 + r], lo[e * 2 + r]);
         }
       }
@@ -394,8 +420,8 @@ gla_chunk_output_kernel(const GlaChunkParams p) {
     if (!odd)
       each([&](float& x, float& y, int t, int s) {
         const float2 o = *reinterpret_cast<const float2*>(part + t * ap + s);
-        x = s <= t ? x + o.x : 0.f;
-        y = s + 1 <= t ? y + o.y : 0.f;
+        x = s + kBonus <= t ? x + o.x : (kBonus && s == t ? ss_s[t] : 0.f);
+        y = s + 1 + kBonus <= t ? y + o.y : (kBonus && s + 1 == t ? ss_s[t] : 0.f);
       });
     __syncthreads();
     if (!odd)
@@ -408,8 +434,9 @@ gla_chunk_output_kernel(const GlaChunkParams p) {
       const int t = (i >> 8) * 16 + ((i >> 4) & 15), s = (i >> 8) * 16 + (i & 15);
       if (s > t) continue;
       float x = 0.f;
+      if (kBonus && s == t) continue;  // as it is
       for (int c = 0; c < dk; ++c)
-        x += __bfloat162float(q_s[t * kp + c]) * __bfloat162float(k_s[s * kp + c]) * gc_exp2(b_s[t * bp + c] - b_s[s * bp + c]);
+        x += __bfloat162float(q_s[t * kp + c]) * __bfloat162float(k_s[s * kp + c]) * gc_exp2(b_s[(t - kBonus) * bp + c] - b_s[s * bp + c]);
       x *= p.s.scale;
       const __nv_bfloat16 hi = __float2bfloat16(x);
       a_hi[t * ap + s] = hi;
@@ -421,7 +448,7 @@ gla_chunk_output_kernel(const GlaChunkParams p) {
   {
     for (int t = warp; t < kGc; t += kGcWarps)
       for (int c = lane * 2; c < dk; c += 64) {
-        const float2 q = gc_pair(q_s + t * kp + c), b = *reinterpret_cast<const float2*>(b_s + t * bp + c);
+        const float2 q = gc_pair(q_s + t * kp + c), b = b_query(t, c);
         gc_split(q.x * p.s.scale * gc_exp2(b.x), q.y * p.s.scale * gc_exp2(b.y), *reinterpret_cast<uint32_t*>(q_s + t * kp + c),
                  *reinterpret_cast<uint32_t*>(k_s + t * kp + c));
       }
@@ -523,7 +550,7 @@ gla_chunk_output_kernel(const GlaChunkParams p) {
     for (int nt = 0; nt < NT; ++nt) {
       if (nt < tiles) {
         const int c = col(nt) + t4 * 2;
-        const float2 gt = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gate[r][nt])), w = *reinterpret_cast<const float2*>(p.norm_w + c);
+        const float2 gt = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gate[r][nt])), w = *reinterpret_cast<const float2*>(p.norm_w + h * p.s.norm_stride + c);
         *reinterpret_cast<__nv_bfloat162*>(y + c) =
             __floats2bfloat162_rn(o[nt][2 * r] * f * w.x * gc_silu(gt.x), o[nt][2 * r + 1] * f * w.y * gc_silu(gt.y));
       }
@@ -531,15 +558,15 @@ gla_chunk_output_kernel(const GlaChunkParams p) {
   }
 }
 
-template <int NT>
+template <int NT, bool kBonus>
 int launch_gla_output(const GlaChunkParams& p, dim3 grid, cudaStream_t stream) {
   const int smem = gc_output_smem(p.s.dk, p.s.dv).bytes;
   static int allowed = 0;
   if (smem > allowed) {
-    if (cudaFuncSetAttribute(gla_chunk_output_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -6;
+    if (cudaFuncSetAttribute(gla_chunk_output_kernel<NT, kBonus>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -6;
     allowed = smem;
   }
-  return launch_kernel(gla_chunk_output_kernel<NT>, grid, dim3(kGcThreads), smem, stream, p) == cudaSuccess ? 0 : -7;
+  return launch_kernel(gla_chunk_output_kernel<NT, kBonus>, grid, dim3(kGcThreads), smem, stream, p) == cudaSuccess ? 0 : -7;
 }
 
 }  // namespace
@@ -552,12 +579,14 @@ using namespace mfq;
 // Returns -5 for sizes that do not fit (callers use the token-by-token kernel).
 extern "C" int mfq_gla_chunk(const void* proj, const void* w2, const float* bias, const float* norm_w, void* y, float* state,
                              const int* slot, const int* starts, float* cum, float* u, float* gam, int B, int max_q, int H, int dk, int dv,
-                             int real_dv, int rank, int row_stride, float scale, float inv_tau, float eps, cudaStream_t stream) {
+                             int real_dv, int rank, int row_stride, float scale, float inv_tau, float eps, int decay, int norm_stride,
+                             const float* bonus, cudaStream_t stream) {
+  if (decay < kGlaSigmoid || decay > kGlaExp || (norm_stride && norm_stride != dv)) return -1;
   if (B <= 0 || B > 65535 || max_q <= 0 || H <= 0 || H > 65535 || dk <= 0 || dv <= 0 || dk % 16 || dv % 16 || rank <= 0 || rank % 8) return -1;
   if (real_dv <= 0 || real_dv > dv || row_stride < 2 * H * (dk + dv) + rank || row_stride % 8) return -1;
   const int local = gc_local_smem(dk, dv, rank).bytes;
   if (dk > kGcMaxDk || dv > kGcMaxDv || local > 227 * 1024 || gc_output_smem(dk, dv).bytes > 227 * 1024) return -5;
-  const GlaChunkParams p{GlaShape{H, dk, dv, rank, row_stride, scale, inv_tau, 1.f / float(real_dv), eps}, static_cast<const __nv_bfloat16*>(proj),
+  const GlaChunkParams p{GlaShape{H, dk, dv, rank, row_stride, scale, inv_tau, 1.f / float(real_dv), eps, decay, norm_stride, bonus}, static_cast<const __nv_bfloat16*>(proj),
                          static_cast<const __nv_bfloat16*>(w2), bias, norm_w, static_cast<__nv_bfloat16*>(y), starts, slot, state, cum, u, gam};
   const dim3 grid((max_q + kGc - 1) / kGc, H, B);
   static int allowed = 0;
@@ -567,7 +596,11 @@ extern "C" int mfq_gla_chunk(const void* proj, const void* w2, const float* bias
   }
   launch_kernel(gla_chunk_local_kernel, grid, dim3(kGcThreads), local, stream, p);
   launch_kernel(gla_chunk_state_kernel, dim3((dk * dv / 8 + 127) / 128, H, B), dim3(128), 0, stream, p);
-  const int rc = dv <= 128 ? launch_gla_output<4>(p, grid, stream) : dv <= 256 ? launch_gla_output<8>(p, grid, stream)
-                                                                          : launch_gla_output<16>(p, grid, stream);
+  auto output = [&](auto with_bonus) {
+    constexpr bool kBonus = decltype(with_bonus)::value;
+    return dv <= 128 ? launch_gla_output<4, kBonus>(p, grid, stream)
+                     : dv <= 256 ? launch_gla_output<8, kBonus>(p, grid, stream) : launch_gla_output<16, kBonus>(p, grid, stream);
+  };
+  const int rc = bonus ? output(std::true_type{}) : output(std::false_type{});
   return rc == 0 && cudaGetLastError() == cudaSuccess ? 0 : (rc ? rc : -7);
 }

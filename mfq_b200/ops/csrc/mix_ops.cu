@@ -1,0 +1,223 @@
+// Stages between the normalised stream and the projections or recurrences of a layer, for activations in bf16 or fp32.
+//
+//   layer_norm_out    h = (x - mean) / sqrt(var + eps) * w + b of the fp32 stream
+//   token_shift       every stream s of a token reads  h + (h' - h) * mu_s,  h' the row of the previous token (zeros before the
+//                     first); the last row of a sequence is kept in its state slot
+//   short_conv        causal convolution over time per channel, then SiLU; the last taps - 1 inputs are kept in the state slot
+//
+// Batches are ragged: sequence b owns rows starts[b] .. starts[b + 1] - 1 (starts null: row b) and state slot slot[b] (< 0: the
+// sequence is skipped).
+#include "dense_common.cuh"
+
+namespace mfq {
+
+constexpr int kMixVecs = 4;  // 8-wide vectors a thread keeps in registers
+
+template <typename T>
+__global__ void __launch_bounds__(512)
+layer_norm_out_kernel(const float* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias, T* __restrict__ out, int W,
+                      int width, float eps) {
+  pdl_trigger();
+  __shared__ float red[33];
+  const size_t row = blockIdx.x;
+  const int nvec = W / 8;
+  pdl_wait();
+  float v[kMixVecs][8];
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < kMixVecs; ++i) {
+    const int vi = threadIdx.x + i * blockDim.x;
+    if (vi < nvec) {
+      load8<float>(x + row * W + vi * 8, v[i]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) s += v[i][j];  // padding columns are zeros
+    }
+  }
+  const float inv = 1.f / float(width), mean = dense_block_sum(s, red) * inv;
+  __syncthreads();
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < kMixVecs; ++i) {
+    const int c = (threadIdx.x + i * blockDim.x) * 8;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      if (c + j < width) {
+        v[i][j] -= mean;
+        ss += v[i][j] * v[i][j];
+      }
+    }
+  }
+  const float rstd = rsqrtf(dense_block_sum(ss, red) * inv + eps);
+#pragma unroll
+  for (int i = 0; i < kMixVecs; ++i) {
+    const int vi = threadIdx.x + i * blockDim.x;
+    if (vi < nvec) {
+      float ww[8], bb[8];
+      load8<float>(w + vi * 8, ww);
+      load8<float>(bias + vi * 8, bb);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[i][j] = fmaf(v[i][j] * rstd, ww[j], bb[j]);
+      store8<T>(out + row * W + vi * 8, v[i]);
+    }
+  }
+}
+
+// h [T, W]; mu [streams, W]; out [T, streams * W]; last [slots, W] fp32.  The CTA of a sequence's first row reads the kept row and
+// replaces it, element by element in the same thread.
+template <typename T>
+__global__ void __launch_bounds__(256)
+token_shift_kernel(const T* __restrict__ h, const float* __restrict__ mu, float* __restrict__ last, const int* __restrict__ slot,
+                   const int* __restrict__ starts, const int* __restrict__ tok_seq, T* __restrict__ out, int W, int streams) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, b = tok_seq ? tok_seq[t] : t, s = slot[b];
+  const int t0 = starts ? starts[b] : t, t1 = starts ? starts[b + 1] : t + 1;
+  for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {
+    float x[8], p[8] = {};
+    load8<T>(h + size_t(t) * W + c, x);
+    if (t > t0) {
+      load8<T>(h + size_t(t - 1) * W + c, p);
+    } else if (s >= 0) {
+      load8<float>(last + size_t(s) * W + c, p);
+      float e[8];
+      load8<T>(h + size_t(t1 - 1) * W + c, e);
+      store8<float>(last + size_t(s) * W + c, e);
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) p[j] -= x[j];
+    for (int i = 0; i < streams; ++i) {
+      float m[8];
+      load8<float>(mu + size_t(i) * W + c, m);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) m[j] = fmaf(p[j], m[j], x[j]);
+      store8<T>(out + (size_t(t) * streams + i) * W + c, m);
+    }
+  }
+}
+
+struct ShortConvParams {
+  const float* w;     // [taps, C], last row for the current token
+  float* state;       // [slots, taps - 1, C], oldest first
+  const int* slot;    // [B]
+  const int* starts;  // [B + 1] or null
+  int C, taps, in_stride, out_stride;
+};
+
+// A thread owns 8 channels and a run of consecutive tokens; TAPS is an upper bound of the taps (missing ones weigh nothing).
+constexpr int kConvRunTokens = 16;
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128)
+short_conv_kernel(const T* __restrict__ x, T* __restrict__ out, const ShortConvParams p) {
+  pdl_trigger();
+  pdl_wait();
+  const int b = blockIdx.z, s = p.slot[b], c = (blockIdx.x * 128 + threadIdx.x) * 8;
+  if (s < 0 || c >= p.C) return;
+  const int r0 = p.starts ? p.starts[b] : b, len = p.starts ? p.starts[b + 1] - r0 : 1;
+  const int n0 = blockIdx.y * kConvRunTokens, n1 = min(len, n0 + kConvRunTokens), hist = p.taps - 1;
+  if (n0 >= len) return;
+  float* st = p.state + size_t(s) * hist * p.C + c;
+  auto in = [&](int n, float(&v)[8]) {  // input n tokens into the portion; n < 0: the kept ones
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = 0.f;
+    if (n >= 0) load8<T>(x + size_t(r0 + n) * p.in_stride + c, v);
+    else if (n + hist >= 0) load8<float>(st + size_t(n + hist) * p.C, v);
+  };
+  float w[TAPS][8], win[TAPS][8];  // win[i]: input i - (TAPS - 1) tokens from the current one
+#pragma unroll
+  for (int i = 0; i < TAPS; ++i) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) w[i][j] = 0.f;
+    if (i - (TAPS - p.taps) >= 0) load8<float>(p.w + size_t(i - (TAPS - p.taps)) * p.C + c, w[i]);
+    if (i > 0) in(n0 + i - TAPS, win[i]);
+  }
+  for (int n = n0; n < n1; ++n) {
+#pragma unroll
+    for (int i = 0; i + 1 < TAPS; ++i)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) win[i][j] = win[i + 1][j];
+    in(n, win[TAPS - 1]);
+    float y[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      float a = 0.f;
+#pragma unroll
+      for (int i = 0; i < TAPS; ++i) a = fmaf(w[i][j], win[i][j], a);
+      y[j] = a / (1.f + expf(-a));
+    }
+    store8<T>(out + size_t(r0 + n) * p.out_stride + c, y);
+  }
+  // Portions of one token: this thread is the only one that reads these kept inputs, so it may replace them.
+  if (!p.starts) {
+#pragma unroll
+    for (int i = 1; i < TAPS; ++i)
+      if (i - (TAPS - p.taps) >= 1) store8<float>(st + size_t(i - (TAPS - p.taps) - 1) * p.C, win[i]);
+  }
+}
+
+// The kept inputs after a portion of any length, as a launch of its own (blocks of the convolution still read the old ones).
+template <typename T>
+__global__ void __launch_bounds__(128)
+short_conv_state_kernel(const T* __restrict__ x, const ShortConvParams p) {
+  pdl_trigger();
+  pdl_wait();
+  const int b = blockIdx.y, s = p.slot[b], c = (blockIdx.x * 128 + threadIdx.x) * 8;
+  if (s < 0 || c >= p.C) return;
+  const int r0 = p.starts[b], len = p.starts[b + 1] - r0, hist = p.taps - 1;
+  float* st = p.state + size_t(s) * hist * p.C + c;
+  for (int i = 0; i < hist; ++i) {  // ascending: place i reads place i + len >= i
+    const int n = len - hist + i;
+    float v[8];
+    if (n >= 0) load8<T>(x + size_t(r0 + n) * p.in_stride + c, v);
+    else load8<float>(st + size_t(n + hist) * p.C, v);
+    store8<float>(st + size_t(i) * p.C, v);
+  }
+}
+
+template <typename T>
+static int launch_short_conv(const void* x, void* out, const ShortConvParams& p, int B, int max_q, cudaStream_t stream) {
+  const T* xt = static_cast<const T*>(x);
+  T* ot = static_cast<T*>(out);
+  const int blocks = (p.C / 8 + 127) / 128;
+  const dim3 grid(blocks, (max_q + kConvRunTokens - 1) / kConvRunTokens, B);
+  if (p.taps <= 4) launch_kernel(short_conv_kernel<T, 4>, grid, dim3(128), 0, stream, xt, ot, p);
+  else launch_kernel(short_conv_kernel<T, 8>, grid, dim3(128), 0, stream, xt, ot, p);
+  if (p.starts && p.taps > 1) launch_kernel(short_conv_state_kernel<T>, dim3(blocks, B), dim3(128), 0, stream, xt, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -7;
+}
+
+}  // namespace mfq
+
+using namespace mfq;
+
+extern "C" int mfq_layer_norm_out(const float* x, const float* w, const float* bias, void* out, int M, int W, int width, float eps, int fp32,
+                                  cudaStream_t stream) {
+  if (M <= 0 || W <= 0 || W % 8 || W > 8 * kMixVecs * 512 || width <= 0 || width > W) return -1;
+  const int nvec = W / 8;
+  int threads = (nvec + 31) / 32 * 32;
+  if (threads > 256) threads = max(256, ((nvec + kMixVecs - 1) / kMixVecs + 31) / 32 * 32);
+  if (fp32) launch_kernel(layer_norm_out_kernel<float>, dim3(M), dim3(threads), 0, stream, x, w, bias, static_cast<float*>(out), W, width, eps);
+  else launch_kernel(layer_norm_out_kernel<__nv_bfloat16>, dim3(M), dim3(threads), 0, stream, x, w, bias, static_cast<__nv_bfloat16*>(out), W, width, eps);
+  return cudaGetLastError() == cudaSuccess ? 0 : -7;
+}
+
+extern "C" int mfq_token_shift(const void* h, const float* mu, float* last, const int* slot, const int* starts, const int* tok_seq, void* out,
+                               int T_, int W, int streams, int fp32, cudaStream_t stream) {
+  if (T_ <= 0 || W <= 0 || W % 8 || streams <= 0 || (starts && !tok_seq)) return -1;
+  const int threads = min(256, (W / 8 + 31) / 32 * 32);
+  if (fp32)
+    launch_kernel(token_shift_kernel<float>, dim3(T_), dim3(threads), 0, stream, static_cast<const float*>(h), mu, last, slot, starts, tok_seq,
+                  static_cast<float*>(out), W, streams);
+  else
+    launch_kernel(token_shift_kernel<__nv_bfloat16>, dim3(T_), dim3(threads), 0, stream, static_cast<const __nv_bfloat16*>(h), mu, last, slot,
+                  starts, tok_seq, static_cast<__nv_bfloat16*>(out), W, streams);
+  return cudaGetLastError() == cudaSuccess ? 0 : -7;
+}
+
+// x: rows of in_stride, channels 0 .. C - 1; w [taps, C]; state [slots, taps - 1, C]; starts null: row b belongs to sequence b
+extern "C" int mfq_short_conv(const void* x, int in_stride, const float* w, float* state, const int* slot, const int* starts, void* out,
+                              int out_stride, int B, int max_q, int C, int taps, int fp32, cudaStream_t stream) {
+  if (B <= 0 || B > 65535 || max_q <= 0 || C <= 0 || C % 8 || taps < 1 || taps > 8 || in_stride % 8 || out_stride % 8) return -1;
+  const ShortConvParams p{w, state, slot, starts, C, taps, in_stride, out_stride};
+  return fp32 ? launch_short_conv<float>(x, out, p, B, starts ? max_q : 1, stream)
+              : launch_short_conv<__nv_bfloat16>(x, out, p, B, starts ? max_q : 1, stream);
+}

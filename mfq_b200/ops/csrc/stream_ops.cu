@@ -104,13 +104,15 @@ norm_out_kernel(const float* __restrict__ x, const float* __restrict__ w, T* __r
 // ---------------------------------------------------------------------------------------------
 // qkv rows [Hq * dk | Hk * maps * dk | Hk * dv] (dk, dv: head widths as stored, multiples of 16; d: the true q / k width the
 // norm averages over; Hq counts every query map).  `L` lanes (a power of two) share a head, 8 channels each; a warp takes 32 / L
-// heads of one token.  The rotation reads (cos, sin) of the token's position from a table [positions][rot / 2]; channel i turns
+// heads of one token.  Queries may also be multiplied by a temperature that grows with the position.  The rotation reads (cos, sin) of the token's position from a table [positions][rot / 2]; channel i turns
 // with i + rot / 2 (read from shared memory), or with its neighbour (`pairs`).  Pages: K [page][Hk][16][maps * dk],
 // V [page][Hk][16][dv]; slot < 0: the token is not cached.  No pages: rows hold queries only.
 // ---------------------------------------------------------------------------------------------
 struct QkvFinishParams {
   int T, Hq, Hk, maps, d, dk, dv, rot, pairs, row_stride, page_size, L, table_rows;
   float eps, lambda;        // lambda: share of the other layer's values
+  float temp;               // queries times 1 + temp * ln(floor((position + 1) / temp_every) + 1)
+  int temp_every;
   int first_stride;         // row stride of `v_first`
   const float* q_norm;
   const float* k_norm;      // [dk] fp32 or null: no norm
@@ -191,6 +193,11 @@ qkv_finish_kernel(const T* __restrict__ qkv, const T* __restrict__ v_first, T* _
     }
   }
   if (is_q) {
+    if (p.temp != 0.f) {
+      const float f = fmaf(p.temp, logf(float((p.positions[t] + 1) / p.temp_every) + 1.f), 1.f);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] *= f;
+    }
     store8<T>(q_out + (size_t(t) * p.Hq + h) * p.dk + c * 8, v);
     return;
   }
@@ -307,7 +314,9 @@ extern "C" int mfq_map_difference(const void* a, void* out, int T_, int H, int p
 extern "C" int mfq_qkv_finish(const void* qkv, int row_stride, const void* v_first, int first_stride, float lambda, void* q_out,
                               void* k_pages, void* v_pages, const int* positions, const int* slots, const float* q_norm,
                               const float* k_norm, const float* rope, int table_rows, int T_, int Hq, int Hk, int maps, int d, int dk,
-                              int dv, int rot, int pairs, int page_size, float eps, int fp32, cudaStream_t stream) {
+                              int dv, int rot, int pairs, int page_size, float eps, float temp, int temp_every, int fp32,
+                              cudaStream_t stream) {
+  if (temp != 0.f && temp_every <= 0) return -1;
   if (!k_pages) { Hk = 0; dv = 0; v_first = nullptr; }
   if (T_ <= 0 || Hq <= 0 || maps <= 0 || dk % 16 || dk <= 0 || dk > 256 || d <= 0 || d > dk) return -1;
   if (k_pages && (Hk <= 0 || Hq % (Hk * maps) || dv % 16 || dv <= 0 || dv > 256 || page_size <= 0 || !v_pages || !slots)) return -1;
@@ -315,7 +324,7 @@ extern "C" int mfq_qkv_finish(const void* qkv, int row_stride, const void* v_fir
   if (rot < 0 || rot % 2 || rot > d || (rot > 0 && (!rope || table_rows <= 0))) return -1;
   int L = 1;
   while (L * 8 < max(dk, dv)) L *= 2;
-  QkvFinishParams p{T_, Hq, Hk, maps, d, dk, dv, rot, pairs, row_stride, page_size, L, table_rows, eps, lambda, first_stride, q_norm, k_norm,
+  QkvFinishParams p{T_, Hq, Hk, maps, d, dk, dv, rot, pairs, row_stride, page_size, L, table_rows, eps, lambda, temp, temp_every, first_stride, q_norm, k_norm,
                     reinterpret_cast<const float2*>(rope), positions, slots};
   const int heads = Hq + Hk * (maps + 1), per_warp = 32 / L;
   const long long warps = (long long)(T_) * ((heads + per_warp - 1) / per_warp);

@@ -1,7 +1,8 @@
 // Sliding-window attention over unquantized pages (K [page][Hk][16][maps * dk], V [page][Hk][16][dv]), one query token per
 // sequence or, in the plain kernel, any number of them.  A query at position i sees the keys j with 0 <= i - j < window, and of
 // the first `keep` keys every one up to i.  With two maps (differential attention) a KV head has two key vectors and one value
-// vector per token; queries are ordered [KV head][map][query head of the KV head].
+// vector per token; queries are ordered [KV head][map][query head of the KV head].  With one map a head may have a score bias by
+// distance and a sink (window_attn.cuh: ScoreExtra).
 //
 //   window_attn_decode_kernel   bf16, one query per sequence.  A CTA serves one (sequence, KV head, KV split); its four warps
 //                               take alternate pages that hold visible keys through private cp.async rings.  The (up to 16)
@@ -29,6 +30,7 @@ struct WindowDecodeParams {
   float* part_ml;       // [B * Hq][splits][2]
   int Hq, Hk, maps, dk, dv, max_pages, window, keep, splits, head_tiles;
   ScoreCap cap;
+  ScoreExtra extra;
 };
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
@@ -144,6 +146,15 @@ window_attn_decode_kernel(const WindowDecodeParams p) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) o[i][j] = 0.f;
   float m[2] = {-FLT_MAX, -FLT_MAX}, l[2] = {0.f, 0.f};
+  const float* bias[2] = {nullptr, nullptr};  // of rows r0 and r0 + 8
+  float far[2] = {0.f, 0.f};
+  if (p.extra.bias) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      bias[r] = p.extra.bias + size_t(head0 + min(r0 + 8 * r, heads - 1)) * (p.extra.last + 1);
+      far[r] = bias[r][p.extra.last] * kLog2e;
+    }
+  }
   const int mat = lane >> 3, mrow = lane & 7;
   const uint32_t k_off = (((mat >> 1) * 8 + mrow) * kpitch + (mat & 1) * 8) * 2;
   const uint32_t v_off = (((mat & 1) * 8 + mrow) * vpitch + (mat >> 1) * 8) * 2;
@@ -166,12 +177,15 @@ window_attn_decode_kernel(const WindowDecodeParams p) {
     const int pg = page0 + warp + kWinWarps * i;
     const int key0 = (pg < kept ? pg : pg + skip) * kWinPage + t4 * 2;
     float mx[2] = {-FLT_MAX, -FLT_MAX};
+    const bool near = pos - (key0 - t4 * 2 + kWinPage - 1) < p.extra.last;  // some key of the page is nearer than the last bias
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = key0 + nt * 8 + (e & 1);
-        s[nt][e] = (key >= lo || key < p.keep) && key <= pos ? score_any(p.cap, s[nt][e]) : -FLT_MAX;
+        float c = score_any(p.cap, s[nt][e]);
+        if (p.extra.bias) c += near ? bias[e >> 1][min(max(pos - key, 0), p.extra.last)] * kLog2e : far[e >> 1];
+        s[nt][e] = (key >= lo || key < p.keep) && key <= pos ? c : -FLT_MAX;
         mx[e >> 1] = fmaxf(mx[e >> 1], s[nt][e]);
       }
     float alpha[2];
@@ -239,13 +253,18 @@ window_attn_decode_kernel(const WindowDecodeParams p) {
     float mw[kWinWarps], mt = -FLT_MAX, lt = 0.f;
 #pragma unroll
     for (int w = 0; w < kWinWarps; ++w) { mw[w] = ml[(w * 16 + r) * 2]; mt = fmaxf(mt, mw[w]); }
+    const bool whole = p.splits == 1 && p.maps == 1;
+    if (whole && p.extra.sink) {
+      const float sink = p.extra.sink[head0 + r] * kLog2e;
+      mt = fmaxf(mt, sink);
+      lt = window_exp2(sink - mt);
+    }
 #pragma unroll
     for (int w = 0; w < kWinWarps; ++w) {
       mw[w] = window_exp2(mw[w] - mt);  // a warp without pages: l = 0, o = 0
       lt += ml[(w * 16 + r) * 2 + 1] * mw[w];
     }
     const size_t orow = size_t(b) * p.Hq + head0 + r;
-    const bool whole = p.splits == 1 && p.maps == 1;
     const float inv = whole ? (lt > 0.f ? 1.f / lt : 0.f) : 1.f;
     for (int c = lane; c < dv; c += 32) {
       float x = 0.f;
@@ -264,6 +283,7 @@ window_attn_decode_kernel(const WindowDecodeParams p) {
 
 // A CTA per (sequence, output head).  Two maps: y = a1 - lambda a2, out = scale * y / sqrt(mean(y^2) + eps).
 struct WindowMergeParams {
+  const float* sink;  // [heads] or null (one map)
   int splits, dv, heads, of_map, maps;  // heads: output heads; of_map: query heads per KV head
   float lambda, scale, eps, inv_d;
 };
@@ -275,16 +295,21 @@ window_attn_merge_kernel(const float* __restrict__ part, const float* __restrict
   pdl_wait();
   __shared__ float red[33];
   const int b = blockIdx.x / p.heads, h = blockIdx.x - b * p.heads, g = h / p.of_map;
-  float y[2] = {0.f, 0.f};  // channels threadIdx.x and threadIdx.x + 128
+  constexpr int kCols = 4;  // channels threadIdx.x + 128 i: values up to 512 wide
+  float y[kCols] = {};
   for (int m = 0; m < p.maps; ++m) {
     const size_t row = (size_t(b) * p.heads + g * p.of_map) * p.maps + m * p.of_map + h - g * p.of_map;
     const float* ml = part_ml + row * p.splits * 2;
     float mt = -FLT_MAX, lt = 0.f;
     for (int z = 0; z < p.splits; ++z) mt = fmaxf(mt, ml[z * 2]);
+    if (p.sink) {
+      mt = fmaxf(mt, p.sink[h] * kLog2e);
+      lt = window_exp2(p.sink[h] * kLog2e - mt);
+    }
     for (int z = 0; z < p.splits; ++z) lt += ml[z * 2 + 1] * window_exp2(ml[z * 2] - mt);
     const float inv = (lt > 0.f ? 1.f / lt : 0.f) * (m == 0 ? 1.f : -p.lambda);
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
+    for (int i = 0; i < kCols; ++i) {
       const int c = threadIdx.x + i * 128;
       if (c >= p.dv) continue;
       float x = 0.f;
@@ -293,12 +318,18 @@ window_attn_merge_kernel(const float* __restrict__ part, const float* __restrict
     }
   }
   float f = 1.f;
-  if (p.maps == 2) f = rsqrtf(dense_block_sum(y[0] * y[0] + y[1] * y[1], red) * p.inv_d + p.eps) * p.scale;
+  if (p.maps == 2) f = rsqrtf(dense_block_sum(y[0] * y[0] + y[1] * y[1] + y[2] * y[2] + y[3] * y[3], red) * p.inv_d + p.eps) * p.scale;
 #pragma unroll
-  for (int i = 0; i < 2; ++i) {
+  for (int i = 0; i < kCols; ++i) {
     const int c = threadIdx.x + i * 128;
     if (c < p.dv) out[size_t(blockIdx.x) * p.dv + c] = __float2bfloat16(y[i] * f);
   }
+}
+
+int launch_attn_merge(const float* part, const float* part_ml, __nv_bfloat16* out, int B, int heads, int splits, int dv, cudaStream_t stream) {
+  const WindowMergeParams mp{nullptr, splits, dv, heads, heads, 1, 0.f, 1.f, 0.f, 0.f};
+  launch_kernel(window_attn_merge_kernel, dim3(B * heads), dim3(128), 0, stream, part, part_ml, out, mp);
+  return cudaGetLastError() == cudaSuccess ? 0 : -7;
 }
 
 template <int DK, int DV>
@@ -324,6 +355,7 @@ struct WindowPlainParams {
   const int* table;
   int T, Hq, Hk, maps, dk, dv, max_pages, window, keep;
   float scale, cap;
+  ScoreExtra extra;
 };
 
 template <typename T>
@@ -348,6 +380,10 @@ window_attn_plain_kernel(const T* __restrict__ q, const T* __restrict__ k, const
   }
   __syncwarp();
   float m = -FLT_MAX, l = 0.f, acc[8] = {};
+  if (p.extra.sink) {  // one more key, without a value
+    m = p.extra.sink[h];
+    l = 1.f;
+  }
   for (int j0 = 0; j0 <= pos - skip; j0 += 32) {  // over the visible keys: the kept ones before the window, then the window
     const int key = j0 + lane < kept ? j0 + lane : j0 + lane + skip;
     float s = -FLT_MAX;
@@ -364,6 +400,7 @@ window_attn_plain_kernel(const T* __restrict__ q, const T* __restrict__ k, const
       }
       s = dot * p.scale;
       if (p.cap > 0.f) s = p.cap * tanhf(s / p.cap);
+      if (p.extra.bias) s += p.extra.bias[size_t(h) * (p.extra.last + 1) + min(pos - key, p.extra.last)];
     }
     float mx = s;
 #pragma unroll
@@ -410,14 +447,16 @@ using namespace mfq;
 extern "C" int mfq_window_attn_decode(const void* q, const void* k, const void* v, const int* table, const int* seq_lens, void* out,
                                       float* part, float* part_ml, int B, int Hq, int Hk, int maps, int dk, int dv, int max_pages, int window,
                                       int keep, float scale, float cap, int splits, float lambda, float out_scale, float eps, int d,
-                                      cudaStream_t stream) {
+                                      const float* bias, int bias_last, const float* sink, cudaStream_t stream) {
   if (B <= 0 || Hq <= 0 || Hk <= 0 || maps < 1 || maps > 2 || Hq % (Hk * maps) || dk % 16 || dv % 16 || dk <= 0 || dv <= 0) return -1;
+  if ((bias || sink) && maps > 1) return -1;
+  if (bias && bias_last < 0) return -1;
   if (dk * maps > 512 || dv > 256 || keep < 0 || (maps > 1 && (d <= 0 || d > dv))) return -1;
   if (window <= 0 || !(scale > 0.f) || splits < 1 || ((splits > 1 || maps > 1) && (!part || !part_ml))) return -1;
   const WindowDecodeParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k), static_cast<const __nv_bfloat16*>(v),
                              table, seq_lens, static_cast<__nv_bfloat16*>(out), part, part_ml, Hq, Hk, maps, dk, dv, max_pages, window, keep,
-                             splits, (Hq / Hk + 15) / 16, make_score_cap(scale, cap)};
-  const WindowMergeParams mp{splits, dv, Hq / maps, Hq / Hk / maps, maps, lambda, out_scale, eps, maps > 1 ? 1.f / float(d) : 0.f};
+                             splits, (Hq / Hk + 15) / 16, make_score_cap(scale, cap), ScoreExtra{bias, nullptr, sink, bias ? bias_last : 0}};
+  const WindowMergeParams mp{sink, splits, dv, Hq / maps, Hq / Hk / maps, maps, lambda, out_scale, eps, maps > 1 ? 1.f / float(d) : 0.f};
   const int kw = dk * maps;
 #define MFQ_WIN_DV(DK)                                                     \
   (dv <= 64 ? launch_window_decode<DK, 64>(p, mp, B, stream)               \
@@ -431,10 +470,12 @@ extern "C" int mfq_window_attn_decode(const void* q, const void* k, const void* 
 // output of every map.
 extern "C" int mfq_window_attn_plain(const void* q, const void* k, const void* v, const int* table, const int* tok_seq,
                                      const int* positions, void* out, int T_, int Hq, int Hk, int maps, int dk, int dv, int max_pages,
-                                     int window, int keep, float scale, float cap, int fp32, cudaStream_t stream) {
+                                     int window, int keep, float scale, float cap, const float* bias, int bias_last, const float* sink,
+                                     int fp32, cudaStream_t stream) {
+  if (((bias || sink) && maps > 1) || (bias && bias_last < 0)) return -1;
   if (T_ <= 0 || Hq <= 0 || Hk <= 0 || maps < 1 || Hq % (Hk * maps) || dk % 8 || dv % 8 || dk > 256 || dv > 256 || window <= 0 || keep < 0)
     return -1;
-  const WindowPlainParams p{positions, tok_seq, table, T_, Hq, Hk, maps, dk, dv, max_pages, window, keep, scale, cap};
+  const WindowPlainParams p{positions, tok_seq, table, T_, Hq, Hk, maps, dk, dv, max_pages, window, keep, scale, cap, ScoreExtra{bias, nullptr, sink, bias ? bias_last : 0}};
   const dim3 grid(unsigned(((long long)(T_) * Hq + 3) / 4));
   if (fp32)
     launch_kernel(window_attn_plain_kernel<float>, grid, dim3(128), 0, stream, static_cast<const float*>(q), static_cast<const float*>(k),

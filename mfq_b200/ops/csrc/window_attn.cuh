@@ -52,4 +52,14 @@ __device__ __forceinline__ float score_any(const ScoreCap& k, float s) {
   return fabsf(s) <= k.small ? score_small(k, s) : score_large(k, s);
 }
 
+// What a head adds to its softmax, in natural units: a score bias by distance, bias[h][min(distance, last)], added to the capped
+// score, and one more term exp(sink[h]) of the denominator.
+struct ScoreExtra {
+  const float* bias;  // [Hq][last + 1] or null
+  const float* top;   // [Hq] largest bias of the head (prefill kernel)
+  const float* sink;  // [Hq] or null
+  int last;
+};
+constexpr float kLog2e = 1.4426950408889634f;
+
 }  // namespace mfq

@@ -13,7 +13,8 @@ import torch
 
 from .lib import Workspace, check, dense_lib, ptr, stream_ptr
 
-BIAS, GLU, GELU, GELU_GLU, SOFTCAP, ADD = range(6)  # epilogues (dense_common.cuh)
+BIAS, GLU, GELU, GELU_GLU, SOFTCAP, ADD, RELU_GLU, SILU_GLU, FLOAT = range(9)  # epilogues (dense_common.cuh)
+UNITS = {"gelu": GELU_GLU, "relu": RELU_GLU, "silu": SILU_GLU}  # act(gate) * up
 GEMV_ROWS, GEMV_MID_ROWS, GEMV_MID_WEIGHTS = 8, 16, 8 << 20
 
 
@@ -63,45 +64,57 @@ def plan(m: int, n: int, k: int, sms: int = 148) -> tuple[int, int]:
 @dataclass
 class DenseLinear:
     """``[rows, cols]`` weight (rows a multiple of 16, cols of 8) with an optional fp32 bias.  ``glu``: the rows alternate
-    between 8 gate and 8 up rows (:func:`interleave_glu`) and the output is the gated unit of the two, half as wide."""
+    between 8 gate and 8 up rows (:func:`interleave_glu`) and the output is the gated unit of the two, half as wide.
+    ``groups`` G > 1: G matrices on top of each other, ``[G * rows, cols]``, each with its own columns of input and output."""
 
     w: torch.Tensor
     bias: torch.Tensor | None = None
-    glu: tuple[float, float] | str | None = None  # (alpha, limit) of the clipped GLU, or "gelu": gelu_tanh(gate) * up
+    glu: tuple[float, float] | str | None = None  # (alpha, limit) of the clipped GLU, or the activation: act(gate) * up
+    groups: int = 1
     input_kind = "dense"
 
     @property
     def out_width(self) -> int:
-        return self.w.shape[0] // (2 if self.glu is not None else 1)
+        return self.w.shape[0] // self.groups // (2 if self.glu is not None else 1)
 
     def __call__(self, x: torch.Tensor, *, table: torch.Tensor | None = None, ids: torch.Tensor | None = None,
-                 softcap: float = 0.0, add_to: torch.Tensor | None = None, out: torch.Tensor | None = None, tile: int | None = None,
+                 softcap: float = 0.0, add_to: torch.Tensor | None = None, scale: float = 1.0, out: torch.Tensor | None = None,
+                 fp32: bool = False, x_step: int | None = None, out_step: int | None = None, tile: int | None = None,
                  splits: int | None = None) -> torch.Tensor:
         """``x [M, cols]``.  ``table`` (``[vocabulary, rows]``) with ``ids [M]``: the result is ``gelu_tanh(y) * table[ids]``;
-        ``softcap`` c > 0: ``c tanh(y / c)``; ``add_to``: ``y`` is added to this fp32 stream, which is also the result."""
-        m, n, k = x.shape[0], self.w.shape[0], self.w.shape[1]
-        assert x.shape[1] == k and x.stride(1) == 1 and x.dtype == self.w.dtype and self.w.is_contiguous()
+        ``softcap`` c > 0: ``c tanh(y / c)``; ``add_to``: ``scale * y`` is added to this fp32 stream, which is also the result;
+        ``fp32``: the result stays fp32.  Groups: matrix g reads ``x`` from column ``g * x_step`` (by default ``cols``) and writes
+        ``out`` from column ``g * out_step`` (by default ``out_width``)."""
+        m, n, k, g = x.shape[0], self.w.shape[0] // self.groups, self.w.shape[1], self.groups
+        x_step, out_step = k if x_step is None else x_step, self.out_width if out_step is None else out_step
+        assert x.shape[1] >= (g - 1) * x_step + k and (g > 1 or x.shape[1] == k)
+        assert x.stride(1) == 1 and x.dtype == self.w.dtype and self.w.is_contiguous()
+        width = (g - 1) * out_step + self.out_width
         if add_to is not None:
-            assert self.glu is None and add_to.dtype == torch.float32 and add_to.shape == (m, n) and add_to.stride(1) == 1
+            assert self.glu is None and add_to.dtype == torch.float32 and add_to.shape == (m, width) and add_to.stride(1) == 1
             out = add_to
         elif out is None:
-            out = torch.empty((m, self.out_width), dtype=x.dtype, device=x.device)
+            out = torch.empty((m, width), dtype=torch.float32 if fp32 else x.dtype, device=x.device)
+        else:
+            assert out.shape[0] == m and out.shape[1] >= width and out.stride(1) == 1 and out.dtype == (torch.float32 if fp32 else x.dtype)
         kind, alpha, limit = BIAS, 0.0, 0.0
-        if self.glu == "gelu":
-            kind = GELU_GLU
+        if isinstance(self.glu, str):
+            kind = UNITS[self.glu]
         elif self.glu is not None:
             kind, (alpha, limit) = GLU, self.glu
         elif add_to is not None:
-            kind = ADD
+            kind, alpha = ADD, scale
+        elif fp32:
+            kind = FLOAT
         elif softcap > 0:
             kind, limit = SOFTCAP, softcap
         elif table is not None:
             assert table.shape[1] == n and table.is_contiguous() and table.dtype == x.dtype and ids.dtype == torch.int32
             kind = GELU
-        t, s = plan(m, n, k)
+        t, s = plan(m, n * g, k)
         t, s = (t if tile is None else tile), (s if splits is None else splits)
-        rc = dense_lib().mfq_dense_linear(ptr(self.w), ptr(x), x.stride(0), ptr(out), out.stride(0), ptr(self.bias), m, n, k, kind,
-                                          alpha, limit, ptr(table), ptr(ids), t, s, is_fp32(x.dtype),
+        rc = dense_lib().mfq_dense_linear(ptr(self.w), ptr(x), x.stride(0), ptr(out), out.stride(0), ptr(self.bias), m, n, k, g, x_step,
+                                          out_step, kind, alpha, limit, ptr(table), ptr(ids), t, s, is_fp32(x.dtype),
                                           ptr(Workspace.get(x.device).status), stream_ptr())
         check(rc, "dense_linear")
         return out
@@ -138,4 +151,13 @@ def norm_out(x: torch.Tensor, weight: torch.Tensor, width: int, eps: float, dtyp
     m, w = x.shape
     out = torch.empty((m, w), dtype=dtype, device=x.device)
     check(dense_lib().mfq_norm_out(ptr(x), ptr(weight), ptr(out), m, w, width, float(eps), is_fp32(dtype), stream_ptr()), "norm_out")
+    return out
+
+
+def layer_norm_out(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, width: int, eps: float, dtype: torch.dtype) -> torch.Tensor:
+    """``(x - mean) / sqrt(var + eps) * weight + bias`` of the fp32 stream (over ``width`` columns), in ``dtype``."""
+    m, w = x.shape
+    out = torch.empty((m, w), dtype=dtype, device=x.device)
+    check(dense_lib().mfq_layer_norm_out(ptr(x), ptr(weight), ptr(bias), ptr(out), m, w, width, float(eps), is_fp32(dtype), stream_ptr()),
+          "layer_norm_out")
     return out

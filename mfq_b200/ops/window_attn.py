@@ -1,8 +1,9 @@
 """Attention over unquantized pages with a sliding window, kept first tokens, an optional score cap and one or two maps
-(``csrc/window_attn*.cu``), and the per-head stage in front of it (``csrc/stream_ops.cu``).
+(``csrc/window_attn*.cu``), with one map also a score bias by distance and a sink per head, and the per-head stage in front of it (``csrc/stream_ops.cu``).
 
 A query at position ``i`` sees the keys ``j <= i`` with ``i - j < window`` or ``j < keep``; a score is ``q . k * scale``, then
-``cap * tanh(score / cap)`` (``cap`` 0: no cap).  Pages: ``k [pages, Hk, 16, maps * dk]``, ``v [pages, Hk, 16, dv]``, widths
+``cap * tanh(score / cap)`` (``cap`` 0: no cap), then plus the head's bias for the distance ``i - j`` (:class:`DistanceBias`).  A sink
+adds ``exp(sink)`` to the head's denominator.  Pages: ``k [pages, Hk, 16, maps * dk]``, ``v [pages, Hk, 16, dv]``, widths
 ``dk`` and ``dv`` multiples of 16 up to 256.  bf16 runs on tensor cores (one kernel for portions of prompts, one for single
 tokens), fp32 on a plain kernel.
 
@@ -23,6 +24,7 @@ from .lib import Workspace, check, dense_lib, ptr, stream_ptr
 
 MAX_HEAD = 256
 NO_WINDOW = 1 << 30
+MAX_BIAS_SPREAD = 60.0  # the prefill kernel adds a head's largest bias to its running maximum: weights must not underflow
 
 
 @dataclass(frozen=True)
@@ -33,6 +35,35 @@ class Difference:
     scale: float
     eps: float
     dim: int  # real value channels
+
+
+@dataclass
+class DistanceBias:
+    """Per head, what a key ``n`` tokens back adds to its score: ``table[h, min(n, last)]``."""
+
+    table: torch.Tensor  # [heads, last + 1] fp32
+    top: torch.Tensor  # [heads] largest entry
+
+    @classmethod
+    def from_table(cls, table: torch.Tensor) -> "DistanceBias":
+        table = table.float().contiguous()
+        if float((table.amax(1) - table.amin(1)).max()) > MAX_BIAS_SPREAD:
+            raise ValueError(f"biases of a head that differ by more than {MAX_BIAS_SPREAD:g} are not supported")
+        return cls(table, table.amax(1).contiguous())
+
+    @property
+    def last(self) -> int:
+        return self.table.shape[1] - 1
+
+
+def log_buckets(rows: int, most: float) -> list[int]:
+    """Row of a table of ``rows`` for the distances 0, 1, ...: one row each up to half of them, then logarithmic up to ``most``; ends
+    where the last row begins."""
+    half, out = rows // 2, []
+    while not out or out[-1] < rows - 1:
+        n = len(out)
+        out.append(n if n < half else min(rows - 1, half + math.floor(math.log(n / half) / math.log(most / half) * (rows - half))))
+    return out
 
 
 @dataclass(frozen=True)
@@ -55,31 +86,37 @@ class FrequencyScaling:
         return (1 - s) * f / self.factor + s * f
 
 
-def rope_table(base: float, dims: int, positions: int, device, scaling: FrequencyScaling | None = None) -> torch.Tensor:
-    """``[positions, dims / 2, 2]`` fp32 (cos, sin) of ``p * f_i``, ``f_i = base^(-2i / dims)`` (scaled), in double precision."""
-    freq = [float(base) ** (-2.0 * i / dims) for i in range(dims // 2)]
-    freq = torch.tensor([scaling(f) for f in freq] if scaling is not None else freq, dtype=torch.float64, device=device)
-    a = torch.arange(positions, dtype=torch.float64, device=device)[:, None] * freq
-    return torch.stack([a.cos(), a.sin()], -1).float().contiguous()
+def rope_table(base: float, dims: int, positions: int, device, scaling=None) -> torch.Tensor:
+    """``[positions, dims / 2, 2]`` fp32 (cos, sin) of ``p * f_i``, ``f_i = base^(-2i / dims)``, in double precision.  ``scaling``: a
+    :class:`FrequencyScaling`, or a :class:`~mfq_b200.models.rope_scaling.YarnScaling`, which also lengthens the rotated pairs."""
+    freq, length = [float(base) ** (-2.0 * i / dims) for i in range(dims // 2)], 1.0
+    if isinstance(scaling, FrequencyScaling):
+        freq = [scaling(f) for f in freq]
+    elif scaling is not None:
+        freq, length = scaling.frequencies(dims, base), scaling.mscale
+    a = torch.arange(positions, dtype=torch.float64, device=device)[:, None] * torch.tensor(freq, dtype=torch.float64, device=device)
+    return (torch.stack([a.cos(), a.sin()], -1) * length).float().contiguous()
 
 
 def qkv_finish(qkv: torch.Tensor, kv, positions, slots, *, heads: int, kv_heads: int, dim: int, q_norm, k_norm, rope, rot: int,
                eps: float, v_first: torch.Tensor | None = None, mix: float = 0.0, maps: int = 1, pairs: bool = False,
-               dk: int | None = None) -> torch.Tensor:
+               dk: int | None = None, temperature: tuple[float, int] | None = None) -> torch.Tensor:
     """Per-head RMS norm of q and k (over ``dim`` channels; no norm without weights), rotation of the leading ``rot`` channels
     (``i`` with ``i + rot / 2``, or with its neighbour: ``pairs``), K and V into their pages; returns ``q [T, maps * heads, dk]``.
     ``v_first`` (``[T, kv_heads * dv]``, rows may be strided): the cached values are ``(1 - mix) v + mix v_first``.  ``kv`` None:
-    the rows hold queries only (of stored width ``dk``)."""
+    the rows hold queries only (of stored width ``dk``).  ``temperature`` (coef, every): queries at position p times
+    ``1 + coef * ln(floor((p + 1) / every) + 1)``."""
     t = qkv.shape[0]
     if kv is not None:
         dk, dv, page = kv.k.shape[-1] // maps, kv.v.shape[-1], kv.page_size
     else:
         dv = page = 0
     q = torch.empty((t, maps * heads, dk), dtype=qkv.dtype, device=qkv.device)
+    temp, every = temperature or (0.0, 1)
     rc = dense_lib().mfq_qkv_finish(ptr(qkv), qkv.stride(0), ptr(v_first), v_first.stride(0) if v_first is not None else 0, float(mix),
                                     ptr(q), ptr(kv.k) if kv is not None else None, ptr(kv.v) if kv is not None else None, ptr(positions),
                                     ptr(slots), ptr(q_norm), ptr(k_norm), ptr(rope), rope.shape[0] if rope is not None else 0, t,
-                                    maps * heads, kv_heads, maps, dim, dk, dv, rot, int(pairs), page, float(eps), is_fp32(qkv.dtype),
+                                    maps * heads, kv_heads, maps, dim, dk, dv, rot, int(pairs), page, float(eps), float(temp), int(every), is_fp32(qkv.dtype),
                                     stream_ptr())
     check(rc, "qkv_finish")
     return q
@@ -108,8 +145,12 @@ def decode_splits(batch: int, kv_heads: int, keys: int) -> int:
     return min(choices, key=lambda s: -(-n * s // slots) * keys / s + 20 * s)
 
 
+def _bias_args(bias: DistanceBias | None) -> tuple:
+    return (ptr(bias.table), bias.last) if bias is not None else (None, 0)
+
+
 def decode(q: torch.Tensor, kv, block_table, seq_lens, *, window: int, scale: float, cap: float, keep: int = 0,
-           diff: Difference | None = None, splits: int = 1, out=None):
+           diff: Difference | None = None, bias: DistanceBias | None = None, sink: torch.Tensor | None = None, splits: int = 1, out=None):
     """One query token per sequence (bf16): ``q [B, Hq, dk]`` -> ``[B, Hq, dv]``, or ``[B, Hq / 2, dv]`` with ``diff``;
     ``seq_lens`` count the query token."""
     b, hq, dk = q.shape
@@ -123,13 +164,13 @@ def decode(q: torch.Tensor, kv, block_table, seq_lens, *, window: int, scale: fl
     how = (diff.weight, diff.scale, diff.eps, diff.dim) if diff is not None else (0.0, 1.0, 0.0, dv)
     rc = dense_lib().mfq_window_attn_decode(ptr(q), ptr(kv.k), ptr(kv.v), ptr(block_table), ptr(seq_lens), ptr(out), ptr(ws.attn_acc),
                                             ptr(ws.attn_ml), b, hq, hk, maps, dk, dv, block_table.stride(0), window, keep, float(scale),
-                                            float(cap), splits, *how, stream_ptr())
+                                            float(cap), splits, *how, *_bias_args(bias), ptr(sink), stream_ptr())
     check(rc, "window_attn_decode", 2 if parts else 1)
     return out
 
 
 def prefill(q: torch.Tensor, kv, block_table, q_starts, seq_lens, max_q: int, *, window: int, scale: float, cap: float, keep: int = 0,
-            maps: int = 1, out=None):
+            maps: int = 1, bias: DistanceBias | None = None, sink: torch.Tensor | None = None, out=None):
     """Portions of several sequences (bf16): rows ``q_starts[b] .. q_starts[b + 1] - 1`` of ``q [T, Hq, dk]`` are the last
     tokens of a sequence of ``seq_lens[b]``.  ``max_q``: the longest portion (host).  Writes the output of every map."""
     t, hq, dk = q.shape
@@ -137,19 +178,21 @@ def prefill(q: torch.Tensor, kv, block_table, q_starts, seq_lens, max_q: int, *,
     out = torch.empty((t, hq, dv), dtype=q.dtype, device=q.device) if out is None else out
     rc = dense_lib().mfq_window_attn_prefill(ptr(q), ptr(kv.k), ptr(kv.v), ptr(block_table), ptr(q_starts), ptr(seq_lens), ptr(out), t,
                                              seq_lens.numel(), max_q, hq, hk, maps, dk, dv, kv.k.shape[0], block_table.stride(0), window,
-                                             keep, float(scale), float(cap), ptr(Workspace.get(q.device).status), stream_ptr())
+                                             keep, float(scale), float(cap), *_bias_args(bias), ptr(bias.top) if bias is not None else None, ptr(sink),
+                                             ptr(Workspace.get(q.device).status), stream_ptr())
     check(rc, "window_attn_prefill")
     return out
 
 
-def plain(q: torch.Tensor, kv, block_table, tok_seq, positions, *, window: int, scale: float, cap: float, keep: int = 0, maps: int = 1):
+def plain(q: torch.Tensor, kv, block_table, tok_seq, positions, *, window: int, scale: float, cap: float, keep: int = 0, maps: int = 1,
+          bias: DistanceBias | None = None, sink: torch.Tensor | None = None):
     """The same in fp32 arithmetic for any mix of tokens: token ``t`` is at ``positions[t]`` of sequence ``tok_seq[t]``."""
     t, hq, dk = q.shape
     hk, dv = kv.k.shape[1], kv.v.shape[-1]
     out = torch.empty((t, hq, dv), dtype=q.dtype, device=q.device)
     rc = dense_lib().mfq_window_attn_plain(ptr(q), ptr(kv.k), ptr(kv.v), ptr(block_table), ptr(tok_seq), ptr(positions), ptr(out), t, hq,
                                            hk, maps, dk, dv, block_table.stride(0), window, keep, float(scale), float(cap),
-                                           is_fp32(q.dtype), stream_ptr())
+                                           *_bias_args(bias), ptr(sink), is_fp32(q.dtype), stream_ptr())
     check(rc, "window_attn_plain")
     return out
 

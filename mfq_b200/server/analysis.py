@@ -105,6 +105,8 @@ def _own_family(cfg: dict):
         from ..models.tepetar import TepetarConfig as Config, tensor_shapes
     elif cfg.get("family") == "kamedra":
         from ..models.kamedra import KamedraConfig as Config, tensor_shapes
+    elif cfg.get("family") == "bufolorn":
+        from ..models.bufolorn import BufolornConfig as Config, tensor_shapes
     else:
         return None
     own = Config.from_dict(cfg)
@@ -120,7 +122,7 @@ def model_parameters(cfg: dict) -> dict:
             groups[group_of(name)] = groups.get(group_of(name), 0) + math.prod(shape)
         total = sum(groups.values())
         return {"groups": groups, "total": total, "active_per_token": total, "experts": None, "top_k": None, "layers": own[0].num_layers,
-                "attention_layers": len(own[0].key_spans())}
+                "attention_layers": getattr(own[0], "attention_layers", len(own[0].key_spans()))}
     h = _cfg_int(cfg, "hidden_size")
     layers = _cfg_int(cfg, "num_layers", "num_hidden_layers")
     hq = _cfg_int(cfg, "num_heads", "num_attention_heads")
