@@ -17,6 +17,7 @@
 // Precision: the recurrence is kept to fp32 level on bf16 tensor cores by splitting every fp32 operand into two bf16 numbers
 // (16 significant bits): 2^(b_C - b) k, 2^b q, the factors of A, A itself and S_0; v is bf16 as projected.  The 16-row
 // products here are too small for 128-row tcgen05 tiles, and their operands are made in registers, so they run as mma.sync.
+#include "chunk_ops.cuh"
 #include "gla.cuh"
 
 #include <type_traits>
@@ -24,8 +25,7 @@
 namespace mfq {
 namespace {
 
-constexpr int kGc = 64, kGcThreads = 512, kGcWarps = kGcThreads / 32, kGcMaxDk = 256, kGcMaxDv = 512;
-constexpr float kGcSpan = 100.f;
+constexpr int kGcThreads = 512, kGcWarps = kGcThreads / 32, kGcMaxDk = 256, kGcMaxDv = 512;
 
 struct GlaChunkParams {
   GlaShape s;
@@ -42,11 +42,6 @@ struct GlaChunkParams {
   float* gam;                 // [chunks, H, dk]     2^b_C
 };
 
-__device__ __forceinline__ float gc_exp2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
 // log2(sigmoid(z)) and silu to a few units of 2^-23 (absolute, relative)
 __device__ __forceinline__ float gc_log2_sigmoid(float z) {
   float y;
@@ -58,32 +53,6 @@ __device__ __forceinline__ float gc_log2_decay(const GlaShape& s, float z) {
   return fmaxf(-1.4426950408889634f * gc_exp2(1.4426950408889634f * z), kGlaFloor);
 }
 __device__ __forceinline__ float gc_silu(float x) { return __fdividef(x, 1.f + gc_exp2(-1.4426950408889634f * fmaxf(x, -80.f))); }
-__device__ __forceinline__ void gc_cp16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void gc_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N>
-__device__ __forceinline__ void gc_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-__device__ __forceinline__ void gc_ldm(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void gc_ldm_t(uint32_t addr, uint32_t (&r)[4]) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void gc_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// (x, y) as a pair of bf16 numbers and the pair of what they leave
-__device__ __forceinline__ void gc_split(float x, float y, uint32_t& hi, uint32_t& lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-  const __nv_bfloat162 l = __floats2bfloat162_rn(x - __low2float(h), y - __high2float(h));
-  hi = *reinterpret_cast<const uint32_t*>(&h);
-  lo = *reinterpret_cast<const uint32_t*>(&l);
-}
-__device__ __forceinline__ float2 gc_pair(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
-
 // A CTA's chunk: tokens t0 .. t0 + n - 1; `index` numbers the chunks of all portions without overlap.
 struct GlaChunkAt {
   int t0, n;
@@ -98,17 +67,6 @@ __device__ __forceinline__ bool gc_locate(const GlaChunkParams& p, int chunk, in
 }
 
 __host__ __device__ constexpr int gc_groups(int dk) { return dk <= 64 ? 8 : dk <= 128 ? 4 : 2; }
-
-// 64 rows of `width` bf16 (a multiple of 16) to shared memory, two rows of a warp at a time; rows from `n` on are zeros.
-__device__ __forceinline__ void gc_rows(__nv_bfloat16* dst, int pitch, const __nv_bfloat16* src, int stride, int width, int n, int warp, int lane) {
-  const int per = width / 8;
-  for (int t0 = warp * 2; t0 < kGc; t0 += 2 * kGcWarps)
-    for (int i = lane; i < 2 * per; i += 32) {
-      const int t = t0 + (i >= per), c = (i >= per ? i - per : i) * 8;
-      if (t < n) gc_cp16(dst + t * pitch + c, src + size_t(t) * stride + c);
-      else *reinterpret_cast<uint4*>(dst + t * pitch + c) = make_uint4(0, 0, 0, 0);
-    }
-}
 
 struct GlaLocalSmem {
   int b, k, lo, v, tot, bytes;
@@ -144,9 +102,9 @@ gla_chunk_local_kernel(const GlaChunkParams p) {
   __nv_bfloat16* k_lo = reinterpret_cast<__nv_bfloat16*>(gc_sm + m.lo);
   const __nv_bfloat16* rows = p.proj + size_t(at.t0) * p.s.row_stride;
   {
-    gc_rows(k_lo, kp, rows + (H + h) * dk, p.s.row_stride, dk, at.n, warp, lane);
+    gc_rows<kGcWarps>(k_lo, kp, rows + (H + h) * dk, p.s.row_stride, dk, at.n, warp, lane);
     gc_commit();
-    gc_rows(v_s, vp, rows + 2 * H * dk + h * dv, p.s.row_stride, dv, at.n, warp, lane);
+    gc_rows<kGcWarps>(v_s, vp, rows + 2 * H * dk + h * dv, p.s.row_stride, dv, at.n, warp, lane);
     gc_commit();
     const __nv_bfloat16* a = rows + 2 * H * (dk + dv);
     const int aper = rank / 8;
@@ -333,9 +291,9 @@ gla_chunk_output_kernel(const GlaChunkParams p) {
     const float* cum = p.cum + size_t(at.t0) * (H * dk) + h * dk;
     for (int t = warp; t < kGc; t += kGcWarps)  // rows past the end repeat the last one
       for (int c = lane * 4; c < dk; c += 128) gc_cp16(b_s + t * bp + c, cum + size_t(min(t, at.n - 1)) * (H * dk) + c);
-    gc_rows(q_s, kp, rows + h * dk, p.s.row_stride, dk, at.n, warp, lane);
-    gc_rows(k_s, kp, rows + (H + h) * dk, p.s.row_stride, dk, at.n, warp, lane);
-    gc_rows(v_s, vp, rows + 2 * H * dk + h * dv, p.s.row_stride, dv, at.n, warp, lane);
+    gc_rows<kGcWarps>(q_s, kp, rows + h * dk, p.s.row_stride, dk, at.n, warp, lane);
+    gc_rows<kGcWarps>(k_s, kp, rows + (H + h) * dk, p.s.row_stride, dk, at.n, warp, lane);
+    gc_rows<kGcWarps>(v_s, vp, rows + 2 * H * dk + h * dv, p.s.row_stride, dv, at.n, warp, lane);
     gc_commit();
   }
   gc_wait<0>();

@@ -19,8 +19,11 @@ from dataclasses import dataclass
 import torch
 
 from .dense import DenseLinear, is_fp32, up
-from .lib import check, dense_lib, ptr, stream_ptr
+from .lib import Workspace, check, dense_lib, ptr, stream_ptr
 
+CHUNK, CHUNK_MAX_DK, CHUNK_MAX_RANK = 64, 128, 64
+CHUNKED_MIN_TOKENS = 16  # a batch whose longest portion is shorter goes token by token
+_scratch: dict[int, torch.Tensor] = {}
 MAX_ROWS, THREADS, MAX_SPLIT = 16, 256, 8  # of the token-by-token kernel
 
 
@@ -50,6 +53,15 @@ class Geometry:
     def width(self) -> int:
         """Columns of a row of projections."""
         return self.channels + self.b_cols + self.rank_a + self.rank_g
+
+    @property
+    def chunkable(self) -> bool:
+        return self.dk <= CHUNK_MAX_DK and self.rank_a <= CHUNK_MAX_RANK
+
+    def chunk_bytes(self) -> int:
+        """Scratch per chunk and head."""
+        rows = CHUNK * (self.dk + 8) * 2
+        return 6 * rows + 2 * CHUNK * 72 * 2 + 4 * self.dk + CHUNK * self.dv * 4
 
 
 @dataclass
@@ -99,6 +111,26 @@ def recurrent(x: torch.Tensor, proj: torch.Tensor, w: Weights, state: torch.Tens
     return out
 
 
+def chunked(x: torch.Tensor, proj: torch.Tensor, w: Weights, state: torch.Tensor, slots: torch.Tensor, geo: Geometry, starts: torch.Tensor,
+            max_q: int, *, first: int = 0, out: torch.Tensor | None = None) -> torch.Tensor:
+    """The same for portions (bf16), 64 tokens at a time; ``max_q``: the longest portion, ``first``: the first row of any (host)."""
+    t, b, dev = x.shape[0], slots.numel(), x.device.index or 0
+    out = torch.empty((t, geo.heads * geo.dv), dtype=x.dtype, device=x.device) if out is None else out
+    chunks = (t - first) // CHUNK + b
+    need = chunks * geo.heads * geo.chunk_bytes()
+    if dev not in _scratch or _scratch[dev].numel() < need:
+        _scratch[dev] = torch.empty(need, dtype=torch.uint8, device=x.device)
+    side = proj[:, geo.channels :]
+    gate = w.g2(side[:, geo.b_cols + geo.rank_a :])
+    raw = torch.empty((t, geo.heads * geo.dv), dtype=torch.float32, device=x.device)
+    rc = dense_lib().mfq_delta_chunk(ptr(x), ptr(side), ptr(w.a2), ptr(gate), ptr(w.dt_bias), ptr(w.rate), ptr(w.norm), ptr(out), ptr(state),
+                                     ptr(slots), ptr(starts), ptr(raw), ptr(_scratch[dev]), chunks, first, t - first, b, max_q, geo.heads,
+                                     geo.key_heads, geo.dk, geo.dv, geo.vdim, geo.b_cols, geo.rank_a, geo.rank_g, x.stride(0), proj.stride(0),
+                                     geo.dim ** -0.5, geo.eps, ptr(Workspace.get(x.device).status), stream_ptr())
+    check(rc, "delta_chunk", 3)
+    return out
+
+
 def ragged(proj: torch.Tensor, w: Weights, state: torch.Tensor, conv_state: torch.Tensor, slots: torch.Tensor, geo: Geometry,
            starts: torch.Tensor | None, max_q: int, singles: int) -> torch.Tensor:
     """Convolution and recurrence of a batch of portions whose first ``singles`` sequences bring one token each (``starts`` None: all)."""
@@ -111,5 +143,8 @@ def ragged(proj: torch.Tensor, w: Weights, state: torch.Tensor, conv_state: torc
     if singles < slots.numel():
         rest, first = slots[singles:], starts[singles:]
         conv(proj, w.conv, conv_state, rest, geo.channels, starts=first, max_q=max_q, out=x)
-        recurrent(x, proj, w, state, rest, geo, starts=first, out=out)
+        if proj.dtype == torch.bfloat16 and max_q >= CHUNKED_MIN_TOKENS and geo.chunkable:
+            chunked(x, proj, w, state, rest, geo, first, max_q, first=singles, out=out)
+        else:
+            recurrent(x, proj, w, state, rest, geo, starts=first, out=out)
     return out

@@ -68,6 +68,7 @@ _DENSE_SIGNATURES = {
     "mfq_latent_pages": [_vp] * 5 + [_i] * 3 + [_vp],
     "mfq_latent_decode": [_vp] * 5 + [_i] + [_vp] * 3 + [_i] * 6 + [_f, _i, _vp],
     "mfq_latent_plain": [_vp] * 6 + [_i] * 6 + [_f, _i, _vp],
+    "mfq_delta_chunk": [_vp] * 13 + [_i] * 15 + [_f, _f, _vp, _vp],
     "mfq_delta_recurrent": [_vp] * 11 + [_i] * 12 + [_f, _f, _i, _vp],
     "mfq_embed_scaled": [_vp, _vp, _f, _vp, _vp, _i, _i, _i, _vp],
     "mfq_norm_add": [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _vp],
