@@ -517,6 +517,36 @@ def run_kamedra(args) -> dict:
     return bench.result()
 
 
+def run_bufolorn(args) -> dict:
+    """The Bufolorn family (bf16; a quarter each latent attention in a window, delta rule, attention with distance bias beside time
+    mixing, and latent attention on shared latents) beside the Kamedra of equal width, depth, feed-forward, heads and window: with
+    dense feed-forwards everywhere, and with routed experts of equal active width in every other layer (``-moe``)."""
+    from mfq_b200.models import bufolorn as bf
+    from mfq_b200.models.kamedra import AttentionSpec, GlaSpec, KamedraConfig, KamedraModel, KamedraWeights, RandomTensors
+    bench = FamilyBench(args)
+    for size in (args.size.split(",") if args.size else ["1b", "8b"]):
+        width, ff, layers, hq, hk, hl, vocab = KAMEDRA_SIZES[size]
+        rank, d = 512, 128
+        if args.tiny:
+            width, ff, layers, hq, hk, hl, vocab, rank, d = 256, 512, 4, 4, 2, 2, 1024, 64, 32
+        for window in (int(w) for w in args.window.split(",")):
+            latent = bf.LatentSpec(hq, d, d // 2, d, rank, (1.5 * d) ** -0.5, rot_base=5e5, window=window)
+            parallel = bf.ParallelSpec(bf.BiasedSpec(hq, hk, d, d, d ** -0.5, 50.0, 512.0, 0.1, 1024, buckets=32), bf.TimeMixSpec(hq, d // 2, 64), 1.0, 1.0)
+            experts = bf.ExpertsSpec(16, 2, 2.5, ff // 4, ff // 2)
+            for tag, mlp in (("", [bf.DenseSpec(ff)]), ("-moe", [bf.DenseSpec(ff), experts])):
+                cfg = bf.BufolornConfig.periodic(vocab_size=vocab, hidden_size=width, num_layers=layers, latent=latent, parallel=parallel,
+                                                 delta_rule=bf.DeltaSpec(hq, hq // 2, d, d, 4, 64, 64), mlp=mlp)
+                weights = bf.BufolornWeights(cfg, bf.RandomTensors(cfg, bench.dev), bench.dev)
+                bench.add(f"bufolorn-{size}{tag}-w{window}", bf.BufolornModel(cfg, weights), vocab, **_facts(cfg, weights))
+                del weights
+            cfg = KamedraConfig.periodic(vocab_size=vocab, hidden_size=width, num_layers=layers, ff=ff, linear=GlaSpec(hl, d, 2 * d, 16.0, rank=16),
+                                         attention=AttentionSpec(hq, hk, d // 2, d, 0.125, 0.5, window=window, keep=64, rot_dims=d // 2, rot_base=5e5))
+            weights = KamedraWeights(cfg, RandomTensors(cfg, bench.dev), bench.dev)
+            bench.add(f"kamedra-{size}-w{window}", KamedraModel(cfg, weights), vocab, **_facts(cfg, weights))
+            del weights
+    return bench.result()
+
+
 def run_reference(args) -> dict:
     from baseline import reference_arm
     return reference_arm.run(args)
@@ -542,19 +572,20 @@ def main() -> None:
     ap.add_argument("--profile-steps", type=int, default=0,
                     help="after the timed region, run this many batched decode steps between cudaProfilerStart/Stop")
     ap.add_argument("--tiny", action="store_true", help="tiny model, for checking the harness itself")
-    ap.add_argument("--model", choices=["llama8b", "hybrid80b", "tepetar", "kamedra"], default="llama8b",
+    ap.add_argument("--model", choices=["llama8b", "hybrid80b", "tepetar", "kamedra", "bufolorn"], default="llama8b",
                     help="llama8b: the flagship; hybrid80b: the Gated-DeltaNet + MoE hybrid with an MTP head (one GPU); "
                          "tepetar: that family in bf16 beside the FP8 Llama of equal geometry (one GPU); "
-                         "kamedra: that family in bf16 beside the Tepetar of equal geometry (one GPU)")
-    ap.add_argument("--size", default="", help="tepetar, kamedra: comma separated sizes out of " + ", ".join(TEPETAR_SIZES) + " (default 1b,8b)")
-    ap.add_argument("--window", default="4096,1024", help="tepetar, kamedra: comma separated window sizes")
+                         "kamedra: that family in bf16 beside the Tepetar of equal geometry (one GPU); "
+                         "bufolorn: that family in bf16 beside the Kamedra of equal geometry (one GPU)")
+    ap.add_argument("--size", default="", help="tepetar, kamedra, bufolorn: comma separated sizes out of " + ", ".join(TEPETAR_SIZES) + " (default 1b,8b)")
+    ap.add_argument("--window", default="4096,1024", help="tepetar, kamedra, bufolorn: comma separated window sizes")
     args = ap.parse_args()
     if args.warmup < 3:
         args.warmup = 3
     if args.impl == "reference":
         out = run_reference(args)
     else:
-        out = {"hybrid80b": run_hybrid, "tepetar": run_tepetar, "kamedra": run_kamedra}.get(args.model, run_ours)(args)
+        out = {"hybrid80b": run_hybrid, "tepetar": run_tepetar, "kamedra": run_kamedra, "bufolorn": run_bufolorn}.get(args.model, run_ours)(args)
     if out:
         print(json.dumps(out), flush=True)
 

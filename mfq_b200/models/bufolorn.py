@@ -323,6 +323,17 @@ class BufolornConfig:
     def from_dict(cls, raw: dict) -> "BufolornConfig":
         return cls(**{k: v for k, v in raw.items() if k in cls.__dataclass_fields__})
 
+    @classmethod
+    def periodic(cls, *, vocab_size: int, hidden_size: int, num_layers: int, latent: LatentSpec, delta_rule: DeltaSpec, parallel: ParallelSpec,
+                 mlp: list, embed_scale: float = 1.0, residual_mult: float = 1.0, norm_eps: float = 1e-5, name: str = "bufolorn") -> "BufolornConfig":
+        """Latent, delta rule, parallel, and latent attention on the latents of three layers before, again and again; the feed-forwards
+        go round in a period of their own (benchmarks)."""
+        layers = []
+        for i in range(num_layers):
+            again = LatentSpec(**{**vars(latent), "kv_from": i - 3})
+            layers.append(LayerSpec((latent, delta_rule, parallel, again)[i % 4], mlp[i % len(mlp)]))
+        return cls(vocab_size, hidden_size, layers, embed_scale, residual_mult, norm_eps, name)
+
 
 def tensor_shapes(cfg: BufolornConfig) -> dict[str, tuple[int, ...]]:
     """Canonical names and shapes of a checkpoint of this design (ranks and distance tables as far as the configuration knows them)."""

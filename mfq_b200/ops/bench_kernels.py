@@ -301,12 +301,143 @@ def bench_gdn(batch: int, tokens: int, reps: int) -> dict:
     return {"kernel": "gdn_recurrent" if tokens == 1 else "gdn_chunk (three kernels)", "batch": batch, "t": tokens, "us": ms * 1e3, "gbs": bytes_ / ms / 1e6}
 
 
+def bench_bias(batch: int, ctx: int, hq: int, hk: int, d: int, most: int, reps: int) -> dict:
+    """Attention with a score cap, a distance bias up to ``most`` and a sink: one token per sequence, or for batch 0 one prompt."""
+    from . import window_attn
+    table = torch.randn((hq, len(window_attn.log_buckets(32, most))), device="cuda")
+    how = dict(window=1 << 30, scale=0.088, cap=50.0, bias=window_attn.DistanceBias.from_table(table), sink=torch.zeros(hq, device="cuda"))
+    layers = max(1, min(32, math.ceil(4 * L2_BYTES / (batch * ctx * hk * d * 4)))) if batch else 1
+    cache = _plain_cache(max(1, batch), ctx, hk, d, d, layers)
+    shape = {"batch": batch, "ctx": ctx, "hq": hq, "hk": hk, "d": d, "bias_max": most}
+    q = torch.randn((batch or ctx, hq, d), device="cuda").to(torch.bfloat16)
+    out = torch.empty_like(q)
+    if batch:
+        sl, splits = torch.full((batch,), ctx, dtype=torch.int32, device="cuda"), window_attn.decode_splits(batch, hk, ctx)
+        ms = time_ms(lambda i: window_attn.decode(q, cache.layer(i % layers), cache.block_table, sl, splits=splits, out=out, **how), reps)
+        return {"kernel": "window_attn_decode (bias, sink)", **shape, "splits": splits, "us": ms * 1e3, "gbs": batch * ctx * hk * d * 4 / ms / 1e6}
+    starts, lens = (torch.tensor(v, dtype=torch.int32, device="cuda") for v in ([0, ctx], [ctx]))
+    ms = time_ms(lambda _: window_attn.prefill(q, cache.layer(0), cache.block_table, starts, lens, ctx, out=out, **how), reps)
+    return {"kernel": "window_attn_prefill (bias, sink)", **shape, "us": ms * 1e3, "tflops": 2 * ctx * (ctx + 1) * hq * d / ms / 1e9}
+
+
+def bench_latent(batch: int, ctx: int, heads: int, window: int, reps: int, splits=None) -> list[dict]:
+    """Latent attention at rank 512, 128 + 64 query channels, values of 128: a decode step (attention and the products into and out of
+    latent space), or for batch 0 one prompt (copy of the rows, expansion, attention)."""
+    from . import dense, latent_attn
+    d, rot, e, rank, seen = 128, 64, 128, 512, min(ctx, window)
+    r, layers = rank + rot, max(1, min(32, math.ceil(4 * L2_BYTES / (max(1, batch) * seen * 576 * 2))))
+    cache = _plain_cache(max(1, batch), ctx, 1, r, 0, layers)
+    shape = {"batch": batch, "ctx": ctx, "heads": heads, "window": window}
+    if batch:
+        q = torch.randn((batch, heads, r), device="cuda").to(torch.bfloat16)
+        sl = torch.full((batch,), ctx, dtype=torch.int32, device="cuda")
+        splits = latent_attn.decode_splits(batch, heads, seen) if splits is None else splits
+        ms = time_ms(lambda i: latent_attn.decode(q, cache.layer(i % layers).k, cache.block_table, sl, rank=rank, window=window, scale=0.07, splits=splits), reps)
+        rows = [{"kernel": "latent_decode", **shape, "splits": splits, "us": ms * 1e3, "gbs": batch * seen * r * 2 / ms / 1e6,
+                 "tile_gbs": batch * seen * r * 2 * math.ceil(heads / 16) / ms / 1e6}]
+        copies = 16
+        for name, n, k in (("into latent space", rank, d), ("out of it", e, rank)):
+            lin = [dense.DenseLinear(torch.randn((heads * n, k), device="cuda").to(torch.bfloat16), groups=heads) for _ in range(copies)]
+            x, out = torch.randn((batch, heads * k), device="cuda").to(torch.bfloat16), torch.empty((batch, heads * n), device="cuda", dtype=torch.bfloat16)
+            ms = time_ms(lambda i: lin[i % copies](x, out=out), reps)
+            rows.append({"kernel": f"product per head, {name}", "batch": batch, "heads": heads, "us": ms * 1e3,
+                         "gbs": 2 * (heads * n * k + batch * heads * (n + k)) / ms / 1e6})
+        return rows
+    seq, shift = (torch.tensor(v, dtype=torch.int32, device="cuda") for v in latent_attn.visible_pages([(0, ctx)], window))
+    rows_ = latent_attn.visible_rows(cache.layer(0).k, cache.block_table, seq, shift)
+    ms = time_ms(lambda _: latent_attn.visible_rows(cache.layer(0).k, cache.block_table, seq, shift), reps)
+    rows = [{"kernel": "latent_pages", **shape, "us": ms * 1e3, "gbs": ctx * r * 4 / ms / 1e6}]
+    lin = dense.DenseLinear(torch.randn((heads * (d + rot + e), r), device="cuda").to(torch.bfloat16))
+    kv = lin(rows_)
+    ms = time_ms(lambda _: lin(rows_), reps)
+    rows.append({"kernel": "dense_gemm (expansion)", **shape, "us": ms * 1e3, "tflops": 2 * ctx * heads * (d + e) * rank / ms / 1e9})
+    q = torch.randn((ctx, heads, d + rot), device="cuda").to(torch.bfloat16)
+    out = torch.empty((ctx, heads, e), device="cuda", dtype=torch.bfloat16)
+    starts, lens = (torch.tensor(v, dtype=torch.int32, device="cuda") for v in ([0, ctx], [ctx]))
+    ms = time_ms(lambda _: latent_attn.prefill_rows(q, kv, shift, starts, lens, ctx, head0=0, heads=heads, dk=d + rot, dv=e, window=window, scale=0.07,
+                                                    out=out), reps)
+    w = min(window, ctx)
+    pairs = w * (w + 1) // 2 + (ctx - w) * w
+    return rows + [{"kernel": "window_attn_prefill (expanded rows)", **shape, "us": ms * 1e3, "tflops": 2 * pairs * heads * (d + rot + e) / ms / 1e9}]
+
+
+def bench_time_mixing(batch: int, tokens: int, h: int, d: int, reps: int) -> dict:
+    """Time mixing, as :func:`bench_gla`."""
+    from . import gla
+    geo = gla.Geometry(h, d, d, d, d, 64, 1.0, 1e-6, decay="exp", scaled=False)
+    w2, bias = (torch.randn((h * d, 64), device="cuda") * 0.1).to(torch.bfloat16), torch.randn(h * d, device="cuda") - 2
+    norm, bonus, slots = torch.ones((h, d), device="cuda"), torch.ones(h * d, device="cuda"), torch.arange(batch, dtype=torch.int32, device="cuda")
+    proj = torch.randn((batch * tokens, geo.width), device="cuda").to(torch.bfloat16)
+    row = batch * tokens * (geo.width + h * d) * 2
+    if tokens == 1:
+        layers = max(1, min(64, math.ceil(4 * L2_BYTES / (batch * h * d * d * 4))))
+        states = [torch.zeros((batch, h, d, d), device="cuda") for _ in range(layers)]
+        ms = time_ms(lambda i: gla.recurrent(proj, w2, bias, norm, states[i % layers], slots, geo, bonus=bonus), reps)
+        return {"kernel": "gla_recurrent (time mixing)", "batch": batch, "h": h, "d": d, "us": ms * 1e3, "gbs": (batch * h * d * d * 8 + row) / ms / 1e6}
+    state, starts = torch.zeros((1, h, d, d), device="cuda"), torch.tensor([0, tokens], dtype=torch.int32, device="cuda")
+    ms = time_ms(lambda _: gla.chunked(proj, w2, bias, norm, state, slots, geo, starts, tokens, bonus=bonus), reps)
+    return {"kernel": "gla_chunk (time mixing, three kernels)", "t": tokens, "h": h, "d": d, "us": ms * 1e3, "gbs": row / ms / 1e6}
+
+
+def bench_delta(batch: int, tokens: int, h: int, hk: int, d: int, reps: int) -> list[dict]:
+    """Delta rule with a decay per channel (and its convolution), as :func:`bench_gla`."""
+    from . import delta, dense
+    geo = delta.Geometry(h, hk, d, d, d, d, 64, 64, 4, 1e-6)
+    bf = lambda *s: (torch.randn(s, device="cuda") * 0.1).to(torch.bfloat16)
+    w = delta.Weights(torch.randn((4, geo.channels), device="cuda"), bf(h * d, 64), torch.randn(h * d, device="cuda") - 2, torch.ones(h, device="cuda"),
+                      dense.DenseLinear(bf(h * d, 64)), torch.ones(d, device="cuda"))
+    slots, n = torch.arange(batch, dtype=torch.int32, device="cuda"), batch * tokens
+    proj, x = torch.randn((n, geo.width), device="cuda").to(torch.bfloat16), torch.randn((n, geo.channels), device="cuda").to(torch.bfloat16)
+    hist, out = torch.zeros((batch, 3, geo.channels), device="cuda"), torch.empty((n, geo.channels), device="cuda", dtype=torch.bfloat16)
+    row = n * (geo.width + h * d) * 2
+    if tokens == 1:
+        layers = max(1, min(32, math.ceil(4 * L2_BYTES / (batch * h * d * d * 4))))
+        states = [torch.zeros((batch, h, d, d), device="cuda") for _ in range(layers)]
+        ms = time_ms(lambda i: delta.recurrent(x, proj, w, states[i % layers], slots, geo), reps)
+        mc = time_ms(lambda _: delta.conv(proj, w.conv, hist, slots, geo.channels, out=out), reps)
+        return [{"kernel": "delta_recurrent", "batch": batch, "h": h, "d": d, "us": ms * 1e3, "gbs": (batch * h * d * d * 8 + row) / ms / 1e6},
+                {"kernel": "short_conv", "batch": batch, "c": geo.channels, "us": mc * 1e3, "gbs": batch * geo.channels * 28 / mc / 1e6}]
+    state, starts = torch.zeros((1, h, d, d), device="cuda"), torch.tensor([0, tokens], dtype=torch.int32, device="cuda")
+    ms = time_ms(lambda _: delta.chunked(x, proj, w, state, slots, geo, starts, tokens), reps)
+    mc = time_ms(lambda _: delta.conv(proj, w.conv, hist, slots, geo.channels, starts=starts, max_q=tokens, out=out), reps)
+    return [{"kernel": "delta_chunk (four kernels)", "t": tokens, "h": h, "hk": hk, "d": d, "us": ms * 1e3, "gbs": row / ms / 1e6},
+            {"kernel": "short_conv (two kernels)", "t": tokens, "c": geo.channels, "us": mc * 1e3, "gbs": n * geo.channels * 4 / mc / 1e6}]
+
+
+def bench_experts(tokens: int, width: int, ff: int, experts: int, top: int, reps: int) -> list[dict]:
+    """Routed experts of one layer in bf16 (routing, products, addition to the stream), and the same in block-scaled FP8."""
+    from . import dense, dense_moe, moe
+    h, x = torch.randn((tokens, width), device="cuda").to(torch.bfloat16), torch.zeros((tokens, width), device="cuda")
+    logits = torch.randn((tokens, experts), device="cuda")
+    copies = max(1, min(4, math.ceil(4 * L2_BYTES / (experts * 3 * width * ff * 2))))
+    bf = lambda *s: torch.randn(s, device="cuda", dtype=torch.bfloat16) * 0.02
+    banks = [dense_moe.ExpertBank(experts, bf(experts * 2 * ff, width), bf(experts * width, ff)) for _ in range(copies)]
+    bias = torch.zeros(experts, device="cuda")
+    used = len(torch.unique(dense_moe.topk(logits, top, bias, 1.0)[0]))
+
+    def layer(i):
+        ids, wt = dense_moe.topk(logits, top, bias, 2.5)
+        dense_moe.add_experts(h, ids, wt, banks[i % copies], x, 1.0)
+    ms = time_ms(layer, reps)
+    shape = {"tokens": tokens, "width": width, "ff": ff, "experts": experts, "top": top, "used": used}
+    flops = 6 * tokens * top * width * ff
+    rows = [{"kernel": "experts, bf16", **shape, "us": ms * 1e3, "gbs": used * 3 * width * ff * 2 / ms / 1e6, "tflops": flops / ms / 1e9}]
+    del banks
+    f8 = lambda *s: torch.randint(-100, 100, s, device="cuda", dtype=torch.int8).view(torch.float8_e4m3fn)
+    sc = lambda e, n, k: torch.rand((e, math.ceil(n / 128), k // 128), device="cuda") * 0.01
+    gu, dn = [f8(experts, 2 * ff, width) for _ in range(copies)], [f8(experts, width, ff) for _ in range(copies)]
+    gus, dns, xq, xs = sc(experts, 2 * ff, width), sc(experts, width, ff), f8(tokens, width), torch.rand(tokens, device="cuda")
+    ids, wt = dense_moe.topk(logits, top, bias, 2.5)
+    ms = time_ms(lambda i: moe.moe_ffn_fp8(xq, xs, ids, wt, gu[i % copies], gus, dn[i % copies], dns), reps)
+    return rows + [{"kernel": "experts, FP8", **shape, "us": ms * 1e3, "gbs": used * 3 * width * ff / ms / 1e6, "tflops": flops / ms / 1e9}]
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--json", default="")
     ap.add_argument("--reps", type=int, default=20)
     ap.add_argument("--quick", action="store_true")
-    ap.add_argument("--only", default="", help="comma separated kernel families: gemm,w4,attn,mla,small,prefill,dense,maps,gla")
+    ap.add_argument("--only", default="", help="comma separated kernel families: gemm,w4,attn,mla,small,prefill,dense,maps,gla,bias,latent,mixing,delta,experts")
     ap.add_argument("--tp", type=int, default=1, help="time one rank's shard of a tensor-parallel group of this size")
     args = ap.parse_args()
     pk = peaks()
@@ -377,6 +508,39 @@ def main() -> None:
             for h, dk, dv in ((32, 128, 128), (16, 128, 256)):
                 rows.append(bench_gla(batch, tokens, h, dk, dv, args.reps))
             rows.append(bench_gdn(batch, tokens, args.reps))
+    if want("bias"):
+        for batch in (1, 64, 0):
+            for most in (256, 2048):
+                rows.append(bench_bias(batch, 4096, 32, 8, 128, most, args.reps))
+            rows.append(bench_window_decode(batch, 4096, 32, 8, 128, 4096, 50.0, args.reps) if batch else bench_window_prefill(4096, 32, 8, 128, 1 << 30, 50.0, args.reps))
+    if want("latent"):
+        for heads in (16, 32):
+            for batch, window in ((1, 4096), (64, 4096), (64, 1024), (0, 4096), (0, 1024)):
+                rows += bench_latent(batch, 4096, heads, window, args.reps)
+        for batch, splits in ((1, 16), (64, 2)):
+            rows.append(bench_mla_decode(batch, 4096, 16, splits, args.reps))
+        rows += bench_prefill(4096, 32, 32, args.reps, d=256)[:1]  # how the FP8 latent models prefill: heads padded to 256 channels
+    if want("mixing"):
+        from . import dense, gla
+        for batch, tokens in ((1, 1), (64, 1), (1, 2048), (1, 4096)):
+            rows.append(bench_time_mixing(batch, tokens, 64, 64, args.reps))
+            rows.append(bench_gla(batch, tokens, 64, 64, 64, args.reps))
+        for m in (1, 64, 4096):
+            x, w = torch.randn((m, 4096), device="cuda"), torch.ones(4096, device="cuda")
+            ms = time_ms(lambda _: dense.layer_norm_out(x, w, w, 4096, 1e-5, torch.bfloat16), args.reps)
+            rows.append({"kernel": "layer_norm_out", "m": m, "h": 4096, "us": ms * 1e3, "gbs": m * 4096 * 6 / ms / 1e6})
+            h, mu, last = x.to(torch.bfloat16), torch.rand((5, 4096), device="cuda"), torch.zeros((64, 4096), device="cuda")
+            slots = torch.arange(64 if m == 64 else 1, dtype=torch.int32, device="cuda")
+            ragged = (torch.tensor([0, m], dtype=torch.int32, device="cuda"), torch.zeros(m, dtype=torch.int32, device="cuda")) if m > 64 else ()
+            ms = time_ms(lambda _: gla.token_shift(h, mu, last, slots, *ragged), args.reps)
+            rows.append({"kernel": "token_shift", "m": m, "h": 4096, "us": ms * 1e3, "gbs": m * 4096 * 12 / ms / 1e6})
+    if want("delta"):
+        for batch, tokens in ((1, 1), (64, 1), (1, 2048), (1, 4096)):
+            rows += bench_delta(batch, tokens, 32, 16, 128, args.reps)
+            rows.append(bench_gdn(batch, tokens, args.reps))
+    if want("experts"):
+        for tokens in (1, 16, 64, 512, 4096):
+            rows += bench_experts(tokens, 4096, 2048, 32, 4, args.reps)
     for r in rows:
         if "gbs" in r:
             r["hbm_frac"] = r["gbs"] / pk["hbm_gbs"]
