@@ -4,7 +4,8 @@
 //   delta_recurrent_kernel   a CTA per (head, sequence) walks the tokens of the sequence's portion with the state in registers (a
 //                            thread owns four adjacent columns on every R-th row, at most 16 rows).  Unit norms, decays, write
 //                            strength, norm and gate are fused in.  S^T k and S^T q are summed in one pass: o follows from the
-//                            decayed state as S^T q + u (k . q).  The columns of a head may be split over a thread-block cluster,
+//                            decayed state as S^T q + u (k . q).  The low-rank factors of a head's decays and gates are brought to
+//                            shared memory ahead of the dependent-launch wait, if they fit.  The columns of a head may be split over a thread-block cluster,
 //                            which adds its squares for the norm through distributed shared memory.
 #include "delta.cuh"
 
@@ -22,7 +23,22 @@ struct DeltaRecurrentParams {
   const float* rate;     // [H] exp(A_log)
   const float* norm_w;   // [dv]
   int split, rows;    // column split (cluster size); row groups R
+  int staged;         // whether the factors lie in shared memory
 };
+
+__device__ __forceinline__ void delta_cp16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+// n rows of `width` elements (a multiple of 8) to rows 16 bytes further apart
+template <typename T>
+__device__ __forceinline__ void delta_stage(T* dst, const T* src, int n, int width) {
+  constexpr int kVec = 16 / sizeof(T);
+  const int per = width / kVec;
+  for (int i = threadIdx.x; i < n * per; i += blockDim.x) {
+    const int r = i / per, c = (i - r * per) * kVec;
+    delta_cp16(dst + r * (width + kVec) + c, src + size_t(r) * width + c);
+  }
+}
 
 __device__ __forceinline__ void delta_cluster_barrier() {
   asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
@@ -64,6 +80,17 @@ delta_recurrent_kernel(const T* __restrict__ conv, const T* __restrict__ side, c
   float* gate_s = v_s + cols;      // [cols]
   float* part_k = gate_s + cols;   // [R][cols]
   float* part_q = part_k + R * cols;
+  constexpr int kPad = 16 / sizeof(T);
+  const T *a2 = w_a2 + size_t(h) * dk * p.s.ra, *g2 = w_g2 + (size_t(h) * dv + c_base) * p.s.rg;
+  int a2_pitch = p.s.ra, g2_pitch = p.s.rg;
+  if (p.staged) {
+    T* sa = reinterpret_cast<T*>(part_q + R * cols);
+    T* sg = sa + dk * (p.s.ra + kPad);
+    delta_stage<T>(sa, a2, dk, p.s.ra);
+    delta_stage<T>(sg, g2, cols, p.s.rg);
+    a2 = sa; g2 = sg;
+    a2_pitch += kPad; g2_pitch += kPad;
+  }
   __shared__ float red[33];
   __shared__ float dots[8][3];
   __shared__ float ss_own[2];
@@ -72,7 +99,10 @@ delta_recurrent_kernel(const T* __restrict__ conv, const T* __restrict__ side, c
   const int mine = rg < R ? (dk - rg + R - 1) / R : 0;  // my rows: rg + R i
   pdl_wait();
   const int slot = p.slot[b];
-  if (slot < 0) return;  // the whole cluster leaves
+  if (slot < 0) {  // the whole cluster leaves
+    asm volatile("cp.async.wait_all;" ::: "memory");
+    return;
+  }
   const int t0 = p.starts ? p.starts[b] : b, t1 = p.starts ? p.starts[b + 1] : b + 1;
   float* st = p.state + (size_t(slot) * H + h) * dk * dv + c_base + cg * 4;
   float4 s[kDeltaRows];
@@ -101,17 +131,20 @@ delta_recurrent_kernel(const T* __restrict__ conv, const T* __restrict__ side, c
       qk += __shfl_xor_sync(0xffffffffu, qk, o);
     }
     if (lane == 0) { dots[warp][0] = qq; dots[warp][1] = kk; dots[warp][2] = qk; }
+    asm volatile("cp.async.wait_all;" ::: "memory");
     __syncthreads();
     qq = kk = qk = 0.f;
 #pragma unroll
     for (int w = 0; w < 8; ++w) { qq += dots[w][0]; kk += dots[w][1]; qk += dots[w][2]; }
     const float iq = rsqrtf(qq + 1e-6f) * p.s.scale, ik = rsqrtf(kk + 1e-6f), beta = delta_sigmoid(to_float(srow[h]));
-    for (int i = tid; i < dk; i += kDeltaThreads) {
-      const float z = delta_row_dot<T>(w_a2 + size_t(h * dk + i) * p.s.ra, a_s, p.s.ra, p.dt_bias[h * dk + i]);
-      d_s[i] = exp2f(rate * delta_softplus(z));
+    for (int i = tid; i < dk + cols; i += kDeltaThreads) {  // decays of the rows, then gates of my columns
+      if (i < dk) {
+        const float z = delta_row_dot<T>(a2 + i * a2_pitch, a_s, p.s.ra, p.dt_bias[h * dk + i]);
+        d_s[i] = exp2f(fmaxf(rate * delta_softplus(z), kGlaFloor));
+      } else {
+        gate_s[i - dk] = delta_sigmoid(delta_row_dot<T>(g2 + (i - dk) * g2_pitch, g_s, p.s.rg, 0.f));
+      }
     }
-    for (int i = tid; i < cols; i += kDeltaThreads)
-      gate_s[i] = delta_sigmoid(delta_row_dot<T>(w_g2 + size_t(h * dv + c_base + i) * p.s.rg, g_s, p.s.rg, 0.f));
     __syncthreads();
     float4 ak = make_float4(0.f, 0.f, 0.f, 0.f), aq = ak;
 #pragma unroll
@@ -167,10 +200,20 @@ delta_recurrent_kernel(const T* __restrict__ conv, const T* __restrict__ side, c
 }
 
 template <typename T>
-int launch_delta_recurrent(const void* conv, const void* side, const void* w_a2, const void* w_g2, void* y, const DeltaRecurrentParams& p, int B,
+int launch_delta_recurrent(const void* conv, const void* side, const void* w_a2, const void* w_g2, void* y, const DeltaRecurrentParams& p0, int B,
                            cudaStream_t stream) {
-  const int cols = p.s.dv / p.split, smem = (3 * p.s.dk + p.s.ra + p.s.rg + 2 * cols + 2 * p.rows * cols) * 4;
-  if (smem > 48 * 1024) return -5;
+  const int cols = p0.s.dv / p0.split, pad = 16 / int(sizeof(T));
+  const int plain = (3 * p0.s.dk + p0.s.ra + p0.s.rg + 2 * cols + 2 * p0.rows * cols) * 4;
+  const int factors = (p0.s.dk * (p0.s.ra + pad) + cols * (p0.s.rg + pad)) * int(sizeof(T));
+  DeltaRecurrentParams p = p0;
+  p.staged = plain + factors <= 100 * 1024;  // two CTAs per SM
+  const int smem = plain + (p.staged ? factors : 0);
+  if (smem > 200 * 1024) return -5;
+  static int allowed = 48 * 1024;
+  if (smem > allowed) {
+    if (cudaFuncSetAttribute(delta_recurrent_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -6;
+    allowed = smem;
+  }
   const dim3 grid(p.s.H * p.split, B), block(kDeltaThreads);
   const T *c = static_cast<const T*>(conv), *sd = static_cast<const T*>(side), *wa = static_cast<const T*>(w_a2), *wg = static_cast<const T*>(w_g2);
   const cudaError_t rc = p.split > 1
@@ -199,7 +242,7 @@ extern "C" int mfq_delta_recurrent(const void* conv, const void* side, const voi
   const int rows = min(dk, kDeltaThreads / groups);
   if ((dk + rows - 1) / rows > kDeltaRows) return -5;
   const DeltaRecurrentParams p{DeltaShape{H, G, dk, dv, b_cols, ra, rg, conv_stride, side_stride, scale, 1.f / float(real_dv), eps}, starts, slot,
-                               state, dt_bias, rate, norm_w, split, rows};
+                               state, dt_bias, rate, norm_w, split, rows, 0};
   return fp32 ? launch_delta_recurrent<float>(conv, side, w_a2, w_g2, y, p, B, stream)
               : launch_delta_recurrent<__nv_bfloat16>(conv, side, w_a2, w_g2, y, p, B, stream);
 }

@@ -6,9 +6,10 @@
 //   latent_pages    copies the visible pages of portions into consecutive rows, from where keys and values are expanded by a product
 //                   (prefill then runs window_attn_prefill.cuh on them)
 //   latent_decode   bf16, attention in latent space: queries are already mapped there, the value of a token is the latent part of
-//                   its row.  A CTA takes one query token, 16 heads (the rows of m16n8k16 MMAs) and one KV split, eight warps, 64
-//                   tokens (four pages) per step through two cp.async stages.  Scores: warp = (page, half of the channels), summed
-//                   through shared memory; softmax: two rows per warp; values: a warp owns every eighth 16-channel tile.
+//                   its row.  A CTA takes one query token, 16 or 32 heads (one or two row tiles of m16n8k16 MMAs, which share the
+//                   fragments of the cache) and one KV split, eight warps, 64 tokens (four pages) per step through two cp.async
+//                   stages.  Scores: warp = (page, half of the channels), summed through shared memory; softmax: two or four rows
+//                   per warp; values: a warp owns every eighth 16-channel tile.
 //   latent_plain    a warp per (token, head), fp32 arithmetic: the full-precision mode
 #include "window_attn.cuh"
 
@@ -140,50 +141,61 @@ struct LatentDecodeParams {
   float scale_log2;
 };
 
-int la_smem(int R) { return (16 + 2 * kLaStep) * (R + 8) * 2 + 2 * 16 * kLaStep * 4 + 16 * (kLaStep + 8) * 2 + 4 * 16 * 4; }
+int la_smem(int R, int tiles) {
+  const int rows = 16 * tiles;
+  return (rows + 2 * kLaStep) * (R + 8) * 2 + 2 * rows * kLaStep * 4 + rows * (kLaStep + 8) * 2 + 3 * rows * 4;
+}
 
+template <int MT>
 __global__ void __launch_bounds__(kLaThreads)
 latent_decode_kernel(const LatentDecodeParams p) {
   pdl_trigger();
   pdl_wait();
   extern __shared__ __align__(16) uint8_t la_sm[];
+  constexpr int kRows = 16 * MT, kMine = 2 * MT;  // rows of the head tiles; rows whose softmax a warp computes
   const int R = p.R, pitch = R + 8;
-  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(la_sm);                  // [16][pitch]
-  __nv_bfloat16* kv_s = q_s + 16 * pitch;                                         // 2 stages of [64][pitch]
-  float* s_part = reinterpret_cast<float*>(kv_s + 2 * kLaStep * pitch);           // [2][16][64]
-  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(s_part + 2 * 16 * kLaStep);  // [16][72]
-  float* alpha_s = reinterpret_cast<float*>(p_s + 16 * (kLaStep + 8));            // [16], then m, l [16] each
+  __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(la_sm);                      // [rows][pitch]
+  __nv_bfloat16* kv_s = q_s + kRows * pitch;                                          // 2 stages of [64][pitch]
+  float* s_part = reinterpret_cast<float*>(kv_s + 2 * kLaStep * pitch);               // [2][rows][64]
+  __nv_bfloat16* p_s = reinterpret_cast<__nv_bfloat16*>(s_part + 2 * kRows * kLaStep);  // [rows][72]
+  float* alpha_s = reinterpret_cast<float*>(p_s + kRows * (kLaStep + 8));             // [rows], then m, l [rows] each
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3, mat = lane >> 3, mrow = lane & 7;
-  const int t = blockIdx.x, h0 = blockIdx.y * 16, heads = min(16, p.H - h0), split = blockIdx.z;
+  const int t = blockIdx.x, h0 = blockIdx.y * kRows, heads = min(kRows, p.H - h0), split = blockIdx.z;
   const int pos = p.lens[t] + p.len_add - 1, lo = max(0, pos - p.window + 1);
   const int* table = p.table + size_t(p.tok_seq ? p.tok_seq[t] : t) * p.max_pages;
   const int page0 = lo / kLaPage, last = pos / kLaPage;
   const int all = pos >= 0 ? (last - page0) / 4 + 1 : 0, chunk = (all + p.splits - 1) / p.splits;  // steps
   const int step0 = split * chunk, steps = max(0, min(all, step0 + chunk) - step0);
   const int ch = R >> 3;
+  int ids = 0;  // lane j: page j of the next eight steps
   auto fetch = [&](int i) {
-    __nv_bfloat16* dst = kv_s + (i & 1) * kLaStep * pitch;
     const int first = page0 + (step0 + i) * 4;
-    // a warp copies rows of its own: 8 rows per warp and step
-    for (int r = warp; r < kLaStep; r += 8) {
-      const __nv_bfloat16* src = p.kv + (size_t(table[min(first + (r >> 4), last)]) * kLaPage + (r & 15)) * R;
+    if ((i & 7) == 0) ids = table[min(first + lane, last)];
+    __nv_bfloat16* dst = kv_s + (i & 1) * kLaStep * pitch;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {  // a warp copies two rows of every page
+      const int r = k * 8 + warp, page = __shfl_sync(0xffffffffu, ids, (i & 7) * 4 + (k >> 1));
+      const __nv_bfloat16* src = p.kv + (size_t(page) * kLaPage + (r & 15)) * R;
       for (int c = lane; c < ch; c += 32) la_cp16(smem_u32(dst + r * pitch + c * 8), src + c * 8);
     }
   };
-  for (int r = warp; r < 16; r += 8) {
+  for (int r = warp; r < kRows; r += 8) {
     const __nv_bfloat16* src = p.q + (size_t(t) * p.H + h0 + min(r, heads - 1)) * R;
     for (int c = lane; c < ch; c += 32) la_cp16(smem_u32(q_s + r * pitch + c * 8), src + c * 8);
   }
   if (steps > 0) fetch(0);
   la_commit();
-  float o[kLaMaxTiles][2][4];
+  float o[kLaMaxTiles][MT][2][4];
 #pragma unroll
   for (int i = 0; i < kLaMaxTiles; ++i)
 #pragma unroll
-    for (int j = 0; j < 8; ++j) o[i][j >> 2][j & 3] = 0.f;
-  float m_run[2] = {-FLT_MAX, -FLT_MAX}, l_run[2] = {0.f, 0.f};  // of rows 2 warp, 2 warp + 1
+    for (int j = 0; j < MT * 8; ++j) o[i][j >> 3][(j >> 2) & 1][j & 3] = 0.f;
+  float m_run[kMine], l_run[kMine];  // of rows kMine * warp ..
+#pragma unroll
+  for (int e = 0; e < kMine; ++e) { m_run[e] = -FLT_MAX; l_run[e] = 0.f; }
   const int ksteps = R / 16, khalf = (ksteps + 1) / 2, tiles = p.rank / 16;
   const int page = warp & 3, k0 = warp < 4 ? 0 : khalf, k1 = warp < 4 ? khalf : ksteps;
+  const uint32_t a_off = (((mat & 1) * 8 + mrow) * pitch + (mat >> 1) * 8) * 2;
   for (int i = 0; i < steps; ++i) {
     la_wait<0>();
     __syncthreads();  // step i has arrived, everyone is done with step i - 1
@@ -191,103 +203,139 @@ latent_decode_kernel(const LatentDecodeParams p) {
     la_commit();
     const __nv_bfloat16* kv = kv_s + (i & 1) * kLaStep * pitch;
     {
-      float s[2][4] = {};
-      const uint32_t qa = smem_u32(q_s + ((mat & 1) * 8 + mrow) * pitch + (mat >> 1) * 8);
+      float s[MT][2][4] = {};
+      const uint32_t qa = smem_u32(q_s) + a_off;
       const uint32_t ka = smem_u32(kv + (page * 16 + (mat >> 1) * 8 + mrow) * pitch + (mat & 1) * 8);
+#pragma unroll 6
       for (int ks = k0; ks < k1; ++ks) {
-        uint32_t a[4], b[4];
-        la_ldm(qa + ks * 32, a);
+        uint32_t a[MT][4], b[4];
         la_ldm(ka + ks * 32, b);
-        la_mma(s[0], a, b[0], b[1]);
-        la_mma(s[1], a, b[2], b[3]);
-      }
-      float* d = s_part + (warp >> 2) * 16 * kLaStep + page * 16 + t4 * 2;
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt) {
-        *reinterpret_cast<float2*>(d + g * kLaStep + nt * 8) = make_float2(s[nt][0], s[nt][1]);
-        *reinterpret_cast<float2*>(d + (g + 8) * kLaStep + nt * 8) = make_float2(s[nt][2], s[nt][3]);
+        for (int mt = 0; mt < MT; ++mt) la_ldm(qa + mt * 16 * pitch * 2 + ks * 32, a[mt]);
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt) {
+          la_mma(s[mt][0], a[mt], b[0], b[1]);
+          la_mma(s[mt][1], a[mt], b[2], b[3]);
+        }
       }
+      float* d = s_part + (warp >> 2) * kRows * kLaStep + page * 16 + t4 * 2;
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          *reinterpret_cast<float2*>(d + (mt * 16 + g) * kLaStep + nt * 8) = make_float2(s[mt][nt][0], s[mt][nt][1]);
+          *reinterpret_cast<float2*>(d + (mt * 16 + g + 8) * kLaStep + nt * 8) = make_float2(s[mt][nt][2], s[mt][nt][3]);
+        }
     }
     __syncthreads();
     const int key = (page0 + (step0 + i) * 4) * kLaPage + lane * 2;
+    float x[kMine], y[kMine], mx[kMine];
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int r = warp * 2 + e;
+    for (int e = 0; e < kMine; ++e) {
+      const int r = warp * kMine + e;
       const float2 a = *reinterpret_cast<const float2*>(s_part + r * kLaStep + lane * 2);
-      const float2 b = *reinterpret_cast<const float2*>(s_part + (16 + r) * kLaStep + lane * 2);
-      const float x = key >= lo && key <= pos ? (a.x + b.x) * p.scale_log2 : -FLT_MAX;
-      const float y = key + 1 >= lo && key + 1 <= pos ? (a.y + b.y) * p.scale_log2 : -FLT_MAX;
-      float mx = fmaxf(x, y);
+      const float2 b = *reinterpret_cast<const float2*>(s_part + (kRows + r) * kLaStep + lane * 2);
+      x[e] = key >= lo && key <= pos ? (a.x + b.x) * p.scale_log2 : -FLT_MAX;
+      y[e] = key + 1 >= lo && key + 1 <= pos ? (a.y + b.y) * p.scale_log2 : -FLT_MAX;
+      mx[e] = fmaxf(x[e], y[e]);
+    }
 #pragma unroll
-      for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
-      const float mn = fmaxf(m_run[e], mx), al = window_exp2(m_run[e] - mn);  // the step's first page holds a visible key
-      const float px = window_exp2(x - mn), py = window_exp2(y - mn);
-      float sum = px + py;
+    for (int off = 16; off > 0; off >>= 1)
 #pragma unroll
-      for (int off = 16; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
+      for (int e = 0; e < kMine; ++e) mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], off));
+#pragma unroll
+    for (int e = 0; e < kMine; ++e) {
+      const float mn = fmaxf(m_run[e], mx[e]), al = window_exp2(m_run[e] - mn);  // the step's first page holds a visible key
       m_run[e] = mn;
-      l_run[e] = l_run[e] * al + sum;
-      *reinterpret_cast<__nv_bfloat162*>(p_s + r * (kLaStep + 8) + lane * 2) = __floats2bfloat162_rn(px, py);
-      if (lane == 0) alpha_s[r] = al;
+      x[e] = window_exp2(x[e] - mn);
+      y[e] = window_exp2(y[e] - mn);
+      l_run[e] = fmaf(l_run[e], al, x[e] + y[e]);  // of my lane's keys; the lanes meet at the end
+      *reinterpret_cast<__nv_bfloat162*>(p_s + (warp * kMine + e) * (kLaStep + 8) + lane * 2) = __floats2bfloat162_rn(x[e], y[e]);
+      if (lane == 0) alpha_s[warp * kMine + e] = al;
     }
     __syncthreads();
-    const float al0 = alpha_s[g], al1 = alpha_s[g + 8];
-    uint32_t pf[4][4];
 #pragma unroll
-    for (int ks = 0; ks < 4; ++ks) la_ldm(smem_u32(p_s + ((mat & 1) * 8 + mrow) * (kLaStep + 8) + ks * 16 + (mat >> 1) * 8), pf[ks]);
+    for (int mt = 0; mt < MT; ++mt) {
+      const float al0 = alpha_s[mt * 16 + g], al1 = alpha_s[mt * 16 + g + 8];
+      if (__any_sync(0xffffffffu, al0 != 1.f || al1 != 1.f)) {
 #pragma unroll
-    for (int n = 0; n < kLaMaxTiles; ++n) {
-      const int tile = warp + 8 * n;
-      if (tile < tiles) {
+        for (int n = 0; n < kLaMaxTiles; ++n)
 #pragma unroll
-        for (int nt = 0; nt < 2; ++nt) {
-          o[n][nt][0] *= al0; o[n][nt][1] *= al0; o[n][nt][2] *= al1; o[n][nt][3] *= al1;
-        }
+          for (int nt = 0; nt < 2; ++nt) {
+            o[n][mt][nt][0] *= al0; o[n][mt][nt][1] *= al0; o[n][mt][nt][2] *= al1; o[n][mt][nt][3] *= al1;
+          }
+      }
+    }
 #pragma unroll
-        for (int ks = 0; ks < 4; ++ks) {
+    for (int ks = 0; ks < 4; ++ks) {
+      uint32_t pf[MT][4];
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt)
+        la_ldm(smem_u32(p_s + (mt * 16 + (mat & 1) * 8 + mrow) * (kLaStep + 8) + ks * 16 + (mat >> 1) * 8), pf[mt]);
+#pragma unroll
+      for (int n = 0; n < kLaMaxTiles; ++n) {
+        const int tile = warp + 8 * n;
+        if (tile < tiles) {
           uint32_t v[4];
           la_ldm_t(smem_u32(kv + (ks * 16 + (mat & 1) * 8 + mrow) * pitch + tile * 16 + (mat >> 1) * 8), v);
-          la_mma(o[n][0], pf[ks], v[0], v[1]);
-          la_mma(o[n][1], pf[ks], v[2], v[3]);
+#pragma unroll
+          for (int mt = 0; mt < MT; ++mt) {
+            la_mma(o[n][mt][0], pf[mt], v[0], v[1]);
+            la_mma(o[n][mt][1], pf[mt], v[2], v[3]);
+          }
         }
       }
     }
   }
   la_wait<0>();
-  __syncthreads();
-  if (lane == 0) {
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      alpha_s[16 + warp * 2 + e] = m_run[e];
-      alpha_s[32 + warp * 2 + e] = l_run[e];
+  for (int e = 0; e < kMine; ++e) {
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) l_run[e] += __shfl_xor_sync(0xffffffffu, l_run[e], off);
+    if (lane == 0) {
+      alpha_s[kRows + warp * kMine + e] = m_run[e];
+      alpha_s[2 * kRows + warp * kMine + e] = l_run[e];
     }
   }
   __syncthreads();
   const bool whole = p.splits == 1;
 #pragma unroll
-  for (int half = 0; half < 2; ++half) {
-    const int r = g + 8 * half;
+  for (int rr = 0; rr < 2 * MT; ++rr) {
+    const int mt = rr >> 1, half = rr & 1, r = mt * 16 + g + 8 * half;
     if (r >= heads) continue;
     const size_t row = size_t(t) * p.H + h0 + r;
-    const float l = alpha_s[32 + r], f = whole ? (l > 0.f ? 1.f / l : 0.f) : 1.f;
+    const float l = alpha_s[2 * kRows + r], f = whole ? (l > 0.f ? 1.f / l : 0.f) : 1.f;
 #pragma unroll
     for (int n = 0; n < kLaMaxTiles; ++n) {
       const int tile = warp + 8 * n;
       if (tile < tiles) {
 #pragma unroll
         for (int nt = 0; nt < 2; ++nt) {
-          const float x = o[n][nt][2 * half] * f, y = o[n][nt][2 * half + 1] * f;
+          const float a = o[n][mt][nt][2 * half] * f, b = o[n][mt][nt][2 * half + 1] * f;
           const int c = tile * 16 + nt * 8 + t4 * 2;
-          if (whole) *reinterpret_cast<__nv_bfloat162*>(p.out + row * p.rank + c) = __floats2bfloat162_rn(x, y);
-          else *reinterpret_cast<float2*>(p.part + (row * p.splits + split) * p.rank + c) = make_float2(x, y);
+          if (whole) *reinterpret_cast<__nv_bfloat162*>(p.out + row * p.rank + c) = __floats2bfloat162_rn(a, b);
+          else *reinterpret_cast<float2*>(p.part + (row * p.splits + split) * p.rank + c) = make_float2(a, b);
         }
       }
     }
     if (!whole && warp == 0 && t4 == 0) {
-      p.part_ml[(row * p.splits + split) * 2] = alpha_s[16 + r];
+      p.part_ml[(row * p.splits + split) * 2] = alpha_s[kRows + r];
       p.part_ml[(row * p.splits + split) * 2 + 1] = l;
     }
   }
+}
+
+template <int MT>
+int launch_latent_decode(const LatentDecodeParams& p, int T, cudaStream_t stream) {
+  const int smem = la_smem(p.R, MT);
+  if (smem > 227 * 1024) return -5;
+  static int allowed = 48 * 1024;
+  if (smem > allowed) {
+    if (cudaFuncSetAttribute(latent_decode_kernel<MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -6;
+    allowed = smem;
+  }
+  launch_kernel(latent_decode_kernel<MT>, dim3(T, (p.H + 16 * MT - 1) / (16 * MT), p.splits), dim3(kLaThreads), smem, stream, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -7;
 }
 
 struct LatentPlainParams {
@@ -420,17 +468,11 @@ extern "C" int mfq_latent_decode(const void* q, const void* kv, const int* table
                                  float* part, float* part_ml, int T_, int H, int rank, int rot, int max_pages, int window, float scale,
                                  int splits, cudaStream_t stream) {
   if (T_ <= 0 || !la_sizes(H, rank, rot) || rank > 128 * kLaMaxTiles || window <= 0 || splits < 1 || splits > 65535 || (splits > 1 && (!part || !part_ml))) return -1;
-  const int R = rank + rot, smem = la_smem(R);
-  if (smem > 227 * 1024) return -5;
-  static int allowed = 48 * 1024;
-  if (smem > allowed) {
-    if (cudaFuncSetAttribute(latent_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -6;
-    allowed = smem;
-  }
   const LatentDecodeParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(kv), table, tok_seq, lens,
-                             static_cast<__nv_bfloat16*>(out), part, part_ml, H, R, rank, max_pages, window, splits, len_add, scale * kLog2e};
-  launch_kernel(latent_decode_kernel, dim3(T_, (H + 15) / 16, splits), dim3(kLaThreads), smem, stream, p);
-  if (cudaGetLastError() != cudaSuccess) return -7;
+                             static_cast<__nv_bfloat16*>(out), part, part_ml, H, rank + rot, rank, max_pages, window, splits, len_add, scale * kLog2e};
+  const bool two = H > 16 && la_smem(rank + rot, 2) <= 227 * 1024;
+  const int rc = two ? launch_latent_decode<2>(p, T_, stream) : launch_latent_decode<1>(p, T_, stream);
+  if (rc) return rc;
   return splits > 1 ? launch_attn_merge(part, part_ml, static_cast<__nv_bfloat16*>(out), T_, H, splits, rank, stream) : 0;
 }
 

@@ -130,21 +130,28 @@ short_conv_kernel(const T* __restrict__ x, T* __restrict__ out, const ShortConvP
     if (i - (TAPS - p.taps) >= 0) load8<float>(p.w + size_t(i - (TAPS - p.taps)) * p.C + c, w[i]);
     if (i > 0) in(n0 + i - TAPS, win[i]);
   }
-  for (int n = n0; n < n1; ++n) {
+  constexpr int kAhead = 4;  // inputs requested before the first of them is used
+  for (int m = n0; m < n1; m += kAhead) {
+    float next[kAhead][8];
 #pragma unroll
-    for (int i = 0; i + 1 < TAPS; ++i)
+    for (int e = 0; e < kAhead; ++e)
+      if (m + e < n1) in(m + e, next[e]);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) win[i][j] = win[i + 1][j];
-    in(n, win[TAPS - 1]);
-    float y[8];
+    for (int e = 0; e < kAhead; ++e) {
+      if (m + e >= n1) break;
+      float y[8];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      float a = 0.f;
+      for (int j = 0; j < 8; ++j) {
 #pragma unroll
-      for (int i = 0; i < TAPS; ++i) a = fmaf(w[i][j], win[i][j], a);
-      y[j] = a / (1.f + expf(-a));
+        for (int i = 0; i + 1 < TAPS; ++i) win[i][j] = win[i + 1][j];
+        win[TAPS - 1][j] = next[e][j];
+        float a = 0.f;
+#pragma unroll
+        for (int i = 0; i < TAPS; ++i) a = fmaf(w[i][j], win[i][j], a);
+        y[j] = sizeof(T) == 4 ? a / (1.f + expf(-a)) : __fdividef(a, 1.f + __expf(-fmaxf(a, -80.f)));
+      }
+      store8<T>(out + size_t(r0 + m + e) * p.out_stride + c, y);
     }
-    store8<T>(out + size_t(r0 + n) * p.out_stride + c, y);
   }
   // Portions of one token: this thread is the only one that reads these kept inputs, so it may replace them.
   if (!p.starts) {

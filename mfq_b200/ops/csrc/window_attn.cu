@@ -301,21 +301,27 @@ window_attn_merge_kernel(const float* __restrict__ part, const float* __restrict
     const size_t row = (size_t(b) * p.heads + g * p.of_map) * p.maps + m * p.of_map + h - g * p.of_map;
     const float* ml = part_ml + row * p.splits * 2;
     float mt = -FLT_MAX, lt = 0.f;
+#pragma unroll 8
     for (int z = 0; z < p.splits; ++z) mt = fmaxf(mt, ml[z * 2]);
     if (p.sink) {
       mt = fmaxf(mt, p.sink[h] * kLog2e);
       lt = window_exp2(p.sink[h] * kLog2e - mt);
     }
-    for (int z = 0; z < p.splits; ++z) lt += ml[z * 2 + 1] * window_exp2(ml[z * 2] - mt);
+    float x[kCols] = {};
+#pragma unroll 4
+    for (int z = 0; z < p.splits; ++z) {
+      const float w = window_exp2(ml[z * 2] - mt);
+      lt = fmaf(ml[z * 2 + 1], w, lt);
+      const float* src = part + (row * p.splits + z) * p.dv;
+#pragma unroll
+      for (int i = 0; i < kCols; ++i) {
+        const int c = threadIdx.x + i * 128;
+        if (c < p.dv) x[i] = fmaf(src[c], w, x[i]);
+      }
+    }
     const float inv = (lt > 0.f ? 1.f / lt : 0.f) * (m == 0 ? 1.f : -p.lambda);
 #pragma unroll
-    for (int i = 0; i < kCols; ++i) {
-      const int c = threadIdx.x + i * 128;
-      if (c >= p.dv) continue;
-      float x = 0.f;
-      for (int z = 0; z < p.splits; ++z) x += part[(row * p.splits + z) * p.dv + c] * window_exp2(ml[z * 2] - mt);
-      y[i] += x * inv;
-    }
+    for (int i = 0; i < kCols; ++i) y[i] = fmaf(x[i], inv, y[i]);
   }
   float f = 1.f;
   if (p.maps == 2) f = rsqrtf(dense_block_sum(y[0] * y[0] + y[1] * y[1] + y[2] * y[2] + y[3] * y[3], red) * p.inv_d + p.eps) * p.scale;

@@ -35,8 +35,9 @@ def finish(proj: torch.Tensor, pages: torch.Tensor | None, positions, slots, *, 
 
 
 def decode_splits(batch: int, heads: int, keys: int) -> int:
-    """KV splits per (query token, 16 heads) over ``keys`` visible keys: enough CTAs for every SM, 128 keys each at least."""
-    n = max(1, batch * -(-heads // 16))
+    """KV splits per query token and CTA (up to 32 heads) over ``keys`` visible keys: about a CTA for every SM, 128 keys each at
+    least."""
+    n = max(1, batch * -(-heads // 32))
     return max(1, min(148 // n if n <= 148 else 1, keys // 128, 32))
 
 
