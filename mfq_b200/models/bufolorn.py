@@ -653,7 +653,7 @@ class BufolornModel(UnquantizedModel):
                                 step.tok_seq if prefill else None)
         proj = torch.empty((h.shape[0], geo.width), dtype=h.dtype, device=h.device)
         streams = 4 * geo.heads * geo.dk
-        w.rkvg(mixes, out=proj[:, :streams])
+        w.rkvg(mixes[:, : 4 * width], out=proj[:, :streams])
         w.decay_a(mixes[:, 4 * width :], softcap=1.0, out=proj[:, streams:])  # cap 1: tanh
         args = (proj, w.decay_b, w.decay_bias, w.norm, self.state.layer((i, "state")), step.state_slots, geo)
         if prefill:

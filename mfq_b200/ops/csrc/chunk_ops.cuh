@@ -53,4 +53,31 @@ __device__ __forceinline__ void gc_rows(__nv_bfloat16* dst, int pitch, const __n
     }
 }
 
+// z_tc = sum_r a_tr w_cr of a chunk's 64 tokens and the `dk` channels of a head: a [64][pitch] in shared memory, w [dk, rank] in global
+// memory, rank a multiple of 16.  store(t, c, z_tc, z_t(c+1)).
+template <int kWarps, typename Store>
+__device__ __forceinline__ void gc_low_rank(const __nv_bfloat16* a, int pitch, const __nv_bfloat16* w, int rank, int dk, int warp, int lane, Store&& store) {
+  const int g = lane >> 2, t4 = lane & 3, mat = lane >> 3, mrow = lane & 7;
+  const uint32_t frag = smem_u32(a + ((mat & 1) * 8 + mrow) * pitch + (mat >> 1) * 8);
+  for (int n0 = warp * 8; n0 < dk; n0 += kWarps * 8) {
+    const __nv_bfloat16* row = w + size_t(n0 + g) * rank + t4 * 2;
+    float acc[4][4] = {};
+#pragma unroll 4
+    for (int ks = 0; ks < rank / 16; ++ks) {
+      const uint32_t b0 = *reinterpret_cast<const uint32_t*>(row + ks * 16), b1 = *reinterpret_cast<const uint32_t*>(row + ks * 16 + 8);
+#pragma unroll
+      for (int mt = 0; mt < 4; ++mt) {
+        uint32_t f[4];
+        gc_ldm(frag + (mt * 16 * pitch + ks * 16) * 2, f);
+        gc_mma(acc[mt], f, b0, b1);
+      }
+    }
+#pragma unroll
+    for (int mt = 0; mt < 4; ++mt) {
+      store(mt * 16 + g, n0 + t4 * 2, acc[mt][0], acc[mt][1]);
+      store(mt * 16 + g + 8, n0 + t4 * 2, acc[mt][2], acc[mt][3]);
+    }
+  }
+}
+
 }  // namespace mfq

@@ -78,7 +78,7 @@ __host__ __device__ inline DeltaPrepareSmem dc_prepare_smem(int dk) {
   m.b = 0;                                   // [64][dk + 8] fp32
   m.q = m.b + kGc * (dk + 8) * 4;            // q, k [64][dk + 8] bf16
   m.k = m.q + kGc * (dk + 8) * 2;
-  m.l = m.k + kGc * (dk + 8) * 2;            // a^T [rank][68] fp32, then L [64][68] fp32
+  m.l = m.k + kGc * (dk + 8) * 2;            // a [64][rank + 8] bf16, then L [64][68] fp32
   m.misc = m.l + kGc * kDcLp * 4;            // iq, ik, beta [64], totals [256] fp32
   m.bytes = m.misc + (3 * kGc + kDcThreads) * 4;
   return m;
@@ -97,54 +97,41 @@ delta_chunk_prepare_kernel(const DeltaChunkParams p) {
   float* b_s = reinterpret_cast<float*>(dc_sm + m.b);
   __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(dc_sm + m.q);
   __nv_bfloat16* k_s = reinterpret_cast<__nv_bfloat16*>(dc_sm + m.k);
-  float* a_s = reinterpret_cast<float*>(dc_sm + m.l);
-  float* l_s = a_s;
+  __nv_bfloat16* a_s = reinterpret_cast<__nv_bfloat16*>(dc_sm + m.l);
+  float* l_s = reinterpret_cast<float*>(dc_sm + m.l);
   float* iq_s = reinterpret_cast<float*>(dc_sm + m.misc);
   float *ik_s = iq_s + kGc, *beta_s = ik_s + kGc, *tot = beta_s + kGc;
   const int bp = dk + 8, kp = dk + 8;
   const __nv_bfloat16* rows = p.conv + size_t(at.t0) * p.s.conv_stride;
   const __nv_bfloat16* side = p.side + size_t(at.t0) * p.s.side_stride;
+  gc_rows<kDcWarps>(a_s, rank + 8, side + p.s.b_cols, p.s.side_stride, rank, at.n, warp, lane);
+  gc_commit();
   gc_rows<kDcWarps>(q_s, kp, rows + kh * dk, p.s.conv_stride, dk, at.n, warp, lane);
   gc_rows<kDcWarps>(k_s, kp, rows + (G + kh) * dk, p.s.conv_stride, dk, at.n, warp, lane);
   gc_commit();
+  if (tid < kGc) beta_s[tid] = tid < at.n ? delta_sigmoid(__bfloat162float(side[size_t(tid) * p.s.side_stride + h])) : 0.f;
+  gc_wait<1>();
+  __syncthreads();
+  // ----- decays, then their running sum: a thread takes one key channel of 64 / TG tokens -----
   {
-    const int aper = rank / 8;
-    for (int i = tid; i < kGc * aper; i += kDcThreads) {
-      const int t = i / aper, r = (i - t * aper) * 8;
-      float x[8] = {};
-      if (t < at.n) load8<__nv_bfloat16>(side + size_t(t) * p.s.side_stride + p.s.b_cols + r, x);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) a_s[(r + j) * kDcLp + t] = x[j];
-    }
-    if (tid < kGc) beta_s[tid] = tid < at.n ? delta_sigmoid(__bfloat162float(side[size_t(tid) * p.s.side_stride + h])) : 0.f;
+    const float rate = -1.4426950408889634f * p.rate[h];
+    const float* dt = p.dt_bias + h * dk;
+    gc_low_rank<kDcWarps>(a_s, rank + 8, p.w_a2 + size_t(h) * dk * rank, rank, dk, warp, lane, [&](int t, int c, float x, float y) {
+      const float2 bias = *reinterpret_cast<const float2*>(dt + c);
+      const bool in = t < at.n;
+      *reinterpret_cast<float2*>(b_s + t * bp + c) = make_float2(in ? fmaxf(rate * dc_softplus(x + bias.x), kGlaFloor) : 0.f,
+                                                                 in ? fmaxf(rate * dc_softplus(y + bias.y), kGlaFloor) : 0.f);
+    });
   }
   __syncthreads();
-  // ----- decays: a thread takes one key channel of 64 / TG tokens -----
   const int TG = dk <= 32 ? 8 : dk <= 64 ? 4 : 2, len = kGc / TG, c = tid % dk, tg = tid / dk;
   const bool live = tg < TG;
   if (live) {
-    const __nv_bfloat16* w = p.w_a2 + size_t(h * dk + c) * rank;
-    const float bias = p.dt_bias[h * dk + c], rate = -1.4426950408889634f * p.rate[h];
     float run = 0.f;
-    for (int t = tg * len; t < tg * len + len; t += 8) {
-      float z[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) z[j] = bias;
-      for (int r = 0; r < rank; r += 8) {
-        float x[8];
-        load8<__nv_bfloat16>(w + r, x);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const float4 lo = *reinterpret_cast<const float4*>(a_s + (r + e) * kDcLp + t), hi = *reinterpret_cast<const float4*>(a_s + (r + e) * kDcLp + t + 4);
-          z[0] = fmaf(x[e], lo.x, z[0]); z[1] = fmaf(x[e], lo.y, z[1]); z[2] = fmaf(x[e], lo.z, z[2]); z[3] = fmaf(x[e], lo.w, z[3]);
-          z[4] = fmaf(x[e], hi.x, z[4]); z[5] = fmaf(x[e], hi.y, z[5]); z[6] = fmaf(x[e], hi.z, z[6]); z[7] = fmaf(x[e], hi.w, z[7]);
-        }
-      }
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        run += t + j < at.n ? fmaxf(rate * dc_softplus(z[j]), kGlaFloor) : 0.f;
-        b_s[(t + j) * bp + c] = run;
-      }
+#pragma unroll 8
+    for (int t = tg * len; t < tg * len + len; ++t) {
+      run += b_s[t * bp + c];
+      b_s[t * bp + c] = run;
     }
     tot[tg * dk + c] = run;
   }
@@ -224,7 +211,7 @@ delta_chunk_prepare_kernel(const DeltaChunkParams p) {
         }
       }
     }
-    // (the last reader of a^T is behind a barrier: L may take its place)
+    // (the last reader of a is behind a barrier: L may take its place)
 #pragma unroll
     for (int jj = 0; jj < 2; ++jj)
       if (J0 + jj < J1)
@@ -534,32 +521,40 @@ delta_chunk_scan_kernel(const DeltaChunkParams p) {
   }
 }
 
-// y = rms_norm(o) * w * sigmoid(gate); a warp per (token, head)
+// y = rms_norm(o) * w * sigmoid(gate); L lanes (a power of two) per (token, head)
 __global__ void __launch_bounds__(256)
 delta_norm_gate_kernel(const float* __restrict__ o, const __nv_bfloat16* __restrict__ gate, const float* __restrict__ norm_w,
-                       __nv_bfloat16* __restrict__ y, int pairs, int dv, float inv_dv, float eps) {
+                       __nv_bfloat16* __restrict__ y, int pairs, int dv, int L, float inv_dv, float eps) {
   pdl_trigger();
   pdl_wait();
-  const int pair = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (pair >= pairs) return;
-  const size_t at = size_t(pair) * dv;
-  float ss = 0.f, v[8];
-  for (int c = lane * 8; c < dv; c += 256) {
-    load8<float>(o + at + c, v);
+  const int pair = (blockIdx.x * 256 + threadIdx.x) / L, lane = threadIdx.x & (L - 1);
+  const bool live = pair < pairs;
+  const size_t at = size_t(live ? pair : 0) * dv;
+  constexpr int kMost = 4;  // 8-wide vectors per lane: values up to 1024 wide
+  float v[kMost][8], ss = 0.f;
 #pragma unroll
-    for (int j = 0; j < 8; ++j) ss += v[j] * v[j];
+  for (int i = 0; i < kMost; ++i) {
+    const int c = (lane + i * L) * 8;
+    if (c < dv) {
+      load8<float>(o + at + c, v[i]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss += v[i][j] * v[i][j];
+    }
   }
-#pragma unroll
-  for (int i = 16; i > 0; i >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, i);
+  for (int i = L >> 1; i > 0; i >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, i);
+  if (!live) return;
   const float f = rsqrtf(ss * inv_dv + eps);
-  for (int c = lane * 8; c < dv; c += 256) {
-    float w[8], z[8];
-    load8<float>(o + at + c, v);
-    load8<__nv_bfloat16>(gate + at + c, z);
-    load8<float>(norm_w + c, w);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) v[j] *= f * w[j] * delta_sigmoid(z[j]);
-    store8<__nv_bfloat16>(y + at + c, v);
+  for (int i = 0; i < kMost; ++i) {
+    const int c = (lane + i * L) * 8;
+    if (c < dv) {
+      float w[8], z[8];
+      load8<__nv_bfloat16>(gate + at + c, z);
+      load8<float>(norm_w + c, w);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[i][j] *= f * w[j] * __fdividef(1.f, 1.f + __expf(-fmaxf(z[j], -80.f)));
+      store8<__nv_bfloat16>(y + at + c, v[i]);
+    }
   }
 }
 
@@ -583,7 +578,7 @@ extern "C" int mfq_delta_chunk(const void* conv, const void* side, const void* w
   if (B <= 0 || B > 65535 || max_q <= 0 || H <= 0 || H > 65535 || G <= 0 || H % G || dk <= 0 || dv <= 0 || dk % 16 || dv % 16 || real_dv <= 0 || real_dv > dv) return -1;
   if (b_cols < H || b_cols % 8 || ra <= 0 || ra % 8 || conv_stride % 8 || side_stride % 8 || conv_stride < 2 * G * dk + H * dv || chunks <= 0 || count <= 0) return -1;
   const int prep = dc_prepare_smem(dk).bytes, scan = dc_scan_smem(dk).bytes;
-  if (dk > kDcMaxDk || ra > kDcMaxRank || scan > 227 * 1024) return -5;
+  if (dk > kDcMaxDk || dv > 1024 || ra > kDcMaxRank || ra % 16 || scan > 227 * 1024) return -5;
   const size_t tiles = size_t(chunks) * H;
   __nv_bfloat16* wq = static_cast<__nv_bfloat16*>(scratch);
   __nv_bfloat16* kp = wq + tiles * dc_wq(dk);
@@ -604,7 +599,9 @@ extern "C" int mfq_delta_chunk(const void* conv, const void* side, const void* w
   launch_kernel(delta_chunk_scan_kernel, dim3((dv + kDcNs - 1) / kDcNs, H, B), dim3(kDcThreads), scan, stream, p);
   const long long pairs = (long long)(count) * H;
   const size_t skip = size_t(first) * H * dv;
-  launch_kernel(delta_norm_gate_kernel, dim3(unsigned((pairs + 7) / 8)), dim3(256), 0, stream, o_raw + skip, static_cast<const __nv_bfloat16*>(gate) + skip,
-                norm_w, static_cast<__nv_bfloat16*>(y) + skip, int(pairs), dv, 1.f / float(real_dv), eps);
+  int lanes = 1;
+  while (lanes * 8 < dv && lanes < 32) lanes *= 2;
+  launch_kernel(delta_norm_gate_kernel, dim3(unsigned((pairs * lanes + 255) / 256)), dim3(256), 0, stream, o_raw + skip, static_cast<const __nv_bfloat16*>(gate) + skip,
+                norm_w, static_cast<__nv_bfloat16*>(y) + skip, int(pairs), dv, lanes, 1.f / float(real_dv), eps);
   return cudaGetLastError() == cudaSuccess ? 0 : -7;
 }

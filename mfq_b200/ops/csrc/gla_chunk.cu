@@ -74,8 +74,8 @@ struct GlaLocalSmem {
 __host__ __device__ inline GlaLocalSmem gc_local_smem(int dk, int dv, int rank) {
   GlaLocalSmem m{};
   m.b = 0;                                                   // [64][dk + 8] fp32
-  m.k = m.b + kGc * (dk + 8) * 4;                            // a^T [rank][68] fp32, then hi [64][dk + 8] bf16
-  const int half = kGc * (dk + 8) * 2, abytes = rank * 68 * 4;
+  m.k = m.b + kGc * (dk + 8) * 4;                            // a [64][rank + 8] bf16, then hi [64][dk + 8] bf16
+  const int half = kGc * (dk + 8) * 2, abytes = kGc * (rank + 8) * 2;
   m.lo = m.k + (half > abytes ? half : abytes);              // k, then lo [64][dk + 8] bf16
   m.v = m.lo + half;                                         // [64][dv + 8] bf16
   m.tot = m.v + kGc * (dv + 8) * 2;                          // [512] fp32
@@ -94,55 +94,39 @@ gla_chunk_local_kernel(const GlaChunkParams p) {
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const GlaLocalSmem m = gc_local_smem(dk, dv, rank);
   float* b_s = reinterpret_cast<float*>(gc_sm + m.b);
-  float* a_s = reinterpret_cast<float*>(gc_sm + m.k);
+  __nv_bfloat16* a_s = reinterpret_cast<__nv_bfloat16*>(gc_sm + m.k);
   __nv_bfloat16* k_hi = reinterpret_cast<__nv_bfloat16*>(gc_sm + m.k);
   __nv_bfloat16* v_s = reinterpret_cast<__nv_bfloat16*>(gc_sm + m.v);
   float* tot = reinterpret_cast<float*>(gc_sm + m.tot);
   const int bp = dk + 8, kp = dk + 8, vp = dv + 8;
   __nv_bfloat16* k_lo = reinterpret_cast<__nv_bfloat16*>(gc_sm + m.lo);
   const __nv_bfloat16* rows = p.proj + size_t(at.t0) * p.s.row_stride;
+  gc_rows<kGcWarps>(a_s, rank + 8, rows + 2 * H * (dk + dv), p.s.row_stride, rank, at.n, warp, lane);
+  gc_commit();
+  gc_rows<kGcWarps>(k_lo, kp, rows + (H + h) * dk, p.s.row_stride, dk, at.n, warp, lane);
+  gc_commit();
+  gc_rows<kGcWarps>(v_s, vp, rows + 2 * H * dk + h * dv, p.s.row_stride, dv, at.n, warp, lane);
+  gc_commit();
+  gc_wait<2>();
+  __syncthreads();
+  // ----- decays, then their running sum: a thread takes one key channel of 64 / TG tokens -----
   {
-    gc_rows<kGcWarps>(k_lo, kp, rows + (H + h) * dk, p.s.row_stride, dk, at.n, warp, lane);
-    gc_commit();
-    gc_rows<kGcWarps>(v_s, vp, rows + 2 * H * dk + h * dv, p.s.row_stride, dv, at.n, warp, lane);
-    gc_commit();
-    const __nv_bfloat16* a = rows + 2 * H * (dk + dv);
-    const int aper = rank / 8;
-    for (int i = tid; i < kGc * aper; i += kGcThreads) {
-      const int t = i / aper, r = (i - t * aper) * 8;
-      float x[8] = {};
-      if (t < at.n) load8<__nv_bfloat16>(a + size_t(t) * p.s.row_stride + r, x);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) a_s[(r + j) * 68 + t] = x[j];
-    }
+    const float* bias = p.bias + h * dk;
+    gc_low_rank<kGcWarps>(a_s, rank + 8, p.w2 + size_t(h) * dk * rank, rank, dk, warp, lane, [&](int t, int c, float x, float y) {
+      const float2 add = *reinterpret_cast<const float2*>(bias + c);
+      const bool in = t < at.n;
+      *reinterpret_cast<float2*>(b_s + t * bp + c) = make_float2(in ? gc_log2_decay(p.s, x + add.x) : 0.f, in ? gc_log2_decay(p.s, y + add.y) : 0.f);
+    });
   }
   __syncthreads();
-  // ----- decays: a thread takes one key channel of 64 / TG tokens -----
   const int TG = gc_groups(dk), len = kGc / TG, c = tid % dk, tg = tid / dk;
   const bool live = tg < TG;
   if (live) {
-    const __nv_bfloat16* w = p.w2 + size_t(h * dk + c) * rank;
-    const float bias = p.bias[h * dk + c];
     float run = 0.f;
-    for (int t = tg * len; t < tg * len + len; t += 8) {
-      float z[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) z[j] = bias;
-      for (int r = 0; r < rank; r += 8) {
-        float x[8];
-        load8<__nv_bfloat16>(w + r, x);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const float4 lo = *reinterpret_cast<const float4*>(a_s + (r + e) * 68 + t), hi = *reinterpret_cast<const float4*>(a_s + (r + e) * 68 + t + 4);
-          z[0] = fmaf(x[e], lo.x, z[0]); z[1] = fmaf(x[e], lo.y, z[1]); z[2] = fmaf(x[e], lo.z, z[2]); z[3] = fmaf(x[e], lo.w, z[3]);
-          z[4] = fmaf(x[e], hi.x, z[4]); z[5] = fmaf(x[e], hi.y, z[5]); z[6] = fmaf(x[e], hi.z, z[6]); z[7] = fmaf(x[e], hi.w, z[7]);
-        }
-      }
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        run += t + j < at.n ? gc_log2_decay(p.s, z[j]) : 0.f;
-        b_s[(t + j) * bp + c] = run;
-      }
+#pragma unroll 8
+    for (int t = tg * len; t < tg * len + len; ++t) {
+      run += b_s[t * bp + c];
+      b_s[t * bp + c] = run;
     }
     tot[tg * dk + c] = run;
   }
@@ -543,7 +527,7 @@ extern "C" int mfq_gla_chunk(const void* proj, const void* w2, const float* bias
   if (B <= 0 || B > 65535 || max_q <= 0 || H <= 0 || H > 65535 || dk <= 0 || dv <= 0 || dk % 16 || dv % 16 || rank <= 0 || rank % 8) return -1;
   if (real_dv <= 0 || real_dv > dv || row_stride < 2 * H * (dk + dv) + rank || row_stride % 8) return -1;
   const int local = gc_local_smem(dk, dv, rank).bytes;
-  if (dk > kGcMaxDk || dv > kGcMaxDv || local > 227 * 1024 || gc_output_smem(dk, dv).bytes > 227 * 1024) return -5;
+  if (rank % 16 || dk > kGcMaxDk || dv > kGcMaxDv || local > 227 * 1024 || gc_output_smem(dk, dv).bytes > 227 * 1024) return -5;
   const GlaChunkParams p{GlaShape{H, dk, dv, rank, row_stride, scale, inv_tau, 1.f / float(real_dv), eps, decay, norm_stride, bonus}, static_cast<const __nv_bfloat16*>(proj),
                          static_cast<const __nv_bfloat16*>(w2), bias, norm_w, static_cast<__nv_bfloat16*>(y), starts, slot, state, cum, u, gam};
   const dim3 grid((max_q + kGc - 1) / kGc, H, B);

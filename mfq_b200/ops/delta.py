@@ -56,7 +56,7 @@ class Geometry:
 
     @property
     def chunkable(self) -> bool:
-        return self.dk <= CHUNK_MAX_DK and self.rank_a <= CHUNK_MAX_RANK
+        return self.dk <= CHUNK_MAX_DK and self.dv <= 1024 and self.rank_a <= CHUNK_MAX_RANK and self.rank_a % 16 == 0
 
     def chunk_bytes(self) -> int:
         """Scratch per chunk and head."""

@@ -86,8 +86,8 @@ class DenseLinear:
         ``fp32``: the result stays fp32.  Groups: matrix g reads ``x`` from column ``g * x_step`` (by default ``cols``) and writes
         ``out`` from column ``g * out_step`` (by default ``out_width``)."""
         m, n, k, g = x.shape[0], self.w.shape[0] // self.groups, self.w.shape[1], self.groups
+        assert x.shape[1] == g * k if x_step is None else x.shape[1] >= (g - 1) * x_step + k
         x_step, out_step = k if x_step is None else x_step, self.out_width if out_step is None else out_step
-        assert x.shape[1] >= (g - 1) * x_step + k and (g > 1 or x.shape[1] == k)
         assert x.stride(1) == 1 and x.dtype == self.w.dtype and self.w.is_contiguous()
         width = (g - 1) * out_step + self.out_width
         if add_to is not None:

@@ -55,7 +55,7 @@ class Geometry:
 
     @property
     def chunkable(self) -> bool:
-        return self.dk <= 256 and self.dv <= 512 and self.rank <= 64
+        return self.dk <= 256 and self.dv <= 512 and self.rank <= 64 and self.rank % 16 == 0
 
 
 def _space(name: str, floats: int, device) -> torch.Tensor:

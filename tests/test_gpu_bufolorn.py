@@ -45,8 +45,14 @@ def parallel_only():
     return cases.config([cases.parallel(mlp=cases.dense(40)), cases.parallel(heads=20, kv_heads=1, dim=64, vdim=64, rheads=1, rdim=64, bias_max=33, scale=0.2)])
 
 
+def one_head():
+    """A single head of everything."""
+    return cases.config([cases.latent(heads=1, mlp=cases.moe(experts=1, top=1)), cases.delta(heads=1, kv_heads=1), cases.parallel(heads=1, kv_heads=1, rheads=1),
+                         cases.latent(heads=1, kv_from=0)])
+
+
 @BOTH
-@pytest.mark.parametrize("make", [cases.uneven, latent_only, recurrent_only, parallel_only])
+@pytest.mark.parametrize("make", [cases.uneven, latent_only, recurrent_only, parallel_only, one_head])
 def test_whole_prompts_and_every_layer(tmp_path, make, dtype):
     cfg = make()
     w, toks = cases.weights(cfg), cases.tokens(cfg, 150)

@@ -53,7 +53,7 @@ def test_output_stages(m, n, k, dtype):
 
 @BOTH
 @pytest.mark.parametrize("m", [1, 5, 12, 40, 200])
-@pytest.mark.parametrize("g,n,k,x_step,out_step", [(3, 48, 32, 56, 64), (5, 16, 8, 8, 16), (4, 144, 72, 72, 144), (2, 256, 136, 200, 272)])
+@pytest.mark.parametrize("g,n,k,x_step,out_step", [(1, 32, 48, 64, 48), (3, 48, 32, 56, 64), (5, 16, 8, 8, 16), (4, 144, 72, 72, 144), (2, 256, 136, 200, 272)])
 def test_a_matrix_per_head(m, g, n, k, x_step, out_step, dtype):
     from mfq_b200.ops import dense
     x, w, b = rnd(m, (g - 1) * x_step + k + 8, dtype=dtype), rnd(g * n, k, dtype=dtype, scale=k ** -0.5), rnd(g * n, dtype=FP32)
