@@ -8,8 +8,8 @@ Per head, with a fp32 state ``S [dk, dv]`` carried from token to token:
 or, with a bonus ``u`` (time mixing), ``o_t = (S + diag(u) k_t v_t^T)^T (q_t scale)`` from the state before the write.  The decay may
 instead be ``exp(-exp(W_a2 a_t + bias))``, and every head may have norm weights of its own.
 
-A token's projections are one row ``[q: H dk | k: H dk | v: H dv | gate: H dv | a: rank]`` (widths stored as multiples of 16,
-the rank of 8).  bf16 portions of prompts run in 64-token chunks, single tokens, short portions and fp32 token by token.
+A token's projections are one row ``[q: H dk | k: H dk | v: H dv | gate: H dv | a: rank]`` (widths and the
+rank stored as multiples of 16).  bf16 portions of prompts run in 64-token chunks, single tokens, short portions and fp32 token by token.
 """
 
 from __future__ import annotations

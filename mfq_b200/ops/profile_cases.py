@@ -237,7 +237,23 @@ def gla_case(tokens: int, batch: int) -> None:
             gla.chunked(proj, w2, bias, norm, state, slots, geo, starts, tokens)
 
 
-CASES = {"two_maps_decode": two_maps_decode, "two_maps_prefill": two_maps_prefill, "gla_decode": lambda: gla_case(1, 64),
+def latent_case(batch: int) -> None:
+    """32 heads over latents of 512 + 64 channels, windows of 1024 in 4096 tokens: a decode step of `batch` sequences, or (0) a prompt of
+    2048 tokens over expanded rows."""
+    from . import bench_kernels
+    bench_kernels.time_ms = lambda fn, reps, warmup=3: [fn(i) for i in range(3)] and 1.0
+    bench_kernels.bench_latent(batch, 4096 if batch else 2048, 32, 1024, 3)
+
+
+def delta_case(tokens: int, batch: int) -> None:
+    """32 heads with a 128 x 128 state on 16 key heads: a prompt of `tokens` tokens in chunks, or (tokens 1) a decode step."""
+    from . import bench_kernels
+    bench_kernels.time_ms = lambda fn, reps, warmup=3: [fn(i) for i in range(3)] and 1.0
+    bench_kernels.bench_delta(batch, tokens, 32, 16, 128, 3)
+
+
+CASES = {"latent_decode": lambda: latent_case(64), "latent_prefill": lambda: latent_case(0), "delta_decode": lambda: delta_case(1, 64),
+         "delta_prefill": lambda: delta_case(2048, 1), "two_maps_decode": two_maps_decode, "two_maps_prefill": two_maps_prefill, "gla_decode": lambda: gla_case(1, 64),
          "gla_prefill": lambda: gla_case(2048, 1), "gemm_prefill": lambda: gemm(4096, 4096, 4096), "gemm_decode": lambda: gemm(64, 28672, 4096),
          "gemm_decode_splitk": lambda: gemm(64, 4096, 14336),
          "attn_decode": attn_decode, "attn_prefill": attn_prefill, "w4_decode": lambda: w4_gemm(64, 28672, 4096),

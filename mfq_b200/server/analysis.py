@@ -23,6 +23,7 @@ from pathlib import Path
 
 GROUPS = (("predictor", "predictor."), ("routed_experts", ".mlp.experts."), ("shared_experts", ".mlp.shared_expert"),
           ("router", ".mlp.router"), ("attention", ".attention."), ("linear_attention", ".linear_attention."),
+          ("time_mixing", ".time_mixing."),
           ("dense_mlp", ".mlp."), ("embeddings", "token_embedding"), ("head", "model.output.weight"), ("norms", "norm"))
 
 
@@ -121,7 +122,10 @@ def model_parameters(cfg: dict) -> dict:
         for name, shape in own[1].items():
             groups[group_of(name)] = groups.get(group_of(name), 0) + math.prod(shape)
         total = sum(groups.values())
-        return {"groups": groups, "total": total, "active_per_token": total, "experts": None, "top_k": None, "layers": own[0].num_layers,
+        moe = [l.mlp for l in own[0].layers if getattr(getattr(l, "mlp", None), "experts", 0)]
+        idle = sum((m.experts - m.top) * 3 * m.ff * own[0].hidden_size for m in moe)
+        return {"groups": groups, "total": total, "active_per_token": total - idle, "experts": max((m.experts for m in moe), default=None),
+                "top_k": max((m.top for m in moe), default=None), "layers": own[0].num_layers,
                 "attention_layers": getattr(own[0], "attention_layers", len(own[0].key_spans()))}
     h = _cfg_int(cfg, "hidden_size")
     layers = _cfg_int(cfg, "num_layers", "num_hidden_layers")

@@ -292,7 +292,10 @@ def test_memory_of_a_deployment_counts_pages_and_state():
     got = model_memory(cfg, 1000, batch=2, context=64)["per_gpu"]
     assert got["kv_cache"] == (2 * 4 + 1) * 16 * 2 * (64 + 2 * 64 + 64 + 80)
     assert got["recurrent_state"] == 2 * own.state_bytes() and own.state_bytes() == 4 * sum(int(np.prod(s)) for s in own.state_shapes().values())
-    assert model_parameters(cfg)["attention_layers"] == 6
+    counts = model_parameters(cfg)
+    assert counts["attention_layers"] == 6 and counts["experts"] == 7 and counts["top_k"] == 3
+    assert counts["total"] - counts["active_per_token"] == 3 * 104 * 40 * ((7 - 3) + (5 - 1) + (7 - 3))
+    assert counts["groups"]["time_mixing"] > 0 and "other" not in counts["groups"]
 
 
 def test_quantization_keeps_what_is_not_a_projection():
