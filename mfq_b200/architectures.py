@@ -8,7 +8,7 @@ Runtime code consumes canonical names only (``model.block.N.attention.query.weig
 * ``deepseek_v3`` / ``glm4_moe``: latent-attention and shared-expert names, sigmoid router bias, and the next-token
   prediction layer these checkpoints append after the last decoder layer (``model.layers.<L>.{enorm,hnorm,eh_proj,
   shared_head.*}``), which becomes the ``predictor.*`` head;
-* ``tepetar``, ``kamedra``, ``bufolorn``: ``l<N>.{mix,mlp,side}.*`` names (``config.json`` names the design under ``architecture``).
+* ``tepetar``, ``kamedra``, ``bufolorn``, ``gogivik``: ``l<N>.{mix,mlp,side}.*`` names (``config.json`` names the design under ``architecture``).
 
 :func:`detect_family` picks the family from ``config.json`` (``model_type`` / ``architectures``); :func:`to_canonical`
 renames, stacks per-expert matrices, splits fused tensors and moves the appended prediction layer.  Names match the
@@ -161,6 +161,22 @@ BUFOLORN_MIXER = {
     },
 }
 _OWN_EXPERT_RE = re.compile(r"^mlp\.e(\d+)\.(gate|up|down)$")
+# Gogivik: the same short names
+GOGIVIK_TOP = {"embed": "model.token_embedding.weight", "final.norm": "model.output_norm.weight", "head": "model.output.weight"}
+GOGIVIK_LAYER = {
+    "norm1": "attention.norm.weight", "canon1": "attention.input_conv.weight", "norm2": "mlp.norm.weight", "canon2": "mlp.input_conv.weight",
+    "mlp.up": "mlp.up.weight", "mlp.down": "mlp.down.weight",
+}
+GOGIVIK_MIXER = {
+    "latent_attention": {"dq": "attention.query_down.weight", "dq.norm": "attention.query_norm.weight", "uq": "attention.query.weight",
+                         "dkv": "attention.latent.weight", "dkv.norm": "attention.latent_norm.weight", "uk": "attention.key_up.weight",
+                         "uv": "attention.value_up.weight", "sink": "attention.sink", "o": "attention.output.weight"},
+    "attention": {**{k: f"attention.{n}.weight" for k, n in (("q", "query"), ("k", "key"), ("v", "value"), ("o", "output"))},
+                  "q.norm": "attention.query_norm.weight", "k.norm": "attention.key_norm.weight"},
+    "mamba2": {"in": "linear_attention.in.weight", "conv": "linear_attention.in_conv.weight", "conv.b": "linear_attention.in_conv.bias",
+               "dt_bias": "linear_attention.dt_bias", "A_log": "linear_attention.a", "D": "linear_attention.skip",
+               "norm": "linear_attention.norm.weight", "o": "linear_attention.output.weight"},
+}
 _OWN_LAYER_RE = re.compile(r"^l(\d+)\.(.+)$")
 FAMILY_OF_MODEL_TYPE = {
     "llama": "llama", "mistral": "llama", "qwen2": "llama", "qwen3": "llama", "mixtral": "llama", "qwen2_moe": "llama",
@@ -174,7 +190,7 @@ def detect_family(hf_config: dict | None, names=()) -> str:
     """Source naming family of a checkpoint: from ``model_type`` (or the text sub-config's), else from its tensor names."""
     cfg = hf_config or {}
     own = str(cfg.get("architecture", "")).lower()
-    if own in ("tepetar", "kamedra", "bufolorn"):
+    if own in ("tepetar", "kamedra", "bufolorn", "gogivik"):
         return own
     for c in (cfg, cfg.get("text_config") or {}):
         fam = FAMILY_OF_MODEL_TYPE.get(str(c.get("model_type", "")).lower())
@@ -266,6 +282,17 @@ def bufolorn_name(name: str, mixers: list[str]) -> tuple[str, int | None] | None
     return (block + known[m[2]], None) if m[2] in known else None
 
 
+def gogivik_name(name: str, mixers: list[str]) -> str | None:
+    """Source name of a Gogivik tensor -> canonical name (None: not part of the model); ``mixers``: the kind of every layer."""
+    if name in GOGIVIK_TOP:
+        return GOGIVIK_TOP[name]
+    m = _OWN_LAYER_RE.match(name)
+    if not m or int(m[1]) >= len(mixers):
+        return None
+    known = GOGIVIK_LAYER | {"mix." + k: v for k, v in GOGIVIK_MIXER.get(mixers[int(m[1])], {}).items()}
+    return f"model.block.{int(m[1])}.{known[m[2]]}" if m[2] in known else None
+
+
 def split_fused_linear_attention(out: dict[str, np.ndarray], k_heads: int, v_heads: int, head_dim: int) -> None:
     """The hybrid family's fused projections, in place: ``in_proj_qkvz`` holds, per KEY head, the rows
     ``[q (d) | k (d) | v (r d) | z (r d)]`` with ``r = v_heads / k_heads``; ``in_proj_ba`` holds ``[b (r) | a (r)]`` per
@@ -314,9 +341,9 @@ def to_canonical(hf_tensors: dict[str, np.ndarray], hf_config: dict | None = Non
     family = detect_family(hf_config, hf_tensors)
     if family == "tepetar":
         return {c: t for c, t in ((tepetar_name(n), t) for n, t in hf_tensors.items()) if c is not None}
-    if family == "kamedra":
-        mixers = [l.get("type") for l in hf_config["layers"]]
-        return {c: t for c, t in ((kamedra_name(n, mixers), t) for n, t in hf_tensors.items()) if c is not None}
+    if family in ("kamedra", "gogivik"):
+        rename, mixers = {"kamedra": kamedra_name, "gogivik": gogivik_name}[family], [l.get("type") for l in hf_config["layers"]]
+        return {c: t for c, t in ((rename(n, mixers), t) for n, t in hf_tensors.items()) if c is not None}
     if family == "bufolorn":
         mixers = [l.get("type") for l in hf_config["layers"]]
         return _renamed_and_stacked(hf_tensors, lambda n: bufolorn_name(n, mixers))
@@ -365,6 +392,9 @@ def config_from_hf(hf: dict) -> dict:
     if family == "bufolorn":
         from .models.bufolorn import BufolornConfig
         return BufolornConfig.from_source(hf).to_dict()
+    if family == "gogivik":
+        from .models.gogivik import GogivikConfig
+        return GogivikConfig.from_source(hf).to_dict()
     if hf.get("text_config"):
         hf = {**hf, **hf["text_config"]}
     heads = hf.get("num_attention_heads", 32)

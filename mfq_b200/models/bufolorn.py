@@ -23,15 +23,15 @@ from dataclasses import asdict, dataclass, field
 
 import torch
 
-from ..engine.recurrent_state import LayerStates
-from ..ops import delta, dense, dense_moe, gla, latent_attn, window_attn
+from ..ops import delta, dense, dense_moe, gla, window_attn
 from ..ops.dense import DenseLinear, up
 from ..ops.window_attn import NO_WINDOW, DistanceBias
 from ..utils.profiler import scope
-from . import unquantized
+from . import latent, unquantized
+from .latent import LatentUp
 from .llama import StepBuffers
 from .rope_scaling import YarnScaling
-from .unquantized import TensorReader, UnquantizedModel, fit
+from .unquantized import RecurrentModel, TensorReader, fit
 
 
 @dataclass(frozen=True)
@@ -167,12 +167,7 @@ class BufolornConfig:
     def _check(self, i: int, l: LayerSpec) -> None:
         m = l.mixer
         if l.kind == "latent_attention":
-            if min(m.heads, m.dim, m.vdim, m.kv_rank) < 1 or m.rot_dim < 0 or m.rot_dim % 2 or not m.scale > 0 or m.window < 1:
-                raise ValueError(f"unsupported latent attention {m}")
-            if up(m.kv_rank) > latent_attn.MAX_RANK or m.row > latent_attn.MAX_ROW:
-                raise ValueError(f"latents above {latent_attn.MAX_RANK} channels are not supported")
-            if up(m.dim) + up(m.rot_dim) > window_attn.MAX_HEAD or m.vdim > window_attn.MAX_HEAD:
-                raise ValueError(f"heads above {window_attn.MAX_HEAD} channels are not supported")
+            latent.check_sizes(m)
             if m.kv_from is not None:
                 src = self.layers[m.kv_from].mixer if 0 <= m.kv_from < i else None
                 if not isinstance(src, LatentSpec) or src.kv_from is not None:
@@ -391,9 +386,7 @@ class RandomTensors(unquantized.RandomTensors):
 class LatentWeights:
     proj: DenseLinear  # rows [head][dim | rot], then [latent | rot] in a layer with pages of its own
     norm: torch.Tensor | None  # [rank] fp32
-    absorb: DenseLinear  # per head [rank, dim]: queries into latent space
-    value_up: DenseLinear  # per head [vdim, rank]
-    expand: torch.Tensor | None  # per head [dim | rot | vdim, rank + rot]: a row of the cache to keys and values (bf16)
+    up: LatentUp
     o_proj: DenseLinear
 
 
@@ -471,26 +464,14 @@ class BufolornWeights:
     @staticmethod
     def _latent(r: TensorReader, cfg: BufolornConfig, m: LatentSpec, p: str, w: int) -> LatentWeights:
         p += "attention."
-        h, d, rot, e, rank = m.heads, up(m.dim), up(m.rot_dim), up(m.vdim), up(m.kv_rank)
-        q = r.get(p + "query.weight").to(r.dtype).reshape(h, m.dim + m.rot_dim, cfg.hidden_size)
-        parts = [torch.cat([fit(q[:, : m.dim], h, d, w), fit(q[:, m.dim :], h, rot, w)], 1).reshape(-1, w)]
-        norm = None
+        rot, rank = up(m.rot_dim), up(m.kv_rank)
+        parts, norm = [latent.head_rows(r.get(p + "query.weight").to(r.dtype), m, w)], None
         if m.kv_from is None:
             c = r.get(p + "latent.weight").to(r.dtype)
             parts += [fit(c[: m.kv_rank], rank, w), fit(c[m.kv_rank :], rot, w)]
             norm = r.vec(p + "latent_norm.weight", rank)
-        uk = r.heads(p + "key_up.weight", h, m.dim, d, m.kv_rank, rank)
-        uv = r.heads(p + "value_up.weight", h, m.vdim, e, m.kv_rank, rank)
-        expand = None
-        if r.dtype == torch.bfloat16:
-            expand = torch.zeros((h, d + rot + e, rank + rot), dtype=r.dtype, device=r.device)
-            expand[:, :d, :rank], expand[:, d + rot :, :rank] = uk, uv
-            expand[:, d : d + rot, rank:] = torch.eye(rot, dtype=r.dtype, device=r.device)
-            expand = expand.reshape(-1, rank + rot)
-        return LatentWeights(DenseLinear(torch.cat(parts).contiguous()), norm,
-                             DenseLinear(uk.transpose(1, 2).reshape(-1, d).contiguous(), groups=h),
-                             DenseLinear(uv.reshape(-1, rank).contiguous(), groups=h), expand,
-                             DenseLinear(r.from_heads(p + "output.weight", cfg.hidden_size, w, h, m.vdim, e)))
+        return LatentWeights(DenseLinear(torch.cat(parts).contiguous()), norm, LatentUp.read(r, m, p),
+                             DenseLinear(r.from_heads(p + "output.weight", cfg.hidden_size, w, m.heads, m.vdim, up(m.vdim))))
 
     @staticmethod
     def _parallel(r: TensorReader, cfg: BufolornConfig, m: ParallelSpec, p: str, w: int) -> ParallelWeights:
@@ -562,74 +543,26 @@ class BufolornWeights:
         return _tensor_bytes([self.embed, self.lm_head, self.final_norm, self.layers])
 
 
-class BufolornModel(UnquantizedModel):
+class BufolornModel(RecurrentModel):
     def __init__(self, cfg: BufolornConfig, weights: BufolornWeights, collective=None) -> None:
         super().__init__(cfg, weights, collective)
         place = {layer: n for n, layer in enumerate(cfg.owners())}
         self.pages_of = [place.get(getattr(l.mixer, "kv_from", None) if getattr(l.mixer, "kv_from", None) is not None else i)
                          for i, l in enumerate(cfg.layers)]
-        self.state: LayerStates | None = None
-
-    def make_state(self, slots: int) -> LayerStates | None:
-        """Recurrent state for ``slots`` sequences (None if no layer has one)."""
-        shapes = self.cfg.state_shapes()
-        self.state = LayerStates(shapes, slots, self.w.embed.device) if shapes else None
-        return self.state
-
-    def state_bytes_per_row(self) -> int:
-        return self.cfg.state_bytes()
 
     def decode_splits(self, batch: int, longest: int) -> int:
-        latent = (latent_attn.decode_splits(batch, m.heads, min(longest, m.window)) for m in self.cfg.latent)
-        return max(super().decode_splits(batch, longest), max(latent, default=1))
+        return max(super().decode_splits(batch, longest), latent.decode_splits(self.cfg.latent, batch, longest))
 
     # -- mixers -----------------------------------------------------------------------------------------------------
     def _latent_at(self, i: int, h, x, cache, step: StepBuffers, prefill: bool) -> None:
         m, w = self.cfg.layers[i].mixer, self.w.layers[i].mixer
-        pages = cache.layer(self.pages_of[i]).k
-        t, heads, d, rot, e, rank = h.shape[0], m.heads, up(m.dim), up(m.rot_dim), up(m.vdim), up(m.kv_rank)
-        fp32 = h.dtype == torch.float32
-        singles = step.num_decode if prefill else t
-        latent_rows = t if fp32 or step.max_q < latent_attn.EXPAND_MIN_TOKENS else singles
         with scope("latent.proj", x.device):
             proj = w.proj(h)
         with scope("latent.core", x.device):
-            q_latent, q = latent_attn.finish(
-                proj, pages if m.kv_from is None else None, step.positions, step.slots, heads=heads, d=d, rank=rank, rot=rot, real_rank=m.kv_rank,
-                real_rot=m.rot_dim, norm_w=w.norm, rope=self._rope.get(m.rotation), eps=self.cfg.norm_eps, latent_rows=latent_rows)
-            y = torch.empty((t, heads * e), dtype=h.dtype, device=h.device)
-            if latent_rows:
-                w.absorb(proj[:latent_rows], x_step=d + rot, out=q_latent.view(latent_rows, -1), out_step=rank + rot)
-                how = dict(rank=rank, window=m.window, scale=m.scale)
-                if fp32:
-                    a = latent_attn.plain(q_latent, pages, step.block_table, self._sequence_of_rows(step, t), step.positions, **how)
-                else:
-                    each = latent_rows > singles  # several rows of a sequence
-                    how["splits"] = min(self.attn_splits, latent_attn.decode_splits(latent_rows, heads, m.window))
-                    a = latent_attn.decode(q_latent, pages, step.block_table, step.positions if each else step.seq_lens,
-                                           tok_seq=step.tok_seq if each else None, **how)
-                w.value_up(a.view(latent_rows, -1), out=y[:latent_rows])
-            if latent_rows < t:
-                self._attend_expanded(m, w, q, pages, step, singles, y.view(t, heads, e))
+            y = latent.attend(self, m, w.up, proj, cache.layer(self.pages_of[i]).k, step, prefill, rope=self._rope.get(m.rotation),
+                              own_rows=m.kv_from is None, norm=w.norm)
         with scope("latent.o_proj", x.device):
             w.o_proj(y, add_to=x, scale=self.cfg.residual_mult)
-
-    @staticmethod
-    def _attend_expanded(m: LatentSpec, w: LatentWeights, q, pages, step: StepBuffers, singles: int, y) -> None:
-        """Portions of the sequences from ``singles`` on, over keys and values expanded from the visible rows."""
-        table, dk, dv = step.block_table[singles:], q.shape[-1], y.shape[-1]
-        if m.window not in step.plans:
-            seq, shift = latent_attn.visible_pages(step.portions[singles:], m.window)
-            both = torch.tensor(seq + shift, dtype=torch.int32).pin_memory().to(q.device, non_blocking=True)
-            step.plans[m.window] = both.split([len(seq), len(shift)])
-        seq, shift = step.plans[m.window]
-        rows = latent_attn.visible_rows(pages, table, seq, shift)
-        group = max(1, min(m.heads, latent_attn.EXPANDED_BYTES // (rows.shape[0] * (dk + dv) * 2)))
-        for h0 in range(0, m.heads, group):
-            n = min(group, m.heads - h0)
-            kv = DenseLinear(w.expand[h0 * (dk + dv) : (h0 + n) * (dk + dv)])(rows)
-            latent_attn.prefill_rows(q, kv, shift, step.q_starts[singles:], step.seq_lens[singles:], step.max_q, head0=h0, heads=n, dk=dk, dv=dv,
-                                     window=m.window, scale=m.scale, out=y)
 
     def _biased_attention(self, a: BiasedSpec, w: ParallelWeights, h, kv, step: StepBuffers, prefill: bool):
         t = h.shape[0]

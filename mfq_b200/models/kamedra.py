@@ -20,14 +20,13 @@ from dataclasses import asdict, dataclass, field
 
 import torch
 
-from ..engine.recurrent_state import LayerStates
 from ..ops import dense, gla, window_attn
 from ..ops.dense import DenseLinear, up
 from ..ops.window_attn import NO_WINDOW, Difference, FrequencyScaling
 from ..utils.profiler import scope
 from . import unquantized
 from .llama import StepBuffers
-from .unquantized import TensorReader, UnquantizedModel
+from .unquantized import RecurrentModel, TensorReader
 
 
 @dataclass(frozen=True)
@@ -333,21 +332,11 @@ class KamedraWeights:
         return _tensor_bytes([self.embed, self.final_norm, self.layers])
 
 
-class KamedraModel(UnquantizedModel):
+class KamedraModel(RecurrentModel):
     def __init__(self, cfg: KamedraConfig, weights: KamedraWeights, collective=None) -> None:
         super().__init__(cfg, weights, collective)
         place = {layer: n for n, layer in enumerate(cfg.owners())}
         self.pages_of = [None if l.linear else place[i if l.mixer.kv_from is None else l.mixer.kv_from] for i, l in enumerate(cfg.layers)]
-        self.state: LayerStates | None = None
-
-    def make_state(self, slots: int) -> LayerStates | None:
-        """Recurrent state for ``slots`` sequences (None if no layer has one)."""
-        shapes = self.cfg.state_shapes()
-        self.state = LayerStates(shapes, slots, self.w.embed.device) if shapes else None
-        return self.state
-
-    def state_bytes_per_row(self) -> int:
-        return self.cfg.state_bytes()
 
     # -- forward ----------------------------------------------------------------------------------------------------
     def _attend(self, q, kv, m: AttentionSpec, d: Difference, step: StepBuffers, prefill: bool):

@@ -84,6 +84,7 @@ FAMILIES = (
     _unquantized("tepetar", "TepetarConfig", "TepetarWeights", "TepetarModel"),
     _unquantized("kamedra", "KamedraConfig", "KamedraWeights", "KamedraModel"),
     _unquantized("bufolorn", "BufolornConfig", "BufolornWeights", "BufolornModel"),
+    _unquantized("gogivik", "GogivikConfig", "GogivikWeights", "GogivikModel"),
     Family("latent attention", lambda raw: bool(raw.get("kv_lora_rank")), _build_mla),
     Family("decoder", lambda raw: True, _build_moe_decoder),  # dense and mixture-of-experts decoders
 )

@@ -6,6 +6,7 @@ from __future__ import annotations
 import torch
 
 from ..engine.kv_cache import PlainPagedKVCache
+from ..engine.recurrent_state import LayerStates
 from ..ops import dense, window_attn
 from ..ops.dense import DenseLinear
 from .llama import LlamaModel
@@ -112,3 +113,19 @@ class UnquantizedModel(LlamaModel):
         if self._rows is None or self._rows.numel() < t:
             self._rows = torch.arange(max(t, 256), dtype=torch.int32, device=self.w.embed.device)
         return self._rows[:t]
+
+
+class RecurrentModel(UnquantizedModel):
+    """Models some of whose layers carry a state per sequence: ``cfg`` also brings ``state_shapes()`` (layer, or (layer, part), -> shape)
+    and ``state_bytes()``."""
+
+    state: LayerStates | None = None
+
+    def make_state(self, slots: int) -> LayerStates | None:
+        """Recurrent state for ``slots`` sequences (None if no layer has one)."""
+        shapes = self.cfg.state_shapes()
+        self.state = LayerStates(shapes, slots, self.w.embed.device) if shapes else None
+        return self.state
+
+    def state_bytes_per_row(self) -> int:
+        return self.cfg.state_bytes()

@@ -24,7 +24,7 @@ CSRC = HERE / "csrc"
 LIB_PATH = HERE / "_mfq_b200_kernels.so"
 DENSE_LIB_PATH = HERE / "_mfq_b200_dense.so"
 DENSE_SOURCES = ("dense_gemm.cu", "dense_moe.cu", "stream_ops.cu", "mix_ops.cu", "window_attn.cu", "window_attn_prefill.cu",
-                 "window_attn_prefill_bias.cu", "latent_attn.cu", "gla.cu", "gla_chunk.cu", "delta.cu", "delta_chunk.cu", "moe_route.cu")
+                 "window_attn_prefill_bias.cu", "latent_attn.cu", "gla.cu", "gla_chunk.cu", "delta.cu", "delta_chunk.cu", "ssd.cu", "ssd_chunk.cu", "moe_route.cu")
 SHARED_SOURCES = ("moe_route.cu",)  # part of the main library too
 OBJ_DIR = HERE / "build"
 

@@ -69,6 +69,7 @@ enum : int {
   kDenseReluGlu = 6,  // rows packed as for kDenseGlu: out = max(gate, 0) * up, half as wide
   kDenseSiluGlu = 7,  // ... out = silu(gate) * up
   kDenseFloat = 8,    // fp32 out[t, n] = v + bias[n]
+  kDenseRelu2 = 9,    // out[t, n] = max(v + bias[n], 0)^2
 };
 __host__ __device__ constexpr bool dense_is_glu(int kind) {
   return kind == kDenseGlu || kind == kDenseGeluGlu || kind == kDenseReluGlu || kind == kDenseSiluGlu;
@@ -145,6 +146,10 @@ __device__ __forceinline__ void dense_store_item(const DenseEpilogue& e, int t, 
     load8<T>(static_cast<const T*>(e.table) + size_t(e.ids[t]) * e.ldo + n0, g);
 #pragma unroll
     for (int i = 0; i < 8; ++i) v[i] = gelu_tanh(v[i]) * g[i];
+  }
+  if (e.kind == kDenseRelu2) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = fmaxf(v[i], 0.f) * fmaxf(v[i], 0.f);
   }
   if (e.kind == kDenseSoftcap) {
 #pragma unroll

@@ -16,8 +16,8 @@
 // out (a matrix per head), and E matrices whose tokens are runs of rows of x sorted by matrix (experts), a tile list naming
 // (matrix, token tile); the streaming kernel can read those rows through a row -> token map instead of a sorted copy.
 //
-// The output stage (bias, a gated unit over interleaved gate / up rows, GELU times a per-token table row, soft cap, addition to
-// the fp32 stream, plain fp32) is shared by the three kernels (dense_common.cuh).  Waits are bounded as everywhere (common.cuh).
+// The output stage (bias, a gated unit over interleaved gate / up rows, GELU times a per-token table row, soft cap, squared ReLU,
+// addition to the fp32 stream, plain fp32) is shared by the three kernels (dense_common.cuh).  Waits are bounded as everywhere (common.cuh).
 #include "dense_common.cuh"
 
 namespace mfq {
@@ -397,7 +397,7 @@ static int run_dense(const DenseParams& p, const void* w, const void* x, int ldx
                      int fp32, cudaStream_t stream) {
   const int kind = p.epi.kind;
   if (p.M <= 0 || p.N <= 0 || p.K <= 0 || p.N % 16 || p.K % 8 || ldx % 8 || ldx < (p.groups - 1) * p.x_step + p.K || p.epi.ldo % 8) return -1;
-  if (kind < kDenseBias || kind > kDenseFloat || (kind == kDenseGelu && (!p.epi.table || !p.epi.ids))) return -1;
+  if (kind < kDenseBias || kind > kDenseRelu2 || (kind == kDenseGelu && (!p.epi.table || !p.epi.ids))) return -1;
   if (kind == kDenseSoftcap && !(p.epi.limit > 0.f)) return -1;
   if (p.epi.ldo < (p.groups - 1) * p.out_step + (dense_is_glu(kind) ? p.N / 2 : p.N)) return -1;
   if (fp32) {

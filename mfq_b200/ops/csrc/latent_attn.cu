@@ -1,8 +1,10 @@
 // Latent attention over unquantized pages with a sliding window: one row [c: rank | rotated key part: rot] per token serves all
 // heads (pages [page][16][R], R = rank + rot; widths as stored, multiples of 16).  A query at position i sees 0 <= i - j < window.
+// A head may have a sink: one more term exp(sink) of its denominator.
 //
 //   latent_finish   behind the projections: norm of c and rotation of the shared key part into the page; rotation of the queries'
 //                   rotated part, for rows that attend in latent space and for rows that attend to expanded keys
+//   latent_down     the same for the shared row alone, beside the norm of a query latent (queries then come from a product behind it)
 //   latent_pages    copies the visible pages of portions into consecutive rows, from where keys and values are expanded by a product
 //                   (prefill then runs window_attn_prefill.cuh on them)
 //   latent_decode   bf16, attention in latent space: queries are already mapped there, the value of a token is the latent part of
@@ -17,7 +19,7 @@
 
 namespace mfq {
 
-int launch_attn_merge(const float* part, const float* part_ml, __nv_bfloat16* out, int B, int heads, int splits, int dv, cudaStream_t stream);
+int launch_attn_merge(const float* part, const float* part_ml, const float* sink, __nv_bfloat16* out, int B, int heads, int splits, int dv, cudaStream_t stream);
 
 namespace {
 
@@ -51,6 +53,43 @@ struct LatentFinishParams {
   const int* slots;
 };
 
+// 8 channels from c of a rotated part: neighbours turn together.
+template <typename T>
+__device__ __forceinline__ void latent_turned(const T* src, int c, const float2* tab, int real_rot, float (&v)[8]) {
+  load8<T>(src + c, v);
+#pragma unroll
+  for (int j = 0; j < 8; j += 2) {
+    if (tab && c + j < real_rot) {
+      const float2 cs = tab[(c + j) >> 1];
+      const float a = v[j], b = v[j + 1];
+      v[j] = a * cs.x - b * cs.y;
+      v[j + 1] = b * cs.x + a * cs.y;
+    }
+  }
+}
+
+// dst = src / rms(src) * w over `width` stored channels, `real` of which count; a warp.
+template <typename T>
+__device__ __forceinline__ void latent_norm(const T* src, T* dst, const float* w, int width, int real, float eps, int lane) {
+  float v[8], ss = 0.f;
+  for (int c = lane * 8; c < width; c += 256) {
+    load8<T>(src + c, v);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss += v[j] * v[j];
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float f = rsqrtf(ss / float(real) + eps);
+  for (int c = lane * 8; c < width; c += 256) {
+    float ww[8];
+    load8<T>(src + c, v);
+    load8<float>(w + c, ww);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] *= f * ww[j];
+    store8<T>(dst + c, v);
+  }
+}
+
 // proj row: [H][d + rot] queries, then [rank | rot] (has_kv).  A warp per (token, query head or latent row).
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -63,24 +102,12 @@ latent_finish_kernel(const T* __restrict__ proj, T* __restrict__ q_latent, T* __
   const int t = item / per, h = item - t * per, R = p.rank + p.rot, hw = p.d + p.rot;
   const float2* tab = p.rope ? p.rope + size_t(min(p.positions[t], p.table_rows - 1)) * (p.real_rot / 2) : nullptr;
   const T* row = proj + size_t(t) * p.row_stride;
-  auto turned = [&](const T* src, int c, float(&v)[8]) {  // 8 channels from c of a rotated part
-    load8<T>(src + c, v);
-#pragma unroll
-    for (int j = 0; j < 8; j += 2) {
-      if (tab && c + j < p.real_rot) {
-        const float2 cs = tab[(c + j) >> 1];
-        const float a = v[j], b = v[j + 1];
-        v[j] = a * cs.x - b * cs.y;
-        v[j + 1] = b * cs.x + a * cs.y;
-      }
-    }
-  };
   float v[8];
   if (h < p.H) {
     const T* q = row + h * hw;
     T* dst = t < p.latent_rows ? q_latent + (size_t(t) * p.H + h) * R + p.rank : q_full + (size_t(t) * p.H + h) * hw + p.d;
     for (int c = lane * 8; c < p.rot; c += 256) {
-      turned(q + p.d, c, v);
+      latent_turned<T>(q + p.d, c, tab, p.real_rot, v);
       store8<T>(dst + c, v);
     }
     if (t >= p.latent_rows)
@@ -94,25 +121,45 @@ latent_finish_kernel(const T* __restrict__ proj, T* __restrict__ q_latent, T* __
   if (slot < 0) return;
   const T* src = row + p.H * hw;
   T* dst = pages + size_t(slot) * R;  // a page is 16 consecutive rows
-  float ss = 0.f;
-  for (int c = lane * 8; c < p.rank; c += 256) {
-    load8<T>(src + c, v);
-#pragma unroll
-    for (int j = 0; j < 8; ++j) ss += v[j] * v[j];
-  }
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  const float f = rsqrtf(ss / float(p.real_rank) + p.eps);
-  for (int c = lane * 8; c < p.rank; c += 256) {
-    float w[8];
-    load8<T>(src + c, v);
-    load8<float>(p.norm_w + c, w);
-#pragma unroll
-    for (int j = 0; j < 8; ++j) v[j] *= f * w[j];
-    store8<T>(dst + c, v);
-  }
+  latent_norm<T>(src, dst, p.norm_w, p.rank, p.real_rank, p.eps, lane);
   for (int c = lane * 8; c < p.rot; c += 256) {
-    turned(src + p.rank, c, v);
+    latent_turned<T>(src + p.rank, c, tab, p.real_rot, v);
+    store8<T>(dst + p.rank + c, v);
+  }
+}
+
+struct LatentDownParams {
+  int T, q_rank, real_q_rank, rank, real_rank, rot, real_rot, row_stride, table_rows;
+  float eps;
+  const float* q_norm;  // [q_rank]
+  const float* norm_w;  // [rank]
+  const float2* rope;   // [positions][real_rot / 2]
+  const int* positions;
+  const int* slots;
+};
+
+// proj row: [q_rank | rank | rot].  A warp per (token, query latent or shared row).
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_down_kernel(const T* __restrict__ proj, T* __restrict__ q_out, T* __restrict__ pages, const LatentDownParams p) {
+  pdl_trigger();
+  pdl_wait();
+  const int item = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (item >= 2 * p.T) return;
+  const int t = item >> 1;
+  const T* row = proj + size_t(t) * p.row_stride;
+  if (!(item & 1)) {
+    latent_norm<T>(row, q_out + size_t(t) * p.q_rank, p.q_norm, p.q_rank, p.real_q_rank, p.eps, lane);
+    return;
+  }
+  const int slot = p.slots[t];
+  if (slot < 0) return;
+  const float2* tab = p.rope ? p.rope + size_t(min(p.positions[t], p.table_rows - 1)) * (p.real_rot / 2) : nullptr;
+  T* dst = pages + size_t(slot) * (p.rank + p.rot);
+  latent_norm<T>(row + p.q_rank, dst, p.norm_w, p.rank, p.real_rank, p.eps, lane);
+  for (int c = lane * 8; c < p.rot; c += 256) {
+    float v[8];
+    latent_turned<T>(row + p.q_rank + p.rank, c, tab, p.real_rot, v);
     store8<T>(dst + p.rank + c, v);
   }
 }
@@ -139,6 +186,7 @@ struct LatentDecodeParams {
   float* part_ml;
   int H, R, rank, max_pages, window, splits, len_add;
   float scale_log2;
+  const float* sink;  // [H] or null
 };
 
 int la_smem(int R, int tiles) {
@@ -304,7 +352,15 @@ latent_decode_kernel(const LatentDecodeParams p) {
     const int mt = rr >> 1, half = rr & 1, r = mt * 16 + g + 8 * half;
     if (r >= heads) continue;
     const size_t row = size_t(t) * p.H + h0 + r;
-    const float l = alpha_s[2 * kRows + r], f = whole ? (l > 0.f ? 1.f / l : 0.f) : 1.f;
+    float l = alpha_s[2 * kRows + r], f = 1.f;
+    if (whole) {
+      if (p.sink) {  // one more key, without a value
+        const float m = alpha_s[kRows + r], sink = p.sink[h0 + r] * kLog2e, mt = fmaxf(m, sink);
+        f = window_exp2(m - mt);
+        l = fmaf(l, f, window_exp2(sink - mt));
+      }
+      f = l > 0.f ? f / l : 0.f;
+    }
 #pragma unroll
     for (int n = 0; n < kLaMaxTiles; ++n) {
       const int tile = warp + 8 * n;
@@ -344,6 +400,7 @@ struct LatentPlainParams {
   const int* positions;
   int T, H, R, rank, max_pages, window;
   float scale;
+  const float* sink;  // [H] or null
 };
 
 constexpr int kLaPlainMax = 1024, kLaPlainChunks = kLaPlainMax / 256;
@@ -368,6 +425,10 @@ latent_plain_kernel(const T* __restrict__ q, const T* __restrict__ kv, T* __rest
   }
   __syncwarp();
   float m = -FLT_MAX, l = 0.f, acc[kLaPlainChunks][8] = {};
+  if (p.sink) {
+    m = p.sink[gw - t * p.H];
+    l = 1.f;
+  }
   for (int j0 = lo; j0 <= pos; j0 += 32) {
     const int key = j0 + lane;
     float s = -FLT_MAX;
@@ -453,6 +514,24 @@ extern "C" int mfq_latent_finish(const void* proj, int row_stride, void* q_laten
   return cudaGetLastError() == cudaSuccess ? 0 : -7;
 }
 
+// proj [T, row_stride]: [q_rank | rank | rot].  q_out [T, q_rank]: the normed query latents; pages get the shared rows.
+extern "C" int mfq_latent_down(const void* proj, int row_stride, void* q_out, void* pages, const int* positions, const int* slots,
+                               const float* q_norm, const float* norm_w, const float* rope, int table_rows, int T_, int q_rank, int real_q_rank,
+                               int rank, int real_rank, int rot, int real_rot, float eps, int fp32, cudaStream_t stream) {
+  if (T_ <= 0 || T_ > (1 << 29) || !la_sizes(1, rank, rot) || q_rank <= 0 || q_rank % 16 || real_q_rank <= 0 || real_q_rank > q_rank) return -1;
+  if (real_rank <= 0 || real_rank > rank || real_rot % 2 || real_rot > rot || row_stride % 8 || row_stride < q_rank + rank + rot) return -1;
+  if ((real_rot && (!rope || table_rows <= 0)) || !slots || !q_norm || !norm_w) return -1;
+  const LatentDownParams p{T_, q_rank, real_q_rank, rank, real_rank, rot, real_rot, row_stride, table_rows, eps, q_norm, norm_w,
+                           reinterpret_cast<const float2*>(real_rot ? rope : nullptr), positions, slots};
+  const dim3 grid(unsigned((2 * T_ + 7) / 8));
+  if (fp32)
+    launch_kernel(latent_down_kernel<float>, grid, dim3(256), 0, stream, static_cast<const float*>(proj), static_cast<float*>(q_out), static_cast<float*>(pages), p);
+  else
+    launch_kernel(latent_down_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, static_cast<const __nv_bfloat16*>(proj),
+                  static_cast<__nv_bfloat16*>(q_out), static_cast<__nv_bfloat16*>(pages), p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -7;
+}
+
 // Pages of 16 rows of R bf16.  seq [count], shift [B] as in the kernel.
 extern "C" int mfq_latent_pages(const void* pages, const int* table, const int* seq, const int* shift, void* out, int count, int R,
                                 int max_pages, cudaStream_t stream) {
@@ -466,20 +545,21 @@ extern "C" int mfq_latent_pages(const void* pages, const int* table, const int* 
 // * 2 floats (splits > 1).
 extern "C" int mfq_latent_decode(const void* q, const void* kv, const int* table, const int* tok_seq, const int* lens, int len_add, void* out,
                                  float* part, float* part_ml, int T_, int H, int rank, int rot, int max_pages, int window, float scale,
-                                 int splits, cudaStream_t stream) {
+                                 int splits, const float* sink, cudaStream_t stream) {
   if (T_ <= 0 || !la_sizes(H, rank, rot) || rank > 128 * kLaMaxTiles || window <= 0 || splits < 1 || splits > 65535 || (splits > 1 && (!part || !part_ml))) return -1;
   const LatentDecodeParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(kv), table, tok_seq, lens,
-                             static_cast<__nv_bfloat16*>(out), part, part_ml, H, rank + rot, rank, max_pages, window, splits, len_add, scale * kLog2e};
+                             static_cast<__nv_bfloat16*>(out), part, part_ml, H, rank + rot, rank, max_pages, window, splits, len_add, scale * kLog2e, sink};
   const bool two = H > 16 && la_smem(rank + rot, 2) <= 227 * 1024;
   const int rc = two ? launch_latent_decode<2>(p, T_, stream) : launch_latent_decode<1>(p, T_, stream);
   if (rc) return rc;
-  return splits > 1 ? launch_attn_merge(part, part_ml, static_cast<__nv_bfloat16*>(out), T_, H, splits, rank, stream) : 0;
+  return splits > 1 ? launch_attn_merge(part, part_ml, sink, static_cast<__nv_bfloat16*>(out), T_, H, splits, rank, stream) : 0;
 }
 
 extern "C" int mfq_latent_plain(const void* q, const void* kv, const int* table, const int* tok_seq, const int* positions, void* out, int T_,
-                                int H, int rank, int rot, int max_pages, int window, float scale, int fp32, cudaStream_t stream) {
+                                int H, int rank, int rot, int max_pages, int window, float scale, const float* sink, int fp32,
+                                cudaStream_t stream) {
   if (T_ <= 0 || !la_sizes(H, rank, rot) || rank + rot > kLaPlainMax || window <= 0) return -1;
-  const LatentPlainParams p{table, tok_seq, positions, T_, H, rank + rot, rank, max_pages, window, scale};
+  const LatentPlainParams p{table, tok_seq, positions, T_, H, rank + rot, rank, max_pages, window, scale, sink};
   const dim3 grid(unsigned(((long long)(T_) * H + 3) / 4));
   if (fp32)
     launch_kernel(latent_plain_kernel<float>, grid, dim3(128), 0, stream, static_cast<const float*>(q), static_cast<const float*>(kv),

@@ -3,7 +3,10 @@
 //   layer_norm_out    h = (x - mean) / sqrt(var + eps) * w + b of the fp32 stream
 //   token_shift       every stream s of a token reads  h + (h' - h) * mu_s,  h' the row of the previous token (zeros before the
 //                     first); the last row of a sequence is kept in its state slot
-//   short_conv        causal convolution over time per channel, then SiLU; the last taps - 1 inputs are kept in the state slot
+//   short_conv        causal convolution over time per channel (with an optional bias), then SiLU; the last taps - 1 inputs are kept
+//                     in the state slot
+//   norm_conv         g = h + conv(h) with h = rms_norm(x) * w of the fp32 stream and a causal convolution over time per channel; the
+//                     last taps - 1 rows h are kept in the state slot
 //
 // Batches are ragged: sequence b owns rows starts[b] .. starts[b + 1] - 1 (starts null: row b) and state slot slot[b] (< 0: the
 // sequence is skipped).
@@ -97,6 +100,7 @@ token_shift_kernel(const T* __restrict__ h, const float* __restrict__ mu, float*
 
 struct ShortConvParams {
   const float* w;     // [taps, C], last row for the current token
+  const float* bias;  // [C] or null
   float* state;       // [slots, taps - 1, C], oldest first
   const int* slot;    // [B]
   const int* starts;  // [B + 1] or null
@@ -122,7 +126,8 @@ short_conv_kernel(const T* __restrict__ x, T* __restrict__ out, const ShortConvP
     if (n >= 0) load8<T>(x + size_t(r0 + n) * p.in_stride + c, v);
     else if (n + hist >= 0) load8<float>(st + size_t(n + hist) * p.C, v);
   };
-  float w[TAPS][8], win[TAPS][8];  // win[i]: input i - (TAPS - 1) tokens from the current one
+  float w[TAPS][8], win[TAPS][8], add[8] = {};  // win[i]: input i - (TAPS - 1) tokens from the current one
+  if (p.bias) load8<float>(p.bias + c, add);
 #pragma unroll
   for (int i = 0; i < TAPS; ++i) {
 #pragma unroll
@@ -145,7 +150,7 @@ short_conv_kernel(const T* __restrict__ x, T* __restrict__ out, const ShortConvP
 #pragma unroll
         for (int i = 0; i + 1 < TAPS; ++i) win[i][j] = win[i + 1][j];
         win[TAPS - 1][j] = next[e][j];
-        float a = 0.f;
+        float a = add[j];
 #pragma unroll
         for (int i = 0; i < TAPS; ++i) a = fmaf(w[i][j], win[i][j], a);
         y[j] = sizeof(T) == 4 ? a / (1.f + expf(-a)) : __fdividef(a, 1.f + __expf(-fmaxf(a, -80.f)));
@@ -192,6 +197,114 @@ static int launch_short_conv(const void* x, void* out, const ShortConvParams& p,
   return cudaGetLastError() == cudaSuccess ? 0 : -7;
 }
 
+struct NormConvParams {
+  const float* x;       // [T, W] fp32 stream
+  const float* norm_w;  // [W]
+  const float* w;       // [taps, W], last row for the current token
+  float* state;         // [slots, taps - 1, W], oldest first
+  const int* slot;      // [B]
+  const int* starts;    // [B + 1] or null
+  int W, taps;
+  float inv_width, eps;
+};
+
+// A CTA takes a run of tokens of a sequence: first the root mean squares of its rows and of the taps - 1 before them, then every thread
+// walks the run for 8 channels at a time.  The CTA of the sequence's first run is the only one that reads the kept rows, so it also
+// replaces them (by the portion's last rows), channel by channel in the same thread.
+constexpr int kNormRunTokens = 8, kNormMaxTaps = 8;
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256)
+norm_conv_kernel(T* __restrict__ out, const NormConvParams p) {
+  pdl_trigger();
+  pdl_wait();
+  constexpr int kRows = kNormRunTokens + 2 * (kNormMaxTaps - 1);
+  __shared__ float part[kRows * 8], scale[kRows];
+  const int b = blockIdx.y, s = p.slot[b], W = p.W;
+  const int r0 = p.starts ? p.starts[b] : b, len = p.starts ? p.starts[b + 1] - r0 : 1;
+  const int n0 = blockIdx.x * kNormRunTokens, n1 = min(len, n0 + kNormRunTokens), hist = p.taps - 1;
+  if (n0 >= len) return;
+  const int first = max(0, n0 - hist), tail = n0 == 0 ? max(n1, len - hist) : len;  // rows first .. n1 - 1, then tail .. len - 1
+  const int rows = n1 - first + len - tail;
+  auto row_of = [&](int i) { return i < n1 - first ? first + i : tail + i - (n1 - first); };
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5, each = max(1, warps / rows);  // warps per row
+  for (int j = warp; j < rows * each; j += warps) {
+    const int i = j / each;
+    const float* x = p.x + size_t(r0 + row_of(i)) * W;
+    float ss = 0.f;
+#pragma unroll 4
+    for (int c = ((j - i * each) * 32 + lane) * 4; c < W; c += each * 128) {
+      const float4 v = *reinterpret_cast<const float4*>(x + c);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (lane == 0) part[j] = ss;
+  }
+  __syncthreads();
+  if (int(threadIdx.x) < rows) {
+    float ss = 0.f;
+    for (int z = 0; z < each; ++z) ss += part[threadIdx.x * each + z];
+    scale[threadIdx.x] = rsqrtf(ss * p.inv_width + p.eps);
+  }
+  __syncthreads();
+  float* st = s >= 0 && hist > 0 ? p.state + size_t(s) * hist * W : nullptr;
+  for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {
+    float w[TAPS][8], win[TAPS][8], nw[8];
+    load8<float>(p.norm_w + c, nw);
+    auto normed = [&](int n, int place, float(&v)[8]) {
+      load8<float>(p.x + size_t(r0 + n) * W + c, v);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] *= scale[place] * nw[j];
+    };
+#pragma unroll
+    for (int i = 0; i < TAPS; ++i) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) w[i][j] = win[i][j] = 0.f;
+      if (i - (TAPS - p.taps) >= 0) load8<float>(p.w + size_t(i - (TAPS - p.taps)) * W + c, w[i]);
+      const int n = n0 + i - TAPS;  // win[i], i > 0: row n
+      if (i > 0 && i - (TAPS - p.taps) > 0) {
+        if (n >= 0) normed(n, n - first, win[i]);
+        else if (st) load8<float>(st + size_t(n + hist) * W + c, win[i]);
+      }
+    }
+#pragma unroll 4
+    for (int n = n0; n < n1; ++n) {
+      float h[8], y[8];
+      normed(n, n - first, h);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+#pragma unroll
+        for (int i = 0; i + 1 < TAPS; ++i) win[i][j] = win[i + 1][j];
+        win[TAPS - 1][j] = h[j];
+        float a = h[j];
+#pragma unroll
+        for (int i = 0; i < TAPS; ++i) a = fmaf(w[i][j], win[i][j], a);
+        y[j] = a;
+      }
+      store8<T>(out + size_t(r0 + n) * W + c, y);
+    }
+    if (n0 == 0 && st) {
+      for (int i = 0; i < hist; ++i) {  // ascending: place i reads place i + len > i
+        const int n = len - hist + i;
+        float v[8];
+        if (n >= 0) normed(n, n < n1 ? n - first : n1 - first + n - tail, v);
+        else load8<float>(st + size_t(n + hist) * W + c, v);
+        store8<float>(st + size_t(i) * W + c, v);
+      }
+    }
+  }
+}
+
+template <typename T>
+static int launch_norm_conv(void* out, const NormConvParams& p, int B, int max_q, cudaStream_t stream) {
+  const int threads = min(256, (p.W / 8 + 31) / 32 * 32);
+  const dim3 grid((max_q + kNormRunTokens - 1) / kNormRunTokens, B);
+  T* o = static_cast<T*>(out);
+  if (p.taps <= 4) launch_kernel(norm_conv_kernel<T, 4>, grid, dim3(threads), 0, stream, o, p);
+  else launch_kernel(norm_conv_kernel<T, kNormMaxTaps>, grid, dim3(threads), 0, stream, o, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -7;
+}
+
 }  // namespace mfq
 
 using namespace mfq;
@@ -220,11 +333,20 @@ extern "C" int mfq_token_shift(const void* h, const float* mu, float* last, cons
   return cudaGetLastError() == cudaSuccess ? 0 : -7;
 }
 
-// x: rows of in_stride, channels 0 .. C - 1; w [taps, C]; state [slots, taps - 1, C]; starts null: row b belongs to sequence b
-extern "C" int mfq_short_conv(const void* x, int in_stride, const float* w, float* state, const int* slot, const int* starts, void* out,
+// x [T, W] fp32; out [T, W] = h + conv(h); w [taps, W]; state [slots, taps - 1, W]; starts null: row b belongs to sequence b
+extern "C" int mfq_norm_conv(const float* x, const float* norm_w, const float* w, float* state, const int* slot, const int* starts, void* out,
+                             int B, int max_q, int W, int width, int taps, float eps, int fp32, cudaStream_t stream) {
+  if (B <= 0 || B > 65535 || max_q <= 0 || W <= 0 || W % 8 || width <= 0 || width > W || taps < 1 || taps > kNormMaxTaps) return -1;
+  if (taps > 1 && !state) return -1;
+  const NormConvParams p{x, norm_w, w, state, slot, starts, W, taps, 1.f / float(width), eps};
+  return fp32 ? launch_norm_conv<float>(out, p, B, starts ? max_q : 1, stream) : launch_norm_conv<__nv_bfloat16>(out, p, B, starts ? max_q : 1, stream);
+}
+
+// x: rows of in_stride, channels 0 .. C - 1; w [taps, C]; bias [C] or null; state [slots, taps - 1, C]; starts null: row b belongs to sequence b
+extern "C" int mfq_short_conv(const void* x, int in_stride, const float* w, const float* bias, float* state, const int* slot, const int* starts, void* out,
                               int out_stride, int B, int max_q, int C, int taps, int fp32, cudaStream_t stream) {
   if (B <= 0 || B > 65535 || max_q <= 0 || C <= 0 || C % 8 || taps < 1 || taps > 8 || in_stride % 8 || out_stride % 8) return -1;
-  const ShortConvParams p{w, state, slot, starts, C, taps, in_stride, out_stride};
+  const ShortConvParams p{w, bias, state, slot, starts, C, taps, in_stride, out_stride};
   return fp32 ? launch_short_conv<float>(x, out, p, B, starts ? max_q : 1, stream)
               : launch_short_conv<__nv_bfloat16>(x, out, p, B, starts ? max_q : 1, stream);
 }

@@ -5,7 +5,8 @@
 //   norm_add          x += rms_norm(y) * w               -> fp32 stream + copy in the activation type, one pass over y and x
 //   norm_out          h = rms_norm(x) * w                -> activation type (input of a sublayer or of the LM head)
 //   qkv_finish        per head: RMS norm of q and k, rotation of the leading channels, blending of v with the values another
-//                     layer computed for the same token, K / V into their pages
+//                     layer computed for the same token, or RMS norm and rotation of v, K / V into their pages
+//   turn_back         rotation of attention outputs by minus their position (for values that were rotated by theirs)
 //   map_difference    differential attention: rms_norm(a1 - lambda a2) * scale of every head
 //
 // "rms_norm" divides by sqrt(mean(x^2) + eps) over the model's true width; weights arrive in fp32 in the form they multiply
@@ -105,7 +106,8 @@ norm_out_kernel(const float* __restrict__ x, const float* __restrict__ w, T* __r
 // qkv rows [Hq * dk | Hk * maps * dk | Hk * dv] (dk, dv: head widths as stored, multiples of 16; d: the true q / k width the
 // norm averages over; Hq counts every query map).  `L` lanes (a power of two) share a head, 8 channels each; a warp takes 32 / L
 // heads of one token.  Queries may also be multiplied by a temperature that grows with the position.  The rotation reads (cos, sin) of the token's position from a table [positions][rot / 2]; channel i turns
-// with i + rot / 2 (read from shared memory), or with its neighbour (`pairs`).  Pages: K [page][Hk][16][maps * dk],
+// with i + rot / 2 (read from shared memory), or with its neighbour (`pairs`).  With v_d > 0 values are divided by their root mean
+// square over v_d channels and all of these are rotated, from a table of their own.  Pages: K [page][Hk][16][maps * dk],
 // V [page][Hk][16][dv]; slot < 0: the token is not cached.  No pages: rows hold queries only.
 // ---------------------------------------------------------------------------------------------
 struct QkvFinishParams {
@@ -117,6 +119,8 @@ struct QkvFinishParams {
   const float* q_norm;
   const float* k_norm;      // [dk] fp32 or null: no norm
   const float2* rope;       // (cos, sin)
+  const float2* v_rope;
+  int v_d, v_table_rows;    // v_d 0: values stay as they are
   const int* positions;
   const int* slots;
 };
@@ -153,6 +157,11 @@ qkv_finish_kernel(const T* __restrict__ qkv, const T* __restrict__ v_first, T* _
 #pragma unroll
   for (int j = 0; j < 8; ++j) ss += v[j] * v[j];
   for (int o = p.L >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (is_v && p.v_d > 0) {
+    const float inv = rsqrtf(ss / float(p.v_d) + p.eps);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] *= inv;
+  }
   if (mine && nw) {
     const float inv = rsqrtf(ss / float(p.d) + p.eps);
     float ww[8];
@@ -165,13 +174,14 @@ qkv_finish_kernel(const T* __restrict__ qkv, const T* __restrict__ v_first, T* _
   for (int j = 0; j < 8; ++j) mysh[c * 8 + j] = v[j];
   __syncwarp();
   if (!mine) return;
-  if (!is_v && c * 8 < p.rot) {
-    const int half = p.rot >> 1, pos = min(p.positions[t], p.table_rows - 1);
-    const float2* tab = p.rope + size_t(pos) * half;
+  const int rot = is_v ? p.v_d : p.rot;
+  if (c * 8 < rot) {
+    const int half = rot >> 1, pos = min(p.positions[t], (is_v ? p.v_table_rows : p.table_rows) - 1);
+    const float2* tab = (is_v ? p.v_rope : p.rope) + size_t(pos) * half;
     if (p.pairs) {
 #pragma unroll
       for (int j = 0; j < 8; j += 2) {
-        if (c * 8 + j < p.rot) {
+        if (c * 8 + j < rot) {
           const float2 cs = tab[(c * 8 + j) >> 1];
           const float a = v[j], b = v[j + 1];
           v[j] = a * cs.x - b * cs.y;
@@ -186,7 +196,7 @@ qkv_finish_kernel(const T* __restrict__ qkv, const T* __restrict__ v_first, T* _
       if (i < half) {
         const float2 cs = tab[i];
         v[j] = v[j] * cs.x - mysh[i + half] * cs.y;
-      } else if (i < p.rot) {
+      } else if (i < rot) {
         const float2 cs = tab[i - half];
         v[j] = v[j] * cs.x + mysh[i - half] * cs.y;
       }
@@ -254,6 +264,53 @@ map_difference_kernel(const T* __restrict__ a, T* __restrict__ out, int pairs, i
   store8<T>(out + size_t(pair) * dv + lane * 8, y);
 }
 
+// o [T][H][dv] in place: the pairs of the first 2 * half channels turn by minus the angle the table gives for the token's position.
+// A thread takes kVec pairs (i, i + half) of a head, or kVec / 2 pairs of neighbours (`pairs`).
+template <typename T, int kVec>
+__global__ void __launch_bounds__(256)
+turn_back_kernel(T* __restrict__ o, const float2* __restrict__ rope, const int* __restrict__ positions, int T_, int H, int dv, int half,
+                 int table_rows, int pairs) {
+  pdl_trigger();
+  pdl_wait();
+  const int per = (pairs ? 2 * half : half + kVec - 1) / kVec, items = H * per;
+  const long long i = (long long)(blockIdx.x) * 256 + threadIdx.x;
+  if (i >= (long long)(T_) * items) return;
+  const int t = int(i / items), r = int(i - (long long)(t) * items), h = r / per, c = (r - h * per) * kVec;
+  const float2* tab = rope + size_t(min(positions[t], table_rows - 1)) * half;
+  T* head = o + (size_t(t) * H + h) * dv;
+  if constexpr (kVec == 8) {
+    float a[8], b[8];
+    load8<T>(head + c, a);
+    if (pairs) {
+#pragma unroll
+      for (int j = 0; j < 8; j += 2) {
+        const float2 cs = tab[(c + j) >> 1];
+        const float u = a[j], v = a[j + 1];
+        a[j] = fmaf(u, cs.x, v * cs.y);
+        a[j + 1] = fmaf(v, cs.x, -u * cs.y);
+      }
+    } else {
+      load8<T>(head + c + half, b);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float2 cs = tab[c + j];
+        const float u = a[j], v = b[j];
+        a[j] = fmaf(u, cs.x, v * cs.y);
+        b[j] = fmaf(v, cs.x, -u * cs.y);
+      }
+      store8<T>(head + c + half, b);
+    }
+    store8<T>(head + c, a);
+  } else {
+    const int lo = pairs ? c & ~1 : c, hi = pairs ? lo + 1 : c + half;
+    if (pairs && (c & 1)) return;
+    const float2 cs = tab[pairs ? lo >> 1 : lo];
+    const float u = float(head[lo]), v = float(head[hi]);
+    head[lo] = T(fmaf(u, cs.x, v * cs.y));
+    head[hi] = T(fmaf(v, cs.x, -u * cs.y));
+  }
+}
+
 static int stream_threads(int W) {
   const int nvec = W / 8;
   int threads = (nvec + 31) / 32 * 32;
@@ -310,13 +367,31 @@ extern "C" int mfq_map_difference(const void* a, void* out, int T_, int H, int p
   return cudaGetLastError() == cudaSuccess ? 0 : -7;
 }
 
-// k_pages null: the rows hold the Hq query heads only (Hk, dv unused)
+// o [T, H, dv] in place; rope [table_rows][d / 2] (cos, sin), d <= dv
+extern "C" int mfq_turn_back(void* o, const float* rope, const int* positions, int T_, int H, int dv, int d, int table_rows, int pairs,
+                             int fp32, cudaStream_t stream) {
+  if (T_ <= 0 || H <= 0 || dv <= 0 || dv % 8 || d <= 0 || d % 2 || d > dv || !rope || table_rows <= 0) return -1;
+  const int half = d / 2;
+  const bool wide = pairs ? d % 8 == 0 : half % 8 == 0;
+  const long long items = (long long)(T_) * H * (wide ? (pairs ? d / 8 : half / 8) : (pairs ? d : half));
+  if ((items + 255) / 256 > 0x7fffffffLL) return -1;
+  const float2* tab = reinterpret_cast<const float2*>(rope);
+  const dim3 grid(unsigned((items + 255) / 256));
+  if (wide)
+    MFQ_BY_TYPE(fp32, launch_kernel(turn_back_kernel<T, 8>, grid, dim3(256), 0, stream, static_cast<T*>(o), tab, positions, T_, H, dv, half, table_rows, pairs));
+  else
+    MFQ_BY_TYPE(fp32, launch_kernel(turn_back_kernel<T, 1>, grid, dim3(256), 0, stream, static_cast<T*>(o), tab, positions, T_, H, dv, half, table_rows, pairs));
+  return cudaGetLastError() == cudaSuccess ? 0 : -7;
+}
+
+// k_pages null: the rows hold the Hq query heads only (Hk, dv unused).  v_d > 0: values are normed and rotated (v_rope [v_table_rows][v_d / 2])
 extern "C" int mfq_qkv_finish(const void* qkv, int row_stride, const void* v_first, int first_stride, float lambda, void* q_out,
                               void* k_pages, void* v_pages, const int* positions, const int* slots, const float* q_norm,
                               const float* k_norm, const float* rope, int table_rows, int T_, int Hq, int Hk, int maps, int d, int dk,
-                              int dv, int rot, int pairs, int page_size, float eps, float temp, int temp_every, int fp32,
-                              cudaStream_t stream) {
+                              int dv, int rot, int pairs, int page_size, float eps, float temp, int temp_every, const float* v_rope,
+                              int v_d, int v_table_rows, int fp32, cudaStream_t stream) {
   if (temp != 0.f && temp_every <= 0) return -1;
+  if (v_d < 0 || v_d % 2 || (v_d && (!k_pages || v_d > dv || !v_rope || v_table_rows <= 0 || v_first))) return -1;
   if (!k_pages) { Hk = 0; dv = 0; v_first = nullptr; }
   if (T_ <= 0 || Hq <= 0 || maps <= 0 || dk % 16 || dk <= 0 || dk > 256 || d <= 0 || d > dk) return -1;
   if (k_pages && (Hk <= 0 || Hq % (Hk * maps) || dv % 16 || dv <= 0 || dv > 256 || page_size <= 0 || !v_pages || !slots)) return -1;
@@ -325,7 +400,7 @@ extern "C" int mfq_qkv_finish(const void* qkv, int row_stride, const void* v_fir
   int L = 1;
   while (L * 8 < max(dk, dv)) L *= 2;
   QkvFinishParams p{T_, Hq, Hk, maps, d, dk, dv, rot, pairs, row_stride, page_size, L, table_rows, eps, lambda, temp, temp_every, first_stride, q_norm, k_norm,
-                    reinterpret_cast<const float2*>(rope), positions, slots};
+                    reinterpret_cast<const float2*>(rope), reinterpret_cast<const float2*>(v_rope), v_d, v_table_rows, positions, slots};
   const int heads = Hq + Hk * (maps + 1), per_warp = 32 / L;
   const long long warps = (long long)(T_) * ((heads + per_warp - 1) / per_warp);
   MFQ_BY_TYPE(fp32, launch_kernel(qkv_finish_kernel<T>, dim3(unsigned((warps + 7) / 8)), dim3(256), 0, stream, static_cast<const T*>(qkv),

@@ -1,6 +1,7 @@
 // Sliding-window attention over unquantized pages (K [page][Hk][16][maps * dk], V [page][Hk][16][dv]), one query token per
 // sequence or, in the plain kernel, any number of them.  A query at position i sees the keys j with 0 <= i - j < window, and of
-// the first `keep` keys every one up to i.  With two maps (differential attention) a KV head has two key vectors and one value
+// the first `keep` keys every one up to i; with a chunk size it sees the keys j <= i of its own chunk instead of a window.  Outputs may
+// be turned back (window_attn.cuh: ValueTurn).  With two maps (differential attention) a KV head has two key vectors and one value
 // vector per token; queries are ordered [KV head][map][query head of the KV head].  With one map a head may have a score bias by
 // distance and a sink (window_attn.cuh: ScoreExtra).
 //
@@ -28,9 +29,10 @@ struct WindowDecodeParams {
   __nv_bfloat16* out;   // [B, Hq, dv]
   float* part;          // splits > 1 or maps > 1: [B * Hq][splits][dv]
   float* part_ml;       // [B * Hq][splits][2]
-  int Hq, Hk, maps, dk, dv, max_pages, window, keep, splits, head_tiles;
+  int Hq, Hk, maps, dk, dv, max_pages, window, chunk, keep, splits, head_tiles;
   ScoreCap cap;
   ScoreExtra extra;
+  ValueTurn turn;
 };
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
@@ -80,7 +82,7 @@ window_attn_decode_kernel(const WindowDecodeParams p) {
   const int head0 = g * per + ht * 16;
   const int map_dk = p.dk, dk = p.maps * p.dk, dv = p.dv;  // dk: channels of a key row, all maps
   const int pos = p.seq_lens[b] - 1;
-  const int lo = max(0, pos - p.window + 1);
+  const int lo = first_key(pos, p.window, p.chunk);
   // pages are counted over the visible ones: `kept` pages of first tokens that lie before the window, then the window's
   const int first = pos >= 0 ? lo / kWinPage : 0, kept = min((p.keep + kWinPage - 1) / kWinPage, first), skip = first - kept;
   int page0 = 0, page1 = pos >= 0 ? pos / kWinPage + 1 - skip : 0;
@@ -266,13 +268,27 @@ window_attn_decode_kernel(const WindowDecodeParams p) {
     }
     const size_t orow = size_t(b) * p.Hq + head0 + r;
     const float inv = whole ? (lt > 0.f ? 1.f / lt : 0.f) : 1.f;
-    for (int c = lane; c < dv; c += 32) {
+    auto merged = [&](int c) {
       float x = 0.f;
 #pragma unroll
       for (int w = 0; w < kWinWarps; ++w) x += acc[(w * 16 + r) * dv + c] * mw[w];
-      x *= inv;
-      if (whole) p.out[orow * dv + c] = __float2bfloat16(x);
-      else p.part[(orow * p.splits + split) * dv + c] = x;
+      return x * inv;
+    };
+    if (whole && p.turn.rope) {
+      const float2* tab = p.turn.rope + size_t(min(max(pos, 0), p.turn.rows - 1)) * p.turn.half;
+      for (int c = lane; c < p.turn.half; c += 32) {
+        const float2 cs = tab[c];
+        const float x = merged(c), y = merged(c + p.turn.half);
+        p.out[orow * dv + c] = __float2bfloat16(fmaf(x, cs.x, y * cs.y));
+        p.out[orow * dv + c + p.turn.half] = __float2bfloat16(fmaf(y, cs.x, -x * cs.y));
+      }
+      for (int c = 2 * p.turn.half + lane; c < dv; c += 32) p.out[orow * dv + c] = __float2bfloat16(merged(c));
+    } else {
+      for (int c = lane; c < dv; c += 32) {
+        const float x = merged(c);
+        if (whole) p.out[orow * dv + c] = __float2bfloat16(x);
+        else p.part[(orow * p.splits + split) * dv + c] = x;
+      }
     }
     if (!whole && lane == 0) {
       p.part_ml[(orow * p.splits + split) * 2] = mt;
@@ -286,6 +302,8 @@ struct WindowMergeParams {
   const float* sink;  // [heads] or null (one map)
   int splits, dv, heads, of_map, maps;  // heads: output heads; of_map: query heads per KV head
   float lambda, scale, eps, inv_d;
+  ValueTurn turn;       // one map
+  const int* seq_lens;  // for the turn
 };
 
 __global__ void __launch_bounds__(128)
@@ -325,6 +343,22 @@ window_attn_merge_kernel(const float* __restrict__ part, const float* __restrict
   }
   float f = 1.f;
   if (p.maps == 2) f = rsqrtf(dense_block_sum(y[0] * y[0] + y[1] * y[1] + y[2] * y[2] + y[3] * y[3], red) * p.inv_d + p.eps) * p.scale;
+  if (p.turn.rope) {
+    __shared__ float row[512];
+#pragma unroll
+    for (int i = 0; i < kCols; ++i) row[threadIdx.x + i * 128] = y[i];
+    __syncthreads();
+    const float2* tab = p.turn.rope + size_t(min(max(p.seq_lens[b] - 1, 0), p.turn.rows - 1)) * p.turn.half;
+#pragma unroll
+    for (int i = 0; i < kCols; ++i) {
+      const int c = threadIdx.x + i * 128;
+      if (c < 2 * p.turn.half) {
+        const bool low = c < p.turn.half;
+        const float2 cs = tab[low ? c : c - p.turn.half];
+        y[i] = fmaf(y[i], cs.x, low ? row[c + p.turn.half] * cs.y : -row[c - p.turn.half] * cs.y);
+      }
+    }
+  }
 #pragma unroll
   for (int i = 0; i < kCols; ++i) {
     const int c = threadIdx.x + i * 128;
@@ -332,8 +366,9 @@ window_attn_merge_kernel(const float* __restrict__ part, const float* __restrict
   }
 }
 
-int launch_attn_merge(const float* part, const float* part_ml, __nv_bfloat16* out, int B, int heads, int splits, int dv, cudaStream_t stream) {
-  const WindowMergeParams mp{nullptr, splits, dv, heads, heads, 1, 0.f, 1.f, 0.f, 0.f};
+int launch_attn_merge(const float* part, const float* part_ml, const float* sink, __nv_bfloat16* out, int B, int heads, int splits, int dv,
+                      cudaStream_t stream) {
+  const WindowMergeParams mp{sink, splits, dv, heads, heads, 1, 0.f, 1.f, 0.f, 0.f, ValueTurn{}, nullptr};
   launch_kernel(window_attn_merge_kernel, dim3(B * heads), dim3(128), 0, stream, part, part_ml, out, mp);
   return cudaGetLastError() == cudaSuccess ? 0 : -7;
 }
@@ -359,7 +394,7 @@ struct WindowPlainParams {
   const int* positions;  // [T]
   const int* tok_seq;    // [T] row of the block table
   const int* table;
-  int T, Hq, Hk, maps, dk, dv, max_pages, window, keep;
+  int T, Hq, Hk, maps, dk, dv, max_pages, window, chunk, keep;
   float scale, cap;
   ScoreExtra extra;
 };
@@ -376,7 +411,7 @@ window_attn_plain_kernel(const T* __restrict__ q, const T* __restrict__ k, const
   const int gw = blockIdx.x * 4 + warp;
   if (gw >= p.T * p.Hq) return;
   const int t = gw / p.Hq, h = gw - t * p.Hq, per = p.Hq / p.Hk, g = h / per, map = (h - g * per) / (per / p.maps);
-  const int pos = p.positions[t], lo = max(0, pos - p.window + 1), kept = min(p.keep, lo), skip = lo - kept;
+  const int pos = p.positions[t], lo = first_key(pos, p.window, p.chunk), kept = min(p.keep, lo), skip = lo - kept;
   const int* table = p.table + size_t(p.tok_seq[t]) * p.max_pages;
   if (lane * 8 < p.dk) {
     float x[8];
@@ -452,17 +487,20 @@ using namespace mfq;
 // value channels).
 extern "C" int mfq_window_attn_decode(const void* q, const void* k, const void* v, const int* table, const int* seq_lens, void* out,
                                       float* part, float* part_ml, int B, int Hq, int Hk, int maps, int dk, int dv, int max_pages, int window,
-                                      int keep, float scale, float cap, int splits, float lambda, float out_scale, float eps, int d,
-                                      const float* bias, int bias_last, const float* sink, cudaStream_t stream) {
+                                      int chunk, int keep, float scale, float cap, int splits, float lambda, float out_scale, float eps, int d,
+                                      const float* bias, int bias_last, const float* sink, const float* turn, int turn_d, int turn_rows,
+                                      cudaStream_t stream) {
+  if (chunk < 0 || (turn && (maps > 1 || turn_d <= 0 || turn_d % 2 || turn_d > dv || turn_rows <= 0))) return -1;
   if (B <= 0 || Hq <= 0 || Hk <= 0 || maps < 1 || maps > 2 || Hq % (Hk * maps) || dk % 16 || dv % 16 || dk <= 0 || dv <= 0) return -1;
   if ((bias || sink) && maps > 1) return -1;
   if (bias && bias_last < 0) return -1;
   if (dk * maps > 512 || dv > 256 || keep < 0 || (maps > 1 && (d <= 0 || d > dv))) return -1;
   if (window <= 0 || !(scale > 0.f) || splits < 1 || ((splits > 1 || maps > 1) && (!part || !part_ml))) return -1;
+  const ValueTurn back{reinterpret_cast<const float2*>(turn), turn ? turn_d / 2 : 0, turn_rows};
   const WindowDecodeParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k), static_cast<const __nv_bfloat16*>(v),
-                             table, seq_lens, static_cast<__nv_bfloat16*>(out), part, part_ml, Hq, Hk, maps, dk, dv, max_pages, window, keep,
-                             splits, (Hq / Hk + 15) / 16, make_score_cap(scale, cap), ScoreExtra{bias, nullptr, sink, bias ? bias_last : 0}};
-  const WindowMergeParams mp{sink, splits, dv, Hq / maps, Hq / Hk / maps, maps, lambda, out_scale, eps, maps > 1 ? 1.f / float(d) : 0.f};
+                             table, seq_lens, static_cast<__nv_bfloat16*>(out), part, part_ml, Hq, Hk, maps, dk, dv, max_pages, window, chunk, keep,
+                             splits, (Hq / Hk + 15) / 16, make_score_cap(scale, cap), ScoreExtra{bias, nullptr, sink, bias ? bias_last : 0}, back};
+  const WindowMergeParams mp{sink, splits, dv, Hq / maps, Hq / Hk / maps, maps, lambda, out_scale, eps, maps > 1 ? 1.f / float(d) : 0.f, back, seq_lens};
   const int kw = dk * maps;
 #define MFQ_WIN_DV(DK)                                                     \
   (dv <= 64 ? launch_window_decode<DK, 64>(p, mp, B, stream)               \
@@ -476,12 +514,12 @@ extern "C" int mfq_window_attn_decode(const void* q, const void* k, const void* 
 // output of every map.
 extern "C" int mfq_window_attn_plain(const void* q, const void* k, const void* v, const int* table, const int* tok_seq,
                                      const int* positions, void* out, int T_, int Hq, int Hk, int maps, int dk, int dv, int max_pages,
-                                     int window, int keep, float scale, float cap, const float* bias, int bias_last, const float* sink,
+                                     int window, int chunk, int keep, float scale, float cap, const float* bias, int bias_last, const float* sink,
                                      int fp32, cudaStream_t stream) {
   if (((bias || sink) && maps > 1) || (bias && bias_last < 0)) return -1;
-  if (T_ <= 0 || Hq <= 0 || Hk <= 0 || maps < 1 || Hq % (Hk * maps) || dk % 8 || dv % 8 || dk > 256 || dv > 256 || window <= 0 || keep < 0)
+  if (T_ <= 0 || Hq <= 0 || Hk <= 0 || maps < 1 || Hq % (Hk * maps) || dk % 8 || dv % 8 || dk > 256 || dv > 256 || window <= 0 || chunk < 0 || keep < 0)
     return -1;
-  const WindowPlainParams p{positions, tok_seq, table, T_, Hq, Hk, maps, dk, dv, max_pages, window, keep, scale, cap, ScoreExtra{bias, nullptr, sink, bias ? bias_last : 0}};
+  const WindowPlainParams p{positions, tok_seq, table, T_, Hq, Hk, maps, dk, dv, max_pages, window, chunk, keep, scale, cap, ScoreExtra{bias, nullptr, sink, bias ? bias_last : 0}};
   const dim3 grid(unsigned(((long long)(T_) * Hq + 3) / 4));
   if (fp32)
     launch_kernel(window_attn_plain_kernel<float>, grid, dim3(128), 0, stream, static_cast<const float*>(q), static_cast<const float*>(k),

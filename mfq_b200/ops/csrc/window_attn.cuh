@@ -62,4 +62,14 @@ struct ScoreExtra {
 };
 constexpr float kLog2e = 1.4426950408889634f;
 
+// First key that a query at position i sees (kept first keys aside): those of its window, or with chunk > 0 those of its chunk
+// [n chunk, (n + 1) chunk) of the sequence.
+__device__ __forceinline__ int first_key(int i, int window, int chunk) { return chunk > 0 ? i / chunk * chunk : max(0, i - window + 1); }
+
+// Values that carry a rotation by their position: outputs turn back by the query's.  Channel i goes with channel i + half.
+struct ValueTurn {
+  const float2* rope;  // [rows][half] (cos, sin), or null
+  int half, rows;
+};
+
 }  // namespace mfq

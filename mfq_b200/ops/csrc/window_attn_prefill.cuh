@@ -10,7 +10,8 @@
 //   P = softmax    8 warps, two threads per row; the scores' soft cap is a fused polynomial where all of a warp's scores are
 //                  small against the cap, else the exact exponential form; masks only on blocks that need them
 //   O_blk = P V    V as MN-major operand; folded into fp32 registers under the running maximum
-// Only key blocks that some query of the tile can see are visited: the pages of the kept first tokens, then those of the window;
+// Only key blocks that some query of the tile can see are visited: the pages of the kept first tokens, then those of the window (or
+// from the first query's chunk on);
 // blocks count these pages without the gap between the two.  Head widths are multiples of 16 up to 256; channels past a
 // width arrive as zeros (TMA fills them).  Pages past the sequence's last are replaced by the last one, so that every byte the
 // tensor core reads is a number (hidden keys have weight zero, and zero times a number is zero).
@@ -45,7 +46,7 @@ struct WindowPrefillParams {
   const int* table;     // [B, max_pages]
   __nv_bfloat16* out;   // [T, Hq, dv]
   int* status;
-  int Hq, Hk, maps, dk, dv, max_pages, window, keep, per, tokens;  // per: query heads per KV head and map; tokens: query tokens per tile
+  int Hq, Hk, maps, dk, dv, max_pages, window, chunk, keep, per, tokens;  // per: query heads per KV head and map; tokens: query tokens per tile
   int page_rows, head_rows, head_cols;  // rows of K / V per page, between two heads; columns between two heads (token-major form)
   int group0;        // first (KV head, map) among the query heads
   const int* shift;  // [B] token-major form (no table): "page" of a sequence's first page
@@ -78,7 +79,7 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
   const int pos0 = p.seq_lens[seq] - q_len + tok0, pos_last = pos0 + n_tok - 1;
   const int* table = p.table ? p.table + size_t(seq) * p.max_pages : nullptr;
   const int shift = p.table ? 0 : p.shift[seq];
-  const int first_page = max(0, pos0 - p.window + 1) / kWpPage, last_page = pos_last / kWpPage;
+  const int first_page = first_key(pos0, p.window, p.chunk) / kWpPage, last_page = pos_last / kWpPage;
   const int kept = min((p.keep + kWpPage - 1) / kWpPage, first_page), skip = first_page - kept;  // pages before / not visited
   const int nblk = (pos_last - skip * kWpPage) / KB + 1;
 
@@ -194,7 +195,7 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
     const int tok = row / p.per;                 // rows past n_tok * per carry nothing
     const bool row_live = tok < n_tok;
     const int q_pos = pos0 + min(tok, n_tok - 1);
-    const int lo = q_pos - p.window + 1;
+    const int lo = first_key(q_pos, p.window, p.chunk), lo_last = first_key(pos_last, p.window, p.chunk);
     const uint32_t lane_base = uint32_t(quarter * 32) << 16;
     float o[kOut];
 #pragma unroll
@@ -222,8 +223,8 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __g
       tc_fence_after();
       // places count visited keys; the key at place n is n before the gap (n < kept pages), n + gap after it
       const int place0 = j * KB + half * kHalf, split = kept * kWpPage, gap = skip * kWpPage;
-      // a mask is needed where the block holds kept pages, reaches past the FIRST query or starts before the LAST query's window
-      const bool masked = j * KB < split || j * KB + gap + KB - 1 > pos0 || j * KB + gap < pos_last - p.window + 1;
+      // a mask is needed where the block holds kept pages, reaches past the FIRST query or starts before the LAST query's first key
+      const bool masked = j * KB < split || j * KB + gap + KB - 1 > pos0 || j * KB + gap < lo_last;
       const uint32_t tS = tmem_base + sb * KB + lane_base + half * kHalf;
       float mx = -FLT_MAX, big = 0.f;
 #pragma unroll

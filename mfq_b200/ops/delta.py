@@ -85,11 +85,11 @@ def column_split(batch: int, heads: int, dk: int, dv: int) -> int:
 
 
 def conv(proj: torch.Tensor, w: torch.Tensor, state: torch.Tensor, slots: torch.Tensor, channels: int, *, starts: torch.Tensor | None = None,
-         max_q: int = 1, out: torch.Tensor | None = None) -> torch.Tensor:
-    """``silu(causal convolution)`` of the first ``channels`` columns; ``state [slots, taps - 1, channels]`` keeps the last inputs;
+         max_q: int = 1, bias: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
+    """``silu(causal convolution (+ bias))`` of the first ``channels`` columns; ``state [slots, taps - 1, channels]`` keeps the last inputs;
     ``starts [B + 1]``: first row of every portion, or None for one row per sequence."""
     out = torch.empty((proj.shape[0], channels), dtype=proj.dtype, device=proj.device) if out is None else out
-    rc = dense_lib().mfq_short_conv(ptr(proj), proj.stride(0), ptr(w), ptr(state), ptr(slots), ptr(starts), ptr(out), out.stride(0), slots.numel(),
+    rc = dense_lib().mfq_short_conv(ptr(proj), proj.stride(0), ptr(w), ptr(bias), ptr(state), ptr(slots), ptr(starts), ptr(out), out.stride(0), slots.numel(),
                                     max_q, channels, w.shape[0], is_fp32(proj.dtype), stream_ptr())
     check(rc, "short_conv", 2 if starts is not None and w.shape[0] > 1 else 1)
     return out

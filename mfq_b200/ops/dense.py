@@ -13,8 +13,9 @@ import torch
 
 from .lib import Workspace, check, dense_lib, ptr, stream_ptr
 
-BIAS, GLU, GELU, GELU_GLU, SOFTCAP, ADD, RELU_GLU, SILU_GLU, FLOAT = range(9)  # epilogues (dense_common.cuh)
+BIAS, GLU, GELU, GELU_GLU, SOFTCAP, ADD, RELU_GLU, SILU_GLU, FLOAT, RELU2 = range(10)  # epilogues (dense_common.cuh)
 UNITS = {"gelu": GELU_GLU, "relu": RELU_GLU, "silu": SILU_GLU}  # act(gate) * up
+ACTIVATIONS = {"relu2": RELU2}  # max(y, 0)^2
 GEMV_ROWS, GEMV_MID_ROWS, GEMV_MID_WEIGHTS = 8, 16, 8 << 20
 
 
@@ -65,12 +66,14 @@ def plan(m: int, n: int, k: int, sms: int = 148) -> tuple[int, int]:
 class DenseLinear:
     """``[rows, cols]`` weight (rows a multiple of 16, cols of 8) with an optional fp32 bias.  ``glu``: the rows alternate
     between 8 gate and 8 up rows (:func:`interleave_glu`) and the output is the gated unit of the two, half as wide.
-    ``groups`` G > 1: G matrices on top of each other, ``[G * rows, cols]``, each with its own columns of input and output."""
+    ``act``: an activation of the output without a gate (:data:`ACTIVATIONS`).  ``groups`` G > 1: G matrices on top of each other,
+    ``[G * rows, cols]``, each with its own columns of input and output."""
 
     w: torch.Tensor
     bias: torch.Tensor | None = None
     glu: tuple[float, float] | str | None = None  # (alpha, limit) of the clipped GLU, or the activation: act(gate) * up
     groups: int = 1
+    act: str | None = None
     input_kind = "dense"
 
     @property
@@ -102,6 +105,9 @@ class DenseLinear:
             kind = UNITS[self.glu]
         elif self.glu is not None:
             kind, (alpha, limit) = GLU, self.glu
+        elif self.act is not None:
+            assert add_to is None and not fp32 and table is None and softcap == 0
+            kind = ACTIVATIONS[self.act]
         elif add_to is not None:
             kind, alpha = ADD, scale
         elif fp32:
@@ -160,4 +166,23 @@ def layer_norm_out(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, wi
     out = torch.empty((m, w), dtype=dtype, device=x.device)
     check(dense_lib().mfq_layer_norm_out(ptr(x), ptr(weight), ptr(bias), ptr(out), m, w, width, float(eps), is_fp32(dtype), stream_ptr()),
           "layer_norm_out")
+    return out
+
+
+def norm_conv_out(x: torch.Tensor, weight: torch.Tensor, conv: torch.Tensor, state: torch.Tensor | None, slots: torch.Tensor, width: int, eps: float,
+                  dtype: torch.dtype, *, starts: torch.Tensor | None = None, max_q: int = 1, singles: int = 0) -> torch.Tensor:
+    """``h + conv(h)`` in ``dtype``, ``h = x / sqrt(mean(x^2) + eps) * weight`` of the fp32 stream and a causal convolution over time per
+    channel (``conv [taps, W]``, last row for the current token).  ``state [slots, taps - 1, W]`` fp32 keeps every sequence's last rows
+    ``h`` (None with one tap); ``starts [B + 1]``: first row of every portion, whose first ``singles`` have one, or None for one row per
+    sequence; ``max_q``: the longest portion."""
+    out = torch.empty(x.shape, dtype=dtype, device=x.device)
+
+    def run(seqs, first, longest):
+        check(dense_lib().mfq_norm_conv(ptr(x), ptr(weight), ptr(conv), ptr(state), ptr(seqs), ptr(first), ptr(out), seqs.numel(), longest, x.shape[1],
+                                        width, conv.shape[0], float(eps), is_fp32(dtype), stream_ptr()), "norm_conv")
+    singles = slots.numel() if starts is None else singles
+    if singles:
+        run(slots[:singles], None, 1)
+    if singles < slots.numel():
+        run(slots[singles:], starts[singles:], max_q)
     return out

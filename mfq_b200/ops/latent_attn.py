@@ -2,7 +2,7 @@
 all heads of a layer, and of the layers that read its pages.
 
 Single tokens and short portions attend in latent space: queries come mapped there (``W_uk^T q``), the value of a token is the latent
-part of its row.  Longer bf16 portions expand the visible rows to keys and values per head (:func:`visible_rows`, a product, then
+part of its row.  A head may have a sink, one more term of its denominator.  Longer bf16 portions expand the visible rows to keys and values per head (:func:`visible_rows`, a product, then
 :func:`prefill_rows` on the tcgen05 kernel), which costs fewer operations per pair.
 """
 
@@ -34,6 +34,18 @@ def finish(proj: torch.Tensor, pages: torch.Tensor | None, positions, slots, *, 
     return q_latent, q
 
 
+def down(proj: torch.Tensor, pages: torch.Tensor, positions, slots, *, q_rank: int, real_q_rank: int, rank: int, rot: int, real_rank: int, real_rot: int,
+         q_norm, norm_w, rope, eps: float) -> torch.Tensor:
+    """``proj [T, q_rank + rank + rot]``: the shared row as in :func:`finish`, and the normed query latents ``[T, q_rank]``, from which a
+    product makes the queries (:func:`finish` without pages then turns their rotated part)."""
+    t = proj.shape[0]
+    out = torch.empty((t, q_rank), dtype=proj.dtype, device=proj.device)
+    check(dense_lib().mfq_latent_down(ptr(proj), proj.stride(0), ptr(out), ptr(pages), ptr(positions), ptr(slots), ptr(q_norm), ptr(norm_w), ptr(rope),
+                                      rope.shape[0] if rope is not None else 0, t, q_rank, real_q_rank, rank, real_rank, rot, real_rot, float(eps),
+                                      is_fp32(proj.dtype), stream_ptr()), "latent_down")
+    return out
+
+
 def decode_splits(batch: int, heads: int, keys: int) -> int:
     """KV splits per query token and CTA (up to 32 heads) over ``keys`` visible keys: about a CTA for every SM, 128 keys each at
     least."""
@@ -42,7 +54,7 @@ def decode_splits(batch: int, heads: int, keys: int) -> int:
 
 
 def decode(q: torch.Tensor, pages: torch.Tensor, block_table, lens, *, rank: int, window: int, scale: float, splits: int = 1,
-           tok_seq: torch.Tensor | None = None) -> torch.Tensor:
+           tok_seq: torch.Tensor | None = None, sink: torch.Tensor | None = None) -> torch.Tensor:
     """bf16 ``q [T, H, rank + rot]`` -> ``[T, H, rank]``.  ``lens`` count the query token (one row of the table per query), or with
     ``tok_seq`` (query -> row of the table) they are the queries' positions."""
     t, h, r = q.shape
@@ -51,17 +63,18 @@ def decode(q: torch.Tensor, pages: torch.Tensor, block_table, lens, *, rank: int
     splits = max(1, min(splits, ws.attn_acc.numel() // max(1, t * h * rank), ws.attn_ml.numel() // (2 * t * h)))
     rc = dense_lib().mfq_latent_decode(ptr(q), ptr(pages), ptr(block_table), ptr(tok_seq), ptr(lens), 0 if tok_seq is None else 1, ptr(out),
                                        ptr(ws.attn_acc), ptr(ws.attn_ml), t, h, rank, r - rank, block_table.stride(0), window, float(scale),
-                                       splits, stream_ptr())
+                                       splits, ptr(sink), stream_ptr())
     check(rc, "latent_decode", 2 if splits > 1 else 1)
     return out
 
 
-def plain(q: torch.Tensor, pages: torch.Tensor, block_table, tok_seq, positions, *, rank: int, window: int, scale: float) -> torch.Tensor:
+def plain(q: torch.Tensor, pages: torch.Tensor, block_table, tok_seq, positions, *, rank: int, window: int, scale: float,
+          sink: torch.Tensor | None = None) -> torch.Tensor:
     """The same in fp32 arithmetic: query ``t`` is at ``positions[t]`` of sequence ``tok_seq[t]``."""
     t, h, r = q.shape
     out = torch.empty((t, h, rank), dtype=q.dtype, device=q.device)
     rc = dense_lib().mfq_latent_plain(ptr(q), ptr(pages), ptr(block_table), ptr(tok_seq), ptr(positions), ptr(out), t, h, rank, r - rank,
-                                      block_table.stride(0), window, float(scale), is_fp32(q.dtype), stream_ptr())
+                                      block_table.stride(0), window, float(scale), ptr(sink), is_fp32(q.dtype), stream_ptr())
     check(rc, "latent_plain")
     return out
 
@@ -87,11 +100,11 @@ def visible_rows(pages: torch.Tensor, block_table, seq: torch.Tensor, shift: tor
 
 
 def prefill_rows(q: torch.Tensor, kv: torch.Tensor, shift, q_starts, seq_lens, max_q: int, *, head0: int, heads: int, dk: int, dv: int,
-                 window: int, scale: float, out: torch.Tensor) -> None:
+                 window: int, scale: float, out: torch.Tensor, sink: torch.Tensor | None = None) -> None:
     """Portions (bf16) over expanded rows: ``kv [rows, heads * (dk + dv)]`` of the heads ``head0 ..`` of ``q [T, Hq, dk]``; writes those
-    heads of ``out [T, Hq, dv]``."""
+    heads of ``out [T, Hq, dv]``.  ``sink [Hq]``."""
     t, hq, _ = q.shape
     rc = dense_lib().mfq_window_attn_prefill_rows(ptr(q), ptr(kv), ptr(shift), ptr(q_starts), ptr(seq_lens), ptr(out), t, seq_lens.numel(), max_q,
-                                                  hq, head0, heads, dk, dv, kv.shape[0], window, float(scale),
+                                                  hq, head0, heads, dk, dv, kv.shape[0], window, float(scale), ptr(sink),
                                                   ptr(Workspace.get(q.device).status), stream_ptr())
     check(rc, "window_attn_prefill_rows")

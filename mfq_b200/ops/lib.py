@@ -63,22 +63,28 @@ _DENSE_SIGNATURES = {
     "mfq_moe_add_experts": [_vp] * 4 + [_i] * 3 + [_f, _i, _vp],
     "mfq_layer_norm_out": [_vp] * 4 + [_i] * 3 + [_f, _i, _vp],
     "mfq_token_shift": [_vp] * 7 + [_i] * 4 + [_vp],
-    "mfq_short_conv": [_vp, _i] + [_vp] * 5 + [_i] * 6 + [_vp],
+    "mfq_short_conv": [_vp, _i] + [_vp] * 6 + [_i] * 6 + [_vp],
+    "mfq_norm_conv": [_vp] * 7 + [_i] * 5 + [_f, _i, _vp],
+    "mfq_turn_back": [_vp] * 3 + [_i] * 7 + [_vp],
+    "mfq_ssd_recurrent": [_vp] * 9 + [_i] * 9 + [_vp],
+    "mfq_ssd_chunk": [_vp] * 11 + [_i] * 10 + [_vp],
+    "mfq_ssd_gate_norm": [_vp] * 4 + [_i] * 6 + [_f, _i, _vp],
+    "mfq_latent_down": [_vp, _i] + [_vp] * 7 + [_i] * 8 + [_f, _i, _vp],
     "mfq_latent_finish": [_vp, _i] + [_vp] * 7 + [_i] * 9 + [_f, _i, _vp],
     "mfq_latent_pages": [_vp] * 5 + [_i] * 3 + [_vp],
-    "mfq_latent_decode": [_vp] * 5 + [_i] + [_vp] * 3 + [_i] * 6 + [_f, _i, _vp],
-    "mfq_latent_plain": [_vp] * 6 + [_i] * 6 + [_f, _i, _vp],
+    "mfq_latent_decode": [_vp] * 5 + [_i] + [_vp] * 3 + [_i] * 6 + [_f, _i, _vp, _vp],
+    "mfq_latent_plain": [_vp] * 6 + [_i] * 6 + [_f, _vp, _i, _vp],
     "mfq_delta_chunk": [_vp] * 13 + [_i] * 15 + [_f, _f, _vp, _vp],
     "mfq_delta_recurrent": [_vp] * 11 + [_i] * 12 + [_f, _f, _i, _vp],
     "mfq_embed_scaled": [_vp, _vp, _f, _vp, _vp, _i, _i, _i, _vp],
     "mfq_norm_add": [_vp, _vp, _vp, _vp, _i, _i, _i, _f, _i, _vp],
     "mfq_norm_out": [_vp, _vp, _vp, _i, _i, _i, _f, _i, _vp],
-    "mfq_qkv_finish": [_vp, _i, _vp, _i, _f] + [_vp] * 8 + [_i] * 11 + [_f, _f, _i, _i, _vp],
+    "mfq_qkv_finish": [_vp, _i, _vp, _i, _f] + [_vp] * 8 + [_i] * 11 + [_f, _f, _i, _vp, _i, _i, _i, _vp],
     "mfq_map_difference": [_vp, _vp, _i, _i, _i, _i, _i, _f, _f, _f, _i, _vp],
-    "mfq_window_attn_decode": [_vp] * 8 + [_i] * 9 + [_f, _f, _i, _f, _f, _f, _i, _vp, _i, _vp, _vp],
-    "mfq_window_attn_plain": [_vp] * 7 + [_i] * 9 + [_f, _f, _vp, _i, _vp, _i, _vp],
-    "mfq_window_attn_prefill": [_vp] * 7 + [_i] * 12 + [_f, _f, _vp, _i, _vp, _vp, _vp, _vp],
-    "mfq_window_attn_prefill_rows": [_vp] * 6 + [_i] * 10 + [_f, _vp, _vp],
+    "mfq_window_attn_decode": [_vp] * 8 + [_i] * 10 + [_f, _f, _i, _f, _f, _f, _i, _vp, _i, _vp, _vp, _i, _i, _vp],
+    "mfq_window_attn_plain": [_vp] * 7 + [_i] * 10 + [_f, _f, _vp, _i, _vp, _i, _vp],
+    "mfq_window_attn_prefill": [_vp] * 7 + [_i] * 13 + [_f, _f, _vp, _i, _vp, _vp, _vp, _vp],
+    "mfq_window_attn_prefill_rows": [_vp] * 6 + [_i] * 10 + [_f, _vp, _vp, _vp],
     "mfq_gla_recurrent": [_vp] * 8 + [_i] * 8 + [_f, _f, _f, _i, _i, _vp, _i, _vp],
     "mfq_gla_chunk": [_vp] * 11 + [_i] * 8 + [_f, _f, _f, _i, _i, _vp, _vp],
 }

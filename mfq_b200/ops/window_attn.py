@@ -1,7 +1,8 @@
-"""Attention over unquantized pages with a sliding window, kept first tokens, an optional score cap and one or two maps
+"""Attention over unquantized pages with a sliding window or in chunks, kept first tokens, an optional score cap and one or two maps
 (``csrc/window_attn*.cu``), with one map also a score bias by distance and a sink per head, and the per-head stage in front of it (``csrc/stream_ops.cu``).
 
-A query at position ``i`` sees the keys ``j <= i`` with ``i - j < window`` or ``j < keep``; a score is ``q . k * scale``, then
+A query at position ``i`` sees the keys ``j <= i`` with ``i - j < window`` (or, with a ``chunk`` size, those of its own chunk ``i // chunk``)
+or ``j < keep``; a score is ``q . k * scale``, then
 ``cap * tanh(score / cap)`` (``cap`` 0: no cap), then plus the head's bias for the distance ``i - j`` (:class:`DistanceBias`).  A sink
 adds ``exp(sink)`` to the head's denominator.  Pages: ``k [pages, Hk, 16, maps * dk]``, ``v [pages, Hk, 16, dv]``, widths
 ``dk`` and ``dv`` multiples of 16 up to 256.  bf16 runs on tensor cores (one kernel for portions of prompts, one for single
@@ -10,6 +11,8 @@ tokens), fp32 on a plain kernel.
 Two maps (differential attention): every query and KV head has two query / key vectors that attend on their own over the same
 values; a head's output is ``rms(a1 - lambda a2) * scale`` (:class:`Difference`).  Queries are ordered ``[KV head][map][query
 head of the KV head]``.
+
+Values may carry a rotation by their position; a head's output then turns back by the query's (:class:`ValueTurn`).
 """
 
 from __future__ import annotations
@@ -35,6 +38,14 @@ class Difference:
     scale: float
     eps: float
     dim: int  # real value channels
+
+
+@dataclass(frozen=True)
+class ValueTurn:
+    """Values divided by their root mean square over ``dim`` channels and rotated by their position before they are cached."""
+
+    rope: torch.Tensor  # [positions, dim / 2, 2]
+    dim: int
 
 
 @dataclass
@@ -67,6 +78,16 @@ def log_buckets(rows: int, most: float) -> list[int]:
 
 
 @dataclass(frozen=True)
+class LinearScaling:
+    """Every rotation frequency divided by ``factor``."""
+
+    factor: float
+
+    def __call__(self, f: float) -> float:
+        return f / self.factor
+
+
+@dataclass(frozen=True)
 class FrequencyScaling:
     """Rotation frequencies for contexts longer than the original one: frequencies that turn less than ``low`` times over the
     original context are divided by ``factor``, those that turn more than ``high`` times are kept, with a linear blend between."""
@@ -88,9 +109,9 @@ class FrequencyScaling:
 
 def rope_table(base: float, dims: int, positions: int, device, scaling=None) -> torch.Tensor:
     """``[positions, dims / 2, 2]`` fp32 (cos, sin) of ``p * f_i``, ``f_i = base^(-2i / dims)``, in double precision.  ``scaling``: a
-    :class:`FrequencyScaling`, or a :class:`~mfq_b200.models.rope_scaling.YarnScaling`, which also lengthens the rotated pairs."""
+    :class:`FrequencyScaling`, a :class:`LinearScaling`, or a :class:`~mfq_b200.models.rope_scaling.YarnScaling`, which also lengthens the rotated pairs."""
     freq, length = [float(base) ** (-2.0 * i / dims) for i in range(dims // 2)], 1.0
-    if isinstance(scaling, FrequencyScaling):
+    if isinstance(scaling, (FrequencyScaling, LinearScaling)):
         freq = [scaling(f) for f in freq]
     elif scaling is not None:
         freq, length = scaling.frequencies(dims, base), scaling.mscale
@@ -100,12 +121,12 @@ def rope_table(base: float, dims: int, positions: int, device, scaling=None) -> 
 
 def qkv_finish(qkv: torch.Tensor, kv, positions, slots, *, heads: int, kv_heads: int, dim: int, q_norm, k_norm, rope, rot: int,
                eps: float, v_first: torch.Tensor | None = None, mix: float = 0.0, maps: int = 1, pairs: bool = False,
-               dk: int | None = None, temperature: tuple[float, int] | None = None) -> torch.Tensor:
+               dk: int | None = None, temperature: tuple[float, int] | None = None, turn: ValueTurn | None = None) -> torch.Tensor:
     """Per-head RMS norm of q and k (over ``dim`` channels; no norm without weights), rotation of the leading ``rot`` channels
     (``i`` with ``i + rot / 2``, or with its neighbour: ``pairs``), K and V into their pages; returns ``q [T, maps * heads, dk]``.
     ``v_first`` (``[T, kv_heads * dv]``, rows may be strided): the cached values are ``(1 - mix) v + mix v_first``.  ``kv`` None:
     the rows hold queries only (of stored width ``dk``).  ``temperature`` (coef, every): queries at position p times
-    ``1 + coef * ln(floor((p + 1) / every) + 1)``."""
+    ``1 + coef * ln(floor((p + 1) / every) + 1)``.  ``turn``: values are normed and rotated, in the same layout of pairs."""
     t = qkv.shape[0]
     if kv is not None:
         dk, dv, page = kv.k.shape[-1] // maps, kv.v.shape[-1], kv.page_size
@@ -116,8 +137,8 @@ def qkv_finish(qkv: torch.Tensor, kv, positions, slots, *, heads: int, kv_heads:
     rc = dense_lib().mfq_qkv_finish(ptr(qkv), qkv.stride(0), ptr(v_first), v_first.stride(0) if v_first is not None else 0, float(mix),
                                     ptr(q), ptr(kv.k) if kv is not None else None, ptr(kv.v) if kv is not None else None, ptr(positions),
                                     ptr(slots), ptr(q_norm), ptr(k_norm), ptr(rope), rope.shape[0] if rope is not None else 0, t,
-                                    maps * heads, kv_heads, maps, dim, dk, dv, rot, int(pairs), page, float(eps), float(temp), int(every), is_fp32(qkv.dtype),
-                                    stream_ptr())
+                                    maps * heads, kv_heads, maps, dim, dk, dv, rot, int(pairs), page, float(eps), float(temp), int(every), ptr(turn.rope) if turn is not None else None,
+                                    turn.dim if turn is not None else 0, turn.rope.shape[0] if turn is not None else 0, is_fp32(qkv.dtype), stream_ptr())
     check(rc, "qkv_finish")
     return q
 
@@ -129,6 +150,14 @@ def difference(a: torch.Tensor, kv_heads: int, d: Difference, out: torch.Tensor 
     check(dense_lib().mfq_map_difference(ptr(a), ptr(out), t, rows // 2, rows // 2 // kv_heads, dv, d.dim, d.weight, d.scale, d.eps,
                                          is_fp32(a.dtype), stream_ptr()), "map_difference")
     return out
+
+
+def turn_back(o: torch.Tensor, turn: ValueTurn, positions, pairs: bool = False) -> torch.Tensor:
+    """``o [T, H, dv]`` in place: every head's output turned by minus the token's position."""
+    t, h, dv = o.shape
+    check(dense_lib().mfq_turn_back(ptr(o), ptr(turn.rope), ptr(positions), t, h, dv, turn.dim, turn.rope.shape[0], int(pairs), is_fp32(o.dtype),
+                                    stream_ptr()), "turn_back")
+    return o
 
 
 def decode_splits(batch: int, kv_heads: int, keys: int) -> int:
@@ -150,9 +179,10 @@ def _bias_args(bias: DistanceBias | None) -> tuple:
 
 
 def decode(q: torch.Tensor, kv, block_table, seq_lens, *, window: int, scale: float, cap: float, keep: int = 0,
-           diff: Difference | None = None, bias: DistanceBias | None = None, sink: torch.Tensor | None = None, splits: int = 1, out=None):
+           diff: Difference | None = None, bias: DistanceBias | None = None, sink: torch.Tensor | None = None, chunk: int = 0,
+           turn: ValueTurn | None = None, splits: int = 1, out=None):
     """One query token per sequence (bf16): ``q [B, Hq, dk]`` -> ``[B, Hq, dv]``, or ``[B, Hq / 2, dv]`` with ``diff``;
-    ``seq_lens`` count the query token."""
+    ``seq_lens`` count the query token.  ``turn``: outputs turn back (halves; one map)."""
     b, hq, dk = q.shape
     hk, dv = kv.k.shape[1], kv.v.shape[-1]
     maps = 1 if diff is None else 2
@@ -163,21 +193,22 @@ def decode(q: torch.Tensor, kv, block_table, seq_lens, *, window: int, scale: fl
     assert not parts or (b * hq * splits * dv <= ws.attn_acc.numel() and b * hq * splits * 2 <= ws.attn_ml.numel())
     how = (diff.weight, diff.scale, diff.eps, diff.dim) if diff is not None else (0.0, 1.0, 0.0, dv)
     rc = dense_lib().mfq_window_attn_decode(ptr(q), ptr(kv.k), ptr(kv.v), ptr(block_table), ptr(seq_lens), ptr(out), ptr(ws.attn_acc),
-                                            ptr(ws.attn_ml), b, hq, hk, maps, dk, dv, block_table.stride(0), window, keep, float(scale),
-                                            float(cap), splits, *how, *_bias_args(bias), ptr(sink), stream_ptr())
+                                            ptr(ws.attn_ml), b, hq, hk, maps, dk, dv, block_table.stride(0), window, chunk, keep, float(scale),
+                                            float(cap), splits, *how, *_bias_args(bias), ptr(sink), ptr(turn.rope) if turn is not None else None,
+                                            turn.dim if turn is not None else 0, turn.rope.shape[0] if turn is not None else 0, stream_ptr())
     check(rc, "window_attn_decode", 2 if parts else 1)
     return out
 
 
 def prefill(q: torch.Tensor, kv, block_table, q_starts, seq_lens, max_q: int, *, window: int, scale: float, cap: float, keep: int = 0,
-            maps: int = 1, bias: DistanceBias | None = None, sink: torch.Tensor | None = None, out=None):
+            maps: int = 1, bias: DistanceBias | None = None, sink: torch.Tensor | None = None, chunk: int = 0, out=None):
     """Portions of several sequences (bf16): rows ``q_starts[b] .. q_starts[b + 1] - 1`` of ``q [T, Hq, dk]`` are the last
     tokens of a sequence of ``seq_lens[b]``.  ``max_q``: the longest portion (host).  Writes the output of every map."""
     t, hq, dk = q.shape
     hk, dv = kv.k.shape[1], kv.v.shape[-1]
     out = torch.empty((t, hq, dv), dtype=q.dtype, device=q.device) if out is None else out
     rc = dense_lib().mfq_window_attn_prefill(ptr(q), ptr(kv.k), ptr(kv.v), ptr(block_table), ptr(q_starts), ptr(seq_lens), ptr(out), t,
-                                             seq_lens.numel(), max_q, hq, hk, maps, dk, dv, kv.k.shape[0], block_table.stride(0), window,
+                                             seq_lens.numel(), max_q, hq, hk, maps, dk, dv, kv.k.shape[0], block_table.stride(0), window, chunk,
                                              keep, float(scale), float(cap), *_bias_args(bias), ptr(bias.top) if bias is not None else None, ptr(sink),
                                              ptr(Workspace.get(q.device).status), stream_ptr())
     check(rc, "window_attn_prefill")
@@ -185,13 +216,13 @@ def prefill(q: torch.Tensor, kv, block_table, q_starts, seq_lens, max_q: int, *,
 
 
 def plain(q: torch.Tensor, kv, block_table, tok_seq, positions, *, window: int, scale: float, cap: float, keep: int = 0, maps: int = 1,
-          bias: DistanceBias | None = None, sink: torch.Tensor | None = None):
+          bias: DistanceBias | None = None, sink: torch.Tensor | None = None, chunk: int = 0):
     """The same in fp32 arithmetic for any mix of tokens: token ``t`` is at ``positions[t]`` of sequence ``tok_seq[t]``."""
     t, hq, dk = q.shape
     hk, dv = kv.k.shape[1], kv.v.shape[-1]
     out = torch.empty((t, hq, dv), dtype=q.dtype, device=q.device)
     rc = dense_lib().mfq_window_attn_plain(ptr(q), ptr(kv.k), ptr(kv.v), ptr(block_table), ptr(tok_seq), ptr(positions), ptr(out), t, hq,
-                                           hk, maps, dk, dv, block_table.stride(0), window, keep, float(scale), float(cap),
+                                           hk, maps, dk, dv, block_table.stride(0), window, chunk, keep, float(scale), float(cap),
                                            *_bias_args(bias), ptr(sink), is_fp32(q.dtype), stream_ptr())
     check(rc, "window_attn_plain")
     return out

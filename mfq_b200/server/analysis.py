@@ -108,6 +108,8 @@ def _own_family(cfg: dict):
         from ..models.kamedra import KamedraConfig as Config, tensor_shapes
     elif cfg.get("family") == "bufolorn":
         from ..models.bufolorn import BufolornConfig as Config, tensor_shapes
+    elif cfg.get("family") == "gogivik":
+        from ..models.gogivik import GogivikConfig as Config, tensor_shapes
     else:
         return None
     own = Config.from_dict(cfg)

@@ -240,12 +240,12 @@ def test_weights_as_stored_compute_the_same_products(dtype):
                 assert p.norm is None and len(got) == h * (d + r)
             lat, key = rng.standard_normal(m.kv_rank), rng.standard_normal(m.rot_dim)
             k, v = (w[n + "uk"] @ lat).reshape(h, m.dim), (w[n + "uv"] @ lat).reshape(h, m.vdim)
-            a = mat(p.absorb).reshape(h, c, d)
+            a = mat(p.up.absorb).reshape(h, c, d)
             assert np.allclose(np.einsum("hcd,hd,c->h", a, q[:, :d], wide(lat, c)), (q[:, : m.dim] * k).sum(1))
-            assert np.allclose((mat(p.value_up) @ wide(lat, c)).reshape(h, e)[:, : m.vdim], v)
-            assert (p.expand is None) == (dtype == torch.float32)
-            if p.expand is not None:
-                kv = (p.expand.double().numpy() @ np.concatenate([wide(lat, c), wide(key, r)])).reshape(h, d + r + e)
+            assert np.allclose((mat(p.up.value_up) @ wide(lat, c)).reshape(h, e)[:, : m.vdim], v)
+            assert (p.up.expand is None) == (dtype == torch.float32)
+            if p.up.expand is not None:
+                kv = (p.up.expand.double().numpy() @ np.concatenate([wide(lat, c), wide(key, r)])).reshape(h, d + r + e)
                 assert np.allclose(kv[:, : m.dim], k) and np.allclose(kv[:, d : d + m.rot_dim], key[None]) and np.allclose(kv[:, d + r : d + r + m.vdim], v)
             y, yp = rng.standard_normal((h, m.vdim)), np.zeros((h, e))
             yp[:, : m.vdim] = y
