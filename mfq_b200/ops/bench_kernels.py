@@ -320,19 +320,20 @@ def bench_bias(batch: int, ctx: int, hq: int, hk: int, d: int, most: int, reps: 
     return {"kernel": "window_attn_prefill (bias, sink)", **shape, "us": ms * 1e3, "tflops": 2 * ctx * (ctx + 1) * hq * d / ms / 1e9}
 
 
-def bench_latent(batch: int, ctx: int, heads: int, window: int, reps: int, splits=None) -> list[dict]:
+def bench_latent(batch: int, ctx: int, heads: int, window: int, reps: int, splits=None, sink: bool = False) -> list[dict]:
     """Latent attention at rank 512, 128 + 64 query channels, values of 128: a decode step (attention and the products into and out of
     latent space), or for batch 0 one prompt (copy of the rows, expansion, attention)."""
     from . import dense, latent_attn
     d, rot, e, rank, seen = 128, 64, 128, 512, min(ctx, window)
     r, layers = rank + rot, max(1, min(32, math.ceil(4 * L2_BYTES / (max(1, batch) * seen * 576 * 2))))
     cache = _plain_cache(max(1, batch), ctx, 1, r, 0, layers)
-    shape = {"batch": batch, "ctx": ctx, "heads": heads, "window": window}
+    shape = {"batch": batch, "ctx": ctx, "heads": heads, "window": window} | ({"sink": True} if sink else {})
+    sinks = torch.zeros(heads, device="cuda") if sink else None
     if batch:
         q = torch.randn((batch, heads, r), device="cuda").to(torch.bfloat16)
         sl = torch.full((batch,), ctx, dtype=torch.int32, device="cuda")
         splits = latent_attn.decode_splits(batch, heads, seen) if splits is None else splits
-        ms = time_ms(lambda i: latent_attn.decode(q, cache.layer(i % layers).k, cache.block_table, sl, rank=rank, window=window, scale=0.07, splits=splits), reps)
+        ms = time_ms(lambda i: latent_attn.decode(q, cache.layer(i % layers).k, cache.block_table, sl, rank=rank, window=window, scale=0.07, splits=splits, sink=sinks), reps)
         rows = [{"kernel": "latent_decode", **shape, "splits": splits, "us": ms * 1e3, "gbs": batch * seen * r * 2 / ms / 1e6,
                  "tile_gbs": batch * seen * r * 2 * math.ceil(heads / 16) / ms / 1e6}]
         copies = 16
@@ -355,7 +356,7 @@ def bench_latent(batch: int, ctx: int, heads: int, window: int, reps: int, split
     out = torch.empty((ctx, heads, e), device="cuda", dtype=torch.bfloat16)
     starts, lens = (torch.tensor(v, dtype=torch.int32, device="cuda") for v in ([0, ctx], [ctx]))
     ms = time_ms(lambda _: latent_attn.prefill_rows(q, kv, shift, starts, lens, ctx, head0=0, heads=heads, dk=d + rot, dv=e, window=window, scale=0.07,
-                                                    out=out), reps)
+                                                    sink=sinks, out=out), reps)
     w = min(window, ctx)
     pairs = w * (w + 1) // 2 + (ctx - w) * w
     return rows + [{"kernel": "window_attn_prefill (expanded rows)", **shape, "us": ms * 1e3, "tflops": 2 * pairs * heads * (d + rot + e) / ms / 1e9}]
@@ -432,12 +433,97 @@ def bench_experts(tokens: int, width: int, ff: int, experts: int, top: int, reps
     return rows + [{"kernel": "experts, FP8", **shape, "us": ms * 1e3, "gbs": used * 3 * width * ff / ms / 1e6, "tflops": flops / ms / 1e9}]
 
 
+def bench_ssd(batch: int, tokens: int, h: int, groups: int, n: int, p: int, reps: int, chunk=None, heads=None) -> list[dict]:
+    """State-space recurrence with its convolution and gated norm, as :func:`bench_gla`."""
+    from . import ssd
+    geo, t = ssd.Geometry(h, groups, n, p, p, 4, groups, 1e-5), batch * tokens
+    w = ssd.Weights(torch.randn((4, geo.channels), device="cuda"), torch.randn(geo.channels, device="cuda"), torch.randn(h, device="cuda") - 2,
+                    torch.ones(h, device="cuda"), torch.ones(h, device="cuda"), torch.ones(h * p, device="cuda"))
+    proj, x = torch.randn((t, geo.row), device="cuda").to(torch.bfloat16), torch.randn((t, geo.channels), device="cuda").to(torch.bfloat16)
+    slots, hist, out = torch.arange(batch, dtype=torch.int32, device="cuda"), torch.zeros((batch, 3, geo.channels), device="cuda"), torch.empty_like(x)
+    y, row = torch.empty((t, geo.inner), device="cuda", dtype=torch.bfloat16), t * (geo.channels + geo.inner + h) * 2
+    shape = {"batch": batch, "t": tokens, "h": h, "groups": groups, "n": n, "p": p}
+    mn = time_ms(lambda _: ssd.gate_norm(y, proj, w, geo), reps)
+    rows = [{"kernel": "ssd_gate_norm", **shape, "us": mn * 1e3, "gbs": t * geo.inner * 6 / mn / 1e6}]
+    if tokens == 1:
+        layers = max(1, min(32, math.ceil(4 * L2_BYTES / (batch * h * n * p * 4))))
+        states = [torch.zeros((batch, h, n, p), device="cuda") for _ in range(layers)]
+        ms = time_ms(lambda i: ssd.recurrent(x, proj, w, states[i % layers], slots, geo, out=y), reps)
+        mc = time_ms(lambda _: ssd.conv(proj, w.conv, hist, slots, geo.channels, bias=w.conv_bias, out=out), reps)
+        return rows + [{"kernel": "ssd_recurrent", **shape, "us": ms * 1e3, "gbs": (batch * h * n * p * 8 + row) / ms / 1e6},
+                       {"kernel": "short_conv (bias)", "batch": batch, "c": geo.channels, "us": mc * 1e3, "gbs": batch * geo.channels * 28 / mc / 1e6}]
+    state, starts = torch.zeros((1, h, n, p), device="cuda"), torch.tensor([0, tokens], dtype=torch.int32, device="cuda")
+    ms = time_ms(lambda _: ssd.chunked(x, proj, w, state, slots, geo, starts, tokens, out=y, chunk=chunk, heads=heads), reps)
+    mc = time_ms(lambda _: ssd.conv(proj, w.conv, hist, slots, geo.channels, starts=starts, max_q=tokens, bias=w.conv_bias, out=out), reps)
+    plan = ssd.chunk_plan(geo, tokens, tokens)
+    return rows + [{"kernel": "ssd_chunk (three kernels)", **shape, "chunk": chunk or plan[0], "heads": heads or plan[1], "us": ms * 1e3, "gbs": row / ms / 1e6},
+                   {"kernel": "short_conv (bias, two kernels)", "t": tokens, "c": geo.channels, "us": mc * 1e3, "gbs": t * geo.channels * 4 / mc / 1e6}]
+
+
+def bench_sublayer_input(m: int, h: int, reps: int) -> list[dict]:
+    """Norm and convolution of the stream in one kernel, and the norm alone: one row each of ``m`` sequences, and a prompt of ``m``."""
+    from . import dense
+    x, w, k = torch.randn((m, h), device="cuda"), torch.ones(h, device="cuda"), torch.randn((4, h), device="cuda")
+    rows, state, slots = [], torch.zeros((min(m, 64), 3, h), device="cuda"), torch.arange(min(m, 64), dtype=torch.int32, device="cuda")
+    if m <= 64:
+        ms = time_ms(lambda _: dense.norm_conv_out(x, w, k, state, slots, h, 1e-5, torch.bfloat16), reps)
+        rows.append({"kernel": "norm_conv (decode)", "m": m, "h": h, "us": ms * 1e3, "gbs": m * h * 30 / ms / 1e6})
+    else:
+        starts = torch.tensor([0, m], dtype=torch.int32, device="cuda")
+        ms = time_ms(lambda _: dense.norm_conv_out(x, w, k, state, slots[:1], h, 1e-5, torch.bfloat16, starts=starts, max_q=m), reps)
+        rows.append({"kernel": "norm_conv (prompt)", "m": m, "h": h, "us": ms * 1e3, "gbs": m * h * 6 / ms / 1e6})
+    ms = time_ms(lambda _: dense.norm_out(x, w, h, 1e-5, torch.bfloat16), reps)
+    return rows + [{"kernel": "norm_out", "m": m, "h": h, "us": ms * 1e3, "gbs": m * h * 6 / ms / 1e6}]
+
+
+def bench_chunks(batch: int, ctx: int, hq: int, hk: int, d: int, size: int, reps: int) -> list[dict]:
+    """Attention in chunks of ``size`` with rotated values: one token at the end of a chunk per sequence, or for batch 0 one prompt; and
+    the per-head stage in front of it."""
+    from . import window_attn
+    seen, n = min(ctx, size), batch or ctx
+    layers = max(1, min(32, math.ceil(4 * L2_BYTES / (batch * seen * hk * d * 4)))) if batch else 1
+    cache = _plain_cache(max(1, batch), ctx, hk, d, d, layers)
+    shape = {"batch": batch, "ctx": ctx, "hq": hq, "hk": hk, "d": d, "size": size}
+    q, out = torch.randn((n, hq, d), device="cuda").to(torch.bfloat16), torch.empty((n, hq, d), device="cuda", dtype=torch.bfloat16)
+    turn = window_attn.ValueTurn(window_attn.rope_table(5e5, d, ctx, "cuda"), d)
+    how = dict(window=1 << 30, chunk=size, scale=0.088, cap=0.0)
+    pos = torch.arange(n, dtype=torch.int32, device="cuda")
+    qkv, one = torch.randn((n, (hq + 2 * hk) * d), device="cuda").to(torch.bfloat16), torch.ones(d, device="cuda")
+    slots = (cache.slots(0, 0, n) if not batch else torch.cat([cache.slots(b, 0, 1) for b in range(batch)])).cuda()
+    stage = lambda turned: time_ms(lambda _: window_attn.qkv_finish(qkv, cache.layer(0), pos, slots, heads=hq, kv_heads=hk, dim=d, q_norm=one, k_norm=one,
+                                                                    rope=turn.rope, rot=d, eps=1e-5, turn=turn if turned else None), reps)
+    rows = [{"kernel": f"qkv_finish ({name})", **shape, "us": ms * 1e3, "gbs": n * (hq + 2 * hk) * d * 4 / ms / 1e6}
+            for name, ms in (("values normed and rotated", stage(True)), ("plain values", stage(False)))]
+    if batch:
+        sl, splits = torch.full((batch,), ctx, dtype=torch.int32, device="cuda"), window_attn.decode_splits(batch, hk, seen)
+        ms = time_ms(lambda i: window_attn.decode(q, cache.layer(i % layers), cache.block_table, sl, splits=splits, turn=turn, out=out, **how), reps)
+        return rows + [{"kernel": "window_attn_decode (chunks, turned)", **shape, "splits": splits, "us": ms * 1e3, "gbs": batch * seen * hk * d * 4 / ms / 1e6}]
+    starts, lens = (torch.tensor(v, dtype=torch.int32, device="cuda") for v in ([0, ctx], [ctx]))
+    ms = time_ms(lambda _: window_attn.prefill(q, cache.layer(0), cache.block_table, starts, lens, ctx, out=out, **how), reps)
+    mt = time_ms(lambda _: window_attn.turn_back(out, turn, pos), reps)
+    pairs = ctx // seen * (seen * (seen + 1) // 2)
+    return rows + [{"kernel": "window_attn_prefill (chunks)", **shape, "us": ms * 1e3, "tflops": 4 * pairs * hq * d / ms / 1e9},
+                   {"kernel": "turn_back", **shape, "us": mt * 1e3, "gbs": n * hq * d * 4 / mt / 1e6}]
+
+
+def bench_low_queries(m: int, q_rank: int, rank: int, rot: int, reps: int) -> dict:
+    """Norms of the query latent and of the shared latent row, and its page write."""
+    from . import latent_attn, window_attn
+    cache = _plain_cache(1, m, 1, rank + rot, 0, 1)
+    proj, pos = torch.randn((m, q_rank + rank + rot), device="cuda").to(torch.bfloat16), torch.arange(m, dtype=torch.int32, device="cuda")
+    slots, rope = cache.slots(0, 0, m).cuda(), window_attn.rope_table(5e5, rot, m, "cuda")
+    a, b = torch.ones(q_rank, device="cuda"), torch.ones(rank, device="cuda")
+    ms = time_ms(lambda _: latent_attn.down(proj, cache.layer(0).k, pos, slots, q_rank=q_rank, real_q_rank=q_rank, rank=rank, rot=rot, real_rank=rank,
+                                            real_rot=rot, q_norm=a, norm_w=b, rope=rope, eps=1e-5), reps)
+    return {"kernel": "latent_down", "m": m, "q_rank": q_rank, "rank": rank, "us": ms * 1e3, "gbs": m * (q_rank + rank + rot) * 4 / ms / 1e6}
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--json", default="")
     ap.add_argument("--reps", type=int, default=20)
     ap.add_argument("--quick", action="store_true")
-    ap.add_argument("--only", default="", help="comma separated kernel families: gemm,w4,attn,mla,small,prefill,dense,maps,gla,bias,latent,mixing,delta,experts")
+    ap.add_argument("--only", default="", help="comma separated kernel families: gemm,w4,attn,mla,small,prefill,dense,maps,gla,bias,latent,mixing,delta,experts,input,chunks,sink,ssd")
     ap.add_argument("--tp", type=int, default=1, help="time one rank's shard of a tensor-parallel group of this size")
     args = ap.parse_args()
     pk = peaks()
@@ -541,6 +627,26 @@ def main() -> None:
     if want("experts"):
         for tokens in (1, 16, 64, 512, 4096):
             rows += bench_experts(tokens, 4096, 2048, 32, 4, args.reps)
+    if want("input"):
+        for m in (1, 64, 4096):
+            rows += bench_sublayer_input(m, 4096, args.reps)
+            rows.append(bench_low_queries(m, 1536, 512, 64, args.reps))
+    if want("chunks"):
+        for batch in (1, 64, 0):
+            for size in (4096, 1024):
+                rows += bench_chunks(batch, 4096, 32, 8, 128, size, args.reps)
+                rows.append(bench_window_decode(batch, 4096, 32, 8, 128, size, 0.0, args.reps) if batch
+                            else bench_window_prefill(4096, 32, 8, 128, size, 0.0, args.reps))
+    if want("sink"):
+        for batch, window in ((1, 4096), (64, 4096), (64, 1024), (0, 4096), (0, 1024)):
+            for sink in (True, False):
+                rows += bench_latent(batch, 4096, 32, window, args.reps, sink=sink)
+    if want("ssd"):
+        for batch, tokens in ((1, 1), (64, 1), (1, 2048), (1, 4096)):
+            for h, groups in ((64, 1), (64, 8)):
+                rows += bench_ssd(batch, tokens, h, groups, 128, 64, args.reps)
+            rows.append(bench_gla(batch, tokens, 32, 128, 128, args.reps))
+            rows.append(bench_gla(batch, tokens, 64, 128, 64, args.reps))
     for r in rows:
         if "gbs" in r:
             r["hbm_frac"] = r["gbs"] / pk["hbm_gbs"]

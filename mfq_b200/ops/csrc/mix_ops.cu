@@ -209,31 +209,32 @@ struct NormConvParams {
 };
 
 // A CTA takes a run of tokens of a sequence: first the root mean squares of its rows and of the taps - 1 before them, then every thread
-// walks the run for 8 channels at a time.  The CTA of the sequence's first run is the only one that reads the kept rows, so it also
+// walks the run for 4 channels at a time.  The CTA of the sequence's first run is the only one that reads the kept rows, so it also
 // replaces them (by the portion's last rows), channel by channel in the same thread.
-constexpr int kNormRunTokens = 8, kNormMaxTaps = 8;
+constexpr int kNormMaxRun = 32, kNormMaxTaps = 8, kNormThreads = 512;
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256)
-norm_conv_kernel(T* __restrict__ out, const NormConvParams p) {
+__global__ void __launch_bounds__(kNormThreads, TAPS <= 4 ? 2 : 1)
+norm_conv_kernel(T* __restrict__ out, const NormConvParams p, int run) {
   pdl_trigger();
   pdl_wait();
-  constexpr int kRows = kNormRunTokens + 2 * (kNormMaxTaps - 1);
-  __shared__ float part[kRows * 8], scale[kRows];
+  constexpr int kRows = kNormMaxRun + 2 * (kNormMaxTaps - 1), kWarps = kNormThreads / 32, kAhead = TAPS <= 4 ? 4 : 8;
+  __shared__ float part[kRows * kWarps], scale[kRows];
   const int b = blockIdx.y, s = p.slot[b], W = p.W;
   const int r0 = p.starts ? p.starts[b] : b, len = p.starts ? p.starts[b + 1] - r0 : 1;
-  const int n0 = blockIdx.x * kNormRunTokens, n1 = min(len, n0 + kNormRunTokens), hist = p.taps - 1;
+  const int n0 = blockIdx.x * run, n1 = min(len, n0 + run), hist = p.taps - 1;
   if (n0 >= len) return;
   const int first = max(0, n0 - hist), tail = n0 == 0 ? max(n1, len - hist) : len;  // rows first .. n1 - 1, then tail .. len - 1
   const int rows = n1 - first + len - tail;
-  auto row_of = [&](int i) { return i < n1 - first ? first + i : tail + i - (n1 - first); };
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5, each = max(1, warps / rows);  // warps per row
+  const float* x = p.x + size_t(r0) * W;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const int each = rows <= warps ? warps / rows : 2;  // shares of a row
   for (int j = warp; j < rows * each; j += warps) {
-    const int i = j / each;
-    const float* x = p.x + size_t(r0 + row_of(i)) * W;
+    const int i = j / each, n = i < n1 - first ? first + i : tail + i - (n1 - first);
+    const float* row = x + size_t(n) * W;
     float ss = 0.f;
-#pragma unroll 4
+#pragma unroll 8
     for (int c = ((j - i * each) * 32 + lane) * 4; c < W; c += each * 128) {
-      const float4 v = *reinterpret_cast<const float4*>(x + c);
+      const float4 v = *reinterpret_cast<const float4*>(row + c);
       ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
     }
 #pragma unroll
@@ -241,67 +242,181 @@ norm_conv_kernel(T* __restrict__ out, const NormConvParams p) {
     if (lane == 0) part[j] = ss;
   }
   __syncthreads();
-  if (int(threadIdx.x) < rows) {
+  for (int i = threadIdx.x; i < rows; i += blockDim.x) {
     float ss = 0.f;
-    for (int z = 0; z < each; ++z) ss += part[threadIdx.x * each + z];
-    scale[threadIdx.x] = rsqrtf(ss * p.inv_width + p.eps);
+    for (int z = 0; z < each; ++z) ss += part[i * each + z];
+    scale[i] = rsqrtf(fmaf(ss, p.inv_width, p.eps));
   }
   __syncthreads();
   float* st = s >= 0 && hist > 0 ? p.state + size_t(s) * hist * W : nullptr;
-  for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {
-    float w[TAPS][8], win[TAPS][8], nw[8];
-    load8<float>(p.norm_w + c, nw);
-    auto normed = [&](int n, int place, float(&v)[8]) {
-      load8<float>(p.x + size_t(r0 + n) * W + c, v);
-#pragma unroll
-      for (int j = 0; j < 8; ++j) v[j] *= scale[place] * nw[j];
-    };
+  auto load4 = [](const float* src, float (&v)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(src);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+  };
+  for (int c = threadIdx.x * 4; c < W; c += blockDim.x * 4) {
+    float w[TAPS][4], win[TAPS - 1][4], nw[4];  // win: the rows before the current one, oldest first
+    load4(p.norm_w + c, nw);
 #pragma unroll
     for (int i = 0; i < TAPS; ++i) {
+      const bool used = i >= TAPS - p.taps;
+      const int n = n0 + i - (TAPS - 1);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) w[i][j] = win[i][j] = 0.f;
-      if (i - (TAPS - p.taps) >= 0) load8<float>(p.w + size_t(i - (TAPS - p.taps)) * W + c, w[i]);
-      const int n = n0 + i - TAPS;  // win[i], i > 0: row n
-      if (i > 0 && i - (TAPS - p.taps) > 0) {
-        if (n >= 0) normed(n, n - first, win[i]);
-        else if (st) load8<float>(st + size_t(n + hist) * W + c, win[i]);
+      for (int j = 0; j < 4; ++j) w[i][j] = 0.f;
+      if (used) load4(p.w + size_t(i - (TAPS - p.taps)) * W + c, w[i]);
+      if (i < TAPS - 1) {
+        float f = 0.f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) win[i][j] = 0.f;
+        if (used && n >= 0) {
+          load4(x + size_t(n) * W + c, win[i]);
+          f = scale[n - first];
+        } else if (used && st) {
+          load4(st + size_t(n + hist) * W + c, win[i]);
+        }
+        if (n >= 0) {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) win[i][j] *= f * nw[j];
+        }
       }
     }
-#pragma unroll 4
-    for (int n = n0; n < n1; ++n) {
-      float h[8], y[8];
-      normed(n, n - first, h);
+    for (int m = n0; m < n1; m += kAhead) {
+      float h[kAhead][4];
 #pragma unroll
-      for (int j = 0; j < 8; ++j) {
+      for (int e = 0; e < kAhead; ++e)
+        if (m + e < n1) load4(x + size_t(m + e) * W + c, h[e]);
 #pragma unroll
-        for (int i = 0; i + 1 < TAPS; ++i) win[i][j] = win[i + 1][j];
-        win[TAPS - 1][j] = h[j];
-        float a = h[j];
+      for (int e = 0; e < kAhead; ++e) {
+        if (m + e < n1) {
+          const float f = scale[m + e - first];
+          float y[4];
 #pragma unroll
-        for (int i = 0; i < TAPS; ++i) a = fmaf(w[i][j], win[i][j], a);
-        y[j] = a;
+          for (int j = 0; j < 4; ++j) {
+            h[e][j] *= f * nw[j];
+            y[j] = fmaf(w[TAPS - 1][j], h[e][j], h[e][j]);
+#pragma unroll
+            for (int i = 0; i < TAPS - 1; ++i) y[j] = fmaf(w[i][j], i + e < TAPS - 1 ? win[min(i + e, TAPS - 2)][j] : h[max(i + e - (TAPS - 1), 0)][j], y[j]);
+          }
+          T* dst = out + size_t(r0 + m + e) * W + c;
+          if constexpr (sizeof(T) == 4) {
+            *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1], y[2], y[3]);
+          } else {
+            __nv_bfloat162 q[2] = {__floats2bfloat162_rn(y[0], y[1]), __floats2bfloat162_rn(y[2], y[3])};
+            *reinterpret_cast<uint2*>(dst) = *reinterpret_cast<const uint2*>(q);
+          }
+        }
       }
-      store8<T>(out + size_t(r0 + n) * W + c, y);
+#pragma unroll
+      for (int i = 0; i < TAPS - 1; ++i)  // a further batch follows a whole one
+#pragma unroll
+        for (int j = 0; j < 4; ++j) win[i][j] = h[kAhead - (TAPS - 1) + i][j];
     }
     if (n0 == 0 && st) {
       for (int i = 0; i < hist; ++i) {  // ascending: place i reads place i + len > i
         const int n = len - hist + i;
-        float v[8];
-        if (n >= 0) normed(n, n < n1 ? n - first : n1 - first + n - tail, v);
-        else load8<float>(st + size_t(n + hist) * W + c, v);
-        store8<float>(st + size_t(i) * W + c, v);
+        float v[4];
+        if (n >= 0) {
+          const float f = scale[n < n1 ? n - first : n1 - first + n - tail];
+          load4(x + size_t(n) * W + c, v);
+#pragma unroll
+          for (int j = 0; j < 4; ++j) v[j] *= f * nw[j];
+        } else {
+          load4(st + size_t(n + hist) * W + c, v);
+        }
+        *reinterpret_cast<float4*>(st + size_t(i) * W + c) = make_float4(v[0], v[1], v[2], v[3]);
       }
     }
   }
 }
 
+// One row per sequence, up to 4 taps, 8 VECS channels per thread.
+constexpr int kStepTaps = 4;
+template <typename T, int VECS>
+__global__ void __launch_bounds__(kNormThreads, 1)
+norm_conv_step_kernel(T* __restrict__ out, const NormConvParams p) {
+  pdl_trigger();
+  __shared__ float red[33];
+  const int W = p.W, hist = p.taps - 1;
+  const size_t b = blockIdx.x;
+  float w[VECS][kStepTaps][8], nw[VECS][8], x[VECS][8];
+#pragma unroll
+  for (int k = 0; k < VECS; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 8;
+    if (c < W) {
+      load8<float>(p.norm_w + c, nw[k]);
+#pragma unroll
+      for (int i = 0; i < kStepTaps; ++i)
+        if (i < p.taps) load8<float>(p.w + size_t(i) * W + c, w[k][i]);
+    }
+  }
+  pdl_wait();
+  const int s = p.slot[b];
+  float* st = s >= 0 && hist > 0 ? p.state + size_t(s) * hist * W : nullptr;
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < VECS; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 8;
+    if (c < W) {
+      load8<float>(p.x + b * W + c, x[k]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss = fmaf(x[k][j], x[k][j], ss);
+    }
+  }
+  float y[VECS][8];
+#pragma unroll
+  for (int k = 0; k < VECS; ++k) {  // the kept rows, moved up by one
+    const int c = (threadIdx.x + k * blockDim.x) * 8;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) y[k][j] = 0.f;
+    if (c < W && st) {
+#pragma unroll
+      for (int i = 0; i < kStepTaps - 1; ++i) {
+        if (i < hist) {
+          float v[8];
+          load8<float>(st + size_t(i) * W + c, v);
+          if (i > 0) store8<float>(st + size_t(i - 1) * W + c, v);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) y[k][j] = fmaf(w[k][i][j], v[j], y[k][j]);
+        }
+      }
+    }
+  }
+  const float f = rsqrtf(fmaf(dense_block_sum(ss, red), p.inv_width, p.eps));
+#pragma unroll
+  for (int k = 0; k < VECS; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 8;
+    if (c < W) {
+      float last[8];
+#pragma unroll
+      for (int i = 0; i < kStepTaps; ++i)
+        if (i == hist) {
+#pragma unroll
+          for (int j = 0; j < 8; ++j) last[j] = w[k][i][j];
+        }
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        x[k][j] *= f * nw[k][j];
+        y[k][j] = fmaf(last[j], x[k][j], y[k][j]) + x[k][j];
+      }
+      store8<T>(out + b * W + c, y[k]);
+      if (st) store8<float>(st + size_t(hist - 1) * W + c, x[k]);
+    }
+  }
+}
+
 template <typename T>
-static int launch_norm_conv(void* out, const NormConvParams& p, int B, int max_q, cudaStream_t stream) {
-  const int threads = min(256, (p.W / 8 + 31) / 32 * 32);
-  const dim3 grid((max_q + kNormRunTokens - 1) / kNormRunTokens, B);
+static int launch_norm_conv(void* out, const NormConvParams& p, int B, int max_q, int tokens, cudaStream_t stream) {
   T* o = static_cast<T*>(out);
-  if (p.taps <= 4) launch_kernel(norm_conv_kernel<T, 4>, grid, dim3(threads), 0, stream, o, p);
-  else launch_kernel(norm_conv_kernel<T, kNormMaxTaps>, grid, dim3(threads), 0, stream, o, p);
+  const int vecs = p.W / 8;
+  if (!p.starts && p.taps <= kStepTaps && vecs <= 2 * kNormThreads) {
+    if (vecs <= kNormThreads) launch_kernel(norm_conv_step_kernel<T, 1>, dim3(B), dim3((vecs + 31) / 32 * 32), 0, stream, o, p);
+    else launch_kernel(norm_conv_step_kernel<T, 2>, dim3(B), dim3((vecs / 2 + 31) / 32 * 32), 0, stream, o, p);
+    return cudaGetLastError() == cudaSuccess ? 0 : -7;
+  }
+  const int threads = min(kNormThreads, (p.W / 4 + 31) / 32 * 32);
+  const int run = min(kNormMaxRun, max(8, (tokens + 8 * 148 - 1) / (8 * 148) * 4));  // at most a wave of two CTAs per SM, if that many tokens fit
+  const dim3 grid((max_q + run - 1) / run, B);
+  if (p.taps <= 4) launch_kernel(norm_conv_kernel<T, 4>, grid, dim3(threads), 0, stream, o, p, run);
+  else launch_kernel(norm_conv_kernel<T, kNormMaxTaps>, grid, dim3(threads), 0, stream, o, p, run);
   return cudaGetLastError() == cudaSuccess ? 0 : -7;
 }
 
@@ -333,13 +448,15 @@ extern "C" int mfq_token_shift(const void* h, const float* mu, float* last, cons
   return cudaGetLastError() == cudaSuccess ? 0 : -7;
 }
 
-// x [T, W] fp32; out [T, W] = h + conv(h); w [taps, W]; state [slots, taps - 1, W]; starts null: row b belongs to sequence b
+// x [T, W] fp32; out [T, W] = h + conv(h); w [taps, W]; state [slots, taps - 1, W]; starts null: row b belongs to
+// sequence b; tokens: rows of all portions
 extern "C" int mfq_norm_conv(const float* x, const float* norm_w, const float* w, float* state, const int* slot, const int* starts, void* out,
-                             int B, int max_q, int W, int width, int taps, float eps, int fp32, cudaStream_t stream) {
-  if (B <= 0 || B > 65535 || max_q <= 0 || W <= 0 || W % 8 || width <= 0 || width > W || taps < 1 || taps > kNormMaxTaps) return -1;
+                             int B, int max_q, int tokens, int W, int width, int taps, float eps, int fp32, cudaStream_t stream) {
+  if (B <= 0 || B > 65535 || max_q <= 0 || tokens <= 0 || W <= 0 || W % 8 || width <= 0 || width > W || taps < 1 || taps > kNormMaxTaps) return -1;
   if (taps > 1 && !state) return -1;
   const NormConvParams p{x, norm_w, w, state, slot, starts, W, taps, 1.f / float(width), eps};
-  return fp32 ? launch_norm_conv<float>(out, p, B, starts ? max_q : 1, stream) : launch_norm_conv<__nv_bfloat16>(out, p, B, starts ? max_q : 1, stream);
+  return fp32 ? launch_norm_conv<float>(out, p, B, starts ? max_q : 1, tokens, stream)
+              : launch_norm_conv<__nv_bfloat16>(out, p, B, starts ? max_q : 1, tokens, stream);
 }
 
 // x: rows of in_stride, channels 0 .. C - 1; w [taps, C]; bias [C] or null; state [slots, taps - 1, C]; starts null: row b belongs to sequence b

@@ -11,9 +11,9 @@ namespace mfq {
 
 constexpr int kSsdThreads = 256;
 
-// MAXR: rows a thread owns at most
-template <typename T, int MAXR>
-__global__ void __launch_bounds__(kSsdThreads)
+// MAXR: rows a thread owns at most; CTAS per SM: many for a grid of several waves, few where the latency of one CTA counts
+template <typename T, int MAXR, int CTAS>
+__global__ void __launch_bounds__(kSsdThreads, CTAS)
 ssd_recurrent_kernel(const T* __restrict__ x, const T* __restrict__ z, T* __restrict__ y, const SsdShape p, int split, int R) {
   pdl_trigger();
   extern __shared__ __align__(16) float ssd_sm[];
@@ -79,16 +79,16 @@ ssd_recurrent_kernel(const T* __restrict__ x, const T* __restrict__ z, T* __rest
     if (i < mine) *reinterpret_cast<float4*>(st + size_t(rg + R * i) * P) = s[i];
 }
 
-template <typename T, int MAXR>
+template <typename T, int MAXR, int CTAS>
 static int launch_ssd_recurrent(const void* x, const void* z, void* y, const SsdShape& p, int B, int split, int R, cudaStream_t stream) {
   const int smem = (2 * (2 * p.N + p.P / split) + R * (p.P / split)) * 4;
   if (smem > 200 * 1024) return -5;
   static int allowed = 48 * 1024;
   if (smem > allowed) {
-    if (cudaFuncSetAttribute(ssd_recurrent_kernel<T, MAXR>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -6;
+    if (cudaFuncSetAttribute(ssd_recurrent_kernel<T, MAXR, CTAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -6;
     allowed = smem;
   }
-  launch_kernel(ssd_recurrent_kernel<T, MAXR>, dim3(p.H * split, B), dim3(kSsdThreads), smem, stream, static_cast<const T*>(x), static_cast<const T*>(z),
+  launch_kernel(ssd_recurrent_kernel<T, MAXR, CTAS>, dim3(p.H * split, B), dim3(kSsdThreads), smem, stream, static_cast<const T*>(x), static_cast<const T*>(z),
                 static_cast<T*>(y), p, split, R);
   return cudaGetLastError() == cudaSuccess ? 0 : -7;
 }
@@ -153,9 +153,79 @@ ssd_gate_norm_kernel(const T* __restrict__ y, const T* __restrict__ z, const flo
   }
 }
 
+// The same where every part and head is a whole number of 8-channel vectors: a thread keeps its vectors in registers, and only their
+// sums of squares go through shared memory.
+template <typename T, int VECS>
+__global__ void __launch_bounds__(512)
+ssd_gate_norm_vec_kernel(const T* __restrict__ y, const T* __restrict__ z, const float* __restrict__ w, T* __restrict__ out, int H, int P, int d,
+                         int z_stride, int parts, float eps) {
+  pdl_trigger();
+  extern __shared__ __align__(16) float gn_sm[];
+  const int width = H * P, per = H * d / parts / 8, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  float* sum_s = gn_sm;              // [H d / 8] sums of squares of the real vectors
+  float* f_s = sum_s + H * d / 8;    // [parts]
+  const size_t t = blockIdx.x;
+  int place[VECS];                   // of my vectors among the real ones; < 0: padding or none
+  float ww[VECS][8];
+#pragma unroll
+  for (int k = 0; k < VECS; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 8, head = c / P, j = c - head * P;
+    place[k] = c < width && j < d ? (head * d + j) / 8 : -1;
+    if (c < width) load8<float>(w + c, ww[k]);
+  }
+  pdl_wait();
+  float a[VECS][8];
+#pragma unroll
+  for (int k = 0; k < VECS; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 8;
+    if (place[k] >= 0) {
+      float g[8], ss = 0.f;
+      load8<T>(y + t * width + c, a[k]);
+      load8<T>(z + t * z_stride + c, g);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        a[k][j] *= sizeof(T) == 4 ? g[j] / (1.f + expf(-g[j])) : __fdividef(g[j], 1.f + __expf(-fmaxf(g[j], -80.f)));
+        ss = fmaf(a[k][j], a[k][j], ss);
+      }
+      sum_s[place[k]] = ss;
+    }
+  }
+  __syncthreads();
+  for (int i = warp; i < parts; i += warps) {
+    float ss = 0.f;
+    for (int j = lane; j < per; j += 32) ss += sum_s[i * per + j];
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (lane == 0) f_s[i] = rsqrtf(ss / float(per * 8) + eps);
+  }
+  __syncthreads();
+#pragma unroll
+  for (int k = 0; k < VECS; ++k) {
+    const int c = (threadIdx.x + k * blockDim.x) * 8;
+    if (c < width) {
+      const float f = place[k] >= 0 ? f_s[place[k] / per] : 0.f;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) a[k][j] = place[k] >= 0 ? a[k][j] * f * ww[k][j] : 0.f;
+      store8<T>(out + t * width + c, a[k]);
+    }
+  }
+}
+
 template <typename T>
 static int launch_ssd_gate_norm(const void* y, const void* z, const float* w, void* out, int T_, int H, int P, int d, int z_stride, int parts, float eps,
                                 cudaStream_t stream) {
+  const int vecs = H * P / 8;
+  if (d % 8 == 0 && H * d / parts % 8 == 0 && vecs <= 2048) {
+    const int k = vecs <= 256 ? 1 : vecs <= 512 ? 2 : 4, threads = ((vecs + k - 1) / k + 31) / 32 * 32, bytes = (H * d / 8 + parts) * 4;
+    auto run = [&](auto kernel) {
+      launch_kernel(kernel, dim3(T_), dim3(threads), bytes, stream, static_cast<const T*>(y), static_cast<const T*>(z), w, static_cast<T*>(out), H, P, d,
+                    z_stride, parts, eps);
+    };
+    if (k == 1) run(ssd_gate_norm_vec_kernel<T, 1>);
+    else if (k == 2) run(ssd_gate_norm_vec_kernel<T, 2>);
+    else run(ssd_gate_norm_vec_kernel<T, 4>);
+    return cudaGetLastError() == cudaSuccess ? 0 : -7;
+  }
   const int smem = (H * P + parts + max(parts, 8)) * 4;
   if (smem > 200 * 1024) return -5;
   static int allowed = 48 * 1024;
@@ -182,9 +252,10 @@ extern "C" int mfq_ssd_recurrent(const void* x, const void* z, const float* dt_b
   const int R = min(N, kSsdThreads / (P / split / 4)), rows = (N + R - 1) / R;
   if (rows > 16) return -5;
   const SsdShape p{H, groups, N, P, x_stride, z_stride, dt_bias, rate, skip, starts, slot, state};
-  if (rows <= 8)
-    return fp32 ? launch_ssd_recurrent<float, 8>(x, z, y, p, B, split, R, stream) : launch_ssd_recurrent<__nv_bfloat16, 8>(x, z, y, p, B, split, R, stream);
-  return fp32 ? launch_ssd_recurrent<float, 16>(x, z, y, p, B, split, R, stream) : launch_ssd_recurrent<__nv_bfloat16, 16>(x, z, y, p, B, split, R, stream);
+  if (fp32) return launch_ssd_recurrent<float, 16, 1>(x, z, y, p, B, split, R, stream);
+  if (rows > 8) return launch_ssd_recurrent<__nv_bfloat16, 16, 2>(x, z, y, p, B, split, R, stream);
+  return H * split * B <= 4 * 148 ? launch_ssd_recurrent<__nv_bfloat16, 8, 2>(x, z, y, p, B, split, R, stream)
+                                  : launch_ssd_recurrent<__nv_bfloat16, 8, 4>(x, z, y, p, B, split, R, stream);
 }
 
 // y [T, H P], z [T, z_stride], w [H P] fp32 (zero in padding channels), d of the P channels of a head are real; parts divides H * d.

@@ -178,8 +178,8 @@ def norm_conv_out(x: torch.Tensor, weight: torch.Tensor, conv: torch.Tensor, sta
     out = torch.empty(x.shape, dtype=dtype, device=x.device)
 
     def run(seqs, first, longest):
-        check(dense_lib().mfq_norm_conv(ptr(x), ptr(weight), ptr(conv), ptr(state), ptr(seqs), ptr(first), ptr(out), seqs.numel(), longest, x.shape[1],
-                                        width, conv.shape[0], float(eps), is_fp32(dtype), stream_ptr()), "norm_conv")
+        check(dense_lib().mfq_norm_conv(ptr(x), ptr(weight), ptr(conv), ptr(state), ptr(seqs), ptr(first), ptr(out), seqs.numel(), longest, x.shape[0],
+                                        x.shape[1], width, conv.shape[0], float(eps), is_fp32(dtype), stream_ptr()), "norm_conv")
     singles = slots.numel() if starts is None else singles
     if singles:
         run(slots[:singles], None, 1)

@@ -64,7 +64,7 @@ _DENSE_SIGNATURES = {
     "mfq_layer_norm_out": [_vp] * 4 + [_i] * 3 + [_f, _i, _vp],
     "mfq_token_shift": [_vp] * 7 + [_i] * 4 + [_vp],
     "mfq_short_conv": [_vp, _i] + [_vp] * 6 + [_i] * 6 + [_vp],
-    "mfq_norm_conv": [_vp] * 7 + [_i] * 5 + [_f, _i, _vp],
+    "mfq_norm_conv": [_vp] * 7 + [_i] * 6 + [_f, _i, _vp],
     "mfq_turn_back": [_vp] * 3 + [_i] * 7 + [_vp],
     "mfq_ssd_recurrent": [_vp] * 9 + [_i] * 9 + [_vp],
     "mfq_ssd_chunk": [_vp] * 11 + [_i] * 10 + [_vp],
