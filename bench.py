@@ -547,6 +547,36 @@ def run_bufolorn(args) -> dict:
     return bench.result()
 
 
+def run_gogivik(args) -> dict:
+    """The Gogivik family (bf16; a third each state-space recurrence, latent attention in a window, and attention in chunks as long as the
+    window, every sublayer behind a convolution) beside the Bufolorn with dense feed-forwards of equal width, depth, feed-forward
+    parameters, heads and window."""
+    from mfq_b200.models import bufolorn as bf
+    from mfq_b200.models import gogivik as gv
+    bench = FamilyBench(args)
+    for size in (args.size.split(",") if args.size else ["1b", "8b"]):
+        width, ff, layers, hq, hk, hl, vocab = KAMEDRA_SIZES[size]
+        rank, d, state = 512, 128, 128
+        if args.tiny:
+            width, ff, layers, hq, hk, hl, vocab, rank, d, state = 256, 512, 4, 4, 2, 2, 1024, 64, 32, 32
+        for window in (int(w) for w in args.window.split(",")):
+            mixers = [gv.StateSpec(hq * 2, hk, state, d // 2, 4, hk),
+                      gv.LatentSpec(hq, d, d // 2, d, 3 * rank // 2, rank, (1.5 * d) ** -0.5, rot_base=5e5, window=window),
+                      gv.ChunkSpec(hq, hk, d, d, d ** -0.5, chunk=window, rot_dims=d, rot_base=5e5, rot_factor=4.0)]
+            cfg = gv.GogivikConfig.periodic(vocab_size=vocab, hidden_size=width, num_layers=layers, mixers=mixers, ff=3 * ff // 2, logit_scale=0.5)
+            weights = gv.GogivikWeights(cfg, gv.RandomTensors(cfg, bench.dev), bench.dev)
+            bench.add(f"gogivik-{size}-w{window}", gv.GogivikModel(cfg, weights), vocab, **_facts(cfg, weights))
+            del weights
+            latent = bf.LatentSpec(hq, d, d // 2, d, rank, (1.5 * d) ** -0.5, rot_base=5e5, window=window)
+            parallel = bf.ParallelSpec(bf.BiasedSpec(hq, hk, d, d, d ** -0.5, 50.0, 512.0, 0.1, 1024, buckets=32), bf.TimeMixSpec(hq, d // 2, 64), 1.0, 1.0)
+            cfg = bf.BufolornConfig.periodic(vocab_size=vocab, hidden_size=width, num_layers=layers, latent=latent, parallel=parallel,
+                                             delta_rule=bf.DeltaSpec(hq, hq // 2, d, d, 4, 64, 64), mlp=[bf.DenseSpec(ff)])
+            weights = bf.BufolornWeights(cfg, bf.RandomTensors(cfg, bench.dev), bench.dev)
+            bench.add(f"bufolorn-{size}-w{window}", bf.BufolornModel(cfg, weights), vocab, **_facts(cfg, weights))
+            del weights
+    return bench.result()
+
+
 def run_reference(args) -> dict:
     from baseline import reference_arm
     return reference_arm.run(args)
@@ -572,20 +602,21 @@ def main() -> None:
     ap.add_argument("--profile-steps", type=int, default=0,
                     help="after the timed region, run this many batched decode steps between cudaProfilerStart/Stop")
     ap.add_argument("--tiny", action="store_true", help="tiny model, for checking the harness itself")
-    ap.add_argument("--model", choices=["llama8b", "hybrid80b", "tepetar", "kamedra", "bufolorn"], default="llama8b",
+    ap.add_argument("--model", choices=["llama8b", "hybrid80b", "tepetar", "kamedra", "bufolorn", "gogivik"], default="llama8b",
                     help="llama8b: the flagship; hybrid80b: the Gated-DeltaNet + MoE hybrid with an MTP head (one GPU); "
                          "tepetar: that family in bf16 beside the FP8 Llama of equal geometry (one GPU); "
                          "kamedra: that family in bf16 beside the Tepetar of equal geometry (one GPU); "
-                         "bufolorn: that family in bf16 beside the Kamedra of equal geometry (one GPU)")
-    ap.add_argument("--size", default="", help="tepetar, kamedra, bufolorn: comma separated sizes out of " + ", ".join(TEPETAR_SIZES) + " (default 1b,8b)")
-    ap.add_argument("--window", default="4096,1024", help="tepetar, kamedra, bufolorn: comma separated window sizes")
+                         "bufolorn: that family in bf16 beside the Kamedra of equal geometry (one GPU); "
+                         "gogivik: that family in bf16 beside the Bufolorn of equal geometry (one GPU)")
+    ap.add_argument("--size", default="", help="tepetar, kamedra, bufolorn, gogivik: comma separated sizes out of " + ", ".join(TEPETAR_SIZES) + " (default 1b,8b)")
+    ap.add_argument("--window", default="4096,1024", help="tepetar, kamedra, bufolorn, gogivik: comma separated window sizes")
     args = ap.parse_args()
     if args.warmup < 3:
         args.warmup = 3
     if args.impl == "reference":
         out = run_reference(args)
     else:
-        out = {"hybrid80b": run_hybrid, "tepetar": run_tepetar, "kamedra": run_kamedra, "bufolorn": run_bufolorn}.get(args.model, run_ours)(args)
+        out = {"hybrid80b": run_hybrid, "tepetar": run_tepetar, "kamedra": run_kamedra, "bufolorn": run_bufolorn, "gogivik": run_gogivik}.get(args.model, run_ours)(args)
     if out:
         print(json.dumps(out), flush=True)
 

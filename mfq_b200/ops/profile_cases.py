@@ -252,7 +252,21 @@ def delta_case(tokens: int, batch: int) -> None:
     bench_kernels.bench_delta(batch, tokens, 32, 16, 128, 3)
 
 
-CASES = {"latent_decode": lambda: latent_case(64), "latent_prefill": lambda: latent_case(0), "delta_decode": lambda: delta_case(1, 64),
+def ssd_case(tokens: int, batch: int) -> None:
+    """64 heads with a 128 x 64 state in 8 groups: a prompt of `tokens` tokens in chunks, or (tokens 1) a decode step."""
+    from . import bench_kernels
+    bench_kernels.time_ms = lambda fn, reps, warmup=3: [fn(i) for i in range(3)] and 1.0
+    bench_kernels.bench_ssd(batch, tokens, 64, 8, 128, 64, 3)
+
+
+def sublayer_input_case() -> None:
+    """Norm and convolution of 4096 rows of 4096 channels."""
+    from . import bench_kernels
+    bench_kernels.time_ms = lambda fn, reps, warmup=3: [fn(i) for i in range(3)] and 1.0
+    bench_kernels.bench_sublayer_input(4096, 4096, 3)
+
+
+CASES = {"ssd_decode": lambda: ssd_case(1, 64), "ssd_prefill": lambda: ssd_case(2048, 1), "sublayer_input": sublayer_input_case, "latent_decode": lambda: latent_case(64), "latent_prefill": lambda: latent_case(0), "delta_decode": lambda: delta_case(1, 64),
          "delta_prefill": lambda: delta_case(2048, 1), "two_maps_decode": two_maps_decode, "two_maps_prefill": two_maps_prefill, "gla_decode": lambda: gla_case(1, 64),
          "gla_prefill": lambda: gla_case(2048, 1), "gemm_prefill": lambda: gemm(4096, 4096, 4096), "gemm_decode": lambda: gemm(64, 28672, 4096),
          "gemm_decode_splitk": lambda: gemm(64, 4096, 14336),
